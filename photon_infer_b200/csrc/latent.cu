@@ -12,15 +12,30 @@
 //   photon_head_linear      out[t, h, :] = W[h] x[t, h, :] for all heads in one launch (the absorption of W_uk
 //                           into the queries and the application of W_uv to the attention result).
 //
-// Rotation: the first rot_dims numbers of the rotated part, feature i paired with i + rot_dims / 2, angle
-// position * inv_freq[i] in 32-bit; features beyond rot_dims pass unchanged.  All arithmetic is 32-bit.
+// Rotation: the first rot_dims numbers of the rotated part, feature i paired with i + rot_dims / 2 (or, interleaved,
+// feature 2i with 2i + 1), angle position * inv_freq[i] in 32-bit; features beyond rot_dims pass unchanged.  All
+// arithmetic is 32-bit.
 #include "common.cuh"
 #include <math.h>
+
+// Number i of a rotated part x whose token stands at position p.
+template <typename T>
+__device__ __forceinline__ float rotated(const T* x, int i, int rot_dims, int interleaved, float p,
+                                         const float* __restrict__ inv_freq) {
+  if (i >= rot_dims) return to_f32(x[i]);
+  const int half = rot_dims / 2;
+  const bool second = interleaved ? (i & 1) : (i >= half);
+  const int pair = interleaved ? (i >> 1) : (second ? i - half : i);
+  const int mate = interleaved ? (i ^ 1) : (second ? i - half : i + half);
+  float sn, cs;
+  sincosf(p * inv_freq[pair], &sn, &cs);
+  return second ? to_f32(x[i]) * cs + to_f32(x[mate]) * sn : to_f32(x[i]) * cs - to_f32(x[mate]) * sn;
+}
 
 // ---------------------------------------------------------------- norms, rotation, cache write
 template <typename T>
 __global__ void latent_prep_kernel(const T* __restrict__ down, long down_stride, int q_rank, int kv_rank, int rot,
-                                   int rot_dims, const void* __restrict__ qw, int qw_bf16,
+                                   int rot_dims, int interleaved, const void* __restrict__ qw, int qw_bf16,
                                    const void* __restrict__ kw, int kw_bf16, float eps,
                                    const int* __restrict__ positions, const float* __restrict__ inv_freq,
                                    const int* __restrict__ slot_mapping, T* __restrict__ cq, long cq_stride,
@@ -35,6 +50,7 @@ __global__ void latent_prep_kernel(const T* __restrict__ down, long down_stride,
   const float qinv = 1.0f / sqrtf(ss / (float)q_rank + eps);
   for (int i = threadIdx.x; i < q_rank; i += blockDim.x)
     cq[(size_t)t * cq_stride + i] = from_f32<T>(to_f32(row[i]) * qinv * load_w(qw, qw_bf16, i));
+  if (cache == nullptr) return;                         // the layer reads rows that another one has stored
   // key/value latent
   const T* kv = row + q_rank;
   float s2 = 0.f;
@@ -51,29 +67,16 @@ __global__ void latent_prep_kernel(const T* __restrict__ down, long down_stride,
   for (int i = threadIdx.x; i < kv_rank; i += blockDim.x)
     dst[i] = from_f32<T>(to_f32(kv[i]) * kinv * load_w(kw, kw_bf16, i));
   const T* kr = kv + kv_rank;
-  const int half = rot_dims / 2;
   const float p = (float)positions[t];
-  for (int i = threadIdx.x; i < rot; i += blockDim.x) {
-    float y;
-    if (i < half) {
-      float sn, cs;
-      sincosf(p * inv_freq[i], &sn, &cs);
-      y = to_f32(kr[i]) * cs - to_f32(kr[i + half]) * sn;
-    } else if (i < rot_dims) {
-      float sn, cs;
-      sincosf(p * inv_freq[i - half], &sn, &cs);
-      y = to_f32(kr[i]) * cs + to_f32(kr[i - half]) * sn;
-    } else {
-      y = to_f32(kr[i]);
-    }
-    dst[kv_rank + i] = from_f32<T>(y);
-  }
+  for (int i = threadIdx.x; i < rot; i += blockDim.x)
+    dst[kv_rank + i] = from_f32<T>(rotated(kr, i, rot_dims, interleaved, p, inv_freq));
 }
 
 // down [T][q_rank + kv_rank + rot] (row stride in elements): the fused down-projections of a token.
-// cq [T][q_rank]: the normed query latent.  cache: [num_slots][kv_rank + rot], the pages of one layer.
+// cq [T][q_rank]: the normed query latent.  cache: [num_slots][kv_rank + rot], the pages of one layer; null: only the
+// query latent is formed (the row then needs no key/value part, kv_norm_w and slot_mapping are not read).
 PHOTON_API int photon_latent_prep(const void* down, long down_stride, int dtype, int q_rank, int kv_rank, int rot,
-                                  int rot_dims, const void* q_norm_w, int q_norm_dtype, const void* kv_norm_w,
+                                  int rot_dims, int interleaved, const void* q_norm_w, int q_norm_dtype, const void* kv_norm_w,
                                   int kv_norm_dtype, float eps, const int* positions, const float* inv_freq,
                                   const int* slot_mapping, void* cq, long cq_stride, void* cache, long num_slots,
                                   int T_, int* err, cudaStream_t stream) {
@@ -82,11 +85,11 @@ PHOTON_API int photon_latent_prep(const void* down, long down_stride, int dtype,
   const int threads = 128;
   if (dtype == PHOTON_BF16)
     latent_prep_kernel<bf16><<<T_, threads, 0, stream>>>((const bf16*)down, down_stride, q_rank, kv_rank, rot, rot_dims,
-        q_norm_w, q_norm_dtype == PHOTON_BF16, kv_norm_w, kv_norm_dtype == PHOTON_BF16, eps, positions, inv_freq,
+        interleaved, q_norm_w, q_norm_dtype == PHOTON_BF16, kv_norm_w, kv_norm_dtype == PHOTON_BF16, eps, positions, inv_freq,
         slot_mapping, (bf16*)cq, cq_stride, (bf16*)cache, num_slots, err);
   else
     latent_prep_kernel<float><<<T_, threads, 0, stream>>>((const float*)down, down_stride, q_rank, kv_rank, rot, rot_dims,
-        q_norm_w, q_norm_dtype == PHOTON_BF16, kv_norm_w, kv_norm_dtype == PHOTON_BF16, eps, positions, inv_freq,
+        interleaved, q_norm_w, q_norm_dtype == PHOTON_BF16, kv_norm_w, kv_norm_dtype == PHOTON_BF16, eps, positions, inv_freq,
         slot_mapping, (float*)cq, cq_stride, (float*)cache, num_slots, err);
   return launch_status();
 }
@@ -95,40 +98,28 @@ PHOTON_API int photon_latent_prep(const void* down, long down_stride, int dtype,
 // q [T][heads][dim + rot] -> out [T][heads][out_head] at offset out_off: the last rot numbers of every head, rotated.
 template <typename T>
 __global__ void latent_q_rope_kernel(const T* __restrict__ q, long q_stride, int heads, int dim, int rot, int rot_dims,
-                                     const int* __restrict__ positions, const float* __restrict__ inv_freq,
+                                     int interleaved, const int* __restrict__ positions, const float* __restrict__ inv_freq,
                                      T* __restrict__ out, long out_stride, int out_head, int out_off) {
   const int t = blockIdx.x;
   const float p = (float)positions[t];
-  const int half = rot_dims / 2;
   for (int idx = threadIdx.x; idx < heads * rot; idx += blockDim.x) {
     const int h = idx / rot, i = idx - h * rot;
     const T* src = q + (size_t)t * q_stride + (size_t)h * (dim + rot) + dim;
-    float y;
-    if (i < half) {
-      float sn, cs;
-      sincosf(p * inv_freq[i], &sn, &cs);
-      y = to_f32(src[i]) * cs - to_f32(src[i + half]) * sn;
-    } else if (i < rot_dims) {
-      float sn, cs;
-      sincosf(p * inv_freq[i - half], &sn, &cs);
-      y = to_f32(src[i]) * cs + to_f32(src[i - half]) * sn;
-    } else {
-      y = to_f32(src[i]);
-    }
-    out[(size_t)t * out_stride + (size_t)h * out_head + out_off + i] = from_f32<T>(y);
+    out[(size_t)t * out_stride + (size_t)h * out_head + out_off + i] =
+        from_f32<T>(rotated(src, i, rot_dims, interleaved, p, inv_freq));
   }
 }
 
 PHOTON_API int photon_latent_q_rope(const void* q, long q_stride, int dtype, int heads, int dim, int rot, int rot_dims,
-                                    const int* positions, const float* inv_freq, void* out, long out_stride,
+                                    int interleaved, const int* positions, const float* inv_freq, void* out, long out_stride,
                                     int out_head, int out_off, int T_, cudaStream_t stream) {
   if (T_ <= 0 || rot <= 0) return 0;
   if (rot_dims < 0 || rot_dims > rot || (rot_dims & 1)) return PHOTON_ERR_ARGUMENT;
   if (dtype == PHOTON_BF16)
-    latent_q_rope_kernel<bf16><<<T_, 128, 0, stream>>>((const bf16*)q, q_stride, heads, dim, rot, rot_dims, positions,
+    latent_q_rope_kernel<bf16><<<T_, 128, 0, stream>>>((const bf16*)q, q_stride, heads, dim, rot, rot_dims, interleaved, positions,
                                                       inv_freq, (bf16*)out, out_stride, out_head, out_off);
   else
-    latent_q_rope_kernel<float><<<T_, 128, 0, stream>>>((const float*)q, q_stride, heads, dim, rot, rot_dims, positions,
+    latent_q_rope_kernel<float><<<T_, 128, 0, stream>>>((const float*)q, q_stride, heads, dim, rot, rot_dims, interleaved, positions,
                                                        inv_freq, (float*)out, out_stride, out_head, out_off);
   return launch_status();
 }
@@ -143,7 +134,7 @@ PHOTON_API int photon_latent_q_rope(const void* q, long q_stride, int dtype, int
 template <typename T>
 __global__ void __launch_bounds__(256)
 head_linear_kernel(const T* __restrict__ x, long x_row, long x_head, const T* __restrict__ W, T* __restrict__ out,
-                   long o_row, long o_head, int M, int N, int K) {
+                   long o_row, long o_head, int M, int N, int K, const T* __restrict__ gate, long gate_row) {
   __shared__ float As[HL_BK][HL_BM + 4];
   __shared__ float Ws[HL_BK][HL_BN + 4];
   const int h = blockIdx.z;
@@ -187,7 +178,10 @@ head_linear_kernel(const T* __restrict__ x, long x_row, long x_head, const T* __
 #pragma unroll
     for (int j = 0; j < 4; ++j) {
       const int gn = n0 + tx * 4 + j;
-      if (gn < N) out[(size_t)gm * o_row + (size_t)h * o_head + gn] = from_f32<T>(acc[i][j]);
+      if (gn < N) {
+        const float g = gate ? 1.0f + expf(-to_f32(gate[(size_t)gm * gate_row + (size_t)h * N + gn])) : 1.0f;
+        out[(size_t)gm * o_row + (size_t)h * o_head + gn] = from_f32<T>(gate ? acc[i][j] / g : acc[i][j]);
+      }
     }
   }
 }
@@ -197,7 +191,8 @@ head_linear_kernel(const T* __restrict__ x, long x_row, long x_head, const T* __
 #define HLS_ROWS 8
 __global__ void __launch_bounds__(256)
 head_linear_skinny_kernel(const bf16* __restrict__ x, long x_row, long x_head, const bf16* __restrict__ W,
-                          bf16* __restrict__ out, long o_row, long o_head, int M, int N, int K) {
+                          bf16* __restrict__ out, long o_row, long o_head, int M, int N, int K,
+                          const bf16* __restrict__ gate, long gate_row) {
   extern __shared__ __align__(16) bf16 xs[];                 // M x K
   const int h = blockIdx.y, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   for (int i = threadIdx.x * 8; i < M * K; i += blockDim.x * 8) {
@@ -236,77 +231,89 @@ head_linear_skinny_kernel(const bf16* __restrict__ x, long x_row, long x_head, c
 #pragma unroll
     for (int m = 0; m < HLS_ROWS; ++m) {
       if (m < M) {
-        const float v = warp_sum(acc[m]);
+        float v = warp_sum(acc[m]);
+        if (gate) v /= 1.0f + expf(-__bfloat162float(gate[(size_t)m * gate_row + (size_t)h * N + n]));
         if (lane == 0) out[(size_t)m * o_row + (size_t)h * o_head + n] = __float2bfloat16_rn(v);
       }
     }
   }
 }
 
-// x [M][heads][K] and out [M][heads][N] with row and head strides in elements; W [heads][N][K] contiguous.
+// x [M][heads][K] and out [M][heads][N] with row and head strides in elements; W [heads][N][K] contiguous.  gate (may be
+// null; the type of x, [M][heads * N] with row stride gate_row): every output is multiplied by sigmoid(gate) before it
+// is rounded.
 PHOTON_API int photon_head_linear(const void* x, long x_row, long x_head, const void* W, void* out, long o_row,
-                                  long o_head, int dtype, int M, int heads, int N, int K, cudaStream_t stream) {
+                                  long o_head, int dtype, int M, int heads, int N, int K, const void* gate, long gate_row,
+                                  cudaStream_t stream) {
   if (M <= 0 || heads <= 0 || N <= 0) return 0;
   if (K <= 0) return PHOTON_ERR_ARGUMENT;
   if (dtype == PHOTON_BF16 && M <= HLS_ROWS && K % 8 == 0 && x_row % 8 == 0 && x_head % 8 == 0 && (uintptr_t)x % 16 == 0 &&
       (uintptr_t)W % 16 == 0 && heads <= 65535 && (size_t)M * K * 2 <= 48 * 1024) {
     head_linear_skinny_kernel<<<dim3((N + 31) / 32, heads), 256, (size_t)M * K * 2, stream>>>(
-        (const bf16*)x, x_row, x_head, (const bf16*)W, (bf16*)out, o_row, o_head, M, N, K);
+        (const bf16*)x, x_row, x_head, (const bf16*)W, (bf16*)out, o_row, o_head, M, N, K, (const bf16*)gate, gate_row);
     return launch_status();
   }
   dim3 grid((N + HL_BN - 1) / HL_BN, (M + HL_BM - 1) / HL_BM, heads);
   if (grid.y > 65535 || grid.z > 65535) return PHOTON_ERR_UNSUPPORTED;
   if (dtype == PHOTON_BF16)
     head_linear_kernel<bf16><<<grid, 256, 0, stream>>>((const bf16*)x, x_row, x_head, (const bf16*)W, (bf16*)out, o_row,
-                                                      o_head, M, N, K);
+                                                      o_head, M, N, K, (const bf16*)gate, gate_row);
   else
     head_linear_kernel<float><<<grid, 256, 0, stream>>>((const float*)x, x_row, x_head, (const float*)W, (float*)out,
-                                                       o_row, o_head, M, N, K);
+                                                       o_row, o_head, M, N, K, (const float*)gate, gate_row);
   return launch_status();
 }
 
 // ---------------------------------------------------------------- a request's cached rows, in order
-// out[p, :] = cache[table[p / page_size] * page_size + p % page_size, :] for p < count: the latent rows of one
-// request as one dense matrix, the operand of the products that attention over a long prompt portion is made of.
+// out[i, :] = the cached row of position first + i of the request whose pages are `table`, for i < count: its latent
+// rows as one dense matrix, the operand of the products that attention over a long prompt portion is made of.
+// Positions outside [valid_lo, valid_hi) give zero rows (columns of the products that nothing sees).
 template <typename T>
 __global__ void gather_rows_kernel(const T* __restrict__ cache, const int* __restrict__ table, int page_size,
-                                   int num_pages, int width, int count, T* __restrict__ out, int* err) {
-  const int p = blockIdx.x;
-  const int page = table[p / page_size];
+                                   int num_pages, int width, int first, int valid_lo, int valid_hi, T* __restrict__ out,
+                                   int* err) {
+  const int p = first + blockIdx.x;
+  T* dst = out + (size_t)blockIdx.x * width;
+  const bool valid = p >= valid_lo && p < valid_hi;
+  const int page = valid ? table[p / page_size] : -1;
   if (page < 0 || page >= num_pages) {
-    if (threadIdx.x == 0) report_error(err, PHOTON_DEV_BAD_PAGE, 0, p, page);
-    for (int i = threadIdx.x; i < width; i += blockDim.x) out[(size_t)p * width + i] = from_f32<T>(0.f);
+    if (valid && threadIdx.x == 0) report_error(err, PHOTON_DEV_BAD_PAGE, 0, p, page);
+    for (int i = threadIdx.x; i < width; i += blockDim.x) dst[i] = from_f32<T>(0.f);
     return;
   }
   const T* src = cache + ((size_t)page * page_size + p % page_size) * width;
-  for (int i = threadIdx.x; i < width; i += blockDim.x) out[(size_t)p * width + i] = src[i];
+  for (int i = threadIdx.x; i < width; i += blockDim.x) dst[i] = src[i];
 }
 
 PHOTON_API int photon_gather_rows(const void* cache, int dtype, const int* table, int page_size, int num_pages,
-                                  int width, int count, void* out, int* err, cudaStream_t stream) {
+                                  int width, int first, int count, int valid_lo, int valid_hi, void* out, int* err,
+                                  cudaStream_t stream) {
   if (count <= 0) return 0;
-  if (page_size <= 0 || width <= 0) return PHOTON_ERR_ARGUMENT;
+  if (page_size <= 0 || width <= 0 || first < 0 || valid_lo < 0) return PHOTON_ERR_ARGUMENT;
   if (dtype == PHOTON_BF16)
-    gather_rows_kernel<bf16><<<count, 128, 0, stream>>>((const bf16*)cache, table, page_size, num_pages, width, count, (bf16*)out, err);
+    gather_rows_kernel<bf16><<<count, 128, 0, stream>>>((const bf16*)cache, table, page_size, num_pages, width, first, valid_lo, valid_hi, (bf16*)out, err);
   else
-    gather_rows_kernel<float><<<count, 128, 0, stream>>>((const float*)cache, table, page_size, num_pages, width, count, (float*)out, err);
+    gather_rows_kernel<float><<<count, 128, 0, stream>>>((const float*)cache, table, page_size, num_pages, width, first, valid_lo, valid_hi, (float*)out, err);
   return launch_status();
 }
 
 // ---------------------------------------------------------------- causal softmax over rows of scores
-// scores [rows][ld] float: row r belongs to the token at position first_pos + r / heads, which sees the keys
-// 0 .. its own position.  probs [rows][ldp] = softmax(scale * scores) over the visible keys, zero beyond them, up to
-// column `cols`.  One block per row, 32-bit throughout, rounded once on the way out.
+// scores [rows][ld] float: column c is the key at position first_key + c; row r belongs to the token at position
+// first_pos + r / heads, which sees the keys up to its own position and, with window > 0, the last `window` of them.
+// probs [rows][ldp] = softmax(scale * scores) over the visible keys, zero elsewhere, up to column `cols`.  One block per
+// row, 32-bit throughout, rounded once on the way out.
 template <typename T>
 __global__ void causal_softmax_kernel(const float* __restrict__ scores, long ld, T* __restrict__ probs, long ldp,
-                                      int heads, int first_pos, int cols, float scale) {
+                                      int heads, int first_pos, int first_key, int window, int cols, float scale) {
   __shared__ float red[32];
   const int r = blockIdx.x;
-  const int visible = min(cols, first_pos + r / heads + 1);
+  const int pos = first_pos + r / heads;
+  const int hi = min(cols, pos + 1 - first_key);
+  const int lo = window > 0 ? max(0, pos + 1 - window - first_key) : 0;
   const float* s = scores + (size_t)r * ld;
   T* p = probs + (size_t)r * ldp;
   float m = -INFINITY;
-  for (int i = threadIdx.x; i < visible; i += blockDim.x) m = fmaxf(m, s[i] * scale);
+  for (int i = lo + threadIdx.x; i < hi; i += blockDim.x) m = fmaxf(m, s[i] * scale);
   m = warp_max(m);
   __syncthreads();
   if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = m;
@@ -314,28 +321,29 @@ __global__ void causal_softmax_kernel(const float* __restrict__ scores, long ld,
   m = (threadIdx.x & 31) < (blockDim.x >> 5) ? red[threadIdx.x & 31] : -INFINITY;
   m = warp_max(m);
   float sum = 0.f;
-  for (int i = threadIdx.x; i < visible; i += blockDim.x) sum += expf(s[i] * scale - m);
+  for (int i = lo + threadIdx.x; i < hi; i += blockDim.x) sum += expf(s[i] * scale - m);
   sum = block_sum(sum, red);
   const float inv = 1.0f / sum;
   for (int i = threadIdx.x; i < cols; i += blockDim.x)
-    p[i] = from_f32<T>(i < visible ? expf(s[i] * scale - m) * inv : 0.f);
+    p[i] = from_f32<T>(i >= lo && i < hi ? expf(s[i] * scale - m) * inv : 0.f);
 }
 
 PHOTON_API int photon_causal_softmax_rows(const float* scores, long ld, void* probs, long ldp, int dtype, int rows,
-                                          int heads, int first_pos, int cols, float scale, cudaStream_t stream) {
+                                          int heads, int first_pos, int first_key, int window, int cols, float scale,
+                                          cudaStream_t stream) {
   if (rows <= 0 || cols <= 0) return 0;
-  if (heads <= 0 || first_pos < 0) return PHOTON_ERR_ARGUMENT;
+  if (heads <= 0 || first_pos < 0 || first_key < 0 || first_key > first_pos) return PHOTON_ERR_ARGUMENT;
   if (dtype == PHOTON_BF16)
-    causal_softmax_kernel<bf16><<<rows, 256, 0, stream>>>(scores, ld, (bf16*)probs, ldp, heads, first_pos, cols, scale);
+    causal_softmax_kernel<bf16><<<rows, 256, 0, stream>>>(scores, ld, (bf16*)probs, ldp, heads, first_pos, first_key, window, cols, scale);
   else
-    causal_softmax_kernel<float><<<rows, 256, 0, stream>>>(scores, ld, (float*)probs, ldp, heads, first_pos, cols, scale);
+    causal_softmax_kernel<float><<<rows, 256, 0, stream>>>(scores, ld, (float*)probs, ldp, heads, first_pos, first_key, window, cols, scale);
   return launch_status();
 }
 
 // ---------------------------------------------------------------- decoded tokens on the tensor cores
 // All heads of a token attend to the same cached rows, so a decoded token is a (heads x width) by (width x keys)
-// product followed by a (heads x keys) by (keys x kv_rank) one.  Block (t, s) takes token t and the 64 keys
-// s * 64 .. of its request: the rows come into shared memory once (16-byte loads through the block table) and
+// product followed by a (heads x keys) by (keys x kv_rank) one.  Block (t, s) takes token t and the s-th 64 keys of
+// its request, counted from the block of 64 that holds the first key the token sees (key 0 without a window): the rows come into shared memory once (16-byte loads through the block table) and
 // serve every tile of 16 heads; scores = Q C^T with wmma (bfloat16 in, 32-bit accumulate), a softmax over the
 // block's keys in 32-bit, P (rounded to bfloat16) times the first kv_rank columns of the same rows.  Every block
 // leaves its unnormalised sums with the rows' maximum and denominator, in the layout of the general kernel's
@@ -349,7 +357,7 @@ __global__ void __launch_bounds__(128)
 latent_decode_kernel(const bf16* __restrict__ q, long q_stride, const bf16* __restrict__ cache,
                      const int* __restrict__ block_table, int max_pages, const int* __restrict__ token_seq,
                      const int* __restrict__ positions, int heads, int width, int dv, int page_size, int num_pages,
-                     float scale, int splits, float* __restrict__ part, int* err) {
+                     float scale, int window, int splits, float* __restrict__ part, int* err) {
   extern __shared__ __align__(128) unsigned char smem_raw[];
   const int t = blockIdx.x, s = blockIdx.y, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int ldk = width + 8;                                   // bfloat16 elements; rows of 16 keys stay 32-byte aligned
@@ -361,7 +369,9 @@ latent_decode_kernel(const bf16* __restrict__ q, long q_stride, const bf16* __re
   float* rowm = Ot + 4 * 16 * 20;                              // 16
   float* rowl = rowm + 16;                                     // 16
   const int p = positions[t];
-  const int k0 = s * LD_KEYS;
+  const int first = window > 0 ? max(0, p + 1 - window) : 0;   // the first key the token sees
+  const int k0 = (first / LD_KEYS + s) * LD_KEYS;
+  const int nlow = max(0, first - k0);                         // keys of this block that lie before it
   const int nkeys = min(LD_KEYS, p + 1 - k0);                  // keys of this block that the token sees
   if (nkeys <= 0) {                                            // an empty share: the merge skips it
     for (int h = tid; h < heads; h += 128) {
@@ -376,7 +386,7 @@ latent_decode_kernel(const bf16* __restrict__ q, long q_stride, const bf16* __re
   long long* rowbase = reinterpret_cast<long long*>(rowl + 16);
   if (tid < LD_KEYS) {
     long long base = -1;
-    if (tid < nkeys) {
+    if (tid >= nlow && tid < nkeys) {
       const int kk = k0 + tid;
       const int page = table[kk / page_size];
       if (page < 0 || page >= num_pages) report_error(err, PHOTON_DEV_BAD_PAGE, t, kk, page);
@@ -420,7 +430,7 @@ latent_decode_kernel(const bf16* __restrict__ q, long q_stride, const bf16* __re
       float v[8], m = -INFINITY;
 #pragma unroll
       for (int u = 0; u < 8; ++u) {
-        v[u] = c0 + u < nkeys ? Sf[row * 68 + c0 + u] * scale : -INFINITY;
+        v[u] = c0 + u >= nlow && c0 + u < nkeys ? Sf[row * 68 + c0 + u] * scale : -INFINITY;
         m = fmaxf(m, v[u]);
       }
       for (int d = 1; d < 8; d <<= 1) m = fmaxf(m, __shfl_xor_sync(0xffffffffu, m, d));
@@ -485,13 +495,14 @@ __global__ void latent_merge_kernel(const float* __restrict__ part, int splits, 
 }
 
 // q [T][heads * width] bfloat16 (row stride in elements), cache [num_pages * page_size][width] bfloat16, out
-// [T][heads * dv]: token t at position positions[t] of request token_seq[t] sees the rows 0 .. positions[t]; a row's
-// value is its first dv numbers.  width and dv multiples of 16.  splits >= ceil((largest position + 1) / 64);
+// [T][heads * dv]: token t at position positions[t] of request token_seq[t] sees the rows 0 .. positions[t], with
+// window > 0 the last `window` of them; a row's value is its first dv numbers.  width and dv multiples of 16.  splits >=
+// ceil((largest position + 1) / 64), with a window no more than ceil((window - 1) / 64) + 1 are needed;
 // part: float [T * heads * splits * (dv + 2)].
 PHOTON_API int photon_latent_decode_attention(const void* q, long q_stride, const void* cache, const int* block_table,
                                               int max_pages, const int* token_seq, const int* positions, int T_,
                                               int heads, int width, int dv, int page_size, int num_pages, float scale,
-                                              int splits, float* part, void* out, long out_stride, int* err,
+                                              int window, int splits, float* part, void* out, long out_stride, int* err,
                                               cudaStream_t stream) {
   if (T_ <= 0) return 0;
   if (heads <= 0 || splits <= 0 || part == nullptr || dv > width) return PHOTON_ERR_ARGUMENT;
@@ -504,7 +515,7 @@ PHOTON_API int photon_latent_decode_attention(const void* q, long q_stride, cons
     if (e != cudaSuccess) return (int)e;
   }
   latent_decode_kernel<<<dim3(T_, splits), 128, smem, stream>>>((const bf16*)q, q_stride, (const bf16*)cache, block_table,
-      max_pages, token_seq, positions, heads, width, dv, page_size, num_pages, scale, splits, part, err);
+      max_pages, token_seq, positions, heads, width, dv, page_size, num_pages, scale, window, splits, part, err);
   int st = launch_status();
   if (st != 0) return st;
   latent_merge_kernel<<<dim3(T_, heads), 128, 0, stream>>>(part, splits, dv, (bf16*)out, out_stride, heads);

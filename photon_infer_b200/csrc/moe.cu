@@ -81,15 +81,20 @@ __global__ void moe_route_kernel(const T* __restrict__ h, long h_stride, const T
   float* lg = logits + warp * LS;
   const bool first = lane == 0;
   if (first && Wsg) shared_gate[t] = 1.0f / (1.0f + expf(-lg[E]));
-  if (mode == 1 && E <= 32) {
-    // The same rules as the serial form below with one lane per expert: maxima and sums by shuffles, a choice is the
+  if (E <= 32 && (mode == 1 || (mode == 2 && !(n_groups > 1 && keep_groups < n_groups)))) {
+    // The same rules as the serial forms below with one lane per expert: maxima and sums by shuffles, a choice is the
     // lowest lane that holds the maximum (so ties go to the lower index).  top <= E <= 32.
     const unsigned full = 0xffffffffu;
     const bool live = lane < E;
     const float z = live ? lg[lane] : -INFINITY;
-    const float mx = warp_max(z);
-    const float p = live ? expf(z - mx) : 0.f;
-    const float score = p / warp_sum(p);
+    float score;
+    if (mode == 1) {
+      const float mx = warp_max(z);
+      const float p = live ? expf(z - mx) : 0.f;
+      score = p / warp_sum(p);
+    } else {
+      score = 1.0f / (1.0f + expf(-z));                  // every expert by itself
+    }
     float cand = live ? score : -1.f;
     if (n_groups > 1 && keep_groups < n_groups) {
       const int per = E / n_groups;
@@ -116,7 +121,7 @@ __global__ void moe_route_kernel(const T* __restrict__ h, long h_stride, const T
       sum += m;
       if (lane == 0) { ids[(size_t)t * top + j] = best; atomicAdd(&counts[best], 1); }
     }
-    if (lane < top) weights[(size_t)t * top + lane] = mine / (sum + 1e-20f) * route_scale;
+    if (lane < top) weights[(size_t)t * top + lane] = mode == 1 ? mine / (sum + 1e-20f) * route_scale : mine * route_scale;
   } else if (first && (mode == 1 || mode == 2)) {
     // mode 1: scores are the softmax over ALL experts; a group's score is its largest score; the weights are the chosen
     // scores over their sum, times route_scale.  mode 2: scores are sigmoid(logit), each expert by itself; a group's
@@ -307,13 +312,24 @@ __device__ __forceinline__ float moe_act(float g, int act) {
   return g / (1.0f + expf(-g));
 }
 
+// A gated unit of the gate's sum g and the up sum u.  CLAMPED_SWISH bounds both: g from above, u from both sides.
+__device__ __forceinline__ float moe_glu_pair(float g, float u, int act, float limit, float slope) {
+  if (act == PHOTON_ACT_CLAMPED_SWISH) {
+    g = fminf(g, limit);
+    u = fminf(fmaxf(u, -limit), limit);
+    return g / (1.0f + expf(-slope * g)) * (u + 1.0f);
+  }
+  return moe_act(g, act) * u;
+}
+
 // GLU: W holds [gate rows; up rows] per expert (N = 2 * cols); the block computes the gate and the up column of
 // each of its output columns and stores act(gate) * up.
 template <typename T, typename TO, bool GLU>
 __global__ void __launch_bounds__(256)
 moe_gemm_kernel(const T* __restrict__ A, long lda, const int* __restrict__ gather, int gather_div,
                 const T* __restrict__ W, TO* __restrict__ out, long ldo, int N, int K,
-                const int* __restrict__ tiles, const int* __restrict__ num_tiles, int act) {
+                const int* __restrict__ tiles, const int* __restrict__ num_tiles, int act,
+                const float* __restrict__ weights, float limit, float slope) {
   __shared__ float As[MOE_BK][MOE_BM + 4];
   __shared__ float Ws[GLU ? 2 : 1][MOE_BK][MOE_BN + 4];
   __shared__ int arow[MOE_BM];
@@ -372,12 +388,13 @@ moe_gemm_kernel(const T* __restrict__ A, long lda, const int* __restrict__ gathe
   for (int i = 0; i < 2; ++i) {
     const int row = ty * 2 + i;
     if (row >= rows) continue;
+    const float f = weights ? weights[gather[r0 + row]] : 1.0f;      // the row's input factor: products are linear in it
 #pragma unroll
     for (int j = 0; j < 4; ++j) {
       const int gn = n0 + tx * 4 + j;
       if (gn >= cols) continue;
-      float v = acc[0][i][j];
-      v = GLU ? moe_act(v, act) * acc[GLU ? 1 : 0][i][j] : moe_act(v, act);
+      float v = f * acc[0][i][j];
+      v = GLU ? moe_glu_pair(v, f * acc[GLU ? 1 : 0][i][j], act, limit, slope) : moe_act(v, act);
       out[(size_t)(r0 + row) * ldo + gn] = from_f32<TO>(v);
     }
   }
@@ -386,17 +403,20 @@ moe_gemm_kernel(const T* __restrict__ A, long lda, const int* __restrict__ gathe
 // A [*][K] (row stride lda).  gather (may be null): row r of the sorted order reads A row gather[r] / gather_div;
 // null: row r itself.  W [E][N][K] contiguous.  out [n][N] (or [n][N / 2] with glu != 0), rows in sorted order.
 // act: PHOTON_ACT_*; with glu != 0 it is applied to the gate, otherwise to every output (PHOTON_ACT_NONE: plain product).
-// out_dtype: PHOTON_F32 or the input type.  max_tiles: bound of the tile list (the grid's height).
+// out_dtype: PHOTON_F32 or the input type.  max_tiles: bound of the tile list (the grid's height).  weights (may be null;
+// needs gather): row r's sums are multiplied by weights[gather[r]] before the activation, which is the product of the
+// scaled input row.
 PHOTON_API int photon_moe_gemm(const void* A, long lda, int dtype, const int* gather, int gather_div, const void* W,
                                void* out, long ldo, int out_dtype, int N, int K, const int* tiles, const int* num_tiles,
-                               int max_tiles, int glu, int act, cudaStream_t stream) {
+                               int max_tiles, int glu, int act, const float* weights, float limit, float slope,
+                               cudaStream_t stream) {
   if (max_tiles <= 0 || N <= 0) return 0;
-  if (K <= 0 || gather_div <= 0 || (glu && (N & 1))) return PHOTON_ERR_ARGUMENT;
+  if (K <= 0 || gather_div <= 0 || (glu && (N & 1)) || (weights && !gather) || (act == PHOTON_ACT_CLAMPED_SWISH && !glu)) return PHOTON_ERR_ARGUMENT;
   if (max_tiles > 65535) return PHOTON_ERR_UNSUPPORTED;
   const int cols = glu ? N / 2 : N;
   dim3 grid((cols + MOE_BN - 1) / MOE_BN, max_tiles);
 #define MOE_GEMM(T, TO, GLU) moe_gemm_kernel<T, TO, GLU><<<grid, 256, 0, stream>>>((const T*)A, lda, gather, gather_div, \
-      (const T*)W, (TO*)out, ldo, N, K, tiles, num_tiles, act)
+      (const T*)W, (TO*)out, ldo, N, K, tiles, num_tiles, act, weights, limit, slope)
   if (dtype == PHOTON_BF16 && out_dtype == PHOTON_BF16) { if (glu) MOE_GEMM(bf16, bf16, true); else MOE_GEMM(bf16, bf16, false); }
   else if (dtype == PHOTON_BF16 && out_dtype == PHOTON_F32) { if (glu) MOE_GEMM(bf16, float, true); else MOE_GEMM(bf16, float, false); }
   else if (dtype == PHOTON_F32 && out_dtype == PHOTON_F32) { if (glu) MOE_GEMM(float, float, true); else MOE_GEMM(float, float, false); }
@@ -413,7 +433,7 @@ __global__ void moe_combine_kernel(const TY* __restrict__ y, long ldy, const int
   for (int i = threadIdx.x; i < H; i += blockDim.x) {
     float acc = 0.f;
     for (int j = 0; j < top; ++j)
-      acc = fmaf(weights[(size_t)t * top + j],
+      acc = fmaf(weights ? weights[(size_t)t * top + j] : 1.0f,
                  to_f32(y[(size_t)(place ? place[(size_t)t * top + j] : t * top + j) * ldy + i]), acc);
     if (shared_out) acc += shared_gate ? shared_gate[t] * to_f32(shared_out[(size_t)t * H + i]) : to_f32(shared_out[(size_t)t * H + i]);
     out[(size_t)t * H + i] = from_f32<TO>(acc);
@@ -421,7 +441,7 @@ __global__ void moe_combine_kernel(const TY* __restrict__ y, long ldy, const int
 }
 
 // y [n][H] (float or bfloat16): row place[t, j] is the output of token t's j-th expert (place null: row t * top + j);
-// weights [T][top]; shared_out [T][H] (may be null) and out [T][H] of out_dtype.
+// weights [T][top] (null: all 1, experts whose inputs were weighted); shared_out [T][H] (may be null) and out [T][H] of out_dtype.
 PHOTON_API int photon_moe_combine(const void* y, long ldy, int y_dtype, const int* place, const float* weights, int top,
                                   const void* shared_out, void* out, int out_dtype, int T_, int H, cudaStream_t stream) {
   return photon_moe_combine_ex(y, ldy, y_dtype, place, weights, top, shared_out, nullptr, out, out_dtype, T_, H, stream);
@@ -470,6 +490,51 @@ PHOTON_API int photon_moe_gather(const void* x, long ldx, int dtype, const int* 
   return launch_status();
 }
 
+// ---------------------------------------------------------------- gated unit between the library's grouped products
+// gate_up [n][2 I], rows in sorted order -> out [n][I] = act(f gate) * (f up), f the input factor of row r's pair.
+template <typename T>
+__global__ void moe_glu_kernel(const T* __restrict__ gate_up, T* __restrict__ out, int I, int act,
+                               const int* __restrict__ sorted, const float* __restrict__ weights, float limit, float slope,
+                               int vec) {
+  const size_t r = blockIdx.x;
+  const float f = weights ? weights[sorted[r]] : 1.0f;
+  const T* g = gate_up + r * 2 * I;
+  const T* u = g + I;
+  T* o = out + r * I;
+  constexpr int N = 16 / sizeof(T);
+  if (vec) {
+    for (int i = (blockIdx.y * blockDim.x + threadIdx.x) * N; i < I; i += gridDim.y * blockDim.x * N) {
+      const uint4 gv = *reinterpret_cast<const uint4*>(g + i), uv = *reinterpret_cast<const uint4*>(u + i);
+      const T* gp = reinterpret_cast<const T*>(&gv);
+      const T* up = reinterpret_cast<const T*>(&uv);
+      uint4 ov;
+      T* op = reinterpret_cast<T*>(&ov);
+#pragma unroll
+      for (int e = 0; e < N; ++e) op[e] = from_f32<T>(moe_glu_pair(f * to_f32(gp[e]), f * to_f32(up[e]), act, limit, slope));
+      *reinterpret_cast<uint4*>(o + i) = ov;
+    }
+  } else {
+    for (int i = blockIdx.y * blockDim.x + threadIdx.x; i < I; i += gridDim.y * blockDim.x)
+      o[i] = from_f32<T>(moe_glu_pair(f * to_f32(g[i]), f * to_f32(u[i]), act, limit, slope));
+  }
+}
+
+// sorted [n] (pair index of each row) goes with weights [pairs]; weights null: no factors.  act: PHOTON_ACT_*.
+PHOTON_API int photon_moe_glu(const void* gate_up, void* out, int dtype, int n, int I, int act, const int* sorted,
+                              const float* weights, float limit, float slope, cudaStream_t stream) {
+  if (n <= 0 || I <= 0) return 0;
+  if (weights && !sorted) return PHOTON_ERR_ARGUMENT;
+  const int N = dtype == PHOTON_BF16 ? 8 : 4;
+  const int vec = I % N == 0 && (uintptr_t)gate_up % 16 == 0 && (uintptr_t)out % 16 == 0;
+  const int threads = 128, per = threads * (vec ? N : 1);
+  const dim3 grid(n, (I + per - 1) / per < 8 ? (I + per - 1) / per : 8);
+  if (dtype == PHOTON_BF16)
+    moe_glu_kernel<bf16><<<grid, threads, 0, stream>>>((const bf16*)gate_up, (bf16*)out, I, act, sorted, weights, limit, slope, vec);
+  else
+    moe_glu_kernel<float><<<grid, threads, 0, stream>>>((const float*)gate_up, (float*)out, I, act, sorted, weights, limit, slope, vec);
+  return launch_status();
+}
+
 // ---------------------------------------------------------------- few rows: one matrix-vector product per pair
 // A decode step brings a handful of (token, choice) pairs, each to another expert as a rule: nothing is sorted,
 // block (c, p) streams the rows c * 32 .. of pair p's expert matrix once, 16 bytes per lane and load, against the
@@ -479,7 +544,8 @@ PHOTON_API int photon_moe_gather(const void* x, long ldx, int dtype, const int* 
 template <typename TO, bool GLU>
 __global__ void __launch_bounds__(256)
 moe_gemv_kernel(const bf16* __restrict__ x, long ldx, int x_div, const int* __restrict__ ids, const bf16* __restrict__ W,
-                TO* __restrict__ out, long ldo, int N, int K, int act) {
+                TO* __restrict__ out, long ldo, int N, int K, int act, const float* __restrict__ weights, float limit,
+                float slope) {
   extern __shared__ __align__(16) bf16 xs[];
   const int p = blockIdx.y;
   const int e = ids[p];
@@ -519,16 +585,19 @@ moe_gemv_kernel(const bf16* __restrict__ x, long ldx, int x_div, const int* __re
     }
     a0 = warp_sum(a0);
     if (GLU) a1 = warp_sum(a1);
-    if (lane == 0) out[(size_t)p * ldo + col] = from_f32<TO>(GLU ? moe_act(a0, act) * a1 : moe_act(a0, act));
+    if (weights) { const float f = weights[p]; a0 *= f; a1 *= f; }   // the pair's input factor
+    if (lane == 0) out[(size_t)p * ldo + col] = from_f32<TO>(GLU ? moe_glu_pair(a0, a1, act, limit, slope) : moe_act(a0, act));
   }
 }
 
 // x [*][K] bfloat16: pair p reads row p / x_div.  ids [n]: the expert of every pair.  W [E][N][K] bfloat16.
-// out [n][N] float or bfloat16 (glu: [n][N / 2]), rows in the order of the pairs.  K % 8 == 0, 16-byte aligned rows.
+// out [n][N] float or bfloat16 (glu: [n][N / 2]), rows in the order of the pairs.  weights [n] (may be null): pair p's
+// sums are multiplied by weights[p] before the activation.  K % 8 == 0, 16-byte aligned rows.
 PHOTON_API int photon_moe_gemv(const void* x, long ldx, int x_div, const int* ids, int n, const void* W, void* out, long ldo,
-                               int out_dtype, int N, int K, int glu, int act, cudaStream_t stream) {
+                               int out_dtype, int N, int K, int glu, int act, const float* weights, float limit,
+                               float slope, cudaStream_t stream) {
   if (n <= 0 || N <= 0) return 0;
-  if (K <= 0 || x_div <= 0 || (glu && (N & 1))) return PHOTON_ERR_ARGUMENT;
+  if (K <= 0 || x_div <= 0 || (glu && (N & 1)) || (act == PHOTON_ACT_CLAMPED_SWISH && !glu)) return PHOTON_ERR_ARGUMENT;
   if (K % 8 || ldx % 8 || (uintptr_t)x % 16 || (uintptr_t)W % 16 || n > 65535 || (size_t)K * 2 > 96 * 1024) return PHOTON_ERR_UNSUPPORTED;
   const int cols = glu ? N / 2 : N;
   dim3 grid((cols + GEMV_COLS - 1) / GEMV_COLS, n);
@@ -536,7 +605,7 @@ PHOTON_API int photon_moe_gemv(const void* x, long ldx, int x_div, const int* id
 #define MOE_GEMV(TO, GLU) do { \
     if (smem > 48 * 1024) { cudaError_t e_ = cudaFuncSetAttribute(moe_gemv_kernel<TO, GLU>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
                             if (e_ != cudaSuccess) return (int)e_; } \
-    moe_gemv_kernel<TO, GLU><<<grid, 256, smem, stream>>>((const bf16*)x, ldx, x_div, ids, (const bf16*)W, (TO*)out, ldo, N, K, act); } while (0)
+    moe_gemv_kernel<TO, GLU><<<grid, 256, smem, stream>>>((const bf16*)x, ldx, x_div, ids, (const bf16*)W, (TO*)out, ldo, N, K, act, weights, limit, slope); } while (0)
   if (out_dtype == PHOTON_BF16) { if (glu) MOE_GEMV(bf16, true); else MOE_GEMV(bf16, false); }
   else if (out_dtype == PHOTON_F32) { if (glu) MOE_GEMV(float, true); else MOE_GEMV(float, false); }
   else return PHOTON_ERR_ARGUMENT;

@@ -54,6 +54,7 @@ extern "C" {
 #define PHOTON_ACT_GELU_TANH 1
 #define PHOTON_ACT_GELU 2            /* the exact form, 0.5 z (1 + erf(z / sqrt 2)) */
 #define PHOTON_ACT_RELU 3
+#define PHOTON_ACT_CLAMPED_SWISH 4   /* gated only: with g = min(gate, limit), u = clamp(up, -limit, limit): g sigmoid(slope g) (u + 1) */
 #define PHOTON_ACT_NONE (-1)
 
 /* ------------------------------------------------------------------ elementwise.cu */
@@ -138,35 +139,49 @@ PHOTON_EXPORT int photon_paged_attention_ex(const void* q, long q_stride, void* 
 /* One pass over a token's fused down-projection row down[t] = [query latent (q_rank) | key/value latent (kv_rank) |
  * shared key part (rot)]: cq[t] = rmsnorm(query latent) * q_norm_w; the cache row at slot_mapping[t] becomes
  * [rmsnorm(key/value latent) * kv_norm_w | key part with its first rot_dims numbers rotated (i paired with
- * i + rot_dims / 2, angle positions[t] * inv_freq[i])].  cache: [num_slots][kv_rank + rot]. */
+ * i + rot_dims / 2, with interleaved != 0 2i with 2i + 1; angle positions[t] * inv_freq[i])].  cache: [num_slots][kv_rank
+ * + rot]; null: only cq is formed. */
 PHOTON_EXPORT int photon_latent_prep(const void* down, long down_stride, int dtype, int q_rank, int kv_rank, int rot, int rot_dims,
-                       const void* q_norm_w, int q_norm_dtype, const void* kv_norm_w, int kv_norm_dtype, float eps,
+                       int interleaved, const void* q_norm_w, int q_norm_dtype, const void* kv_norm_w, int kv_norm_dtype, float eps,
                        const int* positions, const float* inv_freq, const int* slot_mapping, void* cq, long cq_stride,
                        void* cache, long num_slots, int T_, int* err, cudaStream_t stream);
 /* out[t, h, out_off .. out_off + rot) = the last rot numbers of head h of q [T][heads][dim + rot], rotated as above. */
 PHOTON_EXPORT int photon_latent_q_rope(const void* q, long q_stride, int dtype, int heads, int dim, int rot, int rot_dims,
-                         const int* positions, const float* inv_freq, void* out, long out_stride, int out_head,
+                         int interleaved, const int* positions, const float* inv_freq, void* out, long out_stride, int out_head,
                          int out_off, int T_, cudaStream_t stream);
 /* out[t, h, :] = W[h] x[t, h, :] for every head: x [M][heads][K], out [M][heads][N] (row and head strides in elements),
- * W [heads][N][K]. */
+ * W [heads][N][K]; gate [M][heads * N] (row stride gate_row, may be null): times sigmoid(gate). */
 PHOTON_EXPORT int photon_head_linear(const void* x, long x_row, long x_head, const void* W, void* out, long o_row, long o_head,
-                       int dtype, int M, int heads, int N, int K, cudaStream_t stream);
+                       int dtype, int M, int heads, int N, int K, const void* gate, long gate_row, cudaStream_t stream);
 
-/* out[p, :] = the cache row of position p < count of the request whose pages are table (cache [num_pages * page_size][width]). */
+/* out[i, :] = the cache row of position first + i (i < count) of the request whose pages are table (cache
+ * [num_pages * page_size][width]); zero rows for positions outside [valid_lo, valid_hi). */
 PHOTON_EXPORT int photon_gather_rows(const void* cache, int dtype, const int* table, int page_size, int num_pages, int width,
-                       int count, void* out, int* err, cudaStream_t stream);
-/* probs [rows][ldp] = softmax(scale * scores [rows][ld]) over the keys 0 .. first_pos + r / heads of row r, zero beyond,
- * up to column cols. */
+                       int first, int count, int valid_lo, int valid_hi, void* out, int* err, cudaStream_t stream);
+/* probs [rows][ldp] = softmax(scale * scores [rows][ld]) over the keys that row r sees, zero elsewhere, up to column cols:
+ * column c is the key at first_key + c, row r the token at first_pos + r / heads, which sees the keys up to its own
+ * position, with window > 0 the last window of them. */
 PHOTON_EXPORT int photon_causal_softmax_rows(const float* scores, long ld, void* probs, long ldp, int dtype, int rows, int heads,
-                               int first_pos, int cols, float scale, cudaStream_t stream);
+                               int first_pos, int first_key, int window, int cols, float scale, cudaStream_t stream);
 
 /* Decoded tokens on the tensor cores (bfloat16; width and dv multiples of 16): token t sees the rows 0 .. positions[t] of
- * request token_seq[t]; a row's value is its first dv numbers.  splits >= ceil((largest position + 1) / 64); part: float
+ * request token_seq[t], with window > 0 the last window of them; a row's value is its first dv numbers.  splits >=
+ * ceil((largest position + 1) / 64) (with a window ceil((window - 1) / 64) + 1 are always enough); part: float
  * [T * heads * splits * (dv + 2)]. */
 PHOTON_EXPORT int photon_latent_decode_attention(const void* q, long q_stride, const void* cache, const int* block_table,
                                    int max_pages, const int* token_seq, const int* positions, int T_, int heads, int width,
-                                   int dv, int page_size, int num_pages, float scale, int splits, float* part, void* out,
-                                   long out_stride, int* err, cudaStream_t stream);
+                                   int dv, int page_size, int num_pages, float scale, int window, int splits, float* part,
+                                   void* out, long out_stride, int* err, cudaStream_t stream);
+
+/* ------------------------------------------------------------------ hyper.cu: parallel residual streams */
+/* out [n][H] = norm(u) * w + bias, u = sum_s win[s] X_s (win null: the sum), after the pending write
+ * X_t <- sum_s mix[s][t] X_s + wout[t] y (y null: none) into dst [*][S][H] (may be src, may be null).  Streams of token t
+ * at src + t * src_token, src_stream apart (0: all equal).  center != 0: layer norm, else RMS norm; bias may be null.
+ * rows (may be null): these tokens only, nothing is written back. */
+PHOTON_EXPORT int photon_stream_norm(const float* src, long src_token, long src_stream, float* dst, const void* y, int y_dtype,
+                       const float* mix, const float* wout, const float* win, int S, int H, const void* w, int w_dtype,
+                       const void* bias, int bias_dtype, int center, float eps, void* out, int out_dtype, const int* rows,
+                       int n, cudaStream_t stream);
 
 /* ------------------------------------------------------------------ delta.cu: gated delta rule (recurrent state, short convolutions) */
 /* The state row of a request: S float [H][dim][vdim], then at conv_offset the last taps - 1 projected rows [taps - 1][C],
@@ -324,11 +339,16 @@ PHOTON_EXPORT int photon_moe_align(const int* ids, const int* counts, int n, int
                      int* tiles, int* num_tiles, cudaStream_t stream);
 PHOTON_EXPORT int photon_moe_tile_rows(void);
 /* Grouped product over the sorted rows with W [E][N][K]; gather (may be null): sorted row r reads A row
- * gather[r] / gather_div; glu != 0: W = [gate rows; up rows], out [n][N / 2] = act(gate) * up. */
+ * gather[r] / gather_div; glu != 0: W = [gate rows; up rows], out [n][N / 2] = act(gate) * up.  weights (may be null; needs
+ * gather): the sums of sorted row r are multiplied by weights[gather[r]] first (a factor on the row's input).  limit,
+ * slope: constants of PHOTON_ACT_CLAMPED_SWISH. */
 PHOTON_EXPORT int photon_moe_gemm(const void* A, long lda, int dtype, const int* gather, int gather_div, const void* W, void* out,
                     long ldo, int out_dtype, int N, int K, const int* tiles, const int* num_tiles, int max_tiles, int glu,
-                    int act, cudaStream_t stream);
-/* out[t] = sum_j weights[t, j] * y[place[t, j]] (+ shared_out[t]); y [n][H] float or bfloat16; place null: row t * top + j. */
+                    int act, const float* weights, float limit, float slope, cudaStream_t stream);
+/* out [n][I] = act(w gate) * (w up), gate_up [n][2 I] of one dtype; row r's factor w = weights[sorted[r]] (weights null: 1). */
+PHOTON_EXPORT int photon_moe_glu(const void* gate_up, void* out, int dtype, int n, int I, int act, const int* sorted,
+                   const float* weights, float limit, float slope, cudaStream_t stream);
+/* out[t] = sum_j weights[t, j] * y[place[t, j]] (+ shared_out[t]) (weights null: all 1); y [n][H] float or bfloat16; place null: row t * top + j. */
 PHOTON_EXPORT int photon_moe_combine(const void* y, long ldy, int y_dtype, const int* place, const float* weights, int top,
                        const void* shared_out, void* out, int out_dtype, int T_, int H, cudaStream_t stream);
 /* shared_gate [T] (may be null) multiplies the shared expert's rows. */
@@ -339,9 +359,10 @@ PHOTON_EXPORT int photon_moe_combine_ex(const void* y, long ldy, int y_dtype, co
 PHOTON_EXPORT int photon_moe_gather(const void* x, long ldx, int dtype, const int* sorted, int div, void* out, int n, int H,
                       cudaStream_t stream);
 /* Few pairs (decode steps), bfloat16: out[p] = W[ids[p]] x[p / x_div], one matrix-vector product per pair, unsorted;
- * glu as photon_moe_gemm. */
+ * glu, weights (pair p's factor is weights[p]), limit and slope as photon_moe_gemm. */
 PHOTON_EXPORT int photon_moe_gemv(const void* x, long ldx, int x_div, const int* ids, int n, const void* W, void* out, long ldo,
-                    int out_dtype, int N, int K, int glu, int act, cudaStream_t stream);
+                    int out_dtype, int N, int K, int glu, int act, const float* weights, float limit, float slope,
+                    cudaStream_t stream);
 
 /* ------------------------------------------------------------------ attention_flash.cu (-DHEAD_DIM=d, d % 16 == 0, <= 128; bfloat16) */
 PHOTON_EXPORT int photon_flash_attention_head_dim(void);

@@ -149,6 +149,9 @@ def _check_delta_scale(scale: Optional[torch.Tensor], delta, delta2, H: int) -> 
 
 
 ACTIVATIONS = {"silu": 0, "gelu_tanh": 1, "gelu": 2, "relu": 3}     # gelu: the exact (erf) form
+#: activations of a gated unit that do not split into ``act(gate) * up``; only the routed experts' kernels have them.
+#: ``clamped_swish``: ``g = min(gate, limit)``, ``u = clamp(up, -limit, limit)``, ``g sigmoid(slope g) (u + 1)``
+GATED_ACTIVATIONS = {"clamped_swish": 4}
 ACT_NONE = -1
 
 
@@ -1003,34 +1006,38 @@ def linear(x: torch.Tensor, weight: torch.Tensor, out: Optional[torch.Tensor] = 
 # ----------------------------------------------------------------------------- attention over a cached latent
 
 def latent_prep(down: torch.Tensor, q_rank: int, kv_rank: int, rot: int, rot_dims: int, q_norm_w: torch.Tensor,
-                kv_norm_w: torch.Tensor, eps: float, positions: torch.Tensor, inv_freq: torch.Tensor,
-                slot_mapping: torch.Tensor, cq: torch.Tensor, cache: torch.Tensor, err: Optional[torch.Tensor]) -> None:
+                kv_norm_w: Optional[torch.Tensor], eps: float, positions: torch.Tensor, inv_freq: torch.Tensor,
+                slot_mapping: Optional[torch.Tensor], cq: torch.Tensor, cache: Optional[torch.Tensor],
+                err: Optional[torch.Tensor], interleaved: bool = False) -> None:
     """One pass over the fused down-projection rows ``down [T, q_rank + kv_rank + rot]``: the normed query latent
     goes to ``cq [T, q_rank]``, the normed key/value latent and the rotated shared key part to the cache row
-    ``slot_mapping[t]`` of ``cache [pages, 1, page_size, kv_rank + rot]``."""
+    ``slot_mapping[t]`` of ``cache [pages, 1, page_size, kv_rank + rot]``.  ``interleaved``: rotation pairs are
+    neighbours.  ``cache`` None: only the query latent is formed, from ``down [T, >= q_rank]``."""
     _cuda(down, q_norm_w, kv_norm_w, positions, inv_freq, slot_mapping, cq, cache, err)
     T = down.shape[0]
     width = kv_rank + rot
-    if down.shape[1] != q_rank + width or down.stride(1) != 1 or cq.shape != (T, q_rank) or cq.stride(1) != 1 \
-            or cq.dtype != down.dtype or cache.dtype != down.dtype:
+    if down.shape[1] < q_rank + (width if cache is not None else 0) or down.stride(1) != 1 or cq.shape != (T, q_rank) \
+            or cq.stride(1) != 1 or cq.dtype != down.dtype or (cache is not None and cache.dtype != down.dtype):
         raise PhotonError(ErrorCode.SHAPE_MISMATCH, "latent_prep: down [T, q_rank + kv_rank + rot], cq [T, q_rank], one dtype")
-    if cache.dim() != 4 or cache.shape[1] != 1 or cache.shape[3] != width or not cache.is_contiguous():
+    if cache is not None and (cache.dim() != 4 or cache.shape[1] != 1 or cache.shape[3] != width or not cache.is_contiguous()
+                              or kv_norm_w is None or slot_mapping is None):
         raise PhotonError(ErrorCode.SHAPE_MISMATCH, "latent_prep: the cache must be contiguous [pages, 1, page_size, kv_rank + rot]")
     if inv_freq.dtype != torch.float32 or inv_freq.numel() != rot_dims // 2 or rot_dims % 2 or rot_dims > rot:
         raise PhotonError(ErrorCode.SHAPE_MISMATCH, "latent_prep: inv_freq must be float32 [rot_dims / 2], rot_dims even and <= rot")
     _int32(positions, "positions")
-    _int32(slot_mapping, "slot_mapping")
+    if cache is not None:
+        _int32(slot_mapping, "slot_mapping")
     f = _fn("latent", "photon_latent_prep",
-            [c_void_p, c_long, c_int, c_int, c_int, c_int, c_int, c_void_p, c_int, c_void_p, c_int, c_float, c_void_p,
+            [c_void_p, c_long, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_int, c_void_p, c_int, c_float, c_void_p,
              c_void_p, c_void_p, c_void_p, c_long, c_void_p, c_long, c_int, c_void_p, c_void_p])
-    _check(f(_ptr(down), down.stride(0), _dtype_code(down), q_rank, kv_rank, rot, rot_dims, _ptr(q_norm_w),
-             _dtype_code(q_norm_w), _ptr(kv_norm_w), _dtype_code(kv_norm_w), float(eps), _ptr(positions), _ptr(inv_freq),
-             _ptr(slot_mapping), _ptr(cq), cq.stride(0), _ptr(cache), cache.shape[0] * cache.shape[2], T, _ptr(err),
-             _stream()), "latent_prep")
+    _check(f(_ptr(down), down.stride(0), _dtype_code(down), q_rank, kv_rank, rot, rot_dims, int(interleaved), _ptr(q_norm_w),
+             _dtype_code(q_norm_w), _ptr(kv_norm_w), _dtype_code(kv_norm_w) if kv_norm_w is not None else F32, float(eps),
+             _ptr(positions), _ptr(inv_freq), _ptr(slot_mapping), _ptr(cq), cq.stride(0), _ptr(cache),
+             cache.shape[0] * cache.shape[2] if cache is not None else 0, T, _ptr(err), _stream()), "latent_prep")
 
 
 def latent_q_rope(q: torch.Tensor, heads: int, dim: int, rot: int, rot_dims: int, positions: torch.Tensor,
-                  inv_freq: torch.Tensor, out: torch.Tensor, out_off: int) -> None:
+                  inv_freq: torch.Tensor, out: torch.Tensor, out_off: int, interleaved: bool = False) -> None:
     """The last ``rot`` numbers of every head of ``q [T, heads * (dim + rot)]``, rotated, into
     ``out [T, heads, out_head]`` at offset ``out_off`` of every head."""
     _cuda(q, positions, inv_freq, out)
@@ -1040,10 +1047,10 @@ def latent_q_rope(q: torch.Tensor, heads: int, dim: int, rot: int, rot_dims: int
         raise PhotonError(ErrorCode.SHAPE_MISMATCH, "latent_q_rope: q [T, heads * (dim + rot)], out [T, heads, >= out_off + rot]")
     _int32(positions, "positions")
     f = _fn("latent", "photon_latent_q_rope",
-            [c_void_p, c_long, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_long, c_int, c_int,
+            [c_void_p, c_long, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_long, c_int, c_int,
              c_int, c_void_p])
-    _check(f(_ptr(q), q.stride(0), _dtype_code(q), heads, dim, rot, rot_dims, _ptr(positions), _ptr(inv_freq), _ptr(out),
-             out.stride(0), out.shape[2], out_off, T, _stream()), "latent_q_rope")
+    _check(f(_ptr(q), q.stride(0), _dtype_code(q), heads, dim, rot, rot_dims, int(interleaved), _ptr(positions), _ptr(inv_freq),
+             _ptr(out), out.stride(0), out.shape[2], out_off, T, _stream()), "latent_q_rope")
 
 
 def latent_decode_supported(q: torch.Tensor, width: int, value_dim: int) -> bool:
@@ -1052,13 +1059,20 @@ def latent_decode_supported(q: torch.Tensor, width: int, value_dim: int) -> bool
             and q.stride(0) % 8 == 0 and q.data_ptr() % 16 == 0 and (80 * (width + 8) * 2 + 16384) <= 220 * 1024)
 
 
+def latent_decode_shares(max_context: int, window: Optional[int] = None) -> int:
+    """Blocks of 64 rows that the tokens of a step may see at most: a window touches one block more than it fills."""
+    shares = max(1, -(-int(max_context) // 64))
+    return shares if not window else min(shares, -(-(int(window) - 1) // 64) + 1)
+
+
 def latent_decode_attention(q: torch.Tensor, out: torch.Tensor, cache: torch.Tensor, block_table: torch.Tensor,
                             token_seq: torch.Tensor, positions: torch.Tensor, heads: int, width: int, value_dim: int,
-                            scale: float, max_context: int, err: Optional[torch.Tensor]) -> None:
+                            scale: float, max_context: int, err: Optional[torch.Tensor], window: Optional[int] = None) -> None:
     """Attention of decoded tokens (or of the few tokens of a short portion) over cached latent rows on the tensor
     cores: ``q [T, heads * width]``, ``cache [pages, 1, page_size, width]``, ``out [T, heads * value_dim]``; every token
-    sees the rows up to its own position, a row's value is its first ``value_dim`` numbers.  ``max_context``: an upper
-    bound of the tokens' contexts (sizes the grid: one block per token and 64 rows)."""
+    sees the rows up to its own position (with a ``window`` the last ``window`` of them), a row's value is its first
+    ``value_dim`` numbers.  ``max_context``: an upper bound of the tokens' contexts (sizes the grid: one block per token
+    and 64 rows that it may see)."""
     _cuda(q, out, cache, block_table, token_seq, positions, err)
     T = q.shape[0]
     if not latent_decode_supported(q, width, value_dim) or q.shape[1] != heads * width or q.stride(1) != 1 \
@@ -1067,13 +1081,13 @@ def latent_decode_attention(q: torch.Tensor, out: torch.Tensor, cache: torch.Ten
         raise PhotonError(ErrorCode.UNSUPPORTED_SIZE, "latent_decode_attention: bfloat16, widths that are multiples of 16")
     for name, t in (("block_table", block_table), ("token_seq", token_seq), ("positions", positions)):
         _int32(t, name)
-    splits = max(1, -(-int(max_context) // 64))
+    splits = latent_decode_shares(max_context, window)
     part = torch.empty(T * heads * splits * (value_dim + 2), dtype=torch.float32, device=q.device)
     f = _fn("latent", "photon_latent_decode_attention",
             [c_void_p, c_long, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int,
-             c_float, c_int, c_void_p, c_void_p, c_long, c_void_p, c_void_p])
+             c_float, c_int, c_int, c_void_p, c_void_p, c_long, c_void_p, c_void_p])
     _check(f(_ptr(q), q.stride(0), _ptr(cache), _ptr(block_table), block_table.shape[1], _ptr(token_seq), _ptr(positions), T,
-             heads, width, value_dim, cache.shape[2], cache.shape[0], float(scale), splits, _ptr(part), _ptr(out),
+             heads, width, value_dim, cache.shape[2], cache.shape[0], float(scale), int(window or 0), splits, _ptr(part), _ptr(out),
              out.stride(0), _ptr(err), _stream()), "latent_decode_attention")
     global _launch_count
     _launch_count += 1
@@ -1083,52 +1097,103 @@ def latent_decode_attention(q: torch.Tensor, out: torch.Tensor, cache: torch.Ten
 HEAD_LINEAR_LIBRARY_ROWS = 16
 
 
-def head_linear(x: torch.Tensor, weight: torch.Tensor, out: torch.Tensor) -> None:
+def head_linear(x: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, gate: Optional[torch.Tensor] = None) -> None:
     """``out[t, h, :] = weight[h] @ x[t, h, :]`` for all heads at once: ``x [T, heads, K]`` and
-    ``out [T, heads, N]`` are views with free row and head strides, ``weight [heads, N, K]`` is contiguous.
-    float32 and few rows: this package's kernel (one chain of fused multiply-adds per output); many bfloat16
-    rows: the library's batched product."""
-    _cuda(x, weight, out)
+    ``out [T, heads, N]`` are views with free row and head strides, ``weight [heads, N, K]`` is contiguous.  ``gate
+    [T, heads * N]`` (rows with a stride): every output is multiplied by ``sigmoid(gate)``.
+    float32 and few rows: this package's kernel (one chain of fused multiply-adds per output, the gate in its epilogue);
+    many bfloat16 rows: the library's batched product, then the gate."""
+    _cuda(x, weight, out, gate)
     T, heads, K = x.shape
     N = weight.shape[1]
     if weight.shape != (heads, N, K) or not weight.is_contiguous() or out.shape != (T, heads, N) \
             or x.stride(2) != 1 or out.stride(2) != 1 or x.dtype != weight.dtype or out.dtype != x.dtype:
         raise PhotonError(ErrorCode.SHAPE_MISMATCH, "head_linear: x [T, heads, K], weight [heads, N, K], out [T, heads, N]")
+    if gate is not None and (gate.shape != (T, heads * N) or gate.stride(1) != 1 or gate.dtype != x.dtype):
+        raise PhotonError(ErrorCode.SHAPE_MISMATCH, "head_linear: gate [T, heads * N] of the type of x")
     if x.dtype == torch.bfloat16 and T >= HEAD_LINEAR_LIBRARY_ROWS:
         torch.bmm(x.transpose(0, 1), weight.transpose(1, 2), out=out.transpose(0, 1))
+        if gate is not None:
+            if not out.is_contiguous():
+                raise PhotonError(ErrorCode.SHAPE_MISMATCH, "head_linear: a gated output must be contiguous")
+            gate_mul(out.view(T, heads * N), gate)
         return
     f = _fn("latent", "photon_head_linear",
-            [c_void_p, c_long, c_long, c_void_p, c_void_p, c_long, c_long, c_int, c_int, c_int, c_int, c_int, c_void_p])
+            [c_void_p, c_long, c_long, c_void_p, c_void_p, c_long, c_long, c_int, c_int, c_int, c_int, c_int, c_void_p, c_long,
+             c_void_p])
     _check(f(_ptr(x), x.stride(0), x.stride(1), _ptr(weight), _ptr(out), out.stride(0), out.stride(1), _dtype_code(x),
-             T, heads, N, K, _stream()), "head_linear")
+             T, heads, N, K, _ptr(gate), gate.stride(0) if gate is not None else 0, _stream()), "head_linear")
 
 
-def gather_rows(cache: torch.Tensor, table: torch.Tensor, count: int, err: Optional[torch.Tensor]) -> torch.Tensor:
-    """The first ``count`` cached rows of the request whose pages are ``table`` (one row of a block table), as
-    one dense matrix ``[count, width]``; ``cache [pages, 1, page_size, width]``."""
+def gather_rows(cache: torch.Tensor, table: torch.Tensor, count: int, err: Optional[torch.Tensor], first: int = 0,
+                valid=None) -> torch.Tensor:
+    """``count`` cached rows from position ``first`` on of the request whose pages are ``table`` (one row of a block
+    table), as one dense matrix ``[count, width]``; ``cache [pages, 1, page_size, width]``.  ``valid`` ``(lo, hi)``:
+    positions outside give zero rows."""
     _cuda(cache, table, err)
     _int32(table, "table")
     pages, _, page_size, width = cache.shape
-    if count > table.numel() * page_size or not cache.is_contiguous():
+    lo, hi = valid if valid is not None else (first, first + count)
+    if hi > table.numel() * page_size or min(first, lo) < 0 or not cache.is_contiguous():
         raise PhotonError(ErrorCode.INVALID_ARGUMENT, "gather_rows: more rows asked for than the table's pages hold")
     out = torch.empty((count, width), dtype=cache.dtype, device=cache.device)
-    f = _fn("latent", "photon_gather_rows", [c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p])
-    _check(f(_ptr(cache), _dtype_code(cache), _ptr(table), page_size, pages, width, int(count), _ptr(out), _ptr(err), _stream()),
-           "gather_rows")
+    f = _fn("latent", "photon_gather_rows", [c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p,
+                                             c_void_p, c_void_p])
+    _check(f(_ptr(cache), _dtype_code(cache), _ptr(table), page_size, pages, width, int(first), int(count), int(lo), int(hi),
+             _ptr(out), _ptr(err), _stream()), "gather_rows")
     return out
 
 
-def causal_softmax_rows(scores: torch.Tensor, probs: torch.Tensor, heads: int, first_pos: int, scale: float) -> None:
-    """``probs = softmax(scale * scores)`` row by row over the keys each row may see: row ``r`` belongs to the token
-    at position ``first_pos + r // heads`` and sees the keys up to that position; zero beyond."""
+def causal_softmax_rows(scores: torch.Tensor, probs: torch.Tensor, heads: int, first_pos: int, scale: float,
+                        first_key: int = 0, window: Optional[int] = None) -> None:
+    """``probs = softmax(scale * scores)`` row by row over the keys each row may see: column ``c`` is the key at position
+    ``first_key + c``, row ``r`` belongs to the token at position ``first_pos + r // heads`` and sees the keys up to that
+    position (with a ``window`` the last ``window`` of them); zero elsewhere."""
     _cuda(scores, probs)
     rows, cols = scores.shape
     if scores.dtype != torch.float32 or scores.stride(1) != 1 or probs.shape != scores.shape or probs.stride(1) != 1:
         raise PhotonError(ErrorCode.SHAPE_MISMATCH, "causal_softmax_rows: scores float32 [rows, cols], probs of the same shape")
     f = _fn("latent", "photon_causal_softmax_rows",
-            [c_void_p, c_long, c_void_p, c_long, c_int, c_int, c_int, c_int, c_int, c_float, c_void_p])
+            [c_void_p, c_long, c_void_p, c_long, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_void_p])
     _check(f(_ptr(scores), scores.stride(0), _ptr(probs), probs.stride(0), _dtype_code(probs), rows, int(heads), int(first_pos),
-             cols, float(scale), _stream()), "causal_softmax_rows")
+             int(first_key), int(window or 0), cols, float(scale), _stream()), "causal_softmax_rows")
+
+
+# ----------------------------------------------------------------------------- parallel residual streams
+
+def stream_norm(streams: torch.Tensor, count: int, y: Optional[torch.Tensor], mix: Optional[torch.Tensor],
+                w_out: Optional[torch.Tensor], w_in: Optional[torch.Tensor], weight: torch.Tensor, bias: Optional[torch.Tensor],
+                eps: float, out: torch.Tensor, center: bool = True, new_streams: Optional[torch.Tensor] = None,
+                rows: Optional[torch.Tensor] = None) -> None:
+    """``out = norm(sum_s w_in[s] X_s) * weight (+ bias)`` (``w_in`` None: the plain sum), after the pending write
+    ``X_t <- sum_s mix[s, t] X_s + w_out[t] y`` (``y`` None: nothing pending).  ``streams``: float32 ``[T, count, H]``, or
+    ``[T, H]`` where all ``count`` streams are equal.  ``new_streams [T, count, H]`` receives the written streams (it may be
+    ``streams``; None: they are not kept).  ``center``: layer norm, else RMS norm.  ``rows``: only these tokens are read."""
+    _cuda(streams, y, mix, w_out, w_in, weight, bias, out, new_streams, rows)
+    T, H = streams.shape[0], streams.shape[-1]
+    equal = streams.dim() == 2
+    if streams.dtype != torch.float32 or not streams.is_contiguous() or (not equal and streams.shape != (T, count, H)):
+        raise PhotonError(ErrorCode.SHAPE_MISMATCH, "stream_norm: streams must be contiguous float32 [T, count, H] or [T, H]")
+    if y is not None and (y.shape != (T, H) or not y.is_contiguous() or mix is None or w_out is None):
+        raise PhotonError(ErrorCode.SHAPE_MISMATCH, "stream_norm: a pending output [T, H] comes with its mix and out weights")
+    for t, shape in ((mix, (count, count)), (w_out, (count,)), (w_in, (count,))):
+        if t is not None and (t.dtype != torch.float32 or tuple(t.shape) != shape or not t.is_contiguous()):
+            raise PhotonError(ErrorCode.SHAPE_MISMATCH, f"stream_norm: weights must be float32, one per stream ({count})")
+    if new_streams is not None and (new_streams.dtype != torch.float32 or new_streams.shape != (T, count, H)
+                                    or not new_streams.is_contiguous() or rows is not None):
+        raise PhotonError(ErrorCode.SHAPE_MISMATCH, "stream_norm: new_streams must be contiguous float32 [T, count, H]")
+    if rows is not None:
+        _int32(rows, "rows")
+    n = rows.numel() if rows is not None else T
+    if out.shape != (n, H) or not out.is_contiguous() or weight.numel() != H or (bias is not None and bias.numel() != H):
+        raise PhotonError(ErrorCode.SHAPE_MISMATCH, "stream_norm: out must be [rows, H], weight and bias [H]")
+    f = _fn("hyper", "photon_stream_norm",
+            [c_void_p, c_long, c_long, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p, c_int,
+             c_void_p, c_int, c_int, c_float, c_void_p, c_int, c_void_p, c_int, c_void_p])
+    _check(f(_ptr(streams), H if equal else count * H, 0 if equal else H, _ptr(new_streams), _ptr(y),
+             _dtype_code(y) if y is not None else F32, _ptr(mix), _ptr(w_out), _ptr(w_in), int(count), H, _ptr(weight),
+             _dtype_code(weight), _ptr(bias), _dtype_code(bias) if bias is not None else F32, int(center), float(eps), _ptr(out),
+             _dtype_code(out), _ptr(rows), n, _stream()), "stream_norm")
 
 
 # ----------------------------------------------------------------------------- gated delta rule
@@ -1758,35 +1823,63 @@ def moe_align(ids: torch.Tensor, counts: torch.Tensor):
 
 def moe_gemm(a: torch.Tensor, gather: Optional[torch.Tensor], gather_div: int, weight: torch.Tensor, out: torch.Tensor,
              tiles: torch.Tensor, num_tiles: torch.Tensor, max_tiles: int, glu: bool = False,
-             activation: Optional[str] = None) -> None:
+             activation: Optional[str] = None, weights: Optional[torch.Tensor] = None, limit: float = 0.0,
+             slope: float = 1.0) -> None:
     """Grouped product over rows sorted by expert: ``weight [E, N, K]``; sorted row ``r`` reads row
     ``gather[r] // gather_div`` of ``a`` (``gather`` None: row ``r``).  ``glu``: ``weight`` holds gate rows
     then up rows and ``out [n, N / 2] = act(gate) * up`` (silu unless named).  Without ``glu`` an ``activation`` is
-    applied to every output (None: the plain product)."""
-    _cuda(a, gather, weight, out, tiles, num_tiles)
-    act = ACTIVATIONS[activation or "silu"] if glu or activation else ACT_NONE
+    applied to every output (None: the plain product).  ``weights`` float32 (one per pair, with ``gather``): a factor on
+    the pair's input row.  ``limit``, ``slope``: constants of ``clamped_swish``."""
+    _cuda(a, gather, weight, out, tiles, num_tiles, weights)
+    act = _expert_act(glu, activation)
+    if weights is not None and (gather is None or weights.dtype != torch.float32 or not weights.is_contiguous()):
+        raise PhotonError(ErrorCode.INVALID_ARGUMENT, "moe_gemm: input factors are float32, one per pair, and need the sorted list")
     E, N, K = weight.shape
     if a.shape[1] != K or a.stride(1) != 1 or not weight.is_contiguous() or a.dtype != weight.dtype \
             or out.stride(1) != 1 or out.shape[1] != (N // 2 if glu else N) or out.dtype not in (a.dtype, torch.float32):
         raise PhotonError(ErrorCode.SHAPE_MISMATCH, "moe_gemm: a [*, K], weight [E, N, K], out [n, N or N / 2]")
     f = _fn("moe", "photon_moe_gemm",
             [c_void_p, c_long, c_int, c_void_p, c_int, c_void_p, c_void_p, c_long, c_int, c_int, c_int, c_void_p,
-             c_void_p, c_int, c_int, c_int, c_void_p])
+             c_void_p, c_int, c_int, c_int, c_void_p, c_float, c_float, c_void_p])
     _check(f(_ptr(a), a.stride(0), _dtype_code(a), _ptr(gather), int(gather_div), _ptr(weight), _ptr(out), out.stride(0),
-             _dtype_code(out), N, K, _ptr(tiles), _ptr(num_tiles), int(max_tiles), int(glu), act,
-             _stream()), "moe_gemm")
+             _dtype_code(out), N, K, _ptr(tiles), _ptr(num_tiles), int(max_tiles), int(glu), act, _ptr(weights), float(limit),
+             float(slope), _stream()), "moe_gemm")
 
 
-def moe_combine(y: torch.Tensor, place: Optional[torch.Tensor], weights: torch.Tensor, shared_out: Optional[torch.Tensor],
+def _expert_act(glu: bool, activation: Optional[str]) -> int:
+    if activation in GATED_ACTIVATIONS:
+        if not glu:
+            raise PhotonError(ErrorCode.INVALID_ARGUMENT, f"{activation} is the activation of a gated unit")
+        return GATED_ACTIVATIONS[activation]
+    return ACTIVATIONS[activation or "silu"] if glu or activation else ACT_NONE
+
+
+def moe_glu(gate_up: torch.Tensor, out: torch.Tensor, activation: str, srt: Optional[torch.Tensor] = None,
+            weights: Optional[torch.Tensor] = None, limit: float = 0.0, slope: float = 1.0) -> None:
+    """The gated unit of the routed experts on rows in sorted order: ``gate_up [n, 2 I]`` -> ``out [n, I]``; with
+    ``weights`` float32 (one per pair) and ``srt`` the sums of row ``r`` are multiplied by ``weights[srt[r]]`` first."""
+    _cuda(gate_up, out, srt, weights)
+    n, I2 = gate_up.shape
+    if I2 % 2 or out.shape != (n, I2 // 2) or out.dtype != gate_up.dtype or not gate_up.is_contiguous() or not out.is_contiguous():
+        raise PhotonError(ErrorCode.SHAPE_MISMATCH, "moe_glu: gate_up [n, 2 I] and out [n, I] of one dtype")
+    if weights is not None and (srt is None or weights.numel() != n or weights.dtype != torch.float32 or not weights.is_contiguous()):
+        raise PhotonError(ErrorCode.INVALID_ARGUMENT, "moe_glu: input factors are float32, one per pair, and need the sorted list")
+    f = _fn("moe", "photon_moe_glu", [c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_float, c_float, c_void_p])
+    _check(f(_ptr(gate_up), _ptr(out), _dtype_code(out), n, I2 // 2, _expert_act(True, activation), _ptr(srt), _ptr(weights),
+             float(limit), float(slope), _stream()), "moe_glu")
+
+
+def moe_combine(y: torch.Tensor, place: Optional[torch.Tensor], weights: Optional[torch.Tensor], shared_out: Optional[torch.Tensor],
                 out: torch.Tensor, shared_gate: Optional[torch.Tensor] = None) -> None:
     """``out[t] = sum_j weights[t, j] * y[place[t, j]] (+ shared_out[t])``, summed in 32-bit in the order of ``j``;
     ``place`` None: the rows of ``y`` stand in the order of the pairs.  ``shared_gate`` float32 ``[T]``: the shared
-    expert's row of token ``t`` is multiplied by ``shared_gate[t]``."""
+    expert's row of token ``t`` is multiplied by ``shared_gate[t]``.  ``weights`` None: a plain sum (the experts' inputs
+    carried the weights)."""
     _cuda(y, place, weights, shared_out, out, shared_gate)
-    if shared_gate is not None and (shared_out is None or shared_gate.dtype != torch.float32 or shared_gate.numel() != weights.shape[0]):
+    T, H = out.shape[0], y.shape[1]
+    top = weights.shape[1] if weights is not None else y.shape[0] // max(T, 1)
+    if shared_gate is not None and (shared_out is None or shared_gate.dtype != torch.float32 or shared_gate.numel() != T):
         raise PhotonError(ErrorCode.SHAPE_MISMATCH, "moe_combine: shared_gate float32 [T] goes with shared_out")
-    T, top = weights.shape
-    H = y.shape[1]
     if y.stride(1) != 1 or out.shape != (T, H) or not out.is_contiguous() \
             or (shared_out is not None and (shared_out.shape != (T, H) or not shared_out.is_contiguous()
                                             or shared_out.dtype != out.dtype)):
@@ -1814,11 +1907,15 @@ def moe_gemv_supported(x: torch.Tensor, weight: torch.Tensor) -> bool:
 
 
 def moe_gemv(x: torch.Tensor, x_div: int, ids: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, glu: bool = False,
-             activation: Optional[str] = None) -> None:
+             activation: Optional[str] = None, weights: Optional[torch.Tensor] = None, limit: float = 0.0,
+             slope: float = 1.0) -> None:
     """A decode step's few (token, choice) pairs: ``out[p] = weight[ids[p]] @ x[p // x_div]``, one matrix-vector
-    product per pair in the order of the pairs, the expert's rows streamed once.  bfloat16 in, bfloat16 or float32 out."""
-    _cuda(x, ids, weight, out)
-    act = ACTIVATIONS[activation or "silu"] if glu or activation else ACT_NONE
+    product per pair in the order of the pairs, the expert's rows streamed once.  bfloat16 in, bfloat16 or float32 out.
+    ``weights`` float32 (one per pair): a factor on the pair's input row."""
+    _cuda(x, ids, weight, out, weights)
+    act = _expert_act(glu, activation)
+    if weights is not None and (weights.dtype != torch.float32 or weights.numel() != ids.numel() or not weights.is_contiguous()):
+        raise PhotonError(ErrorCode.SHAPE_MISMATCH, "moe_gemv: input factors are float32, one per pair")
     E, N, K = weight.shape
     n = ids.numel()
     if not moe_gemv_supported(x, weight) or x.shape[1] != K:
@@ -1826,9 +1923,10 @@ def moe_gemv(x: torch.Tensor, x_div: int, ids: torch.Tensor, weight: torch.Tenso
     if out.shape != (n, N // 2 if glu else N) or out.stride(1) != 1:
         raise PhotonError(ErrorCode.SHAPE_MISMATCH, "moe_gemv: out [pairs, N or N / 2]")
     f = _fn("moe", "photon_moe_gemv",
-            [c_void_p, c_long, c_int, c_void_p, c_int, c_void_p, c_void_p, c_long, c_int, c_int, c_int, c_int, c_int, c_void_p])
+            [c_void_p, c_long, c_int, c_void_p, c_int, c_void_p, c_void_p, c_long, c_int, c_int, c_int, c_int, c_int, c_void_p, c_float,
+             c_float, c_void_p])
     _check(f(_ptr(x), x.stride(0), int(x_div), _ptr(ids), n, _ptr(weight), _ptr(out), out.stride(0), _dtype_code(out), N, K,
-             int(glu), act, _stream()), "moe_gemv")
+             int(glu), act, _ptr(weights), float(limit), float(slope), _stream()), "moe_gemv")
 
 
 # ----------------------------------------------------------------------------- sampling

@@ -37,9 +37,8 @@ def _build_layer(ls: LayerSpec, encodings: Dict[str, Part]) -> Block:
     norm2 = create_part("norm", ls.norm2.kind, ls.norm2.params) if ls.norm2 is not None else None
     ff = create_part("feed_forward", ls.feed_forward.kind, ls.feed_forward.params) if ls.feed_forward is not None else None
     params = dict(ls.block.params, norm1=norm1, mixer=mixer, norm2=norm2, feed_forward=ff)
-    for key, ps in (("scale1", ls.scale1), ("scale2", ls.scale2)):
-        if ps is not None:
-            params[key] = create_part("scale", ps.kind, ps.params)
+    for key, table, ps in ls.optional_parts():
+        params[key] = create_part(table, ps.kind, ps.params)
     return create_part("block", ls.block.kind, params)
 
 
@@ -49,9 +48,8 @@ def _layer_part_prefixes(ls: LayerSpec) -> Dict[str, str]:
         out["norm2"] = ls.prefix + ls.norm2.prefix
     if ls.feed_forward is not None:
         out["feed_forward"] = ls.prefix + ls.feed_forward.prefix
-    for key, ps in (("scale1", ls.scale1), ("scale2", ls.scale2)):
-        if ps is not None:
-            out[key] = ls.prefix + ps.prefix
+    for key, _, ps in ls.optional_parts():
+        out[key] = ls.prefix + ps.prefix
     return out
 
 

@@ -29,6 +29,15 @@ class LayerSpec:
     # by channel before it is added to the residual stream
     scale1: Optional[PartSpec] = None
     scale2: Optional[PartSpec] = None
+    # how the mixer and the feed-forward read and write several residual streams (kind "hyper", with a block that has them)
+    connect1: Optional[PartSpec] = None
+    connect2: Optional[PartSpec] = None
+
+    def optional_parts(self):
+        """``(block parameter, part table, spec)`` of the optional parts that this layer has."""
+        return [(key, table, ps) for key, table, ps in (("scale1", "scale", self.scale1), ("scale2", "scale", self.scale2),
+                                                        ("connect1", "connection", self.connect1),
+                                                        ("connect2", "connection", self.connect2)) if ps is not None]
 
 
 @dataclasses.dataclass

@@ -188,6 +188,21 @@ class Normed:
         return self.norm.forward(x, torch.float32)
 
 
+@dataclasses.dataclass
+class Connected:
+    """A pending output of a layer with several residual streams: ``X_t <- sum_s mix[s, t] X_s + out[t] tensor``, with the
+    weights of the sublayer's ``connection``.  Only a norm that reads streams (``Norm.read_streams``) takes it."""
+    tensor: torch.Tensor
+    connection: "ConnectionPart"
+
+    def apply(self, streams: torch.Tensor) -> torch.Tensor:
+        """The new streams ``[T, S, H]`` from the old ones (``[T, S, H]``, or ``[T, H]`` where all are equal), in 32-bit, by
+        plain tensor operations: for a consumer without a kernel of its own."""
+        c = self.connection
+        x = streams if streams.dim() == 3 else streams.unsqueeze(1).expand(-1, c.streams, -1)
+        return torch.einsum("st,nsh->nth", c.mix, x) + c.w_out[None, :, None] * self.tensor.to(torch.float32).unsqueeze(1)
+
+
 def delta_terms(delta) -> Tuple[Optional[torch.Tensor], Optional[torch.Tensor], Optional[torch.Tensor]]:
     """``(d1, d2, scale)``: what is pending on the stream as ``scale * d1 + d2`` (each may be None)."""
     if isinstance(delta, Scaled):
@@ -201,6 +216,8 @@ def delta_pair(delta) -> Tuple[Optional[torch.Tensor], Optional[torch.Tensor]]:
     parallel block (mixer and feed-forward), which are summed with each other first and then into the stream."""
     if delta is None:
         return None, None
+    if isinstance(delta, Connected):
+        raise TypeError("an output pending on several residual streams cannot be added to a single one")
     if isinstance(delta, (Scaled, Normed)):
         return delta.materialize(), None
     if isinstance(delta, (tuple, list)):
@@ -236,6 +253,24 @@ class Norm(Part):
         if out_dtype is None:
             return None
         return residual if out_dtype == residual.dtype else residual.to(out_dtype)
+
+    def read_streams(self, delta: Optional[Connected], streams: torch.Tensor, w_in: Optional[torch.Tensor],
+                     out_dtype: torch.dtype, rows: Optional[torch.Tensor] = None):
+        """Several residual streams: what is pending is written to them, then ``forward(sum_s w_in[s] X_s)`` (``w_in`` None:
+        the plain sum).  ``streams`` float32 ``[T, S, H]``, or ``[T, H]`` where all are equal.  Returns ``(normed rows, new
+        streams)``; with ``rows`` only those tokens' rows, and the streams as they were.  This form uses plain tensor
+        operations; a norm with a kernel for it does everything in one pass."""
+        if rows is not None:
+            idx = rows.long()
+            part = None if delta is None else Connected(delta.tensor.index_select(0, idx), delta.connection)
+            return self.read_streams(part, streams.index_select(0, idx), w_in, out_dtype)[0], streams
+        new = streams if delta is None else delta.apply(streams)
+        if new.dim() == 2:
+            if w_in is None:
+                raise ValueError("the sum of streams that are all equal needs their number")
+            return self.forward(new * w_in.sum(), out_dtype), new
+        x = new.sum(dim=1) if w_in is None else torch.einsum("s,nsh->nh", w_in, new)
+        return self.forward(x.contiguous(), out_dtype), new
 
     def add_forward_rows(self, delta, residual: torch.Tensor, rows: torch.Tensor, out_dtype: torch.dtype) -> torch.Tensor:
         """Same as ``add_forward`` for the listed rows only; returns ``[len(rows), H]``."""
@@ -299,6 +334,15 @@ class ChannelScalePart(Part):
 
     def apply(self, x: torch.Tensor) -> "Scaled":
         return Scaled(x, self.vector)
+
+
+class ConnectionPart(Part):
+    """How a sublayer reads from and writes to several residual streams: ``u = sum_s w_in[s] X_s`` goes into its norm, its
+    output ``y`` comes back as ``X_t <- sum_s mix[s, t] X_s + w_out[t] y``.  All weights are held in 32-bit."""
+    streams: int = 1
+    w_in: Optional[torch.Tensor] = None         # [S]
+    w_out: Optional[torch.Tensor] = None        # [S]
+    mix: Optional[torch.Tensor] = None          # [S, S], [from, to]
 
 
 class StreamPart(Part):

@@ -7,6 +7,9 @@ without a feed-forward adds the mixer's output alone.
 Output norm: ``x += norm1(mixer(x)); x += norm2(ff(x))``: the sublayers read the stream itself and the norms sit on
 their outputs.
 
+Hyper pre-norm: pre-norm over several parallel residual streams, which each sublayer reads and writes through a connection
+of its own.
+
 Each residual sum is handed to the norm that follows it, which does both in one pass over the row, in
 32-bit; a parallel block hands on its two outputs as a pair, and that norm forms their sum first."""
 from __future__ import annotations
@@ -15,7 +18,7 @@ from typing import Dict, Optional, Tuple
 
 import torch
 
-from .base import (Block, ChannelScalePart, FeedForward, LayerCache, Mixer, Norm, Normed, Part, Scaled, StepContext,
+from .base import (Block, ChannelScalePart, Connected, ConnectionPart, FeedForward, LayerCache, Mixer, Norm, Normed, Part, Scaled, StepContext,
                    delta_pair)
 from .registry import register_block
 
@@ -128,6 +131,38 @@ class OutputNormBlock(Block):
         return residual, Normed(self.feed_forward.forward(h2, ctx), self.norm2)
 
 
+class HyperPreNormBlock(Block):
+    """Pre-norm over several residual streams: a sublayer's norm gets ``sum_s in[s] X_s`` and its output is written back into
+    all streams, mixed with each other at the same time (``parts/hyper.py``).  The write stays pending (``Connected``) for
+    the next norm, which writes, reads and norms in one kernel; ``residual`` is ``[T, H]`` while all streams are equal (up
+    to the first write) and ``[T, S, H]`` afterwards."""
+
+    def __init__(self, norm1: Norm, mixer: Mixer, connect1: ConnectionPart, norm2: Optional[Norm] = None,
+                 feed_forward: Optional[FeedForward] = None, connect2: Optional[ConnectionPart] = None):
+        if not (norm2 is None) == (feed_forward is None) == (connect2 is None):
+            raise ValueError("a block has a second norm and connection exactly when it has a feed-forward")
+        self.norm1, self._mixer, self.connect1 = norm1, mixer, connect1
+        self.norm2, self.feed_forward, self.connect2 = norm2, feed_forward, connect2
+
+    def parts(self) -> Dict[str, Part]:
+        p = {"norm1": self.norm1, "mixer": self._mixer, "connect1": self.connect1}
+        if self.feed_forward is not None:
+            p.update(norm2=self.norm2, feed_forward=self.feed_forward, connect2=self.connect2)
+        return p
+
+    def mixer(self) -> Mixer:
+        return self._mixer
+
+    def forward(self, residual: torch.Tensor, delta, ctx: StepContext, cache: LayerCache):
+        h, residual = self.norm1.read_streams(delta, residual, self.connect1.w_in, ctx.dtype)
+        a = Connected(self._mixer.forward(h, ctx, cache), self.connect1)
+        if self.feed_forward is None:
+            return residual, a
+        h2, residual = self.norm2.read_streams(a, residual, self.connect2.w_in, ctx.dtype)
+        return residual, Connected(self.feed_forward.forward(h2, ctx), self.connect2)
+
+
 register_block("pre_norm", PreNormBlock)
 register_block("parallel", ParallelBlock)
 register_block("output_norm", OutputNormBlock)
+register_block("hyper_pre_norm", HyperPreNormBlock)

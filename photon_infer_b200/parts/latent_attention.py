@@ -13,8 +13,15 @@ once per step (``head_linear``), attention runs with ONE key/value head whose ke
 whose values are the first ``kv_rank`` numbers of the same rows, and ``W_uv[h]`` is applied to the head's
 weighted sum of latents.  A prompt portion, a decoded token and a mixed batch are the same case.
 
-The rotation turns the first ``rot_dims`` numbers of the rotated part, feature ``i`` paired with
-``i + rot_dims / 2``, by the angle ``position * base^(-2i / rot_dims)``; the rest passes unchanged.
+The rotation turns the first ``rot_dims`` numbers of the rotated part by the angle ``position * base^(-2i / rot_dims)``,
+feature ``i`` paired with ``i + rot_dims / 2`` or (``rot_interleaved``) feature ``2i`` with ``2i + 1``; the rest passes
+unchanged.
+
+Variants, all by parameter.  ``window``: a token sees its own row and the ``window - 1`` before it.  ``output_gate``: the
+concatenated heads are multiplied by ``sigmoid(W_g h)`` before ``W_o``; ``W_g``'s rows ride in the fused down-projection.
+``own_kv`` False: the layer has no ``W_dkv``; it reads the cached rows of an earlier layer (the run list's ``kv_from``) with
+its own queries, ``W_uk``, ``W_uv``, window and everything else.  ``cache_window``: how many rows the cache must keep for
+this layer AND the layers that read its pages (``"own"``: this layer's window; None: everything).
 """
 from __future__ import annotations
 
@@ -32,7 +39,8 @@ class LatentAttention(Mixer):
     kernel_modules = ("latent", "attention")
 
     def __init__(self, hidden_size: int, heads: int, dim: int, rot_dim: int, vdim: int, kv_rank: int, q_rank: int,
-                 scale: float, eps: float, rot_base: float, rot_dims: Optional[int] = None, window: Optional[int] = None):
+                 scale: float, eps: float, rot_base: float, rot_dims: Optional[int] = None, window: Optional[int] = None,
+                 rot_interleaved: bool = False, cache_window="own", own_kv: bool = True, output_gate: bool = False):
         self.hidden_size, self.heads, self.dim, self.rot_dim, self.vdim = hidden_size, heads, dim, rot_dim, vdim
         self.kv_rank, self.q_rank = kv_rank, q_rank
         self.scale, self.eps = float(scale), float(eps)
@@ -40,7 +48,12 @@ class LatentAttention(Mixer):
         self.rot_dims = rot_dim if rot_dims is None else int(rot_dims)
         if self.rot_dims % 2 or not 0 <= self.rot_dims <= rot_dim:
             raise ValueError("the rotated features must be an even number of at most rot_dim")
-        self.window = window
+        self.rot_interleaved = bool(rot_interleaved)
+        self.window = int(window) if window else None
+        self.cache_window = self.window if cache_window == "own" else (int(cache_window) if cache_window else None)
+        if self.cache_window is not None and (self.window is None or self.window > self.cache_window):
+            raise ValueError("the cache must keep at least the rows that this layer's window sees")
+        self.own_kv, self.output_gate = bool(own_kv), bool(output_gate)
         self.width = kv_rank + rot_dim          # one cached row
         half = self.rot_dims // 2
         self.inv_freq_host = torch.tensor([self.rot_base ** (-2.0 * i / self.rot_dims) for i in range(half)],
@@ -53,20 +66,27 @@ class LatentAttention(Mixer):
         mods = list(self.kernel_modules)
         if dtype == torch.bfloat16:
             mods.extend(["gemm_skinny", "gemm_tc", "gemm_tc2"])
+        if self.output_gate:
+            mods.append("elementwise")
         return mods
 
     def tensor_specs(self) -> List[TensorSpec]:
         H, n, d, r, v = self.hidden_size, self.heads, self.dim, self.rot_dim, self.vdim
-        return [TensorSpec("dq", (self.q_rank, H)), TensorSpec("dq.norm", (self.q_rank,), role="vector", init="norm"),
-                TensorSpec("uq", (n * (d + r), self.q_rank)),
-                TensorSpec("dkv", (self.kv_rank + r, H)), TensorSpec("dkv.norm", (self.kv_rank,), role="vector", init="norm"),
-                TensorSpec("uk", (n * d, self.kv_rank)), TensorSpec("uv", (n * v, self.kv_rank)),
-                TensorSpec("o", (H, n * v))]
+        specs = [TensorSpec("dq", (self.q_rank, H)), TensorSpec("dq.norm", (self.q_rank,), role="vector", init="norm"),
+                 TensorSpec("uq", (n * (d + r), self.q_rank))]
+        if self.own_kv:
+            specs += [TensorSpec("dkv", (self.kv_rank + r, H)), TensorSpec("dkv.norm", (self.kv_rank,), role="vector", init="norm")]
+        specs += [TensorSpec("uk", (n * d, self.kv_rank)), TensorSpec("uv", (n * v, self.kv_rank))]
+        if self.output_gate:
+            specs.append(TensorSpec("g", (n * v, H)))
+        return specs + [TensorSpec("o", (H, n * v))]
 
     def load(self, tensors: Dict[str, torch.Tensor]) -> None:
         n, d, v = self.heads, self.dim, self.vdim
-        self.w_down = torch.cat([tensors["dq"], tensors["dkv"]], dim=0).contiguous()      # h is read once
-        self.q_norm, self.kv_norm = tensors["dq.norm"].contiguous(), tensors["dkv.norm"].contiguous()
+        down = [tensors["dq"]] + ([tensors["dkv"]] if self.own_kv else []) + ([tensors["g"]] if self.output_gate else [])
+        self.w_down = torch.cat(down, dim=0).contiguous()                                 # h is read once
+        self.q_norm = tensors["dq.norm"].contiguous()
+        self.kv_norm = tensors["dkv.norm"].contiguous() if self.own_kv else None
         self.w_uq = tensors["uq"].contiguous()
         # W_uk[h]^T as the [out, in] matrix of the product that takes a head's unrotated query into the latent space
         self.w_absorb = tensors["uk"].view(n, d, self.kv_rank).transpose(1, 2).contiguous()   # [heads, kv_rank, dim]
@@ -79,36 +99,39 @@ class LatentAttention(Mixer):
         return sum(w.numel() * w.element_size() for w in ws)
 
     def cache_spec(self) -> Optional[PagedCacheSpec]:
-        return PagedCacheSpec(1, self.width, self.window, values=False)
+        return PagedCacheSpec(1, self.width, self.cache_window, values=False)
 
     def forward(self, h: torch.Tensor, ctx: StepContext, cache: LayerCache) -> torch.Tensor:
         T = h.shape[0]
         n, d, r, kr = self.heads, self.dim, self.rot_dim, self.kv_rank
         group = ctx.groups[cache.group]
-        down = project(h, self.w_down)                                   # [T, q_rank + kv_rank + rot]
+        down = project(h, self.w_down)                                   # [T, q_rank (+ kv_rank + rot) (+ gate)]
+        gate = down[:, down.shape[1] - n * self.vdim:] if self.output_gate else None
+        store = self.own_kv and not cache.shared
         cq = torch.empty((T, self.q_rank), dtype=h.dtype, device=h.device)
         ops.latent_prep(down, self.q_rank, kr, r, self.rot_dims, self.q_norm, self.kv_norm, self.eps, ctx.positions,
-                        self.inv_freq, group.slot_mapping, cq, cache.k, ctx.error_flag)
+                        self.inv_freq, group.slot_mapping if store else None, cq, cache.k if store else None, ctx.error_flag,
+                        interleaved=self.rot_interleaved)
         q = project(cq, self.w_uq)                                       # [T, heads * (dim + rot)]
         q_lat = torch.empty((T, n, self.width), dtype=h.dtype, device=h.device)
         ops.head_linear(q.view(T, n, d + r)[:, :, :d], self.w_absorb, q_lat[:, :, :kr])
-        ops.latent_q_rope(q, n, d, r, self.rot_dims, ctx.positions, self.inv_freq, q_lat, kr)
+        ops.latent_q_rope(q, n, d, r, self.rot_dims, ctx.positions, self.inv_freq, q_lat, kr, interleaved=self.rot_interleaved)
         o_lat = torch.empty((T, n * kr), dtype=h.dtype, device=h.device)
         self.attend(q_lat, o_lat, ctx, cache)
         o = torch.empty((T, n, self.vdim), dtype=h.dtype, device=h.device)
-        ops.head_linear(o_lat.view(T, n, kr), self.w_uv, o)
+        ops.head_linear(o_lat.view(T, n, kr), self.w_uv, o, gate=gate)
         return project(o.view(T, n * self.vdim), self.w_o)
-
 
     def attend(self, q_lat: torch.Tensor, o_lat: torch.Tensor, ctx: StepContext, cache: LayerCache) -> None:
         """Decoded tokens, short portions and the float32 run: the paged kernel, whose sums depend only on a token's
         position.  A long bfloat16 portion: the request's cached rows are gathered into one matrix and attention
         is three steps per slab of queries, scores = Q C^T (library product, 32-bit out), a causal softmax over the
-        rows, and P C[:, :kv_rank] (library product); a slab ends at the last key its queries may see."""
+        rows, and P C[:, :kv_rank] (library product); a slab starts at the first and ends at the last row its queries
+        may see."""
         T, n, kr = q_lat.shape[0], self.heads, self.kv_rank
         group = ctx.groups[cache.group]
         lens = list(ctx.host_query_lens) or [T]
-        long_rows = [q_lat.dtype == torch.bfloat16 and self.window is None and m >= LIBRARY_MIN_TOKENS for m in lens]
+        long_rows = [q_lat.dtype == torch.bfloat16 and m >= LIBRARY_MIN_TOKENS for m in lens]
         t = 0
         pending = None                                  # a run of neighbouring requests for the paged kernel
         for s, m in enumerate(lens):
@@ -127,19 +150,21 @@ class LatentAttention(Mixer):
         n = self.heads
         group = ctx.groups[cache.group]
         q2 = q_lat[a:b].view(b - a, n * self.width)
-        shares = -(-max(ctx.max_context_len, 1) // 64)
-        if self.window is None and ops.latent_decode_supported(q2, self.width, self.kv_rank) \
+        shares = ops.latent_decode_shares(ctx.max_context_len, self.window)
+        if ops.latent_decode_supported(q2, self.width, self.kv_rank) \
                 and (b - a) * n * shares * (self.kv_rank + 2) * 4 <= DECODE_SHARES_BYTES:
             # bfloat16 with widths that fit the tensor cores' tiles: one block per token and 64 cached rows
             ops.latent_decode_attention(q2, o_lat[a:b], cache.k, group.block_table, ctx.token_seq[a:b], ctx.positions[a:b], n,
-                                        self.width, self.kv_rank, self.scale, ctx.max_context_len, ctx.error_flag)
+                                        self.width, self.kv_rank, self.scale, ctx.max_context_len, ctx.error_flag,
+                                        window=self.window)
             return
         splits = 1
         if q_lat.dtype == torch.bfloat16:
             # few tokens with long contexts: share every token's key tiles out until the GPU is full (the float32 run keeps
             # one block per token, whose sums depend on the token's position alone)
             chunks = -(-n // max(1, min(n, 4096 // self.width)))
-            tiles = -(-max(ctx.max_context_len, 1) // 32)
+            seen = max(ctx.max_context_len, 1) if self.window is None else min(max(ctx.max_context_len, 1), self.window + 31)
+            tiles = -(-seen // 32)
             splits = max(1, min(4 * ops.sm_count(q_lat.device) // max(1, (b - a) * chunks), tiles, 64))
         ops.paged_attention(q_lat[a:b].view(b - a, n * self.width), o_lat[a:b], cache.k, cache.k, group.block_table,
                             ctx.token_seq[a:b], ctx.positions[a:b], n, 1, self.width, self.window, self.scale,
@@ -147,15 +172,26 @@ class LatentAttention(Mixer):
 
     def _dense(self, q, o, start: int, table: torch.Tensor, cache: LayerCache, ctx: StepContext) -> None:
         m, n, kr = q.shape[0], self.heads, self.kv_rank
-        rows = ops.gather_rows(cache.k, table, start + m, ctx.error_flag)            # [context, width]
-        slab = max(1, min(m, SCORE_BYTES // (4 * n * (start + m))))
-        for t0 in range(0, m, slab):
-            t1 = min(m, t0 + slab)
-            keys = start + t1                                                          # the last query of the slab sees these
-            scores = torch.mm(q[t0:t1].view((t1 - t0) * n, self.width), rows[:keys].t(), out_dtype=torch.float32)
+        end, w = start + m, self.window
+        first_seen = 0 if w is None else max(0, start + 1 - w)       # of the portion's first token
+        # the library's products want rows of 16 bytes: the matrix starts and ends at multiples of eight positions (zero
+        # rows where no token of the portion sees, which the softmax leaves out)
+        base = first_seen // 8 * 8
+        rows = ops.gather_rows(cache.k, table, -(-end // 8) * 8 - base, ctx.error_flag, first=base, valid=(first_seen, end))
+        # a window: short slabs, so that few of a slab's products fall outside its tokens' windows
+        most = m if w is None else max(64, -(-w // 256) * 64)
+        t0 = 0
+        while t0 < m:
+            lo = 0 if w is None else max(0, start + t0 + 1 - w) // 8 * 8       # the first row that the slab's first token sees
+            keys = end - lo if w is None else min(end - lo, w + most + 8)
+            t1 = min(m, t0 + max(1, min(most, SCORE_BYTES // (4 * n * keys))))
+            hi = -(-(start + t1) // 8) * 8                                     # behind the last row that its last token sees
+            part = rows[lo - base:hi - base]
+            scores = torch.mm(q[t0:t1].view((t1 - t0) * n, self.width), part.t(), out_dtype=torch.float32)
             probs = torch.empty(scores.shape, dtype=q.dtype, device=q.device)
-            ops.causal_softmax_rows(scores, probs, n, start + t0, self.scale)
-            torch.mm(probs, rows[:keys, :kr], out=o[t0:t1].view((t1 - t0) * n, kr))
+            ops.causal_softmax_rows(scores, probs, n, start + t0, self.scale, first_key=lo, window=w)
+            torch.mm(probs, part[:, :kr], out=o[t0:t1].view((t1 - t0) * n, kr))
+            t0 = t1
 
 
 #: The tensor-core decode kernel leaves one share per token, head and 64 rows of the longest context the step allows;

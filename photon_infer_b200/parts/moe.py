@@ -21,6 +21,10 @@ over their sum times ``route_scale``.  ``shared_gate``: the shared expert's outp
 ``sigmoid(W_sg h)``, one number per token (``shared.sg [1, H]``), computed with the router's logits in 32-bit.
 ``scoring`` ``sigmoid``: scores are ``sigmoid(logit)``, each expert by itself; a group's score is the sum of its two largest
 scores; the weights are the chosen scores times ``route_scale``, not divided by their sum.
+``weight_input``: the weight multiplies the expert's input instead of its output, ``sum_j expert_j(w_j h)``; the first
+products are linear, so their 32-bit sums are scaled in the epilogue (or by the gated unit's kernel) and the outputs are
+added as they are.  ``activation`` ``clamped_swish`` (gated experts): ``g = min(W_gate x, act_limit)``,
+``u = clamp(W_up x, -act_limit, act_limit)``, and the unit is ``g sigmoid(act_slope g) (u + 1)``.
 """
 from __future__ import annotations
 
@@ -44,11 +48,19 @@ class MoEFeedForward(FeedForward):
     def __init__(self, hidden_size: int, experts: int, top: int, expert_size: int, shared_size: Optional[int] = None,
                  activation: str = "silu", shared_activation: Optional[str] = None, gated: bool = True,
                  router_bias: bool = True, scoring: str = "softmax_chosen", groups: int = 1, keep_groups: Optional[int] = None,
-                 route_scale: float = 1.0, shared_gate: bool = False):
+                 route_scale: float = 1.0, shared_gate: bool = False, weight_input: bool = False, act_limit: Optional[float] = None,
+                 act_slope: float = 1.0):
         if not 1 <= top <= experts:
             raise ValueError("a token uses between one and all of the experts")
-        if activation not in ops.ACTIVATIONS:
+        if activation not in ops.ACTIVATIONS and activation not in ops.GATED_ACTIVATIONS:
             raise ValueError(f"unknown activation {activation!r}")
+        self.weight_input = bool(weight_input)
+        self.own_unit = self.weight_input or activation in ops.GATED_ACTIVATIONS   # the unit that the dense kernels lack
+        if self.own_unit and not gated:
+            raise ValueError("input weights and activations of gated units need gated experts")
+        if activation in ops.GATED_ACTIVATIONS and (shared_size or act_limit is None or not act_limit > 0):
+            raise ValueError(f"{activation} needs a positive act_limit and is not an activation of the shared expert")
+        self.act_limit, self.act_slope = float(act_limit or 0.0), float(act_slope)
         self.hidden_size, self.experts, self.top = hidden_size, experts, top
         self.expert_size, self.shared_size = expert_size, shared_size
         self.activation = activation
@@ -135,15 +147,18 @@ class MoEFeedForward(FeedForward):
         glu, act_name = self.gated, self.activation
         out = torch.empty((T, H), dtype=h.dtype, device=h.device)
 
+        # factors on the experts' inputs, and the constants of the gated unit
+        unit = dict(limit=self.act_limit, slope=self.act_slope, weights=weights.view(-1) if self.weight_input else None)
+
         def combine(y, place):
             if shared_done is not None:
                 torch.cuda.current_stream().wait_event(shared_done)      # the shared expert's rows are there
-            ops.moe_combine(y, place, weights, shared, out, sgate)
+            ops.moe_combine(y, place, None if self.weight_input else weights, shared, out, sgate)
 
         if n <= GEMV_MAX_PAIRS and ops.moe_gemv_supported(h, self.w_gate_up) and self.expert_size % 8 == 0:
             # a decode step: nothing is sorted, every pair streams its expert's matrices once
             act = torch.empty((n, self.expert_size), dtype=h.dtype, device=h.device)
-            ops.moe_gemv(h, self.top, ids, self.w_gate_up, act, glu=glu, activation=act_name)
+            ops.moe_gemv(h, self.top, ids, self.w_gate_up, act, glu=glu, activation=act_name, **unit)
             y = torch.empty((n, H), dtype=torch.float32, device=h.device)
             ops.moe_gemv(act, 1, ids, self.w_down, y)
             combine(y, None)
@@ -155,14 +170,18 @@ class MoEFeedForward(FeedForward):
             gate_up = torch._grouped_mm(xs, self.w_gate_up.transpose(1, 2), offs=offsets[1:])
             if glu:
                 act = torch.empty((n, self.expert_size), dtype=h.dtype, device=h.device)
-                ops.swiglu(gate_up, act, act_name)
+                if self.own_unit:
+                    ops.moe_glu(gate_up, act, act_name, srt=srt, **unit)
+                else:
+                    ops.swiglu(gate_up, act, act_name)
             else:
                 act = ops.activation(gate_up, act_name)
             y = torch._grouped_mm(act, self.w_down.transpose(1, 2), offs=offsets[1:])
             combine(y, place)
             return out
         act = torch.empty((n, self.expert_size), dtype=h.dtype, device=h.device)
-        ops.moe_gemm(h, srt, self.top, self.w_gate_up, act, tiles, num_tiles, max_tiles, glu=glu, activation=act_name)
+        ops.moe_gemm(h, srt, self.top, self.w_gate_up, act, tiles, num_tiles, max_tiles, glu=glu, activation=act_name,
+                     **unit)
         y = torch.empty((n, H), dtype=torch.float32, device=h.device)
         ops.moe_gemm(act, None, 1, self.w_down, y, tiles, num_tiles, max_tiles)
         combine(y, place)

@@ -9,8 +9,27 @@ from typing import Dict, List, Optional
 import torch
 
 from ..kernels import ops
-from .base import ChannelScalePart, Norm, Normed, TensorSpec, delta_pair, delta_terms
+from .base import ChannelScalePart, Connected, Norm, Normed, TensorSpec, delta_pair, delta_terms
 from .registry import register_norm, register_scale
+
+
+def _read_streams(norm, center: bool, delta: Optional[Connected], streams: torch.Tensor, w_in, out_dtype, rows):
+    """``Norm.read_streams`` in one kernel: the pending write, the read and the norm."""
+    T, H = streams.shape[0], streams.shape[-1]
+    n = rows.numel() if rows is not None else T
+    out = torch.empty((n, H), dtype=out_dtype, device=streams.device)
+    bias = getattr(norm, "bias", None)
+    if delta is None:
+        count = streams.shape[1] if streams.dim() == 3 else w_in.numel()
+        ops.stream_norm(streams, count, None, None, None, w_in, norm.weight, bias, norm.eps, out, center=center, rows=rows)
+        return out, streams
+    c = delta.connection
+    new = None
+    if rows is None:
+        new = streams if streams.dim() == 3 else torch.empty((T, c.streams, H), dtype=torch.float32, device=streams.device)
+    ops.stream_norm(streams, c.streams, delta.tensor, c.mix, c.w_out, w_in, norm.weight, bias, norm.eps, out, center=center,
+                    new_streams=new, rows=rows)
+    return out, streams if new is None else new
 
 
 class RMSNorm(Norm):
@@ -43,7 +62,12 @@ class RMSNorm(Norm):
         ops.add_rmsnorm(d1, residual, self.weight, self.eps, out, delta2=d2, delta_scale=sc)
         return out
 
+    def read_streams(self, delta, streams, w_in, out_dtype, rows=None):
+        return _read_streams(self, False, delta, streams, w_in, out_dtype, rows)
+
     def add_forward_rows(self, delta, residual, rows, out_dtype):
+        if isinstance(delta, Connected):
+            return self.read_streams(delta, residual, None, out_dtype, rows)[0]
         out = torch.empty((rows.numel(), residual.shape[1]), dtype=out_dtype, device=residual.device)
         d1, d2, sc = delta_terms(delta)
         ops.add_rmsnorm(d1, residual, self.weight, self.eps, out, rows=rows, delta2=d2, delta_scale=sc)
@@ -84,7 +108,12 @@ class LayerNorm(Norm):
         ops.add_layernorm(d1, residual, self.weight, self.bias, self.eps, out, delta2=d2, delta_scale=sc)
         return out
 
+    def read_streams(self, delta, streams, w_in, out_dtype, rows=None):
+        return _read_streams(self, True, delta, streams, w_in, out_dtype, rows)
+
     def add_forward_rows(self, delta, residual, rows, out_dtype):
+        if isinstance(delta, Connected):
+            return self.read_streams(delta, residual, None, out_dtype, rows)[0]
         out = torch.empty((rows.numel(), residual.shape[1]), dtype=out_dtype, device=residual.device)
         d1, d2, sc = delta_terms(delta)
         ops.add_layernorm(d1, residual, self.weight, self.bias, self.eps, out, rows=rows, delta2=d2, delta_scale=sc)

@@ -18,9 +18,11 @@ POSITION_ENCODINGS: Dict[str, Callable] = {}
 BLOCKS: Dict[str, Callable] = {}
 STREAM_PARTS: Dict[str, Callable] = {}
 SCALES: Dict[str, Callable] = {}
+CONNECTIONS: Dict[str, Callable] = {}
 
 _TABLES = {"norm": NORMS, "mixer": MIXERS, "feed_forward": FEED_FORWARDS,
-           "position_encoding": POSITION_ENCODINGS, "block": BLOCKS, "stream": STREAM_PARTS, "scale": SCALES}
+           "position_encoding": POSITION_ENCODINGS, "block": BLOCKS, "stream": STREAM_PARTS, "scale": SCALES,
+           "connection": CONNECTIONS}
 
 
 def _register(table_name: str, kind: str, factory: Callable, replace: bool) -> None:
@@ -36,6 +38,7 @@ def register_feed_forward(kind, factory, replace=False): _register("feed_forward
 def register_position_encoding(kind, factory, replace=False): _register("position_encoding", kind, factory, replace)
 def register_block(kind, factory, replace=False): _register("block", kind, factory, replace)
 def register_stream_part(kind, factory, replace=False): _register("stream", kind, factory, replace)
+def register_connection(kind, factory, replace=False): _register("connection", kind, factory, replace)
 def register_scale(kind, factory, replace=False): _register("scale", kind, factory, replace)
 
 
@@ -50,5 +53,5 @@ def create_part(table_name: str, kind: str, params: dict):
 
 
 def _ensure_builtin() -> None:
-    from . import (attention, block, delta_rule, diff_attention, gla, latent_attention, matrix_memory, mlp, moe,  # noqa: F401
+    from . import (attention, block, delta_rule, diff_attention, gla, hyper, latent_attention, matrix_memory, mlp, moe,  # noqa: F401
                    norm, normed_attention, rope, state_space, stream, talking_attention)                                       # (each registers itself)
