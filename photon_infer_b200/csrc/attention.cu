@@ -51,7 +51,8 @@ paged_attention_kernel(const T* __restrict__ q, long q_stride, T* __restrict__ o
   float* mrun = sc + hb * ATT_TILE;          // hb
   float* lsum = mrun + hb;                   // hb
   float* corr = lsum + hb;                   // hb
-  long long* kbase = (long long*)(corr + hb + ((hb & 1) ? 1 : 0));   // TILE (8-byte aligned)
+  long long* kbase = (long long*)(corr + hb + ((hb & 1) & ((d + 1) & 1)));   // TILE; 8-byte aligned: an odd number of floats
+                                                                            // (hb * (d + 3) of them, mod 2) gets one more
   if (shared_kv) vs = ks;
 
   const int p = positions[t];

@@ -29,7 +29,7 @@ class TensorSpec:
     and are held in the run dtype; ``"vector"`` tensors (norm weights) keep 32-bit
     storage when the file has it; ``"int"`` tensors are integer tables, held as int32.
     ``init`` tells the random-weights mode how to fill it: ``"normal"`` (N(0, std)),
-    ``"norm"`` (ones, or 1 + N(0, norm_std)), ``"zeros"``.
+    ``"norm"`` (ones, or 1 + N(0, norm_std)), ``"eye"`` (identity + N(0, std)), ``"zeros"``.
     A dimension of ``-1`` in ``shape`` is a size that the configuration does not give: the weight file decides it
     (the loader accepts any size there), and the random-weights mode uses ``free_size``.
     """

@@ -34,7 +34,7 @@ class HyperConnection(ConnectionPart):
         i, o, m = self.names
         S = self.streams
         return [TensorSpec(i, (S,), role="vector", init="norm"), TensorSpec(o, (S,), role="vector", init="norm"),
-                TensorSpec(m, (S, S), role="vector", init="normal")]
+                TensorSpec(m, (S, S), role="vector", init="eye")]
 
     def load(self, tensors: Dict[str, torch.Tensor]) -> None:
         self.w_in, self.w_out, self.mix = (tensors[n].to(torch.float32).contiguous() for n in self.names)

@@ -5,7 +5,7 @@ The reference draws N(0, 0.02) for every tensor, norms included, in its tests on
 (tests/model/test_llama_model.cpp:31-42).  Here each tensor has its own generator,
 seeded from (seed, tensor name), so the values of one tensor do not depend on which
 other tensors the model has; matrices are N(0, init_std), norm weights are ones or
-``1 + N(0, norm_std)``.  Values are rounded to the storage dtype (bfloat16 by
+``1 + N(0, norm_std)``, matrices that mix residual streams the identity plus N(0, init_std).  Values are rounded to the storage dtype (bfloat16 by
 default) before writing, so a float32 run and a bfloat16 run read the same numbers.
 """
 from __future__ import annotations
@@ -44,6 +44,8 @@ def random_tensor(spec: TensorSpec, name: str, seed: int, init_std: float, norm_
             t += norm_std * torch.randn(shape, generator=g, dtype=torch.float32)
     elif spec.init == "normal":
         t = init_std * torch.randn(shape, generator=g, dtype=torch.float32)
+    elif spec.init == "eye":
+        t = torch.eye(*shape, dtype=torch.float32) + init_std * torch.randn(shape, generator=g, dtype=torch.float32)
     else:
         raise PhotonError(ErrorCode.INVALID_ARGUMENT, f"tensor {name}: unknown init {spec.init!r}")
     return t.to(dtype)
@@ -100,6 +102,8 @@ def random_tensors_on_device(declared: Dict[str, TensorSpec], run_dtype: torch.d
                 t += norm_std * torch.randn(shape, generator=g, dtype=dtype, device=dev)
         elif spec.init == "normal":
             t = torch.empty(shape, dtype=dtype, device=dev).normal_(0.0, init_std, generator=g)
+        elif spec.init == "eye":
+            t = torch.empty(shape, dtype=dtype, device=dev).normal_(0.0, init_std, generator=g) + torch.eye(*shape, dtype=dtype, device=dev)
         else:
             raise PhotonError(ErrorCode.INVALID_ARGUMENT, f"tensor {name}: unknown init {spec.init!r}")
         out[name] = t

@@ -507,3 +507,90 @@ def pebodra_plain_logits(folder: str, ids: Sequence[int]) -> torch.Tensor:
         cfg, tensors = pebodra_plain_model(folder)
         _pebodra_cache[key] = pebodra_plain.forward(cfg, tensors, list(ids))
     return _pebodra_cache[key]
+
+
+# ----------------------------------------------------------------------------- Milozen
+
+def _zatt(heads, dim, rot_dim, vdim, kv_rank, q_rank, scale, size=None, base=10000.0, kv_from=None):
+    m = dict(heads=heads, dim=dim, rot_dim=rot_dim, vdim=vdim, kv_rank=kv_rank, q_rank=q_rank, scale=scale,
+             rot=dict(base=base, dims=rot_dim))
+    if size:
+        m["mask"] = dict(size=size)
+    if kv_from is not None:
+        m["kv_from"] = kv_from
+    return m
+
+
+def _zmoe(experts, top, ff, limit):
+    return dict(kind="moe", expert=dict(ff=ff, limit=limit), router=dict(experts=experts, top=top))
+
+
+_zlayer = lambda mixer, mlp: dict(type="latent_attention", mixer=mixer, mlp=mlp)
+
+# Tiny Milozen configurations that differ in every size, in the order of the layers and in which optional pieces they
+# have.  Windows are short, so that prompts and decoded tokens alike pass their edges many times.
+TINY_MILOZEN: Dict[str, dict] = {
+    # two streams; a reader with another number of heads, other sizes and a LONGER window than the layer it reads; a layer
+    # without feed-forward
+    "mz_a": dict(
+        config=dict(architecture="Milozen", vocab=150, width=64, streams=2, embedding=dict(scale=4.0), norm=dict(eps=1e-5),
+                    layers=[_zlayer(_zatt(3, 16, 8, 20, 24, 40, 0.3, 40, 5000.0), _zmoe(6, 2, 32, 0.8)),
+                            _zlayer(_zatt(2, 24, 12, 16, 36, 24, 0.25, 17, 100.0), dict(kind="dense", ff=96)),
+                            _zlayer(_zatt(5, 12, 8, 24, 24, 16, 0.2, 56, 5000.0, kv_from=0), None),
+                            _zlayer(_zatt(3, 16, 8, 12, 24, 32, 0.4, 9, 5000.0, kv_from=0), _zmoe(4, 1, 48, 2.0))]),
+        seed=51, init_std=0.1, norm_std=0.1, block_size=16),
+    # four streams; rows and values of 16s (tensor-core decoding in bfloat16) with a window and without; pages of 8
+    "mz_b": dict(
+        config=dict(architecture="Milozen", vocab=210, width=96, streams=4, embedding=dict(scale=1.0), norm=dict(eps=1e-6),
+                    layers=[_zlayer(_zatt(4, 32, 16, 32, 48, 64, 0.2, 70), dict(kind="dense", ff=40)),
+                            _zlayer(_zatt(2, 16, 32, 16, 64, 48, 0.3), _zmoe(8, 3, 24, 1.0)),
+                            _zlayer(_zatt(18, 8, 32, 8, 64, 32, 0.25, 33, kv_from=1), _zmoe(5, 5, 16, 0.5))]),
+        seed=52, init_std=0.08, norm_std=0.15, block_size=8),
+    # sizes that are multiples of nothing; five streams; a window of three keys and of one key; a single head
+    "mz_c": dict(
+        config=dict(architecture="Milozen", vocab=77, width=50, streams=5, embedding=dict(scale=7.5), norm=dict(eps=2e-5),
+                    layers=[_zlayer(_zatt(5, 7, 6, 9, 13, 11, 0.4, 3, 50.0), _zmoe(7, 3, 14, 0.7)),
+                            _zlayer(_zatt(1, 10, 6, 14, 13, 26, 0.3, 37, 50.0, kv_from=0), None),
+                            _zlayer(_zatt(3, 6, 2, 5, 22, 9, 0.5, 1, 1e6), dict(kind="dense", ff=30))]),
+        seed=53, init_std=0.12, norm_std=0.05, block_size=16),
+    # one stream; a latent as wide as a large model's row; a window longer than most requests; pages of 32
+    "mz_d": dict(
+        config=dict(architecture="Milozen", vocab=90, width=32, streams=1, embedding=dict(scale=2.0), norm=dict(eps=1e-5),
+                    layers=[_zlayer(_zatt(2, 64, 64, 128, 256, 24, 0.09, 100, 300000.0), _zmoe(2, 2, 16, 1.5)),
+                            _zlayer(_zatt(4, 8, 64, 16, 256, 96, 0.1, 160, 300000.0, kv_from=0), dict(kind="dense", ff=48))]),
+        seed=54, init_std=0.15, norm_std=0.1, block_size=32),
+    # three streams; two readers, one of them without a window (so everything is kept); more experts than a warp has lanes
+    "mz_e": dict(
+        config=dict(architecture="Milozen", vocab=131, width=48, streams=3, embedding=dict(scale=0.5), norm=dict(eps=1e-5),
+                    layers=[_zlayer(_zatt(2, 16, 16, 24, 32, 20, 0.2, 24, 777.0), _zmoe(40, 2, 8, 3.0)),
+                            _zlayer(_zatt(3, 20, 16, 8, 32, 28, 0.3, None, 777.0, kv_from=0), dict(kind="dense", ff=72)),
+                            _zlayer(_zatt(2, 24, 16, 16, 32, 12, 0.25, 8, 777.0, kv_from=0), _zmoe(3, 1, 36, 0.3))]),
+        seed=55, init_std=0.1, norm_std=0.1, block_size=16),
+}
+
+
+def make_milozen_folder(path: str, name: str, dtype: str = "bfloat16") -> str:
+    from photon_infer_b200.weights import write_random_model
+    t = TINY_MILOZEN[name]
+    write_random_model(path, t["config"], seed=t["seed"], init_std=t["init_std"], norm_std=t["norm_std"], dtype=dtype)
+    return path
+
+
+_milozen_cache: Dict[tuple, torch.Tensor] = {}
+_milozen_models: Dict[str, tuple] = {}
+
+
+def milozen_plain_model(folder: str):
+    from plain import milozen_plain
+    if folder not in _milozen_models:
+        _milozen_models[folder] = milozen_plain.read_folder(folder)
+    return _milozen_models[folder]
+
+
+def milozen_plain_logits(folder: str, ids: Sequence[int]) -> torch.Tensor:
+    from plain import milozen_plain
+    key = (folder, tuple(ids))
+    if key not in _milozen_cache:
+        cfg, tensors = milozen_plain_model(folder)
+        _milozen_cache[key] = milozen_plain.forward(cfg, tensors, list(ids))
+    return _milozen_cache[key]
