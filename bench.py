@@ -378,7 +378,7 @@ def main() -> int:
     ap.add_argument("--layers-3b", type=int, default=0, help="fewer layers for the 3B workload (0: all 28)")
     ap.add_argument("--layers-8b", type=int, default=0, help="fewer layers for the 8B workload (0: all 32)")
     ap.add_argument("--batch-8b", type=int, default=8)
-    ap.add_argument("--design", default=None, choices=["finelix", "fekopel", "lerosun", "pebodra"],
+    ap.add_argument("--design", default=None, choices=["finelix", "fekopel", "lerosun", "pebodra", "milozen"],
                     help="compare this design with a Llama decoder of equal size instead of running the headline")
     ap.add_argument("--design-sizes", default="2048,4096", help="widths to run with --design")
     args = ap.parse_args()

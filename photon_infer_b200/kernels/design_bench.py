@@ -1,8 +1,8 @@
-"""Prefill and decode throughput of another design (the Finelix, the Fekopel, the Lerosun or the Pebodra decoder) beside
-a Llama decoder of equal width, depth and feed-forward size (``python bench.py --design finelix|fekopel|lerosun|pebodra``),
-with the parts of a layer timed alone against their rooflines.  The Lerosun and the Pebodra decoder also run beside the
-Finelix decoder, the other design with a recurrent mixer (a matrix of state per head) and routed experts next to
-attention.
+"""Prefill and decode throughput of another design (the Finelix, the Fekopel, the Lerosun, the Pebodra or the Milozen
+decoder) beside a Llama decoder of equal width, depth and feed-forward size (``python bench.py --design
+finelix|fekopel|lerosun|pebodra|milozen``), with the parts of a layer timed alone against their rooflines.  The Lerosun and
+the Pebodra decoder also run beside the Finelix decoder, the other design with a recurrent mixer (a matrix of state per
+head) and routed experts next to attention, and so does the Milozen decoder, which shares latent attention with it.
 
 Random weights drawn on the device, synthetic token ids, bfloat16.  Per size:
 
@@ -12,7 +12,9 @@ Random weights drawn on the device, synthetic token ids, bfloat16.  Per size:
   events around the call; decode rows as a CUDA graph of the part alone, a buffer larger than L2 written before
   every replay.  ``frac`` is the part's share of its roofline: for decode rows the bytes it must move (the
   weights it reads, the cache rows or state it reads and writes) over the measured copy bandwidth; for prefill rows
-  its arithmetic (the products and the attention or recurrence) over the measured bfloat16 tensor throughput.
+  its arithmetic (the products and the attention or recurrence) over the measured bfloat16 tensor throughput.  ``norm`` and
+  ``streams`` (the residual sum with the norm behind it; the same with several residual streams, which are mixed) are
+  bound by memory in both phases, and their prefill rows are timed with L2 written over as well.
 """
 from __future__ import annotations
 
@@ -101,6 +103,23 @@ def pebodra_config(width: int, layers: int) -> dict:
                 layers=[kinds[i % 4](i) for i in range(layers)])
 
 
+MILOZEN_WINDOW = 1024
+
+
+def milozen_config(width: int, layers: int) -> dict:
+    """Latent attention in every layer with the Finelix sizes (heads of 128 + 64, a latent of 512 + 64), a window of 1,024 and
+    an output gate; every other layer reads the rows of the layer before it.  Four residual streams.  Dense feed-forwards
+    of 4 x width alternate with 16 experts of 2 x width, 2 per token."""
+    heads = width // 128
+    att = lambda extra: dict(heads=heads, dim=128, rot_dim=64, vdim=128, kv_rank=512, q_rank=max(768, width * 3 // 8),
+                             scale=192 ** -0.5, rot=dict(base=10000.0, dims=64), mask=dict(size=MILOZEN_WINDOW), **extra)
+    dense = dict(kind="dense", ff=4 * width)
+    moe = dict(kind="moe", router=dict(experts=16, top=2), expert=dict(ff=2 * width, limit=7.0))
+    return dict(architecture="Milozen", vocab=32000, width=width, streams=4, embedding=dict(scale=1.0), norm=dict(eps=1e-5),
+                layers=[dict(type="latent_attention", mixer=att(dict(kv_from=i - 1) if i % 2 else {}), mlp=moe if i % 2 else dense)
+                        for i in range(layers)])
+
+
 def llama_config(width: int, layers: int, window=None) -> dict:
     cfg = dict(architectures=["LlamaForCausalLM"], hidden_size=width, intermediate_size=4 * width, num_hidden_layers=layers,
                num_attention_heads=width // 128, num_key_value_heads=max(1, width // 512), head_dim=128, vocab_size=32000,
@@ -110,11 +129,14 @@ def llama_config(width: int, layers: int, window=None) -> dict:
     return cfg
 
 
-def _time_events(fn, reps: int = 3) -> float:
+def _time_events(fn, reps: int = 3, flush: bool = False) -> float:
+    """Microseconds of ``fn()``, the best of ``reps``; ``flush``: L2 is written over before each."""
     fn()
     torch.cuda.synchronize()
     best = float("inf")
     for _ in range(reps):
+        if flush:
+            _flush_buffer().zero_()
         e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
         e0.record()
         fn()
@@ -127,11 +149,15 @@ def _time_events(fn, reps: int = 3) -> float:
 _flush = None
 
 
-def _time_graph(fn, reps: int = 8) -> float:
-    """Microseconds of ``fn()`` replayed as a CUDA graph, with L2 written over before every replay."""
+def _flush_buffer() -> torch.Tensor:
     global _flush
     if _flush is None:
         _flush = torch.empty(256 << 20, dtype=torch.uint8, device="cuda")
+    return _flush
+
+
+def _time_graph(fn, reps: int = 8) -> float:
+    """Microseconds of ``fn()`` replayed as a CUDA graph, with L2 written over before every replay."""
     side = torch.cuda.Stream()
     with torch.cuda.stream(side):
         fn()
@@ -141,7 +167,7 @@ def _time_graph(fn, reps: int = 8) -> float:
         fn()
     times = []
     for _ in range(reps):
-        _flush.zero_()
+        _flush_buffer().zero_()
         e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
         e0.record()
         g.replay()
@@ -196,9 +222,9 @@ def _mixer_numbers(m, kind: str, tokens: int, contexts) -> tuple:
         dv = getattr(m, "value_dim", m.head_dim)
         mix = 2 * m.n_q * m.n_q * pairs if kind == "talking" and m.talk else 0       # every head's score from all heads'
         return held * m.n_kv * (m.head_dim + dv) * 2, tokens * (w // 2) * 2 + 2 * m.n_q * (m.head_dim + dv) * pairs + mix
-    pairs = sum(c * (c + 1) // 2 for c in contexts) if tokens > len(contexts) else sum(contexts)
     if kind == "latent":
-        rows = sum(contexts) * m.width * 2
+        pairs = sum(sum(seen_by(p) for p in range(c)) for c in contexts) if tokens > len(contexts) else sum(seen_by(c - 1) for c in contexts)
+        rows = sum(seen_by(c - 1) for c in contexts) * m.width * 2
         flops = tokens * (w // 2) * 2 + 2 * m.heads * (m.width + m.kv_rank) * pairs
         return rows, flops
     raise ValueError(kind)
@@ -245,6 +271,8 @@ def _parts(runner, hbm_peak: float, tf_peak: float) -> Dict[str, dict]:
                     DifferentialAttention: "diff", StateSpaceMixer: "ssm", MatrixMemoryMixer: "memory"}.get(type(m))
             if kind == "normed":                     # the two kinds of layer are timed apart
                 kind_name = "normed_gated" if m.output_gate else "normed_sink"
+            elif kind == "latent":                   # a layer with a latent of its own, and one that reads another's rows
+                kind_name = "latent" if m.own_kv else "latent_reader"
             elif kind == "diff":                     # a layer that owns its keys and values, and one that reads another's
                 kind_name = "diff" if m.own_kv else "diff_reader"
             else:
@@ -254,6 +282,22 @@ def _parts(runner, hbm_peak: float, tf_peak: float) -> Dict[str, dict]:
             if fkind == "dense" and not hasattr(ff, "w_gate_up"):
                 fkind = "polynorm"
             lc = runner._layer_caches[i]
+            streams = getattr(block, "connect1", None)
+            norm_name = "norm" if streams is None else "streams"
+            if (norm_name, phase) not in seen and hasattr(block, "norm2") and not model.spec.layers[e.layer].block.kind == "output_norm":
+                seen.add((norm_name, phase))
+                y = torch.randn(T, H, device=model.device).to(model.dtype)
+                if streams is None:
+                    x = torch.randn(T, H, device=model.device)
+                    step = lambda: block.norm1.add_forward(y, x, model.dtype)
+                    moved = T * H * (2 * 4 + 2 * 2)
+                else:
+                    from ..parts.base import Connected
+                    x = torch.randn(T, streams.streams, H, device=model.device)
+                    step = lambda: block.norm1.read_streams(Connected(y, streams), x, streams.w_in, model.dtype)
+                    moved = T * H * (2 * 4 * streams.streams + 2 * 2)
+                us = _time_events(step, 5, flush=True) if phase == "prefill" else _time_graph(step)
+                out[f"{norm_name}.{phase}"] = {"us": round(us, 1), "frac": round(moved / (us * 1e-6) / (hbm_peak * 1e9), 4)}
             if kind and (kind_name, phase) not in seen:
                 seen.add((kind_name, phase))
                 us = timer(lambda: m.forward(h, ctx, lc))
@@ -326,7 +370,8 @@ def run_design_comparison(design: str, args, hbm_peak: float, tf_peak: float, pe
     steps, warmup = max(8, min(args.steps, 64)), max(args.warmup, 3)
     layers = {2048: 8, 4096: 4}
     make, window = {"finelix": (finelix_config, None), "fekopel": (fekopel_config, FEKOPEL_WINDOW),
-                    "lerosun": (lerosun_config, LEROSUN_WINDOW), "pebodra": (pebodra_config, PEBODRA_WINDOW)}[design]
+                    "lerosun": (lerosun_config, LEROSUN_WINDOW), "pebodra": (pebodra_config, PEBODRA_WINDOW),
+                    "milozen": (milozen_config, MILOZEN_WINDOW)}[design]
     line = {"design": design, "dtype": args.dtype, "data": "synthetic", "peaks": peak_src,
             "workload": {"prefill_tokens": PREFILL, "decode_batch": BATCH, "decode_context": PROMPT, "steps": steps,
                          "warmup": warmup}, "sizes": {}}
@@ -334,7 +379,7 @@ def run_design_comparison(design: str, args, hbm_peak: float, tf_peak: float, pe
         n_layers = layers.get(width, 4)
         point = {"layers": n_layers}
         models = [(design, make(width, n_layers)), ("llama", llama_config(width, n_layers, window))]
-        if design in ("lerosun", "pebodra"):
+        if design in ("lerosun", "pebodra", "milozen"):
             models.append(("finelix", finelix_config(width, n_layers)))
         for name, cfg in models:
             print(f"[bench] {name} width {width}, {n_layers} layers", file=sys.stderr, flush=True)
