@@ -184,7 +184,8 @@ DEFAULT_SPECIALISATIONS = (("attention_flash", {"HEAD_DIM": 64}), ("attention_tc
                            ("attention_decode", {"HEAD_DIM": 64}), ("attention_flash", {"HEAD_DIM": 128}),
                            ("attention_tc", {"HEAD_DIM": 128}), ("attention_decode", {"HEAD_DIM": 128}),
                            ("attention_talk_mma", {"HEAD_DIM": 128, "TALK_H": 16, "TALK_G": 2}),
-                           ("attention_diff_mma", {"DIFF_D": 128, "DIFF_DV": 256}))
+                           ("attention_diff_mma", {"DIFF_D": 128, "DIFF_DV": 256}),
+                           ("attention_latent_tc", {"LT_NU": 2, "LT_NR": 1, "LT_NV": 2}))
 
 
 def build_all(verbose: bool = False) -> None:

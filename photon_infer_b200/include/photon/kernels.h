@@ -173,6 +173,19 @@ PHOTON_EXPORT int photon_latent_decode_attention(const void* q, long q_stride, c
                                    int dv, int page_size, int num_pages, float scale, int window, int splits, float* part,
                                    void* out, long out_stride, int* err, cudaStream_t stream);
 
+/* ------------------------------------------------------------------ attention_latent_tc.cu (-DLT_NU=, -DLT_NR=, -DLT_NV=: 64-wide
+ * chunks of d, r, v; bfloat16): long prompt portions over an expanded latent */
+/* q [T][heads][d + r] (the unrotated parts), q_rot [T][heads][r], kv [rows][>= heads * (d + v)]: heads x d key numbers then
+ * heads x v value numbers per row, rot_rows [rows][r]: the key part all heads share; out [T][heads * v], times sigmoid(gate)
+ * where gate is not null.  seqs (host): S x (first token, tokens, position of the first token, position of the request's
+ * first row, that row).  d, r, v multiples of 8, everything 16-byte aligned. */
+PHOTON_EXPORT int photon_attention_latent_tc_chunks(void);
+PHOTON_EXPORT int photon_attention_latent_tc_max_seqs(void);
+PHOTON_EXPORT int photon_attention_latent_tc(const void* q, long q_stride, const void* q_rot, const void* kv, long kv_stride,
+                               const void* rot_rows, long rot_stride, void* out, long out_stride, const void* gate,
+                               long gate_stride, const int* seqs, int S, int T, int rows, int heads, int d, int r, int v,
+                               int window, float scale, int* err, cudaStream_t stream);
+
 /* ------------------------------------------------------------------ hyper.cu: parallel residual streams */
 /* out [n][H] = norm(u) * w + bias, u = sum_s win[s] X_s (win null: the sum), after the pending write
  * X_t <- sum_s mix[s][t] X_s + wout[t] y (y null: none) into dst [*][S][H] (may be src, may be null).  Streams of token t

@@ -225,7 +225,9 @@ def _mixer_numbers(m, kind: str, tokens: int, contexts) -> tuple:
     if kind == "latent":
         pairs = sum(sum(seen_by(p) for p in range(c)) for c in contexts) if tokens > len(contexts) else sum(seen_by(c - 1) for c in contexts)
         rows = sum(seen_by(c - 1) for c in contexts) * m.width * 2
-        flops = tokens * (w // 2) * 2 + 2 * m.heads * (m.width + m.kv_rank) * pairs
+        # attention to the latents themselves (decoded tokens), or with heads whose keys and values were formed from them (prompts)
+        per_pair = min(m.width + m.kv_rank, m.dim + m.rot_dim + m.vdim)
+        flops = tokens * (w // 2) * 2 + 2 * m.heads * per_pair * pairs
         return rows, flops
     raise ValueError(kind)
 

@@ -1126,7 +1126,7 @@ def head_linear(x: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, gate: 
 
 
 def gather_rows(cache: torch.Tensor, table: torch.Tensor, count: int, err: Optional[torch.Tensor], first: int = 0,
-                valid=None) -> torch.Tensor:
+                valid=None, out: Optional[torch.Tensor] = None) -> torch.Tensor:
     """``count`` cached rows from position ``first`` on of the request whose pages are ``table`` (one row of a block
     table), as one dense matrix ``[count, width]``; ``cache [pages, 1, page_size, width]``.  ``valid`` ``(lo, hi)``:
     positions outside give zero rows."""
@@ -1136,12 +1136,54 @@ def gather_rows(cache: torch.Tensor, table: torch.Tensor, count: int, err: Optio
     lo, hi = valid if valid is not None else (first, first + count)
     if hi > table.numel() * page_size or min(first, lo) < 0 or not cache.is_contiguous():
         raise PhotonError(ErrorCode.INVALID_ARGUMENT, "gather_rows: more rows asked for than the table's pages hold")
-    out = torch.empty((count, width), dtype=cache.dtype, device=cache.device)
+    if out is None:
+        out = torch.empty((count, width), dtype=cache.dtype, device=cache.device)
+    elif out.shape != (count, width) or out.dtype != cache.dtype or not out.is_contiguous():
+        raise PhotonError(ErrorCode.SHAPE_MISMATCH, "gather_rows: out must be contiguous [count, width] of the cache's type")
     f = _fn("latent", "photon_gather_rows", [c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p,
                                              c_void_p, c_void_p])
     _check(f(_ptr(cache), _dtype_code(cache), _ptr(table), page_size, pages, width, int(first), int(count), int(lo), int(hi),
              _ptr(out), _ptr(err), _stream()), "gather_rows")
     return out
+
+
+def latent_prompt_defines(dtype: torch.dtype, d: int, r: int, v: int, kv_rank: int):
+    """The definitions that the tensor-core kernel for long portions over an expanded latent is compiled with, or None for
+    sizes it does not take: bfloat16, sizes that are multiples of 8, keys of at most four 64-wide chunks, values of two."""
+    nu, nr, nv = -(-d // 64), -(-r // 64), -(-v // 64)
+    if dtype != torch.bfloat16 or d % 8 or r % 8 or v % 8 or kv_rank % 8 or nu + nr > 4 or nv > 2:
+        return None
+    return {"LT_NU": nu, "LT_NR": nr, "LT_NV": nv}
+
+
+def latent_prompt_attention(q: torch.Tensor, q_rot: torch.Tensor, kv: torch.Tensor, rot_rows: torch.Tensor, out: torch.Tensor,
+                            seqs, heads: int, d: int, r: int, v: int, window: Optional[int], scale: float,
+                            err: Optional[torch.Tensor], gate: Optional[torch.Tensor] = None) -> None:
+    """Attention of long prompt portions over an expanded latent on the tcgen05 tensor cores.  ``q [T, heads * (d + r)]`` (its
+    unrotated parts are read), ``q_rot [T, heads, r]``; ``kv [rows, heads * (d + v)]``: the heads' keys, then their values;
+    ``rot_rows [rows, r]`` (a view): the key part that all heads share.  ``seqs``: per request ``(first token, tokens, position
+    of the first token, position of its first row, that row)``.  ``out [T, heads * v]`` gets the rows of those tokens, times
+    ``sigmoid(gate)`` when a gate is given."""
+    _cuda(q, q_rot, kv, rot_rows, out, err, gate)
+    T, rows = q.shape[0], kv.shape[0]
+    defines = latent_prompt_defines(q.dtype, d, r, v, 8)
+    if defines is None:
+        raise PhotonError(ErrorCode.UNSUPPORTED_SIZE, f"latent_prompt_attention: heads of {d} + {r} and {v} in {q.dtype}")
+    if q.shape[1] != heads * (d + r) or q.stride(1) != 1 or q_rot.shape != (T, heads, r) or not q_rot.is_contiguous() \
+            or kv.shape[1] != heads * (d + v) or kv.stride(1) != 1 or rot_rows.shape != (rows, r) or rot_rows.stride(1) != 1 \
+            or out.shape != (T, heads * v) or out.stride(1) != 1 \
+            or any(t.dtype != torch.bfloat16 for t in (q_rot, kv, rot_rows, out)):
+        raise PhotonError(ErrorCode.SHAPE_MISMATCH, "latent_prompt_attention: q [T, heads * (d + r)], kv [rows, heads * (d + v)], all bfloat16")
+    if gate is not None and (gate.shape != (T, heads * v) or gate.stride(1) != 1 or gate.dtype != torch.bfloat16):
+        raise PhotonError(ErrorCode.SHAPE_MISMATCH, "latent_prompt_attention: gate [T, heads * v] bfloat16")
+    flat = [int(x) for s in seqs for x in s]
+    host = (ctypes.c_int * len(flat))(*flat)
+    f = _fn("attention_latent_tc", "photon_attention_latent_tc",
+            [c_void_p, c_long, c_void_p, c_void_p, c_long, c_void_p, c_long, c_void_p, c_long, c_void_p, c_long, c_void_p, c_int,
+             c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_void_p, c_void_p], defines=defines)
+    _check(f(_ptr(q), q.stride(0), _ptr(q_rot), _ptr(kv), kv.stride(0), _ptr(rot_rows), rot_rows.stride(0), _ptr(out), out.stride(0),
+             _ptr(gate), gate.stride(0) if gate is not None else 0, ctypes.cast(host, c_void_p), len(flat) // 5, T, rows, heads, d, r,
+             v, int(window or 0), float(scale), _ptr(err), _stream()), "latent_prompt_attention")
 
 
 def causal_softmax_rows(scores: torch.Tensor, probs: torch.Tensor, heads: int, first_pos: int, scale: float,

@@ -202,13 +202,25 @@ SHAPES = [dict(heads=3, dim=16, rot=8, vdim=20, kv_rank=24, q_rank=40),         
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
 @pytest.mark.parametrize("shape", SHAPES)
 @pytest.mark.parametrize("window", [None, 1, 2, 16, 33, 100])
-def test_owner_and_reader_in_portions(dtype, shape, window):
+@pytest.mark.parametrize("expand", [False, True])
+def test_owner_and_reader_in_portions(monkeypatch, dtype, shape, window, expand):
     """A layer with its own latent and one that reads its rows with other heads and another window, two unequal requests
     in portions (from 90 tokens down to one), against whole-sequence attention.  In bfloat16 the long portions take the
-    products-and-softmax path beside short ones in the same step."""
+    products-and-softmax path or (``expand``) keys and values formed from the rows, beside short ones in the same step."""
+    from photon_infer_b200.parts import latent_attention
+    if expand and (dtype == torch.float32 or shape["vdim"] % 8 or shape["dim"] % 8):
+        pytest.skip("only bfloat16 with sizes of 8s expands rows")
+    if expand:                                  # whatever the arithmetic says: small latents would not be worth it
+        def every_long(self, ctx, lens, dtype):
+            assert self._prompt_defines(dtype) is not None
+            starts = ctx.host_start_positions
+            return {i: (starts[i], starts[i] + n - self._first_seen(starts[i])) for i, n in enumerate(lens) if n >= 32}
+        monkeypatch.setattr(latent_attention.LatentAttention, "_expanded_requests", every_long)
+    else:
+        monkeypatch.setattr(latent_attention, "USE_EXPANDED_PROMPTS", False)
     from photon_infer_b200.parts.base import LayerCache
     own, m, w = _mixer(dtype, window=window, **shape)
-    rshape = dict(shape, heads=shape["heads"] + 1, dim=shape["dim"] + 3, vdim=shape["vdim"] + 4, q_rank=shape["q_rank"] + 5)
+    rshape = dict(shape, heads=shape["heads"] + 1, dim=shape["dim"] + (8 if expand else 3), vdim=shape["vdim"] + (8 if expand else 4), q_rank=shape["q_rank"] + 5)
     rwindow = None if window is None else max(1, window - 7)
     reader, rm, rw = _mixer(dtype, window=rwindow, own=False, seed=9, **rshape)
     lens, ps = [150, 77], 8
@@ -286,6 +298,79 @@ def test_a_key_just_inside_and_just_outside_the_window(dtype, window, phase):
                 assert float(p[:, target - lo].min()) > 0.5
             want = p @ kd[lo:asking + 1, :kr]
             assert rel_err(out[-1].float().cpu().view(heads, kr), want) < (2e-5 if dtype == torch.float32 else 2e-2), (asking, back)
+
+
+@pytest.mark.parametrize("sizes", [(64, 32, 64), (128, 64, 128), (16, 16, 24), (72, 8, 80), (136, 40, 104), (192, 64, 8)])
+@pytest.mark.parametrize("window", [None, 1, 63, 64, 65, 200])
+@pytest.mark.parametrize("gated", [False, True])
+def test_long_portions_over_expanded_rows(sizes, window, gated):
+    """The tensor-core kernel alone: three requests of unequal length and start in one call, heads whose sizes fill 64-wide
+    chunks, do not fill them, or need several; for some queries one key is made to stand out, at the window's inner edge,
+    just outside it, at the first visible key and at the query's own position.  Tokens that belong to nobody stay as they
+    are."""
+    from photon_infer_b200.kernels import ops
+    d, r, v = sizes
+    heads = 3
+    g = torch.Generator().manual_seed(d + (window or 0))
+    reqs = [(40, 0), (300, 517), (129, 130)]                        # (tokens, position of the first)
+    gap = 5
+    T = sum(n for n, _ in reqs) + gap * len(reqs)
+    q = torch.randn(T, heads, d + r, generator=g)
+    seqs, kus, krs, vs, t, row = [], [], [], [], 0, 0
+    for n, start in reqs:
+        base = 0 if window is None else max(0, start + 1 - window)
+        L = start + n - base
+        ku, kr, vv = torch.randn(L, heads, d, generator=g), torch.randn(L, r, generator=g), torch.randn(L, heads, v, generator=g)
+        ku, kr = 0.3 * ku, 0.3 * kr
+        for i in range(0, n, 7):
+            pos = start + i
+            lo = 0 if window is None else max(0, pos + 1 - window)
+            back = [0, pos - lo, pos - lo + 1, (window or 40) - 1, (window or 40)][(i // 7) % 5]
+            k = pos - back - base
+            if 0 <= k < L:
+                q[t + i, :, :d] = ku[k] / 0.3 * (5.0 / d ** 0.5)
+                q[t + i, :, d:] = kr[k] / 0.3 * (5.0 / r ** 0.5)
+        seqs.append((t, n, start, base, row))
+        kus.append(ku); krs.append(kr); vs.append(vv)
+        t += n + gap
+        row += L
+    b16 = lambda x: x.bfloat16()
+    q, kus, krs, vs = b16(q), [b16(x) for x in kus], [b16(x) for x in krs], [b16(x) for x in vs]
+    kv = torch.cat([torch.cat([a.reshape(len(a), -1), c.reshape(len(c), -1)], 1) for a, c in zip(kus, vs)])
+    wide = torch.cat([torch.randn(row, 24, generator=g).bfloat16(), torch.cat(krs)], 1).to(DEV)        # the part lies in wider rows
+    gate = (2 * torch.randn(T, heads * v + 16, generator=g)).bfloat16()
+    out = torch.full((T, heads * v), 9.0, dtype=torch.bfloat16, device=DEV)
+    err = torch.zeros(4, dtype=torch.int32, device=DEV)
+    scale = 0.8
+    ops.latent_prompt_attention(q.reshape(T, -1).to(DEV), q[:, :, d:].contiguous().to(DEV), kv.to(DEV), wide[:, 24:], out, seqs, heads, d, r, v,
+                                window, scale, err, gate=gate.to(DEV)[:, 16:] if gated else None)
+    assert err.cpu().tolist()[0] == 0
+    out = out.float().cpu()
+    for (t, n, start, base, row), ku, kr, vv in zip(seqs, kus, krs, vs):
+        p, k = start + torch.arange(n)[:, None], base + torch.arange(len(ku))[None, :]
+        ok = (k <= p) & (p - k < (window or 10 ** 9))
+        qq = q[t:t + n].double()
+        want = plain.attend(qq[..., :d], qq[..., d:], ku.double(), kr.double(), vv.double(), ok, scale)
+        if gated:
+            want = want * torch.sigmoid(gate[t:t + n, 16:].double()).view(n, heads, v)
+        assert rel_err(out[t:t + n].view(n, heads, v), want) < 1.5e-2
+        assert torch.all(out[t + n:t + n + gap] == 9.0)
+
+
+def test_what_the_kernel_of_expanded_rows_refuses():
+    from photon_infer_b200.errors import PhotonError
+    from photon_infer_b200.kernels import ops
+    z = lambda *s: torch.zeros(*s, dtype=torch.bfloat16, device=DEV)
+    call = lambda seqs, d=64, r=32, v=64, rows=64, window=None: ops.latent_prompt_attention(
+        z(40, 2 * (d + r)), z(40, 2, r), z(rows, 2 * (d + v)), z(rows, r), z(40, 2 * v), seqs, 2, d, r, v, window, 1.0, None)
+    call([(0, 40, 24, 0, 0)])
+    for bad in ([(0, 41, 0, 0, 0)], [(0, 40, 25, 0, 0)], [(0, 40, 0, 1, 0)], [(8, 33, 0, 0, 0)], [(0, 40, 0, 0, 25)]):
+        with pytest.raises(PhotonError):
+            call(bad)                           # rows or tokens that do not exist, or a first row behind the first visible one
+    with pytest.raises(PhotonError):
+        call([(0, 40, 0, 0, 0)], d=60)
+    with pytest.raises(PhotonError):
+        call([(0, 40, 0, 0, 0)], v=136)
 
 
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
