@@ -8,11 +8,12 @@
 // joined in memory, and neither are the two parts of a query.
 //
 // A block owns one head and up to 256 tokens of one request as two tiles of 128 rows, and walks the keys that any of
-// them sees in tiles of 64:
-//   * warp 8 brings both query tiles and then the key and value tiles (TMA, 128-byte swizzle, zeros beyond d, r, v and
-//     the matrix' end) into a ring of shared-memory stages;
-//   * one thread of warp 9 issues, for the two query tiles in turn, S = Q K^T (M 128, N 64) into one of two score
-//     buffers and O += P V (M 128, N 64 * LT_NV) with P in tensor memory;
+// them sees in tiles of 128 (a product with N 64 takes the tensor core about as long as one with N 128: tiles of 64 keys
+// measured 50 us where these take 38, at 2,048 tokens, 16 heads of 128 + 64 and a window of 1,024):
+//   * warp 8 brings both query tiles and then the key tiles and the value tiles in halves (TMA, 128-byte swizzle, zeros
+//     beyond d, r, v and the matrix' end) into two rings in shared memory;
+//   * one thread of warp 9 issues, for the two query tiles in turn, O += P V (M 128, N 64 * LT_NV, P in tensor memory) and
+//     the next S = Q K^T (M 128, N 128), which takes the place of that P;
 //   * warps 0-3 and 4-7 own the rows of a query tile each, one row per thread: running maximum and sum in 32-bit, P =
 //     exp2(..) as bfloat16 written back over the scores, O rescaled only when a row's maximum has grown by more than
 //     2^8.  While one tile's softmax runs, the tensor cores work for the other.
@@ -37,17 +38,19 @@
 static_assert(LT_NU >= 1 && LT_NR >= 1 && LT_NK <= 4 && LT_NV >= 1 && LT_NV <= 2, "sizes of the latent prompt attention");
 
 #define LT_ROWS 128                                // rows of a query tile
-#define LT_KT 64                                   // keys per tile
+#define LT_KT 128                                  // keys per tile
+#define LT_VH 64                                   // keys per half of a value tile
 #define LT_THREADS 320
 #define LT_Q_BYTES (LT_ROWS * 128 * LT_NK)         // one query tile
-#define LT_K_BYTES (LT_KT * 128 * LT_NK)
-#define LT_V_BYTES (LT_KT * 128 * LT_NV)
-#define LT_STAGE_BYTES (LT_K_BYTES + LT_V_BYTES)
-#define LT_STAGES (2 * LT_Q_BYTES + 3 * LT_STAGE_BYTES <= 224 * 1024 ? 3 : 2)
-#define LT_SMEM_BYTES (2 * LT_Q_BYTES + LT_STAGES * LT_STAGE_BYTES + 1024 + 256)
+#define LT_K_BYTES (LT_KT * 128 * LT_NK)           // one key tile
+#define LT_V_BYTES (LT_VH * 128 * LT_NV)           // half a value tile
+#define LT_ROOM (224 * 1024)
+#define LT_KST (2 * LT_Q_BYTES + 2 * LT_K_BYTES + 2 * LT_V_BYTES <= LT_ROOM ? 2 : 1)                    // key tiles in the ring
+#define LT_VST (2 * LT_Q_BYTES + LT_KST * LT_K_BYTES + 4 * LT_V_BYTES <= LT_ROOM ? 4 : 2)              // halves of value tiles
+#define LT_SMEM_BYTES (2 * LT_Q_BYTES + LT_KST * LT_K_BYTES + LT_VST * LT_V_BYTES + 1024 + 256)
 static_assert(LT_SMEM_BYTES <= 227 * 1024, "shared memory of a block");
 #define LT_TMEM_COLS 512
-#define LT_O_COL 256                               // scores: 2 tiles x 2 buffers x 64 columns; O: 2 x 128
+#define LT_O_COL 256                               // scores: 2 tiles x 128 columns; O: 2 x 128
 #define LT_RESCALE_STEP 8.0f
 #define LT_MAX_SEQS 64
 
@@ -84,23 +87,26 @@ attention_latent_tc_kernel(const __grid_constant__ CUtensorMap map_qu, const __g
   extern __shared__ unsigned char lt_dyn[];
   unsigned char* base = reinterpret_cast<unsigned char*>(((uintptr_t)lt_dyn + 1023) & ~(uintptr_t)1023);
   unsigned char* q_s = base;                                           // 2 x query tile
-  unsigned char* kv_s = q_s + 2 * LT_Q_BYTES;                          // LT_STAGES x (K | V)
-  uint64_t* bars = reinterpret_cast<uint64_t*>(kv_s + LT_STAGES * LT_STAGE_BYTES);
+  unsigned char* k_s = q_s + 2 * LT_Q_BYTES;                           // LT_KST key tiles
+  unsigned char* v_s = k_s + LT_KST * LT_K_BYTES;                      // LT_VST halves of value tiles
+  uint64_t* bars = reinterpret_cast<uint64_t*>(v_s + LT_VST * LT_V_BYTES);
   uint64_t* q_full = bars;
-  uint64_t* k_full = bars + 1;
-  uint64_t* v_full = k_full + LT_STAGES;
-  uint64_t* kv_empty = v_full + LT_STAGES;
-  uint64_t* s_full = kv_empty + LT_STAGES;          // [tile][buffer] MMA -> softmax
-  uint64_t* p_full = s_full + 4;                    // [tile][buffer] softmax -> MMA (one arrival per warp)
-  uint64_t* pv_done = p_full + 4;                   // [tile][buffer] MMA -> softmax: O is up to date
-  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(pv_done + 4);
+  uint64_t* k_full = bars + 1;                      // [LT_KST] TMA -> MMA
+  uint64_t* k_empty = k_full + LT_KST;              // [LT_KST] MMA -> TMA
+  uint64_t* v_full = k_empty + LT_KST;              // [LT_VST]
+  uint64_t* v_empty = v_full + LT_VST;              // [LT_VST]
+  uint64_t* s_full = v_empty + LT_VST;              // [query tile] MMA -> softmax
+  uint64_t* p_full = s_full + 2;                    // [query tile] softmax -> MMA (one arrival per warp)
+  uint64_t* pv_done = p_full + 2;                   // [query tile] MMA -> softmax: O is up to date
+  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(pv_done + 2);
   volatile int* abort_flag = reinterpret_cast<volatile int*>(tmem_slot + 1);
 
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   if (threadIdx.x == 0) {
     tc_mbar_init(q_full, 1);
-    for (int s = 0; s < LT_STAGES; ++s) { tc_mbar_init(&k_full[s], 1); tc_mbar_init(&v_full[s], 1); tc_mbar_init(&kv_empty[s], 1); }
-    for (int b = 0; b < 4; ++b) { tc_mbar_init(&s_full[b], 1); tc_mbar_init(&p_full[b], 4); tc_mbar_init(&pv_done[b], 1); }
+    for (int s = 0; s < LT_KST; ++s) { tc_mbar_init(&k_full[s], 1); tc_mbar_init(&k_empty[s], 1); }
+    for (int s = 0; s < LT_VST; ++s) { tc_mbar_init(&v_full[s], 1); tc_mbar_init(&v_empty[s], 1); }
+    for (int b = 0; b < 2; ++b) { tc_mbar_init(&s_full[b], 1); tc_mbar_init(&p_full[b], 4); tc_mbar_init(&pv_done[b], 1); }
     *abort_flag = 0;
     asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
   }
@@ -127,30 +133,45 @@ attention_latent_tc_kernel(const __grid_constant__ CUtensorMap map_qu, const __g
 #pragma unroll
         for (int c = 0; c < LT_NR; ++c) tc_tma_load3(qt + (LT_NU + c) * (LT_ROWS * 128), &map_qr, c * 64, head, t, q_full);
       }
-      int issued = 0;
-      for (int i = 0; i < ntiles; ++i) {
-        const int s = i % LT_STAGES;
-        if (!tc_wait(&kv_empty[s], ((i / LT_STAGES) & 1) ^ 1, abort_flag)) break;
-        unsigned char* kst = kv_s + s * LT_STAGE_BYTES;
-        unsigned char* vst = kst + LT_K_BYTES;
-        const int row = row_lo + i * LT_KT;
+      int kn = 0, vn = 0;                           // key tiles and value halves asked for so far
+      auto load_k = [&]() -> bool {
+        const int s = kn % LT_KST;
+        if (!tc_wait(&k_empty[s], ((kn / LT_KST) & 1) ^ 1, abort_flag)) return false;
+        unsigned char* dst = k_s + s * LT_K_BYTES;
+        const int row = row_lo + kn * LT_KT;
         tc_mbar_expect_tx(&k_full[s], LT_K_BYTES);
+#pragma unroll
+        for (int c = 0; c < LT_NU; ++c) tc_tma_load3(dst + c * (LT_KT * 128), &map_ku, c * 64, head, row, &k_full[s]);
+#pragma unroll
+        for (int c = 0; c < LT_NR; ++c) tc_tma_load(dst + (LT_NU + c) * (LT_KT * 128), &map_kr, c * 64, row, &k_full[s]);
+        ++kn;
+        return true;
+      };
+      auto load_v = [&]() -> bool {
+        const int s = vn % LT_VST;
+        if (!tc_wait(&v_empty[s], ((vn / LT_VST) & 1) ^ 1, abort_flag)) return false;
+        unsigned char* dst = v_s + s * LT_V_BYTES;
+        const int row = row_lo + vn * LT_VH;
         tc_mbar_expect_tx(&v_full[s], LT_V_BYTES);
 #pragma unroll
-        for (int c = 0; c < LT_NU; ++c) tc_tma_load3(kst + c * (LT_KT * 128), &map_ku, c * 64, head, row, &k_full[s]);
-#pragma unroll
-        for (int c = 0; c < LT_NR; ++c) tc_tma_load(kst + (LT_NU + c) * (LT_KT * 128), &map_kr, c * 64, row, &k_full[s]);
-#pragma unroll
-        for (int c = 0; c < LT_NV; ++c) tc_tma_load3(vst + c * (LT_KT * 128), &map_v, c * 64, head, row, &v_full[s]);
-        issued = i + 1;
+        for (int c = 0; c < LT_NV; ++c) tc_tma_load3(dst + c * (LT_VH * 128), &map_v, c * 64, head, row, &v_full[s]);
+        ++vn;
+        return true;
+      };
+      // in the order in which room appears: the scores of tile i free a key tile before the products of tile i free values
+      bool ok = true;
+      for (int n = 0; n < LT_KST && n < ntiles && ok; ++n) ok = load_k();
+      for (int i = 0; i < ntiles && ok; ++i) {
+        ok = load_v() && load_v();
+        if (ok && kn < ntiles) ok = load_k();
       }
       if (*abort_flag) {
         // copies already issued still write into this block's shared memory: wait for them, bounded
         for (uint32_t w = 0; w < TC_WAIT_LIMIT && !tc_mbar_try(q_full, 0); ++w) {}
-        for (int j = (issued > LT_STAGES ? issued - LT_STAGES : 0); j < issued; ++j) {
-          for (uint32_t w = 0; w < TC_WAIT_LIMIT && !tc_mbar_try(&k_full[j % LT_STAGES], (j / LT_STAGES) & 1); ++w) {}
-          for (uint32_t w = 0; w < TC_WAIT_LIMIT && !tc_mbar_try(&v_full[j % LT_STAGES], (j / LT_STAGES) & 1); ++w) {}
-        }
+        for (int n = (kn > LT_KST ? kn - LT_KST : 0); n < kn; ++n)
+          for (uint32_t w = 0; w < TC_WAIT_LIMIT && !tc_mbar_try(&k_full[n % LT_KST], (n / LT_KST) & 1); ++w) {}
+        for (int n = (vn > LT_VST ? vn - LT_VST : 0); n < vn; ++n)
+          for (uint32_t w = 0; w < TC_WAIT_LIMIT && !tc_mbar_try(&v_full[n % LT_VST], (n / LT_VST) & 1); ++w) {}
       }
     }
   } else if (warp == 9) {
@@ -158,35 +179,41 @@ attention_latent_tc_kernel(const __grid_constant__ CUtensorMap map_qu, const __g
     if (lane == 0) {
       const uint32_t idesc_s = tc_idesc(LT_ROWS, LT_KT);
       const uint32_t idesc_o = tc_idesc(LT_ROWS, 64 * LT_NV) | TC_IDESC_B_MN;
+      // the scores of key tile i for query tile j; the second query tile is the last to read the keys
       auto issue_scores = [&](int i, int j) -> bool {
-        const int s = i % LT_STAGES;
-        if (!tc_wait(&k_full[s], (i / LT_STAGES) & 1, abort_flag)) return false;
+        const int s = i % LT_KST;
+        if (!tc_wait(&k_full[s], (i / LT_KST) & 1, abort_flag)) return false;
         tc_fence_after();
-        const uint32_t q_addr = tc_smem(q_s + j * LT_Q_BYTES), k_addr = tc_smem(kv_s + s * LT_STAGE_BYTES);
+        const uint32_t q_addr = tc_smem(q_s + j * LT_Q_BYTES), k_addr = tc_smem(k_s + s * LT_K_BYTES);
 #pragma unroll
         for (int kk = 0; kk < LT_NK * 4; ++kk)
-          tc_mma(tmem_base + j * 128 + (i & 1) * LT_KT, tc_desc(q_addr + (kk >> 2) * (LT_ROWS * 128) + (kk & 3) * 32),
+          tc_mma(tmem_base + j * 128, tc_desc(q_addr + (kk >> 2) * (LT_ROWS * 128) + (kk & 3) * 32),
                  tc_desc(k_addr + (kk >> 2) * (LT_KT * 128) + (kk & 3) * 32), idesc_s, kk > 0 ? 1u : 0u);
-        tc_commit(&s_full[j * 2 + (i & 1)]);
+        tc_commit(&s_full[j]);
+        if (j == 1) tc_commit(&k_empty[s]);
         return true;
       };
       bool ok = tc_wait(q_full, 0, abort_flag);
       if (ok) ok = issue_scores(0, 0) && issue_scores(0, 1);
       for (int i = 0; i < ntiles && ok; ++i) {
-        const int s = i % LT_STAGES;
         for (int j = 0; j < 2 && ok; ++j) {
-          // the next tile's scores of these rows first, so that their softmax can start as soon as it is free
-          if (i + 1 < ntiles && !issue_scores(i + 1, j)) { ok = false; break; }
-          if (!tc_wait(&p_full[j * 2 + (i & 1)], (i >> 1) & 1, abort_flag)) { ok = false; break; }
-          if (!tc_wait(&v_full[s], (i / LT_STAGES) & 1, abort_flag)) { ok = false; break; }
-          tc_fence_after();
-          const uint32_t v_addr = tc_smem(kv_s + s * LT_STAGE_BYTES + LT_K_BYTES);
+          if (!tc_wait(&p_full[j], i & 1, abort_flag)) { ok = false; break; }
 #pragma unroll
-          for (int kk = 0; kk < LT_KT / 16; ++kk)
-            at_mma_ts(tmem_base + LT_O_COL + j * 128, tmem_base + j * 128 + (i & 1) * LT_KT + kk * 8,
-                      tc_desc_mn(v_addr + kk * 2048, LT_KT * 128, 1024), idesc_o, (i > 0 || kk > 0) ? 1u : 0u);
-          if (j == 1) tc_commit(&kv_empty[s]);
-          tc_commit(&pv_done[j * 2 + (i & 1)]);
+          for (int half = 0; half < 2; ++half) {
+            const int n = 2 * i + half, s = n % LT_VST;
+            if (!tc_wait(&v_full[s], (n / LT_VST) & 1, abort_flag)) { ok = false; break; }
+            tc_fence_after();
+            const uint32_t v_addr = tc_smem(v_s + s * LT_V_BYTES);
+#pragma unroll
+            for (int kk = 0; kk < LT_VH / 16; ++kk)  // P: 8 columns of packed pairs per 16 keys
+              at_mma_ts(tmem_base + LT_O_COL + j * 128, tmem_base + j * 128 + half * 32 + kk * 8,
+                        tc_desc_mn(v_addr + kk * 2048, LT_VH * 128, 1024), idesc_o, (n > 0 || kk > 0) ? 1u : 0u);
+            if (j == 1) tc_commit(&v_empty[s]);
+          }
+          if (!ok) break;
+          tc_commit(&pv_done[j]);
+          // the next scores go where this tile's P was; the tensor core runs the products in the order of issue
+          if (i + 1 < ntiles) ok = issue_scores(i + 1, j);
         }
       }
       pdl_launch_dependents();                      // all products of this block are issued
@@ -206,26 +233,24 @@ attention_latent_tc_kernel(const __grid_constant__ CUtensorMap map_qu, const __g
     auto wait_all = [&](uint64_t* bar, uint32_t parity) -> bool {
       return __all_sync(0xffffffffu, tc_wait(bar, parity, abort_flag) ? 1 : 0) != 0;
     };
+    const uint32_t s_addr = lane_addr + j * 128, o_addr = lane_addr + LT_O_COL + j * 128;
     for (int i = 0; i < ntiles; ++i) {
-      const int b = j * 2 + (i & 1);
-      if (!wait_all(&s_full[b], (i >> 1) & 1)) { ok = false; break; }
+      if (!wait_all(&s_full[j], i & 1)) { ok = false; break; }
       tc_fence_after();
-      const uint32_t s_addr = lane_addr + j * 128 + (i & 1) * LT_KT;
       const int key_base = key_lo + i * LT_KT;
-      uint32_t sv[64];
-      tc_ld32_issue(s_addr, sv);
-      tc_ld32_issue(s_addr + 32, sv + 32);
+      uint32_t sv[128];
+#pragma unroll
+      for (int u = 0; u < 128; u += 32) tc_ld32_issue(s_addr + u, sv + u);
       tc_ld_wait();
       if (!(key_base + LT_KT - 1 <= pos && key_base >= lo)) {
+        // keys this row does not see: those before offset a or behind offset b of the tile
+        const int a = lo - key_base, b = pos - key_base;
 #pragma unroll
-        for (int u = 0; u < 64; ++u) {
-          const int key = key_base + u;
-          sv[u] = (key >= lo && key <= pos) ? sv[u] : 0xff800000u;       // -inf
-        }
+        for (int u = 0; u < 128; ++u) sv[u] = (u >= a && u <= b) ? sv[u] : 0xff800000u;       // -inf
       }
       float mx4[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
 #pragma unroll
-      for (int u = 0; u < 64; u += 8) {
+      for (int u = 0; u < 128; u += 8) {
 #pragma unroll
         for (int w = 0; w < 4; ++w) mx4[w] = at_max3(mx4[w], __uint_as_float(sv[u + 2 * w]), __uint_as_float(sv[u + 2 * w + 1]));
       }
@@ -236,39 +261,41 @@ attention_latent_tc_kernel(const __grid_constant__ CUtensorMap map_qu, const __g
       const bool grow = cand > m_used + LT_RESCALE_STEP;          // also the first finite maximum
       if (grow) { factor = at_exp2(m_used - cand); m_used = cand; l *= factor; }
       const float nsub = (m_used == -INFINITY) ? 0.f : -m_used;
+      // P = exp2(score * c - max in use), packed pairs over the scores they came from (32 columns per 64 keys)
+      float sum8[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
+#pragma unroll
+      for (int half = 0; half < 2; ++half) {
+        uint32_t pk[32];
+#pragma unroll
+        for (int u = 0; u < 64; u += 2) {
+          float x0, x1;
+          at_fma2(x0, x1, __uint_as_float(sv[half * 64 + u]), __uint_as_float(sv[half * 64 + u + 1]), c, nsub);
+          const float p0 = at_exp2(x0), p1 = at_exp2(x1);
+          at_add2(sum8[u & 6], sum8[(u & 6) + 1], p0, p1);
+          pk[u >> 1] = at_pack(p0, p1);
+        }
+        tc_st32(s_addr + half * 32, pk);
+      }
+      l += ((sum8[0] + sum8[1]) + (sum8[2] + sum8[3])) + ((sum8[4] + sum8[5]) + (sum8[6] + sum8[7]));
       if (i > 0 && __any_sync(0xffffffffu, grow)) {
         // O rescale: the products of the tile before must have landed
-        if (!wait_all(&pv_done[j * 2 + ((i - 1) & 1)], ((i - 1) >> 1) & 1)) { ok = false; break; }
+        if (!wait_all(&pv_done[j], (i - 1) & 1)) { ok = false; break; }
         tc_fence_after();
 #pragma unroll 1
         for (int cc = 0; cc < 64 * LT_NV; cc += 32) {
           uint32_t ov[32];
-          tc_ld32(lane_addr + LT_O_COL + j * 128 + cc, ov);
+          tc_ld32(o_addr + cc, ov);
 #pragma unroll
           for (int u = 0; u < 32; ++u) ov[u] = __float_as_uint(__uint_as_float(ov[u]) * factor);
-          tc_st32(lane_addr + LT_O_COL + j * 128 + cc, ov);
+          tc_st32(o_addr + cc, ov);
         }
-        tc_st_wait();
       }
-      // P = exp2(score * c - max in use), packed pairs over the scores they came from
-      float sum8[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
-      uint32_t pk[32];
-#pragma unroll
-      for (int u = 0; u < 64; u += 2) {
-        float x0, x1;
-        at_fma2(x0, x1, __uint_as_float(sv[u]), __uint_as_float(sv[u + 1]), c, nsub);
-        const float p0 = at_exp2(x0), p1 = at_exp2(x1);
-        at_add2(sum8[u & 6], sum8[(u & 6) + 1], p0, p1);
-        pk[u >> 1] = at_pack(p0, p1);
-      }
-      tc_st32(s_addr, pk);
-      l += ((sum8[0] + sum8[1]) + (sum8[2] + sum8[3])) + ((sum8[4] + sum8[5]) + (sum8[6] + sum8[7]));
       tc_st_wait();
       tc_fence_before();
       __syncwarp();
-      if (lane == 0) tc_mbar_arrive(&p_full[b]);
+      if (lane == 0) tc_mbar_arrive(&p_full[j]);
     }
-    if (ok && wait_all(&pv_done[j * 2 + ((ntiles - 1) & 1)], ((ntiles - 1) >> 1) & 1)) {
+    if (ok && wait_all(&pv_done[j], (ntiles - 1) & 1)) {
       tc_fence_after();
       const float inv = l > 0.f ? 1.f / l : 0.f;
       bf16* dst = P.out + (size_t)(q.tok0 + t) * P.out_stride + (size_t)head * P.dv;
@@ -276,7 +303,7 @@ attention_latent_tc_kernel(const __grid_constant__ CUtensorMap map_qu, const __g
 #pragma unroll 1
       for (int cc = 0; cc < 64 * LT_NV; cc += 32) {
         uint32_t ov[32];
-        tc_ld32(lane_addr + LT_O_COL + j * 128 + cc, ov);
+        tc_ld32(o_addr + cc, ov);
         if (valid) {
 #pragma unroll
           for (int u = 0; u < 32; u += 8) {
@@ -348,7 +375,7 @@ PHOTON_API int photon_attention_latent_tc(const void* q, long q_stride, const vo
   int st = lt_map3(&map_qu, q, d, heads, T, d + r, q_stride, LT_ROWS);
   if (st == 0) st = lt_map3(&map_qr, q_rot, r, heads, T, r, (long)heads * r, LT_ROWS);
   if (st == 0) st = lt_map3(&map_ku, kv, d, heads, rows, d, kv_stride, LT_KT);
-  if (st == 0) st = lt_map3(&map_v, (const bf16*)kv + (long)heads * d, v, heads, rows, v, kv_stride, LT_KT);
+  if (st == 0) st = lt_map3(&map_v, (const bf16*)kv + (long)heads * d, v, heads, rows, v, kv_stride, LT_VH);
   if (st == 0) st = make_map(&map_kr, rot_rows, rows, r, rot_stride, LT_KT);
   if (st != 0) return st;
   static bool attr_done = false;

@@ -154,6 +154,11 @@ PHOTON_EXPORT int photon_latent_q_rope(const void* q, long q_stride, int dtype, 
 PHOTON_EXPORT int photon_head_linear(const void* x, long x_row, long x_head, const void* W, void* out, long o_row, long o_head,
                        int dtype, int M, int heads, int N, int K, const void* gate, long gate_row, cudaStream_t stream);
 
+/* A decode step's queries in one launch (bfloat16, M <= 16, dim a multiple of 8, else PHOTON_ERR_UNSUPPORTED): out[m, h, :N] =
+ * W[h] q[m, h, :dim] and out[m, h, out_off ..] = the rotated last rot numbers of the head. */
+PHOTON_EXPORT int photon_latent_absorb(const void* q, long q_stride, int dtype, const void* W, int M, int heads, int dim, int rot,
+                         int rot_dims, int interleaved, const int* positions, const float* inv_freq, int N, void* out,
+                         long out_stride, int out_head, int out_off, cudaStream_t stream);
 /* out[i, :] = the cache row of position first + i (i < count) of the request whose pages are table (cache
  * [num_pages * page_size][width]); zero rows for positions outside [valid_lo, valid_hi). */
 PHOTON_EXPORT int photon_gather_rows(const void* cache, int dtype, const int* table, int page_size, int num_pages, int width,

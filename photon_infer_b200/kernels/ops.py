@@ -1056,7 +1056,7 @@ def latent_q_rope(q: torch.Tensor, heads: int, dim: int, rot: int, rot_dims: int
 def latent_decode_supported(q: torch.Tensor, width: int, value_dim: int) -> bool:
     """The tensor-core kernel for decoded tokens over a cached latent: bfloat16, row and value widths multiples of 16."""
     return (q.dtype == torch.bfloat16 and width % 16 == 0 and value_dim % 16 == 0 and value_dim <= width
-            and q.stride(0) % 8 == 0 and q.data_ptr() % 16 == 0 and (80 * (width + 8) * 2 + 16384) <= 220 * 1024)
+            and q.stride(0) % 8 == 0 and q.data_ptr() % 16 == 0 and (80 * (width + 8) * 2 + 24576) <= 220 * 1024)
 
 
 def latent_decode_shares(max_context: int, window: Optional[int] = None) -> int:
@@ -1123,6 +1123,31 @@ def head_linear(x: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, gate: 
              c_void_p])
     _check(f(_ptr(x), x.stride(0), x.stride(1), _ptr(weight), _ptr(out), out.stride(0), out.stride(1), _dtype_code(x),
              T, heads, N, K, _ptr(gate), gate.stride(0) if gate is not None else 0, _stream()), "head_linear")
+
+
+def latent_absorb_supported(q: torch.Tensor, dim: int, rot: int) -> bool:
+    """One launch takes a decode step's queries into the latent space: bfloat16, few rows, sizes of 8s."""
+    return (q.dtype == torch.bfloat16 and q.shape[0] < HEAD_LINEAR_LIBRARY_ROWS and dim % 8 == 0 and rot % 8 == 0
+            and q.stride(0) % 8 == 0 and q.data_ptr() % 16 == 0)
+
+
+def latent_absorb(q: torch.Tensor, weight: torch.Tensor, dim: int, rot: int, rot_dims: int, positions: torch.Tensor,
+                  inv_freq: torch.Tensor, out: torch.Tensor, interleaved: bool = False) -> None:
+    """``head_linear`` of the unrotated parts of ``q [T, heads * (dim + rot)]`` with ``weight [heads, N, dim]`` into the first
+    ``N`` numbers of every head of ``out [T, heads, N + rot]``, and ``latent_q_rope`` of the rest behind them, in one launch."""
+    _cuda(q, weight, positions, inv_freq, out)
+    T = q.shape[0]
+    heads, N, K = weight.shape
+    if not latent_absorb_supported(q, dim, rot) or K != dim or q.shape[1] != heads * (dim + rot) or q.stride(1) != 1 \
+            or out.shape != (T, heads, N + rot) or not out.is_contiguous() or not weight.is_contiguous() \
+            or weight.dtype != q.dtype or out.dtype != q.dtype:
+        raise PhotonError(ErrorCode.SHAPE_MISMATCH, "latent_absorb: q [T, heads * (dim + rot)], weight [heads, N, dim], out [T, heads, N + rot]")
+    _int32(positions, "positions")
+    f = _fn("latent", "photon_latent_absorb",
+            [c_void_p, c_long, c_int, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_int, c_void_p, c_long,
+             c_int, c_int, c_void_p])
+    _check(f(_ptr(q), q.stride(0), _dtype_code(q), _ptr(weight), T, heads, dim, rot, rot_dims, int(interleaved), _ptr(positions),
+             _ptr(inv_freq), N, _ptr(out), out.stride(0), out.shape[2], N, _stream()), "latent_absorb")
 
 
 def gather_rows(cache: torch.Tensor, table: torch.Tensor, count: int, err: Optional[torch.Tensor], first: int = 0,

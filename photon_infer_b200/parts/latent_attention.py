@@ -147,9 +147,12 @@ class LatentAttention(Mixer):
         """Requests ``s0 .. s1 - 1`` (tokens from ``t0`` on) in the latent space: queries in, weighted latents out."""
         T, n, d, r, kr = q.shape[0], self.heads, self.dim, self.rot_dim, self.kv_rank
         q_lat = torch.empty((T, n, self.width), dtype=q.dtype, device=q.device)
-        ops.head_linear(q.view(T, n, d + r)[:, :, :d], self.w_absorb, q_lat[:, :, :kr])
-        ops.latent_q_rope(q, n, d, r, self.rot_dims, ctx.positions[t0:t0 + T], self.inv_freq, q_lat, kr,
-                          interleaved=self.rot_interleaved)
+        positions = ctx.positions[t0:t0 + T]
+        if ops.latent_absorb_supported(q, d, r):        # few rows: both parts of the queries in one launch
+            ops.latent_absorb(q, self.w_absorb, d, r, self.rot_dims, positions, self.inv_freq, q_lat, interleaved=self.rot_interleaved)
+        else:
+            ops.head_linear(q.view(T, n, d + r)[:, :, :d], self.w_absorb, q_lat[:, :, :kr])
+            ops.latent_q_rope(q, n, d, r, self.rot_dims, positions, self.inv_freq, q_lat, kr, interleaved=self.rot_interleaved)
         o_lat = torch.empty((T, n * kr), dtype=q.dtype, device=q.device)
         self.attend(q_lat, o_lat, ctx, cache, s0, s1, t0, lens)
         ops.head_linear(o_lat.view(T, n, kr), self.w_uv, o.view(T, n, self.vdim), gate=gate)
