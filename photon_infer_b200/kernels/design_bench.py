@@ -129,7 +129,7 @@ def llama_config(width: int, layers: int, window=None) -> dict:
     return cfg
 
 
-def _time_events(fn, reps: int = 3, flush: bool = False) -> float:
+def _time_events(fn, reps: int = 10, flush: bool = False) -> float:
     """Microseconds of ``fn()``, the best of ``reps``; ``flush``: L2 is written over before each."""
     fn()
     torch.cuda.synchronize()
@@ -298,7 +298,7 @@ def _parts(runner, hbm_peak: float, tf_peak: float) -> Dict[str, dict]:
                     x = torch.randn(T, streams.streams, H, device=model.device)
                     step = lambda: block.norm1.read_streams(Connected(y, streams), x, streams.w_in, model.dtype)
                     moved = T * H * (2 * 4 * streams.streams + 2 * 2)
-                us = _time_events(step, 5, flush=True) if phase == "prefill" else _time_graph(step)
+                us = _time_events(step, flush=True) if phase == "prefill" else _time_graph(step)
                 out[f"{norm_name}.{phase}"] = {"us": round(us, 1), "frac": round(moved / (us * 1e-6) / (hbm_peak * 1e9), 4)}
             if kind and (kind_name, phase) not in seen:
                 seen.add((kind_name, phase))

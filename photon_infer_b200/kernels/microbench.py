@@ -4,6 +4,9 @@
     python -m photon_infer_b200.kernels.microbench decode-products [--rows 1 8 16]
     python -m photon_infer_b200.kernels.microbench attention-prefill [--tokens 2048 8192]
     python -m photon_infer_b200.kernels.microbench attention-decode [--batch 1 8 64] [--context 640 4096]
+    python -m photon_infer_b200.kernels.microbench latent-prefill [--tokens 2048 8192] [--heads 16] [--window 1024]
+    python -m photon_infer_b200.kernels.microbench latent-decode [--batch 8] [--context 512 4096] [--heads 16] [--window 1024]
+    python -m photon_infer_b200.kernels.microbench streams [--rows 8 2048] [--hidden 2048] [--streams 4]
 
 The shapes are those of the Llama 3.2 1B layer unless ``--hidden/--intermediate/--heads/--kv-heads/
 --head-dim`` say otherwise.  Decode kernels are timed inside a CUDA graph of ten launches over ten
@@ -182,9 +185,60 @@ def attention_decode(a) -> None:
             print(line, flush=True)
 
 
+LATENT = dict(d=128, r=64, v=128, kr=512)       # the latent sizes of the design comparison
+
+
+def latent_prefill(a) -> None:
+    """One prompt portion from position 0 over expanded latent rows (the attention alone)."""
+    dev, (d, r, v, kr), n = torch.device("cuda", 0), LATENT.values(), a.heads
+    for T in a.tokens or [2048, 8192]:
+        b16 = lambda *shape: torch.randn(*shape, device=dev).bfloat16()
+        q, q_rot, kv, rows = b16(T, n * (d + r)), b16(T, n, r), b16(T, n * (d + v)), b16(T, kr + r)
+        out = torch.empty(T, n * v, device=dev, dtype=torch.bfloat16)
+        err = torch.zeros(4, dtype=torch.int32, device=dev)
+        pairs = sum(min(i + 1, a.window or T) for i in range(T))
+        fl = 2.0 * n * (d + r + v) * pairs
+        t = _events(lambda: ops.latent_prompt_attention(q, q_rot, kv, rows[:, kr:], out, [(0, T, 0, 0, 0)], n, d, r, v, a.window,
+                                                        (d + r) ** -0.5, err))
+        print(f"tokens {T:6d} heads {n} window {a.window}: {t:8.1f} us ({fl / t / 1e6:4.0f} TFLOP/s)", flush=True)
+
+
+def latent_decode(a) -> None:
+    """One token per request over cached latent rows: the attention and the merge of its shares."""
+    dev, (d, r, v, kr), n = torch.device("cuda", 0), LATENT.values(), a.heads
+    for B in a.batch or [8]:
+        for ctx in a.context or [512, 4096]:
+            per = -(-ctx // a.page_size)
+            caches = [torch.randn(B * per, 1, a.page_size, kr + r, device=dev).bfloat16() for _ in range(10)]
+            table = torch.randperm(B * per).to(torch.int32).reshape(B, per).to(dev)
+            q = torch.randn(B, n * (kr + r), device=dev).bfloat16()
+            out = torch.empty(B, n * kr, device=dev, dtype=torch.bfloat16)
+            seq, pos = torch.arange(B, dtype=torch.int32, device=dev), torch.full((B,), ctx - 1, dtype=torch.int32, device=dev)
+            err = torch.zeros(4, dtype=torch.int32, device=dev)
+            t = _graph(lambda i: ops.latent_decode_attention(q, out, caches[i], table, seq, pos, n, kr + r, kr, (d + r) ** -0.5, ctx, err,
+                                                             window=a.window), 10)
+            mb = B * min(ctx, a.window or ctx) * (kr + r) * 2 / 1e6
+            print(f"batch {B} context {ctx} heads {n} window {a.window}: {t:6.1f} us, {mb:.1f} MB of rows ({mb / t:5.2f} TB/s)", flush=True)
+
+
+def streams(a) -> None:
+    """The pending write, the read and the layer norm of parallel residual streams."""
+    dev, H, S = torch.device("cuda", 0), a.hidden, a.streams
+    f32 = lambda *shape: torch.randn(*shape, device=dev)
+    w, mix, w_out, w_in = f32(H), f32(S, S) * 0.1, f32(S), f32(S)
+    for T in a.rows or [8, 2048]:
+        copies = 10 if T * S * H * 4 < 1 << 20 else 4
+        xs, ys = [f32(T, S, H) for _ in range(copies)], [f32(T, H).bfloat16() for _ in range(copies)]
+        out = torch.empty(T, H, device=dev, dtype=torch.bfloat16)
+        t = _graph(lambda i: ops.stream_norm(xs[i], S, ys[i], mix, w_out, w_in, w, None, 1e-5, out, new_streams=xs[i]), copies)
+        mb = T * H * (8 * S + 4) / 1e6
+        print(f"rows {T} streams {S} width {H}: {t:6.1f} us, {mb:.1f} MB ({mb / t:5.2f} TB/s)", flush=True)
+
+
 def main(argv=None) -> int:
     ap = argparse.ArgumentParser(description=__doc__, formatter_class=argparse.RawDescriptionHelpFormatter)
-    ap.add_argument("what", choices=["products", "decode-products", "attention-prefill", "attention-decode"])
+    ap.add_argument("what", choices=["products", "decode-products", "attention-prefill", "attention-decode", "latent-prefill",
+                                     "latent-decode", "streams"])
     ap.add_argument("--rows", type=int, nargs="*")
     ap.add_argument("--tokens", type=int, nargs="*")
     ap.add_argument("--batch", type=int, nargs="*")
@@ -194,11 +248,14 @@ def main(argv=None) -> int:
     ap.add_argument("--heads", type=int, default=32)
     ap.add_argument("--kv-heads", type=int, default=8)
     ap.add_argument("--head-dim", type=int, default=64)
+    ap.add_argument("--window", type=int, default=None)
+    ap.add_argument("--streams", type=int, default=4)
     ap.add_argument("--page-size", type=int, default=16)
     a = ap.parse_args(argv)
     torch.manual_seed(0)
     {"products": products, "decode-products": decode_products, "attention-prefill": attention_prefill,
-     "attention-decode": attention_decode}[a.what](a)
+     "attention-decode": attention_decode, "latent-prefill": latent_prefill, "latent-decode": latent_decode,
+     "streams": streams}[a.what](a)
     return 0
 
 

@@ -58,7 +58,8 @@ def _ptr(t: Optional[torch.Tensor]) -> c_void_p:
 
 
 def _stream() -> c_void_p:
-    return c_void_p(torch.cuda.current_stream().cuda_stream)
+    # what torch.cuda.current_stream() wraps, without building a Stream object at every launch
+    return c_void_p(torch._C._cuda_getCurrentRawStream(torch._C._cuda_getDevice()))
 
 
 def _check(status: int, what: str) -> None:
