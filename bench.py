@@ -27,7 +27,9 @@ decoder with the same window.  ``--design lerosun`` does it for the Lerosun deco
 are mixed before the softmax, with a window, a sink and an output gate; layers of the gated delta rule; feed-forwards
 with a relu gate), beside a Llama decoder with the same window and the Finelix decoder.  ``--design pebodra`` does it for
 the Pebodra decoder (norms on the sublayers' outputs; differential attention, some layers reading another layer's keys
-and values; state-space and matrix-memory layers; PolyNorm and routed feed-forwards), beside the same two.
+and values; state-space and matrix-memory layers; PolyNorm and routed feed-forwards), beside the same two.  ``--design milozen``
+does it for the Milozen decoder (parallel residual streams; attention over a cached latent with a window and an output
+gate, some layers reading another layer's latent; experts with bounded activations), beside the same two.
 
 ``--impl reference`` runs lumia431/photon_infer itself where it could be built (``baseline/``); else it
 prints an ``unavailable`` line.
