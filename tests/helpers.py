@@ -556,7 +556,7 @@ TINY_MILOZEN: Dict[str, dict] = {
     # one stream; a latent as wide as a large model's row; a window longer than most requests; pages of 32
     "mz_d": dict(
         config=dict(architecture="Milozen", vocab=90, width=32, streams=1, embedding=dict(scale=2.0), norm=dict(eps=1e-5),
-                    layers=[_zlayer(_zatt(2, 64, 64, 128, 256, 24, 0.09, 100, 300000.0), _zmoe(2, 2, 16, 1.5)),
+                    layers=[_zlayer(_zatt(2, 64, 64, 128, 256, 24, 0.09, 100, 300000.0), _zmoe(2, 2, 16, 1.4)),
                             _zlayer(_zatt(4, 8, 64, 16, 256, 96, 0.1, 160, 300000.0, kv_from=0), dict(kind="dense", ff=48))]),
         seed=54, init_std=0.15, norm_std=0.1, block_size=32),
     # three streams; two readers, one of them without a window (so everything is kept); more experts than a warp has lanes
