@@ -22,7 +22,7 @@
 // no tensor-core kernel and no causal mask inside a portion (src/ops/kernels/cuda/
 // paged_attention.cu:90-194, src/arch/transformer_block.cpp:486-509).
 //
-// Compiled per model with -DHEAD_DIM=<d>.
+// Compiled per model with -DHEAD_DIM=<d> and, where a value has another width than a key, -DVALUE_DIM=<dv>.
 #include "common.cuh"
 #include <math.h>
 
@@ -30,10 +30,15 @@
 #define HEAD_DIM 64
 #endif
 
+#ifndef VALUE_DIM
+#define VALUE_DIM HEAD_DIM
+#endif
+
 #define FA_TILE_K 64                      // keys per tile
 #ifndef FA_ROWS
 #define FA_ROWS 128                       // rows per block in ROWS mode (16 per warp)
 #endif
+#define FA_LOG2E 1.4426950408889634f
 #define FA_KEYS_THREADS 128               // KEYS mode: four warps, 16 keys of every tile each
 #define FA_ROWS_THREADS (FA_ROWS * 2)
 #ifndef FA_STAGES
@@ -41,10 +46,13 @@
 #endif
 #define FA_TABLE_SMEM 256                 // block-table entries the KEYS kernel copies to shared memory up front
 #define FA_LD (HEAD_DIM + 8)              // padded row length in shared memory (elements): conflict-free ldmatrix
+#define FA_LDV (VALUE_DIM + 8)            // the same for a row of values
 #define FA_KD (HEAD_DIM / 16)             // k-steps over the head dimension
-#define FA_ND (HEAD_DIM / 8)              // n-tiles over the head dimension
+#define FA_ND (VALUE_DIM / 8)             // n-tiles over a value
+#define FA_STAGE (FA_TILE_K * (FA_LD + FA_LDV))   // elements of one stage: a K tile, then a V tile
 
 static_assert(HEAD_DIM % 16 == 0 && HEAD_DIM >= 16 && HEAD_DIM <= 128, "head size");
+static_assert(VALUE_DIM % 16 == 0 && VALUE_DIM >= 16 && VALUE_DIM <= 128, "size of a value");
 
 __device__ __forceinline__ uint32_t fa_smem(const void* p) { return (uint32_t)__cvta_generic_to_shared(p); }
 __device__ __forceinline__ void cp_async16(void* dst, const void* src, bool valid) {
@@ -78,8 +86,8 @@ __device__ __forceinline__ uint32_t pack_bf16(float lo, float hi) {
 
 struct FlashParams {
   const bf16* q; long q_stride;           // [T, n_q * d] view
-  bf16* out; long out_stride;             // [T, n_q * d]
-  const bf16* k_cache; const bf16* v_cache;   // [pages, n_kv, page_size, d]
+  bf16* out; long out_stride;             // [T, n_q * dv]
+  const bf16* k_cache; const bf16* v_cache;   // [pages, n_kv, page_size, d], [pages, n_kv, page_size, dv]
   const int* block_table; int max_pages;  // [S, max_pages]
   const int* cu_tokens;                   // [S + 1] first token of each request in the step
   const int* positions;                   // [T]
@@ -90,11 +98,12 @@ struct FlashParams {
   float scale_log2;                       // scale * log2(e); with bounded scores log2(e) alone
   int* err;
   // Three more rules (all off at 0).  keep_first: with a window, keys 0 .. keep_first - 1 stay visible behind it.
-  // sink: the softmax has one more key with score 0 and no value.  softcap: scores become
+  // sinks [n_q]: a head's softmax has one more key with this score and no value.  softcap: scores become
   // softcap * tanh(score * scale / softcap); cap_in = scale / softcap.
-  int keep_first, sink;
+  int keep_first;
+  const float* sinks;                     // may be null
   float softcap, cap_in;
-  const bf16* gate; long gate_stride;     // may be null: [T, n_q * d]; every output is multiplied by sigmoid(gate)
+  const bf16* gate; long gate_stride;     // may be null: [T, n_q * dv]; every output is multiplied by sigmoid(gate)
 };
 
 // tanh through one exponential and one reciprocal: 1 - 2 / (2^(2 x log2 e) + 1); absolute error about 1e-7.
@@ -110,12 +119,13 @@ __device__ __forceinline__ void load_kv_tile(const FlashParams& P, const int* ta
                                              int key0, int lo, int hi, bf16* ks, bf16* vs, int t_for_err,
                                              int tid, int nthreads) {
   const int kept = P.keep_first;
-  constexpr int CPR = HEAD_DIM / 8;                       // 16-byte chunks per row
+  constexpr int CPK = HEAD_DIM / 8, CPV = VALUE_DIM / 8;  // 16-byte chunks per row
+  constexpr int CPR = CPK > CPV ? CPK : CPV;
   for (int c = tid; c < FA_TILE_K * CPR; c += nthreads) {
     const int r = c / CPR, cc = c - r * CPR;
     const int key = key0 + r;
     bool valid = (key >= lo || key < kept) && key <= hi;
-    size_t src = 0;
+    size_t row = 0;
     if (valid) {
       const int pidx = P.page_shift >= 0 ? (key >> P.page_shift) : key / P.page_size;
       const int slot = P.page_shift >= 0 ? (key & (P.page_size - 1)) : key - pidx * P.page_size;
@@ -124,11 +134,11 @@ __device__ __forceinline__ void load_kv_tile(const FlashParams& P, const int* ta
         if (cc == 0) report_error(P.err, PHOTON_DEV_BAD_PAGE, t_for_err, key, page);
         valid = false;
       } else {
-        src = (((size_t)page * P.n_kv + g) * P.page_size + slot) * HEAD_DIM + cc * 8;
+        row = ((size_t)page * P.n_kv + g) * P.page_size + slot;
       }
     }
-    cp_async16(ks + r * FA_LD + cc * 8, P.k_cache + src, valid);
-    cp_async16(vs + r * FA_LD + cc * 8, P.v_cache + src, valid);
+    if (CPK == CPR || cc < CPK) cp_async16(ks + r * FA_LD + cc * 8, P.k_cache + (valid ? row * HEAD_DIM + cc * 8 : 0), valid);
+    if (CPV == CPR || cc < CPV) cp_async16(vs + r * FA_LDV + cc * 8, P.v_cache + (valid ? row * VALUE_DIM + cc * 8 : 0), valid);
   }
 }
 
@@ -214,7 +224,7 @@ __device__ __forceinline__ void warp_tile(const uint32_t (&qa)[FA_KD][4], const 
       uint32_t b[4];
       const int key = krow + kk * 16 + (lane & 7) + (((lane >> 3) & 1) << 3);
       const int dim = n * 8 + ((lane >> 4) << 3);
-      ldsm4t(b, vs + key * FA_LD + dim);
+      ldsm4t(b, vs + key * FA_LDV + dim);
       mma_bf16(o[n], pa[kk], b[0], b[1]);
       mma_bf16(o[n + 1], pa[kk], b[2], b[3]);
     }
@@ -232,11 +242,11 @@ __global__ void __launch_bounds__(KEYS_MODE ? FA_KEYS_THREADS * NSUB : FA_ROWS_T
 flash_attention_kernel(const FlashParams P) {
   extern __shared__ __align__(16) unsigned char fa_dyn[];
   constexpr int Q_ELEMS = (KEYS_MODE ? 16 : FA_ROWS) * FA_LD;
-  constexpr int RING_ELEMS = STAGES * 2 * FA_TILE_K * FA_LD;
+  constexpr int RING_ELEMS = STAGES * FA_STAGE;
   const int sub = KEYS_MODE ? (int)(threadIdx.x >> 7) : 0;                  // group of four warps
   const int stid = KEYS_MODE ? (int)(threadIdx.x & 127) : (int)threadIdx.x; // thread index inside the group
   const int sthreads = KEYS_MODE ? FA_KEYS_THREADS : FA_ROWS_THREADS;
-  // per group: Q rows (KEYS: 16, ROWS: FA_ROWS) x FA_LD, then STAGES x (K | V) x 64 x FA_LD
+  // per group: Q rows (KEYS: 16, ROWS: FA_ROWS) x FA_LD, then STAGES x (64 x FA_LD of K | 64 x FA_LDV of V)
   bf16* qs = reinterpret_cast<bf16*>(fa_dyn) + (size_t)sub * (Q_ELEMS + RING_ELEMS);
   bf16* kv = qs + Q_ELEMS;
   auto group_sync = [&]() {
@@ -308,8 +318,8 @@ flash_attention_kernel(const FlashParams P) {
                  P.q + (size_t)(tok0 + tk) * P.q_stride + (size_t)(g * G + h) * HEAD_DIM + cc * 8, valid);
     }
   }
-  auto stage_k = [&](int st) { return kv + (size_t)st * 2 * FA_TILE_K * FA_LD; };
-  auto stage_v = [&](int st) { return kv + (size_t)st * 2 * FA_TILE_K * FA_LD + FA_TILE_K * FA_LD; };
+  auto stage_k = [&](int st) { return kv + (size_t)st * FA_STAGE; };
+  auto stage_v = [&](int st) { return kv + (size_t)st * FA_STAGE + FA_TILE_K * FA_LD; };
   // prologue: the first STAGES - 1 tiles (the Q copy joins the first group)
 #pragma unroll
   for (int i = 0; i < STAGES - 1; ++i) {
@@ -403,10 +413,10 @@ flash_attention_kernel(const FlashParams P) {
       const int row = row0 + wrow + (lane >> 2) + h2 * 8;
       if (row >= rows) continue;
       const int tk = row / G, h = row - tk * G;
-      if (P.sink) l[h2] += exp2f(-m[h2]);                                   // the sink's weight, relative to the running maximum
+      if (P.sinks) l[h2] += exp2f(fmaf(P.sinks[g * G + h], FA_LOG2E, -m[h2]));   // the sink's weight, relative to the running maximum
       const float inv = l[h2] > 0.f ? 1.f / l[h2] : 0.f;
-      bf16* dst = P.out + (size_t)(tok0 + tk) * P.out_stride + (size_t)(g * G + h) * HEAD_DIM + (lane & 3) * 2;
-      const bf16* gt = P.gate ? P.gate + (size_t)(tok0 + tk) * P.gate_stride + (size_t)(g * G + h) * HEAD_DIM + (lane & 3) * 2 : nullptr;
+      bf16* dst = P.out + (size_t)(tok0 + tk) * P.out_stride + (size_t)(g * G + h) * VALUE_DIM + (lane & 3) * 2;
+      const bf16* gt = P.gate ? P.gate + (size_t)(tok0 + tk) * P.gate_stride + (size_t)(g * G + h) * VALUE_DIM + (lane & 3) * 2 : nullptr;
 #pragma unroll
       for (int n = 0; n < FA_ND; ++n) {
         float y0 = o[n][h2 * 2] * inv, y1 = o[n][h2 * 2 + 1] * inv;
@@ -425,21 +435,21 @@ flash_attention_kernel(const FlashParams P) {
   __syncthreads();                                                         // all warps are done with the rings
   float* wm = reinterpret_cast<float*>(fa_dyn);                            // [NW][16]
   float* wl = wm + NW * 16;                                                // [NW][16]
-  float* wo = wl + NW * 16;                                                // [NW][16][HEAD_DIM]
+  float* wo = wl + NW * 16;                                                // [NW][16][VALUE_DIM]
 #pragma unroll
   for (int h2 = 0; h2 < 2; ++h2) {
     const int r = (lane >> 2) + h2 * 8;
     if ((lane & 3) == 0) { wm[warp * 16 + r] = m[h2]; wl[warp * 16 + r] = l[h2]; }
 #pragma unroll
     for (int n = 0; n < FA_ND; ++n) {
-      wo[(warp * 16 + r) * HEAD_DIM + n * 8 + (lane & 3) * 2] = o[n][h2 * 2];
-      wo[(warp * 16 + r) * HEAD_DIM + n * 8 + (lane & 3) * 2 + 1] = o[n][h2 * 2 + 1];
+      wo[(warp * 16 + r) * VALUE_DIM + n * 8 + (lane & 3) * 2] = o[n][h2 * 2];
+      wo[(warp * 16 + r) * VALUE_DIM + n * 8 + (lane & 3) * 2 + 1] = o[n][h2 * 2 + 1];
     }
   }
   __syncthreads();
   const int n_q = P.n_kv * G;
-  for (int e = threadIdx.x; e < nrows * HEAD_DIM; e += blockDim.x) {
-    const int r = e / HEAD_DIM, d = e - r * HEAD_DIM;
+  for (int e = threadIdx.x; e < nrows * VALUE_DIM; e += blockDim.x) {
+    const int r = e / VALUE_DIM, d = e - r * VALUE_DIM;
     float M = -INFINITY;
 #pragma unroll
     for (int w = 0; w < NW; ++w) M = fmaxf(M, wm[w * 16 + r]);
@@ -450,19 +460,19 @@ flash_attention_kernel(const FlashParams P) {
         const float mw = wm[w * 16 + r];
         const float sc = (mw == -INFINITY) ? 0.f : exp2f(mw - M);
         L += wl[w * 16 + r] * sc;
-        A += wo[(w * 16 + r) * HEAD_DIM + d] * sc;
+        A += wo[(w * 16 + r) * VALUE_DIM + d] * sc;
       }
     }
     const int tk = r / G, h = r - tk * G;
     const int head = g * G + h;
     if (P.num_splits == 1) {
-      if (P.sink && M != -INFINITY) L += exp2f(-M);
+      if (P.sinks && M != -INFINITY) L += exp2f(fmaf(P.sinks[head], FA_LOG2E, -M));
       float y = L > 0.f ? A / L : 0.f;
-      if (P.gate) y = __fdividef(y, 1.0f + __expf(-__bfloat162float(P.gate[(size_t)(tok0 + tk) * P.gate_stride + (size_t)head * HEAD_DIM + d])));
-      P.out[(size_t)(tok0 + tk) * P.out_stride + (size_t)head * HEAD_DIM + d] = __float2bfloat16_rn(y);
+      if (P.gate) y = __fdividef(y, 1.0f + __expf(-__bfloat162float(P.gate[(size_t)(tok0 + tk) * P.gate_stride + (size_t)head * VALUE_DIM + d])));
+      P.out[(size_t)(tok0 + tk) * P.out_stride + (size_t)head * VALUE_DIM + d] = __float2bfloat16_rn(y);
     } else {
       const size_t slot = ((size_t)(tok0 + tk) * n_q + head) * P.num_splits + split;
-      __stcg(P.part_acc + slot * HEAD_DIM + d, A);
+      __stcg(P.part_acc + slot * VALUE_DIM + d, A);
       if (d == 0) { __stcg(P.part_ml + slot * 2, M); __stcg(P.part_ml + slot * 2 + 1, L); }
     }
   }
@@ -475,8 +485,8 @@ flash_attention_kernel(const FlashParams P) {
   if (!s_flag) return;
   __threadfence();
   if (threadIdx.x == 0) P.tickets[(size_t)seq * P.n_kv + g] = 0;
-  for (int e = threadIdx.x; e < nrows * HEAD_DIM; e += blockDim.x) {
-    const int r = e / HEAD_DIM, d = e - r * HEAD_DIM;
+  for (int e = threadIdx.x; e < nrows * VALUE_DIM; e += blockDim.x) {
+    const int r = e / VALUE_DIM, d = e - r * VALUE_DIM;
     const int tk = r / G, h = r - tk * G;
     const int head = g * G + h;
     const size_t base = ((size_t)(tok0 + tk) * n_q + head) * P.num_splits;
@@ -488,19 +498,19 @@ flash_attention_kernel(const FlashParams P) {
         const float ms = __ldcg(P.part_ml + (base + s2) * 2);
         const float sc = (ms == -INFINITY) ? 0.f : exp2f(ms - M);
         L += __ldcg(P.part_ml + (base + s2) * 2 + 1) * sc;
-        A += __ldcg(P.part_acc + (base + s2) * HEAD_DIM + d) * sc;
+        A += __ldcg(P.part_acc + (base + s2) * VALUE_DIM + d) * sc;
       }
-      if (P.sink) L += exp2f(-M);
+      if (P.sinks) L += exp2f(fmaf(P.sinks[head], FA_LOG2E, -M));
     }
     float y = L > 0.f ? A / L : 0.f;
-    if (P.gate) y = __fdividef(y, 1.0f + __expf(-__bfloat162float(P.gate[(size_t)(tok0 + tk) * P.gate_stride + (size_t)head * HEAD_DIM + d])));
-    P.out[(size_t)(tok0 + tk) * P.out_stride + (size_t)head * HEAD_DIM + d] = __float2bfloat16_rn(y);
+    if (P.gate) y = __fdividef(y, 1.0f + __expf(-__bfloat162float(P.gate[(size_t)(tok0 + tk) * P.gate_stride + (size_t)head * VALUE_DIM + d])));
+    P.out[(size_t)(tok0 + tk) * P.out_stride + (size_t)head * VALUE_DIM + d] = __float2bfloat16_rn(y);
   }
 }
 
 PHOTON_API int photon_flash_attention_head_dim() { return HEAD_DIM; }
 // Groups of four warps (each with a ring of stages of its own) that fit into the shared memory of one block.
-constexpr int FA_GROUP_BYTES = (16 * FA_LD + FA_STAGES * 2 * FA_TILE_K * FA_LD) * 2;
+constexpr int FA_GROUP_BYTES = (16 * FA_LD + FA_STAGES * FA_STAGE) * 2;
 constexpr int FA_MAX_GROUPS = (4 * FA_GROUP_BYTES + 2048 <= 232448) ? 4 : ((2 * FA_GROUP_BYTES + 2048 <= 232448) ? 2 : 1);
 PHOTON_API int photon_flash_attention_max_groups() { return FA_MAX_GROUPS; }
 
@@ -510,7 +520,7 @@ PHOTON_API int photon_flash_attention_max_groups() { return FA_MAX_GROUPS; }
 // key tiles (at most photon_flash_attention_max_groups(), which depends on the head size).
 // context_lens (may be null): tokens of each request after this step; with it the KEYS kernel does not read
 // `positions` (the tokens a request brings are then taken to be its last ones, in order).
-// Scratch (KEYS mode with num_splits > 1): part_acc float [T * n_q * num_splits * d], part_ml float
+// Scratch (KEYS mode with num_splits > 1): part_acc float [T * n_q * num_splits * dv], part_ml float
 // [T * n_q * num_splits * 2], tickets int [S * n_kv] all zero between launches.  Launches that share scratch
 // must not overlap on the device.
 PHOTON_API int photon_flash_attention(const void* q, long q_stride, void* out, long out_stride, const void* k_cache,
@@ -522,12 +532,12 @@ PHOTON_API int photon_flash_attention(const void* q, long q_stride, void* out, l
                                       int nsub, int mode, int* err, cudaStream_t stream) {
   return photon_flash_attention_ex(q, q_stride, out, out_stride, k_cache, v_cache, block_table, max_pages, cu_tokens, positions,
                                    context_lens, part_acc, part_ml, tickets, S, max_tokens_per_seq, n_q, n_kv, d, page_size,
-                                   num_pages, window, scale, num_splits, nsub, mode, err, 0, 0, 0.f, nullptr, 0, stream);
+                                   num_pages, window, scale, num_splits, nsub, mode, err, 0, nullptr, 0.f, nullptr, 0, stream);
 }
 
-// The same with kept first keys (with a window, keys 0 .. keep_first - 1 stay visible behind it), a sink (one more
-// key with score 0 and no value in the softmax) and bounded scores (softcap * tanh(score * scale / softcap); 0: off).
-// gate (may be null): bfloat16 [T, n_q * d] with row stride gate_stride (a multiple of 2, 4-byte aligned rows); every
+// The same with kept first keys (with a window, keys 0 .. keep_first - 1 stay visible behind it), sinks (float [n_q], may
+// be null: one more key with this score and no value in head h's softmax) and bounded scores (softcap * tanh(score * scale / softcap); 0: off).
+// gate (may be null): bfloat16 [T, n_q * dv] with row stride gate_stride (a multiple of 2, 4-byte aligned rows); every
 // output is multiplied by sigmoid(gate) before it is rounded.
 PHOTON_API int photon_flash_attention_ex(const void* q, long q_stride, void* out, long out_stride, const void* k_cache,
                                          const void* v_cache, const int* block_table, int max_pages,
@@ -535,7 +545,7 @@ PHOTON_API int photon_flash_attention_ex(const void* q, long q_stride, void* out
                                          float* part_acc, float* part_ml,
                                          int* tickets, int S, int max_tokens_per_seq, int n_q, int n_kv, int d,
                                          int page_size, int num_pages, int window, float scale, int num_splits,
-                                         int nsub, int mode, int* err, int keep_first, int sink, float softcap,
+                                         int nsub, int mode, int* err, int keep_first, const float* sinks, float softcap,
                                          const void* gate, long gate_stride, cudaStream_t stream) {
   if (S <= 0) return 0;
   if (keep_first < 0 || softcap < 0.f) return PHOTON_ERR_ARGUMENT;
@@ -553,13 +563,13 @@ PHOTON_API int photon_flash_attention_ex(const void* q, long q_stride, void* out
   P.n_q = n_q; P.n_kv = n_kv; P.group = n_q / n_kv; P.page_size = page_size; P.num_pages = num_pages;
   P.page_shift = -1;
   for (int sh = 0; sh < 20; ++sh) if ((1 << sh) == page_size) P.page_shift = sh;
-  P.window = window; P.scale_log2 = scale * 1.4426950408889634f; P.err = err;
-  P.keep_first = window > 0 ? keep_first : 0; P.sink = sink; P.softcap = softcap; P.cap_in = 0.f;
-  if (softcap > 0.f) { P.cap_in = scale / softcap; P.scale_log2 = 1.4426950408889634f; }
+  P.window = window; P.scale_log2 = scale * FA_LOG2E; P.err = err;
+  P.keep_first = window > 0 ? keep_first : 0; P.sinks = sinks; P.softcap = softcap; P.cap_in = 0.f;
+  if (softcap > 0.f) { P.cap_in = scale / softcap; P.scale_log2 = FA_LOG2E; }
   if (gate != nullptr && (((uintptr_t)gate & 3) || (gate_stride & 1))) return PHOTON_ERR_ARGUMENT;
   P.gate = (const bf16*)gate; P.gate_stride = gate_stride;
-  const size_t ring = (size_t)FA_STAGES * 2 * FA_TILE_K * FA_LD;
-  const size_t ring2 = (size_t)2 * 2 * FA_TILE_K * FA_LD;                   // two stages
+  const size_t ring = (size_t)FA_STAGES * FA_STAGE;
+  const size_t ring2 = (size_t)2 * FA_STAGE;                   // two stages
   const size_t smem_rows = ((size_t)FA_ROWS * FA_LD + ring) * sizeof(bf16);
   const size_t smem_keys = ((size_t)16 * FA_LD + ring) * sizeof(bf16);      // per group of four warps
   const size_t smem_keys2 = ((size_t)16 * FA_LD + ring2) * sizeof(bf16);

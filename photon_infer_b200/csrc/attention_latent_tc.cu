@@ -63,6 +63,8 @@ struct LatentTcSeq {
 struct LatentTcParams {
   bf16* out; long out_stride;                      // [T, heads * v]
   const bf16* gate; long gate_stride;              // may be null: every output times sigmoid(gate)
+  int gate_heads;                                  // the gate is one number per head: [T, heads]
+  const float* sinks;                              // may be null: [heads], one more key with this score and no value
   int dv, window, tiles_per_seq;
   float scale_log2;
   int* err;
@@ -297,9 +299,12 @@ attention_latent_tc_kernel(const __grid_constant__ CUtensorMap map_qu, const __g
     }
     if (ok && wait_all(&pv_done[j], (ntiles - 1) & 1)) {
       tc_fence_after();
-      const float inv = l > 0.f ? 1.f / l : 0.f;
+      if (P.sinks && valid) l += exp2f(fmaf(P.sinks[head], 1.4426950408889634f, -m_used));   // relative to the maximum in use
+      float inv = l > 0.f ? 1.f / l : 0.f;
+      if (P.gate && P.gate_heads && valid)
+        inv = __fdividef(inv, 1.0f + __expf(-__bfloat162float(P.gate[(size_t)(q.tok0 + t) * P.gate_stride + head])));
       bf16* dst = P.out + (size_t)(q.tok0 + t) * P.out_stride + (size_t)head * P.dv;
-      const bf16* gt = P.gate ? P.gate + (size_t)(q.tok0 + t) * P.gate_stride + (size_t)head * P.dv : nullptr;
+      const bf16* gt = P.gate && !P.gate_heads ? P.gate + (size_t)(q.tok0 + t) * P.gate_stride + (size_t)head * P.dv : nullptr;
 #pragma unroll 1
       for (int cc = 0; cc < 64 * LT_NV; cc += 32) {
         uint32_t ov[32];
@@ -357,19 +362,22 @@ PHOTON_API int photon_attention_latent_tc_max_seqs(void) { return LT_MAX_SEQS; }
 
 // q [T][heads][d + r] (row stride q_stride; the d unrotated numbers of every head), q_rot [T][heads][r] contiguous; kv
 // [rows][kv_stride]: every row holds heads x d key numbers, then heads x v value numbers; rot_rows: the r shared key numbers of
-// every row (row stride rot_stride).  out [T][heads * v]; gate (may be null) [T][heads * v].  seqs (host memory): S x (tok0,
+// every row (row stride rot_stride).  out [T][heads * v]; gate (may be null) [T][heads * v] or, with gate_heads != 0,
+// [T][heads] (one number per head, any alignment); sinks (may be null) float [heads].  seqs (host memory): S x (tok0,
 // ntok, start, base, row0), see LatentTcSeq; a token at position p sees the rows of positions max(0, p - window + 1) .. p
 // (window <= 0: from 0), all of which must be in the matrix.  d, r, v multiples of 8; all pointers and strides 16-byte aligned.
 PHOTON_API int photon_attention_latent_tc(const void* q, long q_stride, const void* q_rot, const void* kv, long kv_stride,
                                           const void* rot_rows, long rot_stride, void* out, long out_stride, const void* gate,
-                                          long gate_stride, const int* seqs, int S, int T, int rows, int heads, int d, int r,
-                                          int v, int window, float scale, int* err, cudaStream_t stream) {
+                                          long gate_stride, int gate_heads, const float* sinks, const int* seqs, int S, int T,
+                                          int rows, int heads, int d, int r, int v, int window, float scale, int* err,
+                                          cudaStream_t stream) {
   if (S <= 0 || T <= 0) return 0;
   if (rows <= 0 || heads <= 0 || heads > 65535 || !(scale > 0.f)) return PHOTON_ERR_ARGUMENT;
   if ((d & 7) || (r & 7) || (v & 7) || (d + 63) / 64 != LT_NU || (r + 63) / 64 != LT_NR || (v + 63) / 64 != LT_NV)
     return PHOTON_ERR_UNSUPPORTED;
   if (((uintptr_t)q & 15) || ((uintptr_t)q_rot & 15) || ((uintptr_t)kv & 15) || ((uintptr_t)rot_rows & 15) || ((uintptr_t)out & 15) ||
-      ((uintptr_t)gate & 15) || (q_stride & 7) || (kv_stride & 7) || (rot_stride & 7) || (out_stride & 7) || (gate && (gate_stride & 7)))
+      (q_stride & 7) || (kv_stride & 7) || (rot_stride & 7) || (out_stride & 7) ||
+      (gate && !gate_heads && (((uintptr_t)gate & 15) || (gate_stride & 7))))
     return PHOTON_ERR_ARGUMENT;
   CUtensorMap map_qu, map_qr, map_ku, map_kr, map_v;
   int st = lt_map3(&map_qu, q, d, heads, T, d + r, q_stride, LT_ROWS);
@@ -388,6 +396,7 @@ PHOTON_API int photon_attention_latent_tc(const void* q, long q_stride, const vo
     const int n = S - s0 < LT_MAX_SEQS ? S - s0 : LT_MAX_SEQS;
     LatentTcParams P;
     P.out = (bf16*)out; P.out_stride = out_stride; P.gate = (const bf16*)gate; P.gate_stride = gate_stride;
+    P.gate_heads = gate_heads; P.sinks = sinks;
     P.dv = v; P.window = window; P.scale_log2 = scale * 1.4426950408889634f; P.err = err;
     int most = 0;
     for (int i = 0; i < n; ++i) {

@@ -1,5 +1,6 @@
 // Paged causal attention for prompt portions on the fifth-generation tensor cores
-// (tcgen05, accumulators in tensor memory), bfloat16, head size 64 or 128.
+// (tcgen05, accumulators in tensor memory), bfloat16, heads of up to 128 numbers (a multiple of 8; tiles are 64 or 128
+// wide, zeros behind the head), values of another width where VALUE_DIM says so.
 //
 // A block owns up to 128 query rows of one request that share a key/value head
 // (row = token_in_step * GROUP + head_in_group, as in attention_flash.cu; floor(128 / GROUP)
@@ -33,14 +34,18 @@
 // that all roles poll, records PHOTON_DEV_WAIT_TIMEOUT, waits (bounded) for the copies it
 // has in flight, frees its tensor memory and returns.
 //
-// Compiled per model with -DHEAD_DIM=<64|128>.
+// Compiled per model with -DHEAD_DIM=<d> and, where a value has another width than a key, -DVALUE_DIM=<dv>.
 #include "attention_tc.cuh"
 #include <math.h>
 
 #ifndef HEAD_DIM
 #define HEAD_DIM 64
 #endif
-static_assert(HEAD_DIM == 64 || HEAD_DIM == 128, "head size of the tcgen05 attention");
+#ifndef VALUE_DIM
+#define VALUE_DIM HEAD_DIM
+#endif
+static_assert(HEAD_DIM % 8 == 0 && HEAD_DIM >= 16 && HEAD_DIM <= 128, "head size of the tcgen05 attention");
+static_assert(VALUE_DIM % 8 == 0 && VALUE_DIM >= 16 && VALUE_DIM <= 128, "size of a value of the tcgen05 attention");
 
 #define AT_ROWS 128
 // Keys per tile.  -DAT_KT=128 (heads of 64 only: two stages of such tiles leave room for two blocks per SM) halves the
@@ -49,43 +54,47 @@ static_assert(HEAD_DIM == 64 || HEAD_DIM == 128, "head size of the tcgen05 atten
 #ifndef AT_KT
 #define AT_KT 64
 #endif
-static_assert(AT_KT == 64 || HEAD_DIM == 64, "tiles of 128 keys only at heads of 64");
+static_assert(AT_KT == 64 || (HEAD_DIM == 64 && VALUE_DIM == 64), "tiles of 128 keys only at heads of 64");
 static_assert(AT_KT == 64 || AT_KT == 128, "keys per tile");
 #define AT_NBUF (AT_KT == 128 ? 1 : 2)             // score buffers in tensor memory (128 columns in all)
+#define AT_DH ((HEAD_DIM + 63) / 64)               // 64-wide halves of the head dimension
+#define AT_VH ((VALUE_DIM + 63) / 64)              // ... and of a value
 #ifndef AT_STAGES
-#define AT_STAGES (HEAD_DIM * AT_KT == 64 * 64 ? 3 : 2)   // two blocks per SM either way (81 KB, or 97 KB at heads of 128)
+#define AT_STAGES (AT_DH * AT_KT == 64 && AT_VH == 1 ? 3 : 2)   // two blocks per SM either way (81 KB, or 97 KB at heads of 128)
 #endif
 #ifndef AT_BLOCKS_PER_SM
 #define AT_BLOCKS_PER_SM 2
 #endif
 #define AT_THREADS 192                             // warps 0-3: softmax, warp 4: TMA, warp 5: MMA + TMEM
-#define AT_DH (HEAD_DIM / 64)                      // 64-wide halves of the head dimension
-#define AT_Q_BYTES (AT_ROWS * HEAD_DIM * 2)
-#define AT_KV_BYTES (AT_KT * HEAD_DIM * 2)         // one K tile or one V tile
+#define AT_Q_BYTES (AT_ROWS * 128 * AT_DH)
+#define AT_K_BYTES (AT_KT * 128 * AT_DH)           // one K tile
+#define AT_V_BYTES (AT_KT * 128 * AT_VH)           // one V tile
 #define AT_HALF_BYTES (AT_KT * 128)                // one 64-wide half of a K or V tile
 #ifndef AT_P_TMEM
 #define AT_P_TMEM 1                                // 1: P stays in tensor memory (it takes the place of the scores it came from)
 #endif
 #define AT_P_BYTES (AT_P_TMEM ? 0 : AT_ROWS * AT_KT * 2)
 static_assert(AT_P_TMEM || AT_KT == 64, "P in shared memory only with tiles of 64 keys");
-#define AT_SMEM_BYTES (AT_Q_BYTES + AT_STAGES * 2 * AT_KV_BYTES + 2 * AT_P_BYTES + 1024 + 256)
+#define AT_STAGE_BYTES (AT_K_BYTES + AT_V_BYTES)
+#define AT_SMEM_BYTES (AT_Q_BYTES + AT_STAGES * AT_STAGE_BYTES + 2 * AT_P_BYTES + 1024 + 256)
 #define AT_TMEM_COLS 256                           // scores 2 x 64 or 1 x 128 columns, O from column 128
 #define AT_O_COL 128
 #define AT_RESCALE_STEP 8.0f                       // log2 units a maximum may lag behind before O is rescaled
 
 struct AttnTcParams {
-  bf16* out; long out_stride;                      // [T, n_q * d]
+  bf16* out; long out_stride;                      // [T, n_q * dv]
   const int* block_table; int max_pages;           // [S, max_pages]
   const int* cu_tokens;                            // [S + 1]
   const int* positions;                            // [T]
   int n_kv, group, tile_rows, page_size, num_pages, box_rows, window, tiles_per_seq, total_rows;
   float scale_log2;                                // scale * log2(e); with bounded scores log2(e) alone
   int* err;
-  // keep_first: with a window, keys 0 .. keep_first - 1 stay visible behind it.  sink: one more key with score 0 and no
-  // value in the softmax.  softcap > 0: scores become softcap * tanh(score * cap_in), cap_in = scale / softcap.
-  int keep_first, sink;
+  // keep_first: with a window, keys 0 .. keep_first - 1 stay visible behind it.  sinks [n_q] (may be null): one more key
+  // with this score and no value in a head's softmax.  softcap > 0: scores become softcap * tanh(score * cap_in), cap_in = scale / softcap.
+  int keep_first;
+  const float* sinks;
   float softcap, cap_in;
-  const bf16* gate; long gate_stride;              // may be null: [T, n_q * d]; every output is multiplied by sigmoid(gate)
+  const bf16* gate; long gate_stride;              // may be null: [T, n_q * dv]; every output is multiplied by sigmoid(gate)
 };
 
 __global__ void __launch_bounds__(AT_THREADS, AT_BLOCKS_PER_SM)
@@ -116,7 +125,7 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
   unsigned char* base = reinterpret_cast<unsigned char*>(((uintptr_t)at_dyn + 1023) & ~(uintptr_t)1023);
   unsigned char* q_s = base;
   unsigned char* kv_s = q_s + AT_Q_BYTES;                              // AT_STAGES x (K tile | V tile)
-  unsigned char* p_s = kv_s + AT_STAGES * 2 * AT_KV_BYTES;             // 2 x P
+  unsigned char* p_s = kv_s + AT_STAGES * AT_STAGE_BYTES;              // 2 x P
   uint64_t* bars = reinterpret_cast<uint64_t*>(p_s + 2 * AT_P_BYTES);
   uint64_t* q_full = bars;                          // TMA -> MMA
   uint64_t* k_full = bars + 1;                      // [AT_STAGES] TMA -> MMA
@@ -173,15 +182,15 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
       if (lane == 0) ok = tc_wait(&kv_empty[s], ((i / AT_STAGES) & 1) ^ 1, abort_flag) ? 1 : 0;
       ok = __shfl_sync(0xffffffffu, ok, 0);
       if (!ok) break;
-      if (lane == 0) { tc_mbar_expect_tx(&k_full[s], AT_KV_BYTES); tc_mbar_expect_tx(&v_full[s], AT_KV_BYTES); }
+      if (lane == 0) { tc_mbar_expect_tx(&k_full[s], AT_K_BYTES); tc_mbar_expect_tx(&v_full[s], AT_V_BYTES); }
       __syncwarp();
       if (lane < boxes) {
-        unsigned char* kst = kv_s + s * 2 * AT_KV_BYTES + lane * P.box_rows * 128;
-        unsigned char* vst = kst + AT_KV_BYTES;
+        unsigned char* kst = kv_s + s * AT_STAGE_BYTES + lane * P.box_rows * 128;
+        unsigned char* vst = kst + AT_K_BYTES;
 #pragma unroll
         for (int h = 0; h < AT_DH; ++h) tc_tma_load(kst + h * AT_HALF_BYTES, &map_k, h * 64, rowc, &k_full[s]);
 #pragma unroll
-        for (int h = 0; h < AT_DH; ++h) tc_tma_load(vst + h * AT_HALF_BYTES, &map_v, h * 64, rowc, &v_full[s]);
+        for (int h = 0; h < AT_VH; ++h) tc_tma_load(vst + h * AT_HALF_BYTES, &map_v, h * 64, rowc, &v_full[s]);
       }
       issued = i + 1;
     }
@@ -197,15 +206,15 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
     // ---------------- MMA issuer
     if (lane == 0) {
       const uint32_t idesc_s = tc_idesc(AT_ROWS, AT_KT);
-      const uint32_t idesc_o = tc_idesc(AT_ROWS, HEAD_DIM) | TC_IDESC_B_MN;
+      const uint32_t idesc_o = tc_idesc(AT_ROWS, 64 * AT_VH) | TC_IDESC_B_MN;
       const uint32_t q_addr = tc_smem(q_s);
       auto issue_scores = [&](int i) -> bool {
         const int s = i % AT_STAGES;
         if (!tc_wait(&k_full[s], (i / AT_STAGES) & 1, abort_flag)) return false;
         tc_fence_after();
-        const uint32_t k_addr = tc_smem(kv_s + s * 2 * AT_KV_BYTES);
+        const uint32_t k_addr = tc_smem(kv_s + s * AT_STAGE_BYTES);
 #pragma unroll
-        for (int kk = 0; kk < HEAD_DIM / 16; ++kk)
+        for (int kk = 0; kk < (HEAD_DIM + 15) / 16; ++kk)
           tc_mma(tmem_base + (i % AT_NBUF) * AT_KT, tc_desc(q_addr + (kk >> 2) * (AT_ROWS * 128) + (kk & 3) * 32),
                  tc_desc(k_addr + (kk >> 2) * AT_HALF_BYTES + (kk & 3) * 32), idesc_s, kk > 0 ? 1u : 0u);
         tc_commit(&s_full[i % AT_NBUF]);
@@ -222,7 +231,7 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
         if (!tc_wait(&v_full[s], (i / AT_STAGES) & 1, abort_flag)) { ok = false; break; }
         tc_fence_after();
         const uint32_t p_addr = tc_smem(p_s + (i & 1) * AT_P_BYTES);
-        const uint32_t v_addr = tc_smem(kv_s + s * 2 * AT_KV_BYTES + AT_KV_BYTES);
+        const uint32_t v_addr = tc_smem(kv_s + s * AT_STAGE_BYTES + AT_K_BYTES);
 #pragma unroll
         for (int kk = 0; kk < AT_KT / 16; ++kk) {  // 16 keys: two groups of 8 rows of V
           if (AT_P_TMEM)                           // P: 8 columns of packed pairs per 16 keys, where the tile's scores were
@@ -306,7 +315,7 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
         if (!wait_all(&pv_done[(i - 1) % AT_NBUF], ((i - 1) / AT_NBUF) & 1)) { ok = false; break; }
         tc_fence_after();
 #pragma unroll 1
-        for (int cc = 0; cc < HEAD_DIM; cc += 32) {
+        for (int cc = 0; cc < VALUE_DIM; cc += 32) {
           uint32_t ov[32];
           tc_ld32(lane_addr + AT_O_COL + cc, ov);
 #pragma unroll
@@ -320,8 +329,8 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
         const int nvalid = pos_last - key_base + 1, nzero = AT_KT - nvalid;
         const int s = i % AT_STAGES;
         if (!wait_all(&v_full[s], (i / AT_STAGES) & 1)) { ok = false; break; }
-        unsigned char* vst = kv_s + s * 2 * AT_KV_BYTES + AT_KV_BYTES;
-        for (int e = r; e < nzero * 8 * AT_DH; e += AT_ROWS) {
+        unsigned char* vst = kv_s + s * AT_STAGE_BYTES + AT_K_BYTES;
+        for (int e = r; e < nzero * 8 * AT_VH; e += AT_ROWS) {
           const int half = e / (nzero * 8), rem = e - half * (nzero * 8);
           *reinterpret_cast<uint4*>(vst + half * AT_HALF_BYTES + (nvalid + (rem >> 3)) * 128 + ((rem & 7) << 4)) = make_uint4(0, 0, 0, 0);
         }
@@ -368,18 +377,20 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
     }
     if (ok && ntiles > 0 && wait_all(&pv_done[(ntiles - 1) % AT_NBUF], ((ntiles - 1) / AT_NBUF) & 1)) {
       tc_fence_after();
-      if (P.sink && valid) l += exp2f(-m_used);     // the sink's weight, relative to the maximum in use
-      const float inv = l > 0.f ? 1.f / l : 0.f;
       const int tk = valid ? row / G : 0, h = valid ? row - tk * G : 0;
-      bf16* dst = P.out + (size_t)(tok0 + tk) * P.out_stride + (size_t)(g * G + h) * HEAD_DIM;
-      const bf16* gt = P.gate ? P.gate + (size_t)(tok0 + tk) * P.gate_stride + (size_t)(g * G + h) * HEAD_DIM : nullptr;
+      // the sink's weight, relative to the maximum in use
+      if (P.sinks && valid) l += exp2f(fmaf(P.sinks[g * G + h], 1.4426950408889634f, -m_used));
+      const float inv = l > 0.f ? 1.f / l : 0.f;
+      bf16* dst = P.out + (size_t)(tok0 + tk) * P.out_stride + (size_t)(g * G + h) * VALUE_DIM;
+      const bf16* gt = P.gate ? P.gate + (size_t)(tok0 + tk) * P.gate_stride + (size_t)(g * G + h) * VALUE_DIM : nullptr;
 #pragma unroll 1
-      for (int cc = 0; cc < HEAD_DIM; cc += 32) {
+      for (int cc = 0; cc < VALUE_DIM; cc += 32) {
         uint32_t ov[32];
         tc_ld32(lane_addr + AT_O_COL + cc, ov);
         if (valid) {
 #pragma unroll
           for (int j = 0; j < 32; j += 8) {
+            if (VALUE_DIM % 32 != 0 && cc + j >= VALUE_DIM) continue;
             if (gt) {
               // eight gates of this row (16 bytes): the output times sigmoid(gate), folded into the numbers before `inv`
               const uint4 gz = *reinterpret_cast<const uint4*>(gt + cc + j);
@@ -415,8 +426,8 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
 PHOTON_API int photon_attention_tc_head_dim() { return HEAD_DIM; }
 
 // Runs the requests of the step that bring more than 16 rows (tokens x group); the others are left
-// untouched.  q [T, n_q * d] with row stride q_stride, out [T, n_q * d]; k_cache, v_cache
-// [num_pages, n_kv, page_size, d] contiguous.  group at most 128, page_size a multiple of 8 that
+// untouched.  q [T, n_q * d] with row stride q_stride, out [T, n_q * dv]; k_cache
+// [num_pages, n_kv, page_size, d] and v_cache [num_pages, n_kv, page_size, dv] contiguous.  group at most 128, page_size a multiple of 8 that
 // divides 64 or is a multiple of 64.
 PHOTON_API int photon_attention_tc(const void* q, long q_stride, void* out, long out_stride, const void* k_cache,
                                    const void* v_cache, const int* block_table, int max_pages, const int* cu_tokens,
@@ -424,17 +435,17 @@ PHOTON_API int photon_attention_tc(const void* q, long q_stride, void* out, long
                                    int page_size, int num_pages, int window, float scale, int* err,
                                    cudaStream_t stream) {
   return photon_attention_tc_ex(q, q_stride, out, out_stride, k_cache, v_cache, block_table, max_pages, cu_tokens, positions,
-                                S, max_tokens_per_seq, T, n_q, n_kv, d, page_size, num_pages, window, scale, err, 0, 0, 0.f,
+                                S, max_tokens_per_seq, T, n_q, n_kv, d, page_size, num_pages, window, scale, err, 0, nullptr, 0.f,
                                 nullptr, 0, stream);
 }
 
-// The same with kept first keys, a sink and bounded scores (see AttnTcParams), and an optional gate: bfloat16
-// [T, n_q * d] with row stride gate_stride (16-byte aligned rows); every output is multiplied by sigmoid(gate).
+// The same with kept first keys, sinks and bounded scores (see AttnTcParams), and an optional gate: bfloat16
+// [T, n_q * dv] with row stride gate_stride (16-byte aligned rows); every output is multiplied by sigmoid(gate).
 PHOTON_API int photon_attention_tc_ex(const void* q, long q_stride, void* out, long out_stride, const void* k_cache,
                                       const void* v_cache, const int* block_table, int max_pages, const int* cu_tokens,
                                       const int* positions, int S, int max_tokens_per_seq, int T, int n_q, int n_kv, int d,
                                       int page_size, int num_pages, int window, float scale, int* err, int keep_first,
-                                      int sink, float softcap, const void* gate, long gate_stride, cudaStream_t stream) {
+                                      const float* sinks, float softcap, const void* gate, long gate_stride, cudaStream_t stream) {
   if (S <= 0 || T <= 0) return 0;
   if (keep_first < 0 || softcap < 0.f) return PHOTON_ERR_ARGUMENT;
   if (d != HEAD_DIM || n_kv <= 0 || n_q % n_kv || !(scale > 0.f)) return PHOTON_ERR_UNSUPPORTED;
@@ -462,7 +473,7 @@ PHOTON_API int photon_attention_tc_ex(const void* q, long q_stride, void* out, l
   }
   int st = make_map(&map_k, k_cache, total_rows, d, d, box_rows);
   if (st != 0) return st;
-  st = make_map(&map_v, v_cache, total_rows, d, d, box_rows);
+  st = make_map(&map_v, v_cache, total_rows, VALUE_DIM, VALUE_DIM, box_rows);
   if (st != 0) return st;
   AttnTcParams P;
   P.out = (bf16*)out; P.out_stride = out_stride; P.block_table = block_table; P.max_pages = max_pages;
@@ -470,7 +481,7 @@ PHOTON_API int photon_attention_tc_ex(const void* q, long q_stride, void* out, l
   P.page_size = page_size;
   P.num_pages = num_pages; P.box_rows = box_rows; P.window = window; P.total_rows = (int)total_rows;
   P.scale_log2 = scale * 1.4426950408889634f; P.err = err;
-  P.keep_first = window > 0 ? keep_first : 0; P.sink = sink; P.softcap = softcap; P.cap_in = 0.f;
+  P.keep_first = window > 0 ? keep_first : 0; P.sinks = sinks; P.softcap = softcap; P.cap_in = 0.f;
   if (softcap > 0.f) { P.cap_in = scale / softcap; P.scale_log2 = 1.4426950408889634f; }
   if (gate != nullptr && (((uintptr_t)gate & 15) || (gate_stride & 7))) return PHOTON_ERR_ARGUMENT;
   P.gate = (const bf16*)gate; P.gate_stride = gate_stride;

@@ -56,7 +56,7 @@ def build_dir() -> str:
     for c in candidates:
         try:
             os.makedirs(c, exist_ok=True)
-            probe = os.path.join(c, f".probe_{os.getpid()}")
+            probe = os.path.join(c, f".probe_{os.getpid()}_{threading.get_ident()}")
             with open(probe, "w") as f:
                 f.write("x")
             os.remove(probe)

@@ -192,6 +192,129 @@ PHOTON_API int photon_add_rmsnorm(const void* delta, int delta_dtype, const void
   return photon_add_rmsnorm_scaled(delta, delta_dtype, delta2, residual, w, w_dtype, out, out_dtype, rows, n, H, eps, nullptr, stream);
 }
 
+// ---------------------------------------------------------------- norm of a sublayer's output, sum, next norm
+// A sublayer between two norms leaves y; residual (float, in place) += pw * (y / rms(y)), out = w * (residual / rms(residual)),
+// rms(x) = sqrt(mean(x^2) + eps) with an eps of its own for each.  rows as in add_rmsnorm_kernel: only the listed rows are
+// read and nothing is written back.  A thread keeps QUADS groups of four numbers of the row in registers; the row's order
+// of summation depends on H alone.
+template <typename TY, typename TO, int QUADS>
+__global__ void __launch_bounds__(1024)
+add_normed_rmsnorm_kernel(const TY* y, const void* __restrict__ pw, int pw_bf16, float peps, float* residual,
+                          const void* __restrict__ w, int w_bf16, float eps, TO* out, const int* rows, int H) {
+  __shared__ float red[32];
+  pdl_wait();
+  const int r = rows ? rows[blockIdx.x] : blockIdx.x;
+  const TY* yr = y + (size_t)r * H;
+  float* res = residual + (size_t)r * H;
+  float v[QUADS][4], x[QUADS][4];
+  float ss = 0.f;
+#pragma unroll
+  for (int u = 0; u < QUADS; ++u) {
+    const int i = (u * blockDim.x + threadIdx.x) * 4;
+#pragma unroll
+    for (int e = 0; e < 4; ++e) v[u][e] = x[u][e] = 0.f;
+    if (i < H) { Quad<TY>::load(yr + i, v[u]); Quad<float>::load(res + i, x[u]); }
+#pragma unroll
+    for (int e = 0; e < 4; ++e) ss += v[u][e] * v[u][e];
+  }
+  ss = block_sum(ss, red);
+  const float pinv = 1.0f / sqrtf(ss / (float)H + peps);
+  ss = 0.f;
+#pragma unroll
+  for (int u = 0; u < QUADS; ++u) {
+    const int i = (u * blockDim.x + threadIdx.x) * 4;
+    if (i < H) {
+      float p[4];
+      if (pw_bf16) Quad<bf16>::load((const bf16*)pw + i, p); else Quad<float>::load((const float*)pw + i, p);
+#pragma unroll
+      for (int e = 0; e < 4; ++e) { x[u][e] += p[e] * (v[u][e] * pinv); ss += x[u][e] * x[u][e]; }
+    }
+  }
+  ss = block_sum(ss, red);
+  pdl_launch_dependents();
+  const float inv = 1.0f / sqrtf(ss / (float)H + eps);
+  TO* o = out + (size_t)blockIdx.x * H;
+#pragma unroll
+  for (int u = 0; u < QUADS; ++u) {
+    const int i = (u * blockDim.x + threadIdx.x) * 4;
+    if (i < H) {
+      float wv[4], z[4];
+      if (w_bf16) Quad<bf16>::load((const bf16*)w + i, wv); else Quad<float>::load((const float*)w + i, wv);
+      if (!rows) Quad<float>::store(res + i, x[u]);
+#pragma unroll
+      for (int e = 0; e < 4; ++e) z[e] = wv[e] * (x[u][e] * inv);
+      Quad<TO>::store(o + i, z);
+    }
+  }
+}
+
+// Rows whose width is not a multiple of four, or that are wider than the registers hold: the row waits in shared memory.
+template <typename TY, typename TO>
+__global__ void add_normed_rmsnorm_any_kernel(const TY* y, const void* __restrict__ pw, int pw_bf16, float peps, float* residual,
+                                              const void* __restrict__ w, int w_bf16, float eps, TO* out, const int* rows, int H) {
+  __shared__ float red[32];
+  extern __shared__ __align__(16) float stash[];
+  pdl_wait();
+  const int r = rows ? rows[blockIdx.x] : blockIdx.x;
+  const TY* yr = y + (size_t)r * H;
+  float* res = residual + (size_t)r * H;
+  float ss = 0.f;
+  for (int i = threadIdx.x; i < H; i += blockDim.x) { const float v = to_f32(yr[i]); stash[i] = v; ss += v * v; }
+  ss = block_sum(ss, red);
+  const float pinv = 1.0f / sqrtf(ss / (float)H + peps);
+  ss = 0.f;
+  for (int i = threadIdx.x; i < H; i += blockDim.x) {
+    const float x = res[i] + load_w(pw, pw_bf16, i) * (stash[i] * pinv);
+    stash[i] = x;
+    if (!rows) res[i] = x;
+    ss += x * x;
+  }
+  ss = block_sum(ss, red);
+  pdl_launch_dependents();
+  const float inv = 1.0f / sqrtf(ss / (float)H + eps);
+  for (int i = threadIdx.x; i < H; i += blockDim.x) out[(size_t)blockIdx.x * H + i] = from_f32<TO>(load_w(w, w_bf16, i) * (stash[i] * inv));
+}
+
+template <typename TY, typename TO>
+static int add_normed_rmsnorm_launch(const void* y, const void* pw, int pb, float peps, float* residual, const void* w, int wb,
+                                     float eps, void* out, const int* rows, int n, int H, cudaStream_t stream) {
+  const bool vec = H % 4 == 0 && H <= 16384 && (uintptr_t)y % 16 == 0 && (uintptr_t)residual % 16 == 0 && (uintptr_t)pw % 16 == 0 &&
+                   (uintptr_t)w % 16 == 0 && (uintptr_t)out % 16 == 0;
+  if (vec) {
+    int threads = 128;
+    while (threads < 1024 && threads * 8 < H) threads <<= 1;   // depends on H only
+#define ANR_GO(Q) return launch_pdl(add_normed_rmsnorm_kernel<TY, TO, Q>, dim3(n), dim3(threads), 0, stream, (const TY*)y, pw, pb, \
+                                    peps, residual, w, wb, eps, (TO*)out, rows, H)
+    if (H <= threads * 4) ANR_GO(1);
+    if (H <= threads * 8) ANR_GO(2);
+    ANR_GO(4);
+  }
+  const size_t smem = (size_t)H * sizeof(float);
+  if (smem > 200 * 1024) return PHOTON_ERR_UNSUPPORTED;
+  if (smem > 48 * 1024) {
+    cudaError_t e = cudaFuncSetAttribute(add_normed_rmsnorm_any_kernel<TY, TO>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    if (e != cudaSuccess) return (int)e;
+  }
+  return launch_pdl(add_normed_rmsnorm_any_kernel<TY, TO>, dim3(n), dim3(256), smem, stream, (const TY*)y, pw, pb, peps, residual, w,
+                    wb, eps, (TO*)out, rows, H);
+}
+
+// y [*, H] of y_dtype, pw and w [H] of their dtypes, residual float [*, H], out [n, H] of out_dtype.  rows (int [n], may be
+// null): only these rows of y and residual are read, and the residual stays as it is.
+PHOTON_API int photon_add_normed_rmsnorm(const void* y, int y_dtype, const void* pw, int pw_dtype, float post_eps, float* residual,
+                                         const void* w, int w_dtype, float eps, void* out, int out_dtype, const int* rows, int n,
+                                         int H, cudaStream_t stream) {
+  if (n <= 0) return 0;
+  if (H <= 0 || y == nullptr || pw == nullptr || w == nullptr || residual == nullptr || out == nullptr) return PHOTON_ERR_ARGUMENT;
+  const int pb = pw_dtype == PHOTON_BF16, wb = w_dtype == PHOTON_BF16;
+#define ANR_T(TY, TO) return add_normed_rmsnorm_launch<TY, TO>(y, pw, pb, post_eps, residual, w, wb, eps, out, rows, n, H, stream)
+  if (y_dtype == PHOTON_BF16 && out_dtype == PHOTON_BF16) ANR_T(bf16, bf16);
+  if (y_dtype == PHOTON_F32 && out_dtype == PHOTON_F32) ANR_T(float, float);
+  if (y_dtype == PHOTON_F32 && out_dtype == PHOTON_BF16) ANR_T(float, bf16);
+  if (y_dtype == PHOTON_BF16 && out_dtype == PHOTON_F32) ANR_T(bf16, float);
+  return PHOTON_ERR_ARGUMENT;
+}
+
 // The same with a layer norm: out = (x - mean(x)) / sqrt(var(x) + eps) * w + b, x = residual + delta (+ delta2).
 // b may be null.
 PHOTON_API int photon_add_layernorm_scaled(const void* delta, int delta_dtype, const void* delta2, float* residual, const void* w,
@@ -388,16 +511,16 @@ PHOTON_API int photon_activation(const void* x, void* out, int dtype, long total
   return launch_status();
 }
 
-// x [T, W] (row stride ldx, in place) *= sigmoid(g [T, W]) (row stride ldg; its own type): the gate of a mixer's
-// output.  The sigmoid and the product are 32-bit, the result is rounded once.
+// x [T, W] (row stride ldx, in place) *= sigmoid(g [T, W / span]) (row stride ldg; its own type): the gate of a mixer's
+// output, one number for `span` neighbouring columns.  The sigmoid and the product are 32-bit, the result is rounded once.
 template <typename TX, typename TG>
-__global__ void gate_mul_kernel(TX* x, long ldx, const TG* g, long ldg, int W, size_t total) {
+__global__ void gate_mul_kernel(TX* x, long ldx, const TG* g, long ldg, int W, int span, size_t total) {
   size_t idx = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
   const size_t stride = (size_t)gridDim.x * blockDim.x;
   for (; idx < total; idx += stride) {
     const size_t t = idx / W;
     const int i = (int)(idx - t * W);
-    const float z = to_f32(g[t * ldg + i]);
+    const float z = to_f32(g[t * ldg + i / span]);
     x[t * ldx + i] = from_f32<TX>(to_f32(x[t * ldx + i]) / (1.0f + expf(-z)));
   }
 }
@@ -421,11 +544,12 @@ __global__ void gate_mul_vec_kernel(TX* x, long ldx, const TG* g, long ldg, int 
   }
 }
 
-PHOTON_API int photon_gate_mul(void* x, long ldx, int x_dtype, const void* g, long ldg, int g_dtype, int T, int W,
+PHOTON_API int photon_gate_mul(void* x, long ldx, int x_dtype, const void* g, long ldg, int g_dtype, int T, int W, int span,
                                cudaStream_t stream) {
+  if (span < 1 || W % span) return PHOTON_ERR_ARGUMENT;
   const size_t total = (size_t)T * W;
   if (total == 0) return 0;
-  const bool vec = (W % 4 == 0) && (ldx % 4 == 0) && (ldg % 4 == 0) && ((uintptr_t)x % 16 == 0) && ((uintptr_t)g % 16 == 0);
+  const bool vec = span == 1 && (W % 4 == 0) && (ldx % 4 == 0) && (ldg % 4 == 0) && ((uintptr_t)x % 16 == 0) && ((uintptr_t)g % 16 == 0);
   size_t blocks = ((vec ? total / 4 : total) + 255) / 256;
   const size_t cap = (size_t)photon_sm_count() * 16;
   if (blocks > cap) blocks = cap;
@@ -436,9 +560,9 @@ PHOTON_API int photon_gate_mul(void* x, long ldx, int x_dtype, const void* g, lo
     else return PHOTON_ERR_ARGUMENT;
     return launch_status();
   }
-  if (x_dtype == PHOTON_BF16 && g_dtype == PHOTON_BF16) gate_mul_kernel<bf16, bf16><<<(int)blocks, 256, 0, stream>>>((bf16*)x, ldx, (const bf16*)g, ldg, W, total);
-  else if (x_dtype == PHOTON_BF16 && g_dtype == PHOTON_F32) gate_mul_kernel<bf16, float><<<(int)blocks, 256, 0, stream>>>((bf16*)x, ldx, (const float*)g, ldg, W, total);
-  else if (x_dtype == PHOTON_F32 && g_dtype == PHOTON_F32) gate_mul_kernel<float, float><<<(int)blocks, 256, 0, stream>>>((float*)x, ldx, (const float*)g, ldg, W, total);
+  if (x_dtype == PHOTON_BF16 && g_dtype == PHOTON_BF16) gate_mul_kernel<bf16, bf16><<<(int)blocks, 256, 0, stream>>>((bf16*)x, ldx, (const bf16*)g, ldg, W, span, total);
+  else if (x_dtype == PHOTON_BF16 && g_dtype == PHOTON_F32) gate_mul_kernel<bf16, float><<<(int)blocks, 256, 0, stream>>>((bf16*)x, ldx, (const float*)g, ldg, W, span, total);
+  else if (x_dtype == PHOTON_F32 && g_dtype == PHOTON_F32) gate_mul_kernel<float, float><<<(int)blocks, 256, 0, stream>>>((float*)x, ldx, (const float*)g, ldg, W, span, total);
   else return PHOTON_ERR_ARGUMENT;
   return launch_status();
 }

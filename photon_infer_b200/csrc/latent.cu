@@ -144,7 +144,7 @@ PHOTON_API int photon_latent_q_rope(const void* q, long q_stride, int dtype, int
 template <typename T>
 __global__ void __launch_bounds__(256)
 head_linear_kernel(const T* __restrict__ x, long x_row, long x_head, const T* __restrict__ W, T* __restrict__ out,
-                   long o_row, long o_head, int M, int N, int K, const T* __restrict__ gate, long gate_row) {
+                   long o_row, long o_head, int M, int N, int K, const T* __restrict__ gate, long gate_row, int gate_heads) {
   __shared__ float As[HL_BK][HL_BM + 4];
   __shared__ float Ws[HL_BK][HL_BN + 4];
   const int h = blockIdx.z;
@@ -189,7 +189,7 @@ head_linear_kernel(const T* __restrict__ x, long x_row, long x_head, const T* __
     for (int j = 0; j < 4; ++j) {
       const int gn = n0 + tx * 4 + j;
       if (gn < N) {
-        const float g = gate ? 1.0f + expf(-to_f32(gate[(size_t)gm * gate_row + (size_t)h * N + gn])) : 1.0f;
+        const float g = gate ? 1.0f + expf(-to_f32(gate[(size_t)gm * gate_row + (gate_heads ? h : (size_t)h * N + gn)])) : 1.0f;
         out[(size_t)gm * o_row + (size_t)h * o_head + gn] = from_f32<T>(gate ? acc[i][j] / g : acc[i][j]);
       }
     }
@@ -219,7 +219,7 @@ template <int GROUPS>
 __global__ void __launch_bounds__(128)
 head_linear_skinny_kernel(const bf16* __restrict__ x, long x_row, long x_head, const bf16* __restrict__ W,
                           bf16* __restrict__ out, long o_row, long o_head, int M, int N, int K,
-                          const bf16* __restrict__ gate, long gate_row, int ksplit, int feature_blocks, HeadRope R) {
+                          const bf16* __restrict__ gate, long gate_row, int gate_heads, int ksplit, int feature_blocks, HeadRope R) {
   __shared__ float part[4][16][GROUPS * 8];
   const int h = blockIdx.y, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   if ((int)blockIdx.x >= feature_blocks) {
@@ -272,13 +272,13 @@ head_linear_skinny_kernel(const bf16* __restrict__ x, long x_row, long x_head, c
     if (n >= N) continue;
     float v = 0.f;
     for (int u = 0; u < ksplit; ++u) v += part[tile * ksplit + u][f][m];
-    if (gate) v /= 1.0f + expf(-__bfloat162float(gate[(size_t)m * gate_row + (size_t)h * N + n]));
+    if (gate) v /= 1.0f + expf(-__bfloat162float(gate[(size_t)m * gate_row + (gate_heads ? h : (size_t)h * N + n)]));
     out[(size_t)m * o_row + (size_t)h * o_head + n] = __float2bfloat16_rn(v);
   }
 }
 
 static int head_linear_skinny_launch(const void* x, long x_row, long x_head, const void* W, void* out, long o_row, long o_head,
-                                     int M, int heads, int N, int K, const void* gate, long gate_row, const HeadRope* rope,
+                                     int M, int heads, int N, int K, const void* gate, long gate_row, int gate_heads, const HeadRope* rope,
                                      cudaStream_t stream) {
   // few features: cut k over the warps of a block, so that there are blocks for most SMs
   int ksplit = 1;
@@ -289,10 +289,10 @@ static int head_linear_skinny_launch(const void* x, long x_row, long x_head, con
   if (rope) r = *rope;
   if (M <= 8)
     head_linear_skinny_kernel<1><<<grid, 128, 0, stream>>>((const bf16*)x, x_row, x_head, (const bf16*)W, (bf16*)out, o_row, o_head, M,
-                                                         N, K, (const bf16*)gate, gate_row, ksplit, feature_blocks, r);
+                                                         N, K, (const bf16*)gate, gate_row, gate_heads, ksplit, feature_blocks, r);
   else
     head_linear_skinny_kernel<2><<<grid, 128, 0, stream>>>((const bf16*)x, x_row, x_head, (const bf16*)W, (bf16*)out, o_row, o_head, M,
-                                                         N, K, (const bf16*)gate, gate_row, ksplit, feature_blocks, r);
+                                                         N, K, (const bf16*)gate, gate_row, gate_heads, ksplit, feature_blocks, r);
   return launch_status();
 }
 
@@ -311,27 +311,27 @@ PHOTON_API int photon_latent_absorb(const void* q, long q_stride, int dtype, con
   if (dim <= 0 || rot <= 0 || rot_dims < 0 || rot_dims > rot || (rot_dims & 1)) return PHOTON_ERR_ARGUMENT;
   if (!head_linear_skinny_ok(q, q_stride, dim + rot, W, dtype, M, heads, dim)) return PHOTON_ERR_UNSUPPORTED;
   const HeadRope r = {(const bf16*)q, q_stride, positions, inv_freq, (bf16*)out, out_stride, out_head, out_off, dim, rot, rot_dims, interleaved};
-  return head_linear_skinny_launch(q, q_stride, dim + rot, W, out, out_stride, out_head, M, heads, N, dim, nullptr, 0, &r, stream);
+  return head_linear_skinny_launch(q, q_stride, dim + rot, W, out, out_stride, out_head, M, heads, N, dim, nullptr, 0, 0, &r, stream);
 }
 
 // x [M][heads][K] and out [M][heads][N] with row and head strides in elements; W [heads][N][K] contiguous.  gate (may be
 // null; the type of x, [M][heads * N] with row stride gate_row): every output is multiplied by sigmoid(gate) before it
-// is rounded.
+// is rounded.  gate_heads != 0: gate is [M][heads], one number for all outputs of a head.
 PHOTON_API int photon_head_linear(const void* x, long x_row, long x_head, const void* W, void* out, long o_row,
                                   long o_head, int dtype, int M, int heads, int N, int K, const void* gate, long gate_row,
-                                  cudaStream_t stream) {
+                                  int gate_heads, cudaStream_t stream) {
   if (M <= 0 || heads <= 0 || N <= 0) return 0;
   if (K <= 0) return PHOTON_ERR_ARGUMENT;
   if (head_linear_skinny_ok(x, x_row, x_head, W, dtype, M, heads, K))
-    return head_linear_skinny_launch(x, x_row, x_head, W, out, o_row, o_head, M, heads, N, K, gate, gate_row, nullptr, stream);
+    return head_linear_skinny_launch(x, x_row, x_head, W, out, o_row, o_head, M, heads, N, K, gate, gate_row, gate_heads, nullptr, stream);
   dim3 grid((N + HL_BN - 1) / HL_BN, (M + HL_BM - 1) / HL_BM, heads);
   if (grid.y > 65535 || grid.z > 65535) return PHOTON_ERR_UNSUPPORTED;
   if (dtype == PHOTON_BF16)
     head_linear_kernel<bf16><<<grid, 256, 0, stream>>>((const bf16*)x, x_row, x_head, (const bf16*)W, (bf16*)out, o_row,
-                                                      o_head, M, N, K, (const bf16*)gate, gate_row);
+                                                      o_head, M, N, K, (const bf16*)gate, gate_row, gate_heads);
   else
     head_linear_kernel<float><<<grid, 256, 0, stream>>>((const float*)x, x_row, x_head, (const float*)W, (float*)out,
-                                                       o_row, o_head, M, N, K, (const float*)gate, gate_row);
+                                                       o_row, o_head, M, N, K, (const float*)gate, gate_row, gate_heads);
   return launch_status();
 }
 
@@ -371,11 +371,12 @@ PHOTON_API int photon_gather_rows(const void* cache, int dtype, const int* table
 // ---------------------------------------------------------------- causal softmax over rows of scores
 // scores [rows][ld] float: column c is the key at position first_key + c; row r belongs to the token at position
 // first_pos + r / heads, which sees the keys up to its own position and, with window > 0, the last `window` of them.
-// probs [rows][ldp] = softmax(scale * scores) over the visible keys, zero elsewhere, up to column `cols`.  One block per
-// row, 32-bit throughout, rounded once on the way out.
+// probs [rows][ldp] = softmax(scale * scores) over the visible keys, zero elsewhere, up to column `cols`.  sinks [heads]
+// (may be null): row r's denominator also holds exp(sinks[r % heads]).  One block per row, 32-bit throughout, rounded once on the way out.
 template <typename T>
 __global__ void causal_softmax_kernel(const float* __restrict__ scores, long ld, T* __restrict__ probs, long ldp,
-                                      int heads, int first_pos, int first_key, int window, int cols, float scale) {
+                                      int heads, int first_pos, int first_key, int window, int cols, float scale,
+                                      const float* __restrict__ sinks) {
   __shared__ float red[32];
   const int r = blockIdx.x;
   const int pos = first_pos + r / heads;
@@ -394,6 +395,7 @@ __global__ void causal_softmax_kernel(const float* __restrict__ scores, long ld,
   float sum = 0.f;
   for (int i = lo + threadIdx.x; i < hi; i += blockDim.x) sum += expf(s[i] * scale - m);
   sum = block_sum(sum, red);
+  if (sinks) sum += expf(sinks[r % heads] - m);
   const float inv = 1.0f / sum;
   for (int i = threadIdx.x; i < cols; i += blockDim.x)
     p[i] = from_f32<T>(i >= lo && i < hi ? expf(s[i] * scale - m) * inv : 0.f);
@@ -401,13 +403,13 @@ __global__ void causal_softmax_kernel(const float* __restrict__ scores, long ld,
 
 PHOTON_API int photon_causal_softmax_rows(const float* scores, long ld, void* probs, long ldp, int dtype, int rows,
                                           int heads, int first_pos, int first_key, int window, int cols, float scale,
-                                          cudaStream_t stream) {
+                                          const float* sinks, cudaStream_t stream) {
   if (rows <= 0 || cols <= 0) return 0;
   if (heads <= 0 || first_pos < 0 || first_key < 0 || first_key > first_pos) return PHOTON_ERR_ARGUMENT;
   if (dtype == PHOTON_BF16)
-    causal_softmax_kernel<bf16><<<rows, 256, 0, stream>>>(scores, ld, (bf16*)probs, ldp, heads, first_pos, first_key, window, cols, scale);
+    causal_softmax_kernel<bf16><<<rows, 256, 0, stream>>>(scores, ld, (bf16*)probs, ldp, heads, first_pos, first_key, window, cols, scale, sinks);
   else
-    causal_softmax_kernel<float><<<rows, 256, 0, stream>>>(scores, ld, (float*)probs, ldp, heads, first_pos, first_key, window, cols, scale);
+    causal_softmax_kernel<float><<<rows, 256, 0, stream>>>(scores, ld, (float*)probs, ldp, heads, first_pos, first_key, window, cols, scale, sinks);
   return launch_status();
 }
 
@@ -555,7 +557,8 @@ latent_decode_kernel(const bf16* __restrict__ q, long q_stride, const bf16* __re
 // One block per (token, head).  A token's shares that hold keys come first, so the sums run over those alone.
 #define LM_THREADS 128
 __global__ void __launch_bounds__(LM_THREADS)
-latent_merge_kernel(const float* __restrict__ part, int splits, int dv, bf16* __restrict__ out, long out_stride, int heads) {
+latent_merge_kernel(const float* __restrict__ part, int splits, int dv, bf16* __restrict__ out, long out_stride, int heads,
+                    const float* __restrict__ sinks) {
   __shared__ float wgt[LM_THREADS];
   const int t = blockIdx.x, h = blockIdx.y, lane = threadIdx.x & 31;
   const size_t row = (size_t)t * heads + h;
@@ -572,6 +575,7 @@ latent_merge_kernel(const float* __restrict__ part, int splits, int dv, bf16* __
     if (ms != -INFINITY) { l += ml[2 * s + 1] * expf(ms - m); ++used; }
   }
   l = warp_sum(l);
+  if (sinks) l += expf(sinks[h] - m);                          // one more key with this score and no value
   for (int d = 16; d > 0; d >>= 1) used += __shfl_xor_sync(0xffffffffu, used, d);
   const float inv = l > 0.f ? 1.0f / l : 0.f;
   for (int j0 = 0; j0 < dv; j0 += LM_THREADS * 4) {
@@ -603,12 +607,13 @@ latent_merge_kernel(const float* __restrict__ part, int splits, int dv, bf16* __
 // [T][heads * dv]: token t at position positions[t] of request token_seq[t] sees the rows 0 .. positions[t], with
 // window > 0 the last `window` of them; a row's value is its first dv numbers.  width and dv multiples of 16.  splits >=
 // ceil((largest position + 1) / 64), with a window no more than ceil((window - 1) / 64) + 1 are needed;
-// part: float [T * heads * splits * (dv + 2)].
+// part: float [T * heads * splits * (dv + 2)].  sinks (float [heads], may be null): the softmax of head h has one more key
+// with the score sinks[h] (not scaled) and no value.
 PHOTON_API int photon_latent_decode_attention(const void* q, long q_stride, const void* cache, const int* block_table,
                                               int max_pages, const int* token_seq, const int* positions, int T_,
                                               int heads, int width, int dv, int page_size, int num_pages, float scale,
-                                              int window, int splits, float* part, void* out, long out_stride, int* err,
-                                              cudaStream_t stream) {
+                                              int window, int splits, float* part, void* out, long out_stride,
+                                              const float* sinks, int* err, cudaStream_t stream) {
   if (T_ <= 0) return 0;
   if (heads <= 0 || splits <= 0 || part == nullptr || dv > width) return PHOTON_ERR_ARGUMENT;
   if (width % 16 || dv % 16 || q_stride % 8 || (uintptr_t)q % 16 || (uintptr_t)cache % 16 || (uintptr_t)part % 32 || splits > 65535 || heads > 65535)
@@ -623,6 +628,6 @@ PHOTON_API int photon_latent_decode_attention(const void* q, long q_stride, cons
       max_pages, token_seq, positions, heads, width, dv, page_size, num_pages, scale, window, splits, part, err);
   int st = launch_status();
   if (st != 0) return st;
-  latent_merge_kernel<<<dim3(T_, heads), LM_THREADS, 0, stream>>>(part, splits, dv, (bf16*)out, out_stride, heads);
+  latent_merge_kernel<<<dim3(T_, heads), LM_THREADS, 0, stream>>>(part, splits, dv, (bf16*)out, out_stride, heads, sinks);
   return launch_status();
 }

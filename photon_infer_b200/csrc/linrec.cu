@@ -1,9 +1,9 @@
 // Recurrent mixers whose state is one matrix per head, S [N][dv] in 32-bit, that decays by ONE number per head and
-// token and takes a rank-one update:
+// token (modes 0 and 1) or by a number per row (mode 2) and takes a rank-one update:
 //
 //   S_t = keep_t S_(t-1) + take_t k_t v_t^T,      o_t = S_t^T q_t                        (per head)
 //
-// Two mixers are this recurrence with different gates.
+// Three mixers are this recurrence with different gates.
 //
 //   state-space (mode 0):  k = B_t, q = C_t (of the head's group), v = x_t;  dt = softplus(dt_raw + dt_bias[h]);
 //                          keep = exp(-exp(A_log[h]) dt), take = dt;  y_t = o_t + D[h] x_t.
@@ -11,11 +11,17 @@
 //                          a running maximum m (from 0): m_t = max(f + m_(t-1), i); keep = exp(f + m_(t-1) - m_t),
 //                          take = exp(i - m_t); a vector n_t = keep n_(t-1) + take k_t rides along as one more
 //                          column of S (with v = 1);  y_t = o_t / (max(|n_t . q_t|, exp(-m_t)) + 1e-6).
+//   forget-and-write (mode 2): a gate per row f = l + (1 - l) sigmoid(z + b) keeps and 1 - f writes, so that a row of the
+//                          state is a running mean of the values: S_t = S_(t-1) + k_t (v_t^T - S_(t-1)) with the write gate
+//                          k = (1 - l) / (1 + exp(z + b)), formed without the cancellation in 1 - f;  y_t = o_t.  q enters
+//                          as silu(q).
 //
 //   photon_conv_silu        y = silu(bias + causal convolution over `taps` tokens per channel); the taps before the
 //                           step's first token of a request come from the request's state.
 //   photon_conv_state       the last taps - 1 input rows of every request of the step go into its state.
 //   photon_linrec           the recurrence over the tokens of a step, for all requests and heads.
+//   photon_linrec_gates     mode 2: silu(q) and the write gates of all tokens side by side, for long portions, whose blocks
+//                           would otherwise form them once per sixteen columns (few tokens: photon_linrec does it itself).
 //
 // A request's state is one float row per layer; S [H][N][dv] comes first, then (mode 1) n [H][N] and m [H]; the
 // convolution's rows live at an offset the caller gives.  A state slot of -1 starts from zeros and stores nothing.
@@ -138,6 +144,29 @@ __device__ __forceinline__ void lr_cp16(float* dst, const float* src) {
 __device__ __forceinline__ void lr_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
 template <int K> __device__ __forceinline__ void lr_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(K) : "memory"); }
 
+// Mode 2's inputs.
+__device__ __forceinline__ float lr_silu(float x) { return x / (1.0f + expf(-x)); }
+__device__ __forceinline__ float lr_write_gate(float z, float bias, float lower) { return (1.0f - lower) / (1.0f + expf(z + bias)); }
+
+__global__ void linrec_gates_kernel(const float* __restrict__ q, long q_stride, const float* __restrict__ z, long z_stride,
+                                    const float* __restrict__ bias, const float* __restrict__ lower, float* __restrict__ q_out,
+                                    float* __restrict__ k_out, long out_stride, int C) {
+  const int t = blockIdx.y, c = blockIdx.x * blockDim.x + threadIdx.x;
+  if (c >= C) return;
+  q_out[(size_t)t * out_stride + c] = lr_silu(q[(size_t)t * q_stride + c]);
+  k_out[(size_t)t * out_stride + c] = lr_write_gate(z[(size_t)t * z_stride + c], bias[c], lower[c]);
+}
+
+// q, z float [T][C] views, bias and lower float [C]; q_out = silu(q), k_out = (1 - lower) sigmoid(-(z + bias)).
+PHOTON_API int photon_linrec_gates(const float* q, long q_stride, const float* z, long z_stride, const float* bias,
+                                   const float* lower, float* q_out, float* k_out, long out_stride, int T, int C,
+                                   cudaStream_t stream) {
+  if (T <= 0 || C <= 0) return 0;
+  if (T > 65535) return PHOTON_ERR_UNSUPPORTED;
+  linrec_gates_kernel<<<dim3((C + 255) / 256, T), 256, 0, stream>>>(q, q_stride, z, z_stride, bias, lower, q_out, k_out, out_stride, C);
+  return launch_status();
+}
+
 // Eight shares of one sum, added in a fixed order.
 __device__ __forceinline__ float lr_sum8(const float* p) {
   const float4 a = *reinterpret_cast<const float4*>(p), b = *reinterpret_cast<const float4*>(p + 4);
@@ -197,6 +226,7 @@ linrec_kernel(const float* __restrict__ q, long q_stride, const float* __restric
   __syncthreads();
   const int t0 = cu_tokens[s], t1 = cu_tokens[s + 1];
   const float a_h = MODE == 0 ? expf(p0[h]) : 0.f;     // the head's decay rate
+  const bool raw_gates = MODE == 2 && p0 != nullptr;   // mode 2: q and k arrive as projected
 
   auto issue = [&](int base, int stage) {
     const int cnt = min(LR_CHUNK, t1 - base);
@@ -225,7 +255,7 @@ linrec_kernel(const float* __restrict__ q, long q_stride, const float* __restric
       lr_cp4(vd + tt * LR_COLS + cc, v + (size_t)(base + tt) * v_stride + (size_t)h * dv + c0 + cc);
     }
     float* rd = raw + (size_t)stage * 2 * LR_CHUNK;
-    if (tid < cnt) lr_cp4(rd + tid, ga + (size_t)(base + tid) * g_stride + h);
+    if (MODE != 2 && tid < cnt) lr_cp4(rd + tid, ga + (size_t)(base + tid) * g_stride + h);
     else if (MODE == 1 && tid >= 32 && tid < 32 + cnt) lr_cp4(rd + LR_CHUNK + tid - 32, gb + (size_t)(base + tid - 32) * g_stride + h);
     lr_commit();
   };
@@ -237,8 +267,8 @@ linrec_kernel(const float* __restrict__ q, long q_stride, const float* __restric
     __syncthreads();                                   // the chunk before is written out: the other stage is free
     if (base + LR_CHUNK < t1) { issue(base + LR_CHUNK, stage ^ 1); lr_wait<1>(); } else lr_wait<0>();
     __syncthreads();                                   // this chunk has landed for every thread
-    const float* kd = ks + (size_t)stage * LR_CHUNK * NPS;
-    const float* qd = qs + (size_t)stage * LR_CHUNK * NPS;
+    float* kd = ks + (size_t)stage * LR_CHUNK * NPS;
+    float* qd = qs + (size_t)stage * LR_CHUNK * NPS;
     const float* vd = vs + (size_t)stage * LR_CHUNK * LR_COLS;
     const float* rd = raw + (size_t)stage * 2 * LR_CHUNK;
     if (MODE == 0) {
@@ -246,6 +276,14 @@ linrec_kernel(const float* __restrict__ q, long q_stride, const float* __restric
         const float dt = lr_softplus(rd[tid] + p1[h]);
         keep_s[tid] = expf(-a_h * dt);
         take_s[tid] = dt;
+      }
+    } else if (MODE == 2) {
+      if (raw_gates) {
+        for (int i = tid; i < cnt * N; i += LR_THREADS) {
+          const int tt = i / N, r = i - tt * N, at = tt * NPS + r + (r / RPL) * 4;
+          qd[at] = lr_silu(qd[at]);
+          kd[at] = lr_write_gate(kd[at], p0[(size_t)hq * N + r], p1[(size_t)hq * N + r]);
+        }
       }
     } else if (warp == 0) {
       float gi = 0.f, gf = 0.f;
@@ -269,17 +307,24 @@ linrec_kernel(const float* __restrict__ q, long q_stride, const float* __restric
     const float* ql = qd + sub * (RPL + 4);
 #pragma unroll 4
     for (int tt = 0; tt < cnt; ++tt) {
-      const float keep = keep_s[tt];
-      const float w = take_s[tt] * vd[tt * LR_COLS + col];
+      const float keep = MODE == 2 ? 0.f : keep_s[tt];
+      const float w = MODE == 2 ? vd[tt * LR_COLS + col] : take_s[tt] * vd[tt * LR_COLS + col];
       float a0 = 0.f, a1 = 0.f, a2 = 0.f, a3 = 0.f;
 #pragma unroll
       for (int j = 0; j < RPL / 4; ++j) {
         const float4 k4 = *reinterpret_cast<const float4*>(kl + tt * NPS + 4 * j);
         const float4 q4 = *reinterpret_cast<const float4*>(ql + tt * NPS + 4 * j);
-        S[4 * j + 0] = fmaf(k4.x, w, keep * S[4 * j + 0]);
-        S[4 * j + 1] = fmaf(k4.y, w, keep * S[4 * j + 1]);
-        S[4 * j + 2] = fmaf(k4.z, w, keep * S[4 * j + 2]);
-        S[4 * j + 3] = fmaf(k4.w, w, keep * S[4 * j + 3]);
+        if (MODE == 2) {
+          S[4 * j + 0] = fmaf(k4.x, w - S[4 * j + 0], S[4 * j + 0]);
+          S[4 * j + 1] = fmaf(k4.y, w - S[4 * j + 1], S[4 * j + 1]);
+          S[4 * j + 2] = fmaf(k4.z, w - S[4 * j + 2], S[4 * j + 2]);
+          S[4 * j + 3] = fmaf(k4.w, w - S[4 * j + 3], S[4 * j + 3]);
+        } else {
+          S[4 * j + 0] = fmaf(k4.x, w, keep * S[4 * j + 0]);
+          S[4 * j + 1] = fmaf(k4.y, w, keep * S[4 * j + 1]);
+          S[4 * j + 2] = fmaf(k4.z, w, keep * S[4 * j + 2]);
+          S[4 * j + 3] = fmaf(k4.w, w, keep * S[4 * j + 3]);
+        }
         a0 = fmaf(S[4 * j + 0], q4.x, a0);
         a1 = fmaf(S[4 * j + 1], q4.y, a1);
         a2 = fmaf(S[4 * j + 2], q4.z, a2);
@@ -293,7 +338,7 @@ linrec_kernel(const float* __restrict__ q, long q_stride, const float* __restric
       if (c0 + cc >= dv) continue;
       float y = lr_sum8(os[tt][cc]) * q_scale;         // the queries' factor, taken out of the sums
       if (MODE == 0) y = fmaf(p2[h], vd[tt * LR_COLS + cc], y);
-      else y = y / (fmaxf(fabsf(lr_sum8(os[tt][LR_COLS - 1]) * q_scale), floor_s[tt]) + 1e-6f);
+      else if (MODE == 1) y = y / (fmaxf(fabsf(lr_sum8(os[tt][LR_COLS - 1]) * q_scale), floor_s[tt]) + 1e-6f);
       out[(size_t)(base + tt) * out_stride + (size_t)h * dv + c0 + cc] = y;
     }
   }
@@ -350,7 +395,8 @@ static int linrec_launch(int rpl, dim3 grid, cudaStream_t stream, const float* q
 // q, k: float [T][qk_heads * N] views (row strides in elements); v float [T][H * dv]; ga, gb: float [T][H] views with row
 // stride g_stride, the raw gate inputs (mode 0: ga = dt_raw, gb unused; mode 1: ga = i_raw, gb = f_raw).  p0, p1, p2: float
 // [H] (mode 0: A_log, dt_bias, D; mode 1: the input gate's bias, the forget gate's bias, unused).  cap: the gates' bound
-// (mode 1).  q_scale multiplies the queries.  out float [T][H * dv] (row stride out_stride).  Head h reads query/key head
+// (mode 1).  Mode 2: k holds the raw gates z, p0 and p1 float [qk_heads * N] their biases and lower bounds; p0 null: q and k
+// hold silu(q) and the write gates already (photon_linrec_gates); ga, gb are not read.  q_scale multiplies the queries.  out float [T][H * dv] (row stride out_stride).  Head h reads query/key head
 // h / (H / qk_heads).  state: float [num_slots][state_stride], see the top of the file.
 PHOTON_API int photon_linrec(int mode, const float* q, long q_stride, const float* k, long k_stride, const float* v,
                              long v_stride, const float* ga, const float* gb, long g_stride, const float* p0, const float* p1,
@@ -358,7 +404,7 @@ PHOTON_API int photon_linrec(int mode, const float* q, long q_stride, const floa
                              float* state, long state_stride, int num_slots, float* out, long out_stride, int S, int H,
                              int qk_heads, int N, int dv, int* err, cudaStream_t stream) {
   if (S <= 0) return 0;
-  if (mode != 0 && mode != 1) return PHOTON_ERR_ARGUMENT;
+  if (mode < 0 || mode > 2 || (mode == 2 && (p0 == nullptr) != (p1 == nullptr))) return PHOTON_ERR_ARGUMENT;
   if (H <= 0 || qk_heads <= 0 || H % qk_heads || N <= 0 || dv <= 0) return PHOTON_ERR_ARGUMENT;
   if (mode == 1 && !(cap > 0.f)) return PHOTON_ERR_ARGUMENT;
   if (N > 512 || H > 65535 || S > 65535) return PHOTON_ERR_UNSUPPORTED;
@@ -367,6 +413,9 @@ PHOTON_API int photon_linrec(int mode, const float* q, long q_stride, const floa
   dim3 grid((dv + real - 1) / real, H, S);
   if (mode == 0)
     return linrec_launch<0>(rpl, grid, stream, q, q_stride, k, k_stride, v, v_stride, ga, gb, g_stride, p0, p1, p2, cap, q_scale,
+                            cu_tokens, state_slots, state, state_stride, num_slots, out, out_stride, H, qk_heads, N, dv, err);
+  if (mode == 2)
+    return linrec_launch<2>(rpl, grid, stream, q, q_stride, k, k_stride, v, v_stride, ga, gb, g_stride, p0, p1, p2, cap, q_scale,
                             cu_tokens, state_slots, state, state_stride, num_slots, out, out_stride, H, qk_heads, N, dv, err);
   return linrec_launch<1>(rpl, grid, stream, q, q_stride, k, k_stride, v, v_stride, ga, gb, g_stride, p0, p1, p2, cap, q_scale,
                           cu_tokens, state_slots, state, state_stride, num_slots, out, out_stride, H, qk_heads, N, dv, err);

@@ -11,6 +11,10 @@
 //   photon_moe_combine   out[t] = sum_j weight[t, j] * y[place(t, j)] (+ the shared expert's output), the sum in
 //                        32-bit in the order of j.
 //
+// Identity experts: the last outputs of the router may stand for experts without matrices whose output is the token's own
+// row.  Their pairs carry ids from the number of real experts on; they take the last places of the sorted order, no product
+// touches them, and the weighted sum adds the token's row.
+//
 // Every output of a product is one chain of K fused multiply-adds in ascending k, accumulated in 32-bit, so a
 // token's result depends neither on the other tokens of the step nor on its place in the sorted order.
 #include "common.cuh"
@@ -30,12 +34,13 @@ __global__ void moe_route_kernel(const T* __restrict__ h, long h_stride, const T
                                  const void* __restrict__ bias, int bias_bf16, int H, int E, int top,
                                  int* __restrict__ ids, float* __restrict__ weights, int* __restrict__ counts, int T_,
                                  int mode, int n_groups, int keep_groups, float route_scale,
-                                 const T* __restrict__ Wsg, float* __restrict__ shared_gate, int tok) {
-  extern __shared__ float logits[];                     // per token: E (+ 1: the shared expert's gate) + n_groups flags
+                                 const T* __restrict__ Wsg, float* __restrict__ shared_gate, int tok,
+                                 const float* __restrict__ correction, int real) {
+  extern __shared__ float logits[];                     // per token: E (+ 1: the shared expert's gate) + n_groups flags (mode 3: + E)
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nwarp = blockDim.x >> 5;
   const int t0 = blockIdx.x * tok;
   const int ntok = min(tok, T_ - t0);
-  const int LS = E + 1 + n_groups;
+  const int LS = E + 1 + n_groups + (mode == 3 ? E : 0);
   constexpr int V = 16 / sizeof(T);                      // elements of a 16-byte load
   const bool vec = (H % V == 0) && ((uintptr_t)h % 16 == 0) && (h_stride % V == 0) && ((uintptr_t)Wr % 16 == 0) &&
                    ((uintptr_t)Wsg % 16 == 0);
@@ -81,7 +86,41 @@ __global__ void moe_route_kernel(const T* __restrict__ h, long h_stride, const T
   float* lg = logits + warp * LS;
   const bool first = lane == 0;
   if (first && Wsg) shared_gate[t] = 1.0f / (1.0f + expf(-lg[E]));
-  if (E <= 32 && (mode == 1 || (mode == 2 && !(n_groups > 1 && keep_groups < n_groups)))) {
+  if (mode == 3) {
+    // Scores are the softmax over all experts; the choice goes by score + correction, the weights are the chosen scores as
+    // they are, times route_scale.  Lane i keeps the experts i, i + 32, ..; equal choice scores: the lower index.
+    float* choice = lg + E + 1 + n_groups;
+    float mx = -INFINITY;
+    for (int e = lane; e < E; e += 32) mx = fmaxf(mx, lg[e]);
+    mx = warp_max(mx);
+    float den = 0.f;
+    for (int e = lane; e < E; e += 32) den += expf(lg[e] - mx);
+    den = warp_sum(den);
+    for (int e = lane; e < E; e += 32) {
+      const float p = expf(lg[e] - mx) / den;
+      lg[e] = p;
+      choice[e] = p + (correction ? correction[e] : 0.f);
+    }
+    for (int j = 0; j < top; ++j) {
+      float bv = -INFINITY;
+      int best = 0x7fffffff;
+      for (int e = lane; e < E; e += 32)
+        if (choice[e] > bv) { bv = choice[e]; best = e; }
+#pragma unroll
+      for (int o = 16; o > 0; o >>= 1) {
+        const float ov = __shfl_xor_sync(0xffffffffu, bv, o);
+        const int oe = __shfl_xor_sync(0xffffffffu, best, o);
+        if (ov > bv || (ov == bv && oe < best)) { bv = ov; best = oe; }
+      }
+      if (best >= E) best = 0;                           // no score is a number: any expert in range
+      if (lane == (best & 31)) {                         // the lane that keeps it
+        ids[(size_t)t * top + j] = best;
+        weights[(size_t)t * top + j] = lg[best] * route_scale;
+        atomicAdd(&counts[min(best, real)], 1);
+        choice[best] = -INFINITY;
+      }
+    }
+  } else if (E <= 32 && (mode == 1 || (mode == 2 && !(n_groups > 1 && keep_groups < n_groups)))) {
     // The same rules as the serial forms below with one lane per expert: maxima and sums by shuffles, a choice is the
     // lowest lane that holds the maximum (so ties go to the lower index).  top <= E <= 32.
     const unsigned full = 0xffffffffu;
@@ -211,48 +250,54 @@ PHOTON_API int photon_moe_route(const void* h, long h_stride, int dtype, const v
                                 int T_, int H, int E, int top, int* ids, float* weights, int* counts,
                                 cudaStream_t stream) {
   return photon_moe_route_ex(h, h_stride, dtype, Wr, bias, bias_dtype, T_, H, E, top, ids, weights, counts, 0, 1, 1, 1.0f,
-                             nullptr, nullptr, stream);
+                             nullptr, nullptr, nullptr, 0, stream);
 }
 
 // mode 0: as above.  mode 1: scores are the softmax over all experts; with n_groups > 1 the experts form that many
 // equal groups of neighbours and only experts of the keep_groups groups with the largest best score can be chosen; the
 // weights are the chosen scores divided by their sum (+ 1e-20) times route_scale.  mode 2: scores are sigmoid(logit); a
 // group's score is the sum of its two largest scores; the weights are the chosen scores times route_scale, not divided
-// by their sum.  Wsg (may be null): one more row
+// by their sum.  mode 3: scores are the softmax over all experts, those with the largest score + correction [E] (may be
+// null) are chosen, the weights are the chosen scores without the correction times route_scale, not divided by their sum.
+// identity (mode 3): the last `identity` of the E router outputs are identity experts; counts has E - identity + 1 entries
+// then, the last of which counts all their pairs.  Wsg (may be null): one more row
 // [H] of the router's type; shared_gate [T] then gets sigmoid(Wsg . h), the gate of a shared expert.
 PHOTON_API int photon_moe_route_ex(const void* h, long h_stride, int dtype, const void* Wr, const void* bias, int bias_dtype,
                                    int T_, int H, int E, int top, int* ids, float* weights, int* counts, int mode,
                                    int n_groups, int keep_groups, float route_scale, const void* Wsg, float* shared_gate,
-                                   cudaStream_t stream) {
+                                   const float* correction, int identity, cudaStream_t stream) {
   if (T_ <= 0) return 0;
   if (E <= 0 || top <= 0 || top > E || H <= 0) return PHOTON_ERR_ARGUMENT;
-  if (mode < 0 || mode > 2) return PHOTON_ERR_ARGUMENT;
+  if (mode < 0 || mode > 3) return PHOTON_ERR_ARGUMENT;
+  if (identity < 0 || identity >= E || (mode != 3 && (identity > 0 || correction)) || (mode == 3 && n_groups > 1)) return PHOTON_ERR_ARGUMENT;
   if (n_groups < 1 || keep_groups < 1 || keep_groups > n_groups || E % n_groups) return PHOTON_ERR_ARGUMENT;
   if (mode != 0 && n_groups > 1 && (long)keep_groups * (E / n_groups) < top) return PHOTON_ERR_ARGUMENT;
   if ((Wsg == nullptr) != (shared_gate == nullptr)) return PHOTON_ERR_ARGUMENT;
   const int warps = E >= 8 ? 8 : (E >= 4 ? 4 : 2);
   // few tokens (a decode step): one per block, so that every token's logits form on an SM of their own
   const int tok = T_ >= 64 ? (warps < 4 ? warps : 4) : 1;
-  const size_t smem = (size_t)tok * (E + 1 + n_groups) * sizeof(float);
+  const size_t smem = (size_t)tok * (E + 1 + n_groups + (mode == 3 ? E : 0)) * sizeof(float);
+  const int buckets = identity > 0 ? E - identity + 1 : E, real = identity > 0 ? E - identity : E;
   if (smem > 48 * 1024) return PHOTON_ERR_UNSUPPORTED;
-  cudaError_t e = cudaMemsetAsync(counts, 0, (size_t)E * sizeof(int), stream);
+  cudaError_t e = cudaMemsetAsync(counts, 0, (size_t)buckets * sizeof(int), stream);
   if (e != cudaSuccess) return (int)e;
   const int blocks = (T_ + tok - 1) / tok;
   if (dtype == PHOTON_BF16)
     moe_route_kernel<bf16><<<blocks, warps * 32, smem, stream>>>((const bf16*)h, h_stride, (const bf16*)Wr, bias,
                                                                 bias_dtype == PHOTON_BF16, H, E, top, ids, weights, counts, T_,
-                                                                mode, n_groups, keep_groups, route_scale, (const bf16*)Wsg, shared_gate, tok);
+                                                                mode, n_groups, keep_groups, route_scale, (const bf16*)Wsg, shared_gate, tok, correction, real);
   else
     moe_route_kernel<float><<<blocks, warps * 32, smem, stream>>>((const float*)h, h_stride, (const float*)Wr, bias,
                                                                  bias_dtype == PHOTON_BF16, H, E, top, ids, weights, counts, T_,
-                                                                 mode, n_groups, keep_groups, route_scale, (const float*)Wsg, shared_gate, tok);
+                                                                 mode, n_groups, keep_groups, route_scale, (const float*)Wsg, shared_gate, tok, correction, real);
   return launch_status();
 }
 
 // ---------------------------------------------------------------- sort by expert
 // One block per expert e: its first row in the sorted order is the number of pairs of the experts before it, and
-// its pairs take the following places in the order in which they stand in `ids`.
-__global__ void moe_align_kernel(const int* __restrict__ ids, const int* __restrict__ counts, int n, int E,
+// its pairs take the following places in the order in which they stand in `ids`.  Ids from `real` on (identity experts)
+// are one bucket behind the others, without row tiles.
+__global__ void moe_align_kernel(const int* __restrict__ ids, const int* __restrict__ counts, int n, int E, int real,
                                  int* __restrict__ offsets, int* __restrict__ sorted, int* __restrict__ place,
                                  int* __restrict__ tiles, int* __restrict__ num_tiles) {
   __shared__ int warp_tot[32];
@@ -264,19 +309,19 @@ __global__ void moe_align_kernel(const int* __restrict__ ids, const int* __restr
     for (int i = 0; i < e; ++i) { off += counts[i]; tl += (counts[i] + MOE_BM - 1) / MOE_BM; }
     base_s = off;
     offsets[e] = off;
-    const int own = counts[e];
-    for (int i = 0; i * MOE_BM < own; ++i) {
+    const int own = counts[e], tiled = e < real ? own : 0;
+    for (int i = 0; i * MOE_BM < tiled; ++i) {
       tiles[3 * (tl + i)] = e;
       tiles[3 * (tl + i) + 1] = off + i * MOE_BM;
       tiles[3 * (tl + i) + 2] = min(MOE_BM, own - i * MOE_BM);
     }
-    if (e == E - 1) { offsets[E] = off + own; *num_tiles = tl + (own + MOE_BM - 1) / MOE_BM; }
+    if (e == E - 1) { offsets[E] = off + own; *num_tiles = tl + (tiled + MOE_BM - 1) / MOE_BM; }
   }
   __syncthreads();
   int running = base_s;
   for (int i0 = 0; i0 < n; i0 += blockDim.x) {
     const int i = i0 + threadIdx.x;
-    const bool mine = i < n && ids[i] == e;
+    const bool mine = i < n && min(ids[i], real) == e;
     const unsigned ballot = __ballot_sync(0xffffffffu, mine);
     const int before = __popc(ballot & ((1u << lane) - 1u));
     if (lane == 0) warp_tot[warp] = __popc(ballot);
@@ -291,11 +336,13 @@ __global__ void moe_align_kernel(const int* __restrict__ ids, const int* __restr
 
 // ids [n] (n = T * top), counts [E] -> offsets [E + 1], sorted [n] (pair index at each sorted row), place [n]
 // (sorted row of each pair), tiles [3 * max_tiles] (expert, first row, rows), num_tiles [1].
-// max_tiles >= n / MOE_BM + E always suffices.
-PHOTON_API int photon_moe_align(const int* ids, const int* counts, int n, int E, int* offsets, int* sorted, int* place,
+// max_tiles >= n / MOE_BM + E always suffices.  real = E: every bucket is an expert; real = E - 1: the last bucket holds the
+// pairs whose id is real or more (identity experts), behind the others and without row tiles.
+PHOTON_API int photon_moe_align(const int* ids, const int* counts, int n, int E, int real, int* offsets, int* sorted, int* place,
                                 int* tiles, int* num_tiles, cudaStream_t stream) {
   if (n <= 0 || E <= 0) return 0;
-  moe_align_kernel<<<E, 256, 0, stream>>>(ids, counts, n, E, offsets, sorted, place, tiles, num_tiles);
+  if (real != E && real != E - 1) return PHOTON_ERR_ARGUMENT;
+  moe_align_kernel<<<E, 256, 0, stream>>>(ids, counts, n, E, real, offsets, sorted, place, tiles, num_tiles);
   return launch_status();
 }
 
@@ -428,13 +475,18 @@ PHOTON_API int photon_moe_gemm(const void* A, long lda, int dtype, const int* ga
 template <typename TY, typename TO>
 __global__ void moe_combine_kernel(const TY* __restrict__ y, long ldy, const int* __restrict__ place,
                                    const float* __restrict__ weights, int top, const TO* __restrict__ shared_out,
-                                   TO* __restrict__ out, int H, const float* __restrict__ shared_gate) {
+                                   TO* __restrict__ out, int H, const float* __restrict__ shared_gate,
+                                   const int* __restrict__ ids, int real, const TO* __restrict__ x, long ldx) {
   const int t = blockIdx.x;
   for (int i = threadIdx.x; i < H; i += blockDim.x) {
     float acc = 0.f;
-    for (int j = 0; j < top; ++j)
-      acc = fmaf(weights ? weights[(size_t)t * top + j] : 1.0f,
-                 to_f32(y[(size_t)(place ? place[(size_t)t * top + j] : t * top + j) * ldy + i]), acc);
+    for (int j = 0; j < top; ++j) {
+      const float w = weights ? weights[(size_t)t * top + j] : 1.0f;
+      if (ids && ids[(size_t)t * top + j] >= real)       // an identity expert: the token's own row
+        acc = fmaf(w, to_f32(x[(size_t)t * ldx + i]), acc);
+      else
+        acc = fmaf(w, to_f32(y[(size_t)(place ? place[(size_t)t * top + j] : t * top + j) * ldy + i]), acc);
+    }
     if (shared_out) acc += shared_gate ? shared_gate[t] * to_f32(shared_out[(size_t)t * H + i]) : to_f32(shared_out[(size_t)t * H + i]);
     out[(size_t)t * H + i] = from_f32<TO>(acc);
   }
@@ -444,21 +496,24 @@ __global__ void moe_combine_kernel(const TY* __restrict__ y, long ldy, const int
 // weights [T][top] (null: all 1, experts whose inputs were weighted); shared_out [T][H] (may be null) and out [T][H] of out_dtype.
 PHOTON_API int photon_moe_combine(const void* y, long ldy, int y_dtype, const int* place, const float* weights, int top,
                                   const void* shared_out, void* out, int out_dtype, int T_, int H, cudaStream_t stream) {
-  return photon_moe_combine_ex(y, ldy, y_dtype, place, weights, top, shared_out, nullptr, out, out_dtype, T_, H, stream);
+  return photon_moe_combine_ex(y, ldy, y_dtype, place, weights, top, shared_out, nullptr, nullptr, 0, nullptr, 0, out, out_dtype, T_, H, stream);
 }
 
-// The same; shared_gate [T] (may be null): the shared expert's output of token t is multiplied by shared_gate[t].
+// The same; shared_gate [T] (may be null): the shared expert's output of token t is multiplied by shared_gate[t].  ids
+// [T][top] (may be null): a pair whose id is real or more adds row t of x [T][H] (of out_dtype, row stride ldx) instead of
+// its row of y, which is not read.
 PHOTON_API int photon_moe_combine_ex(const void* y, long ldy, int y_dtype, const int* place, const float* weights, int top,
-                                     const void* shared_out, const float* shared_gate, void* out, int out_dtype, int T_,
-                                     int H, cudaStream_t stream) {
+                                     const void* shared_out, const float* shared_gate, const int* ids, int real, const void* x,
+                                     long ldx, void* out, int out_dtype, int T_, int H, cudaStream_t stream) {
   if (T_ <= 0) return 0;
+  if (ids != nullptr && x == nullptr) return PHOTON_ERR_ARGUMENT;
   const int threads = H >= 1024 ? 256 : 128;
   if (out_dtype == PHOTON_BF16 && y_dtype == PHOTON_F32)
-    moe_combine_kernel<float, bf16><<<T_, threads, 0, stream>>>((const float*)y, ldy, place, weights, top, (const bf16*)shared_out, (bf16*)out, H, shared_gate);
+    moe_combine_kernel<float, bf16><<<T_, threads, 0, stream>>>((const float*)y, ldy, place, weights, top, (const bf16*)shared_out, (bf16*)out, H, shared_gate, ids, real, (const bf16*)x, ldx);
   else if (out_dtype == PHOTON_BF16 && y_dtype == PHOTON_BF16)
-    moe_combine_kernel<bf16, bf16><<<T_, threads, 0, stream>>>((const bf16*)y, ldy, place, weights, top, (const bf16*)shared_out, (bf16*)out, H, shared_gate);
+    moe_combine_kernel<bf16, bf16><<<T_, threads, 0, stream>>>((const bf16*)y, ldy, place, weights, top, (const bf16*)shared_out, (bf16*)out, H, shared_gate, ids, real, (const bf16*)x, ldx);
   else if (out_dtype == PHOTON_F32 && y_dtype == PHOTON_F32)
-    moe_combine_kernel<float, float><<<T_, threads, 0, stream>>>((const float*)y, ldy, place, weights, top, (const float*)shared_out, (float*)out, H, shared_gate);
+    moe_combine_kernel<float, float><<<T_, threads, 0, stream>>>((const float*)y, ldy, place, weights, top, (const float*)shared_out, (float*)out, H, shared_gate, ids, real, (const float*)x, ldx);
   else
     return PHOTON_ERR_ARGUMENT;
   return launch_status();
@@ -545,10 +600,11 @@ template <typename TO, bool GLU>
 __global__ void __launch_bounds__(256)
 moe_gemv_kernel(const bf16* __restrict__ x, long ldx, int x_div, const int* __restrict__ ids, const bf16* __restrict__ W,
                 TO* __restrict__ out, long ldo, int N, int K, int act, const float* __restrict__ weights, float limit,
-                float slope) {
+                float slope, int experts) {
   extern __shared__ __align__(16) bf16 xs[];
   const int p = blockIdx.y;
   const int e = ids[p];
+  if (e >= experts) return;                              // an identity expert: nothing to multiply
   const int cols = GLU ? N / 2 : N;
   const bf16* xr = x + (size_t)(p / x_div) * ldx;
   for (int i = threadIdx.x * 8; i < K; i += blockDim.x * 8)
@@ -592,8 +648,9 @@ moe_gemv_kernel(const bf16* __restrict__ x, long ldx, int x_div, const int* __re
 
 // x [*][K] bfloat16: pair p reads row p / x_div.  ids [n]: the expert of every pair.  W [E][N][K] bfloat16.
 // out [n][N] float or bfloat16 (glu: [n][N / 2]), rows in the order of the pairs.  weights [n] (may be null): pair p's
-// sums are multiplied by weights[p] before the activation.  K % 8 == 0, 16-byte aligned rows.
-PHOTON_API int photon_moe_gemv(const void* x, long ldx, int x_div, const int* ids, int n, const void* W, void* out, long ldo,
+// sums are multiplied by weights[p] before the activation.  experts: E; the rows of pairs whose id is E or more are left as
+// they are.  K % 8 == 0, 16-byte aligned rows.
+PHOTON_API int photon_moe_gemv(const void* x, long ldx, int x_div, const int* ids, int n, const void* W, int experts, void* out, long ldo,
                                int out_dtype, int N, int K, int glu, int act, const float* weights, float limit,
                                float slope, cudaStream_t stream) {
   if (n <= 0 || N <= 0) return 0;
@@ -605,7 +662,7 @@ PHOTON_API int photon_moe_gemv(const void* x, long ldx, int x_div, const int* id
 #define MOE_GEMV(TO, GLU) do { \
     if (smem > 48 * 1024) { cudaError_t e_ = cudaFuncSetAttribute(moe_gemv_kernel<TO, GLU>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
                             if (e_ != cudaSuccess) return (int)e_; } \
-    moe_gemv_kernel<TO, GLU><<<grid, 256, smem, stream>>>((const bf16*)x, ldx, x_div, ids, (const bf16*)W, (TO*)out, ldo, N, K, act, weights, limit, slope); } while (0)
+    moe_gemv_kernel<TO, GLU><<<grid, 256, smem, stream>>>((const bf16*)x, ldx, x_div, ids, (const bf16*)W, (TO*)out, ldo, N, K, act, weights, limit, slope, experts); } while (0)
   if (out_dtype == PHOTON_BF16) { if (glu) MOE_GEMV(bf16, true); else MOE_GEMV(bf16, false); }
   else if (out_dtype == PHOTON_F32) { if (glu) MOE_GEMV(float, true); else MOE_GEMV(float, false); }
   else return PHOTON_ERR_ARGUMENT;

@@ -1,8 +1,10 @@
-// Per-head RMS norm of queries and keys, rotation of their first dimensions, and the write of keys and values into
-// the paged cache, in one pass over the projected row of a token.
+// RMS norm of queries and keys, rotation of their first dimensions, and the write of keys and values into the paged
+// cache, in one pass over the projected row of a token.
 //
-//   y = x / sqrt(mean(x^2) + eps) [* w]           per head, over its d numbers; w [d] is shared by all heads
-//   (y[j], y[j + r/2]) <- (y[j] c - y[j + r/2] s, y[j + r/2] c + y[j] s),  j < r/2, angle = position * inv_freq[j]
+//   y = x / sqrt(mean(x^2) + eps) [* w]           per head, over its d numbers, w [d] shared by all heads; or (whole_row)
+//                                                 over all numbers of q (and of k) at once, w [n_q d] and [n_kv d]
+//   (y[a], y[b]) <- (y[a] c - y[b] s, y[b] c + y[a] s),  j < r/2, angle = position * inv_freq[j], where the pair (a, b) of a
+//                                                 head is (j, j + r/2) or (interleaved) (2j, 2j + 1)
 //
 // r = rot_dims <= d; the other d - r numbers of a head pass unrotated.  Norm and rotation are 32-bit, the angle and its
 // sine and cosine 64-bit (a position of a few thousand times a frequency near 1 leaves 1e-4 of an angle's error in
@@ -40,7 +42,7 @@ qk_norm_rope_write_kernel(const TI* q, long q_stride, const TI* k, long k_stride
                           int w_bf16, float eps, const int* __restrict__ positions,
                           const double* __restrict__ inv_freq, int rot_dims, const int* __restrict__ slot_mapping,
                           TO* __restrict__ k_cache, TO* __restrict__ v_cache, int n_q, int n_kv, int d, int dv,
-                          int page_size, long num_slots, int* err) {
+                          int page_size, long num_slots, int* err, int interleaved) {
   extern __shared__ __align__(16) float qkn_smem[];
   pdl_wait();
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -102,9 +104,10 @@ qk_norm_rope_write_kernel(const TI* q, long q_stride, const TI* k, long k_stride
       double sn, cs;
       sincos(pos * inv_freq[j], &sn, &cs);
       const float c = (float)cs, s = (float)sn;
-      const float a = xs[j], b = xs[j + half];
-      xs[j] = a * c - b * s;
-      xs[j + half] = b * c + a * s;
+      const int ia = interleaved ? 2 * j : j, ib = interleaved ? 2 * j + 1 : j + half;
+      const float a = xs[ia], b = xs[ib];
+      xs[ia] = a * c - b * s;
+      xs[ib] = b * c + a * s;
     }
     __syncwarp();
   }
@@ -120,9 +123,107 @@ qk_norm_rope_write_kernel(const TI* q, long q_stride, const TI* k, long k_stride
   }
 }
 
+// The norm over the whole projection: one block per token.  The row (q, then k) waits in shared memory as 32-bit numbers
+// while its two sums of squares form; the sines and cosines of the token's position are computed once for all heads.
+#define QKR_THREADS 256
+template <typename TI, typename TO, bool VEC>
+__global__ void __launch_bounds__(QKR_THREADS)
+qk_row_norm_rope_write_kernel(const TI* q, long q_stride, const TI* k, long k_stride, const TI* v, long v_stride,
+                              TO* q_out, long qo_stride, const void* __restrict__ q_w, const void* __restrict__ k_w,
+                              int w_bf16, float eps, const int* __restrict__ positions,
+                              const double* __restrict__ inv_freq, int rot_dims, const int* __restrict__ slot_mapping,
+                              TO* __restrict__ k_cache, TO* __restrict__ v_cache, int n_q, int n_kv, int d, int dv,
+                              int page_size, long num_slots, int* err, int interleaved) {
+  extern __shared__ __align__(16) float qkn_smem[];
+  __shared__ float red[2][QKR_THREADS / 32];
+  const int t = blockIdx.x, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+  const int nq = n_q * d, nk = k_cache ? n_kv * d : 0, half = rot_dims >> 1;
+  float* xs = qkn_smem;                                // nq + nk numbers, then cosines, then sines
+  float* cs = xs + ((nq + nk + 3) & ~3);
+  float* sn = cs + half;
+  pdl_wait();
+  const double pos = (double)positions[t];
+  for (int j = tid; j < half; j += QKR_THREADS) {
+    double s, c;
+    sincos(pos * inv_freq[j], &s, &c);
+    cs[j] = (float)c;
+    sn[j] = (float)s;
+  }
+  float sq = 0.f, sk = 0.f;
+  const TI* qr = q + (size_t)t * q_stride;
+  const TI* kr = k_cache ? k + (size_t)t * k_stride : nullptr;
+  if (VEC) {
+    for (int i = tid * 4; i < nq; i += QKR_THREADS * 4) {
+      float f[4];
+      qkn_load4(qr + i, f);
+      qkn_store4(xs + i, f);
+      sq += (f[0] * f[0] + f[1] * f[1]) + (f[2] * f[2] + f[3] * f[3]);
+    }
+    for (int i = tid * 4; i < nk; i += QKR_THREADS * 4) {
+      float f[4];
+      qkn_load4(kr + i, f);
+      qkn_store4(xs + nq + i, f);
+      sk += (f[0] * f[0] + f[1] * f[1]) + (f[2] * f[2] + f[3] * f[3]);
+    }
+  } else {
+    for (int i = tid; i < nq; i += QKR_THREADS) { const float x = to_f32(qr[i]); xs[i] = x; sq += x * x; }
+    for (int i = tid; i < nk; i += QKR_THREADS) { const float x = to_f32(kr[i]); xs[nq + i] = x; sk += x * x; }
+  }
+  sq = warp_sum(sq);
+  sk = warp_sum(sk);
+  if (lane == 0) { red[0][warp] = sq; red[1][warp] = sk; }
+  __syncthreads();
+  sq = 0.f; sk = 0.f;
+#pragma unroll
+  for (int u = 0; u < QKR_THREADS / 32; ++u) { sq += red[0][u]; sk += red[1][u]; }
+  const float qinv = 1.0f / sqrtf(sq / (float)nq + eps);
+  const float kinv = nk ? 1.0f / sqrtf(sk / (float)nk + eps) : 0.f;
+
+  long slot = -1, page = 0;
+  int at = 0;
+  if (k_cache) {
+    slot = slot_mapping[t];
+    if (slot >= num_slots || slot < -1) {
+      if (tid == 0) report_error(err, PHOTON_DEV_BAD_SLOT, t, (int)slot, (int)num_slots);
+      slot = -1;
+    }
+    if (slot >= 0) { page = slot / page_size; at = (int)(slot - page * page_size); }
+  }
+  // number j of the head whose first number is xs[base], normed and rotated
+  auto value = [&](int base, int j, float inv, const void* w, int wbase) -> float {
+    auto normed = [&](int i) { return w ? xs[base + i] * inv * load_w(w, w_bf16, wbase + i) : xs[base + i] * inv; };
+    if (j >= rot_dims) return normed(j);
+    const int pair = interleaved ? (j >> 1) : (j >= half ? j - half : j);
+    const bool second = interleaved ? (j & 1) : (j >= half);
+    const int mate = interleaved ? (j ^ 1) : (second ? j - half : j + half);
+    const float own = normed(j), other = normed(mate);
+    return second ? own * cs[pair] + other * sn[pair] : own * cs[pair] - other * sn[pair];
+  };
+  constexpr int STEP = VEC ? 4 : 1;
+  const int last = slot >= 0 ? nq + nk : nq;
+  for (int i = tid * STEP; i < last; i += QKR_THREADS * STEP) {
+    const bool is_q = i < nq;
+    const int off = is_q ? i : i - nq, h = off / d, j = off - h * d;      // a head's first number is a multiple of STEP
+    TO* dst = is_q ? q_out + (size_t)t * qo_stride + off : k_cache + (((size_t)page * n_kv + h) * page_size + at) * d + j;
+    float f[STEP];
+#pragma unroll
+    for (int u = 0; u < STEP; ++u) f[u] = value(i - j, j + u, is_q ? qinv : kinv, is_q ? q_w : k_w, h * d);
+    if constexpr (VEC) qkn_store4(dst, f); else *dst = from_f32<TO>(f[0]);
+  }
+  if (slot >= 0) {
+    const TI* vr = v + (size_t)t * v_stride;
+    for (int i = tid * STEP; i < n_kv * dv; i += QKR_THREADS * STEP) {
+      const int h = i / dv, j = i - h * dv;
+      TO* dst = v_cache + (((size_t)page * n_kv + h) * page_size + at) * dv + j;
+      if constexpr (VEC) { float f[4]; qkn_load4(vr + i, f); qkn_store4(dst, f); } else *dst = from_f32<TO>(to_f32(vr[i]));
+    }
+  }
+}
+
 // q [T, n_q * d], k [T, n_kv * d], v [T, n_kv * dv] of in_dtype, each with its own row stride in elements (sections of
-// one fused row as a rule).  q_out [T, n_q * d] of out_dtype (row stride qo_stride).  q_w, k_w: norm weights [d] of
-// w_dtype, or null for a norm without a weight.  inv_freq: double [rot_dims / 2], null or rot_dims 0: no rotation.
+// one fused row as a rule).  q_out [T, n_q * d] of out_dtype (row stride qo_stride).  q_w, k_w: norm weights [d] (whole_row:
+// [n_q * d] and [n_kv * d]) of w_dtype, or null for a norm without a weight.  whole_row != 0: one norm over all of q and
+// one over all of k.  interleaved != 0: rotation pairs are neighbours.  inv_freq: double [rot_dims / 2], null or rot_dims 0: no rotation.
 // k_cache [pages, n_kv, page_size, d], v_cache [pages, n_kv, page_size, dv] of out_dtype; both null: nothing is stored
 // (an entry that reads another entry's pages), and k and v are not read.
 PHOTON_API int photon_qk_norm_rope_write(const void* q, long q_stride, const void* k, long k_stride, const void* v,
@@ -130,26 +231,34 @@ PHOTON_API int photon_qk_norm_rope_write(const void* q, long q_stride, const voi
                                          const void* q_w, const void* k_w, int w_dtype, float eps, const int* positions,
                                          const double* inv_freq, int rot_dims, const int* slot_mapping, void* k_cache,
                                          void* v_cache, int T, int n_q, int n_kv, int d, int dv, int page_size,
-                                         long num_slots, int* err, cudaStream_t stream) {
+                                         long num_slots, int whole_row, int interleaved, int* err, cudaStream_t stream) {
   if (T <= 0) return 0;
   if (d <= 0 || dv <= 0 || n_q <= 0 || n_kv <= 0 || rot_dims < 0 || (rot_dims & 1) || rot_dims > d) return PHOTON_ERR_ARGUMENT;
   if ((k_cache == nullptr) != (v_cache == nullptr)) return PHOTON_ERR_ARGUMENT;
   if (T > 65535 || d > 8192) return PHOTON_ERR_UNSUPPORTED;
   if (inv_freq == nullptr) rot_dims = 0;
   const int items = n_q + (k_cache ? 2 * n_kv : 0);
-  dim3 grid((items + QKN_WARPS - 1) / QKN_WARPS, T);
-  const size_t smem = (size_t)QKN_WARPS * d * sizeof(float);
+  const dim3 grid = whole_row ? dim3(T) : dim3((items + QKN_WARPS - 1) / QKN_WARPS, T);
+  const size_t smem = whole_row ? ((((size_t)n_q + (k_cache ? n_kv : 0)) * d + 3) / 4 * 4 + rot_dims) * sizeof(float)
+                                : (size_t)QKN_WARPS * d * sizeof(float);
+  if (smem > 220 * 1024) return PHOTON_ERR_UNSUPPORTED;
   const int wb = (w_dtype == PHOTON_BF16);
   const uintptr_t ia = in_dtype == PHOTON_F32 ? 16 : 8, oa = out_dtype == PHOTON_F32 ? 16 : 8;   // bytes of four elements
   const bool vec = d % 4 == 0 && dv % 4 == 0 && q_stride % 4 == 0 && k_stride % 4 == 0 && v_stride % 4 == 0 && qo_stride % 4 == 0 &&
                    (uintptr_t)q % ia == 0 && (uintptr_t)k % ia == 0 && (uintptr_t)v % ia == 0 && (uintptr_t)q_out % oa == 0 &&
                    (uintptr_t)k_cache % oa == 0 && (uintptr_t)v_cache % oa == 0;
-#define QKN_GO(TI, TO, VEC) do { \
-    if (smem > 48 * 1024) { cudaError_t e_ = cudaFuncSetAttribute(qk_norm_rope_write_kernel<TI, TO, VEC>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
+#define QKN_RUN(KERNEL, THREADS) do { \
+    if (smem > 48 * 1024) { cudaError_t e_ = cudaFuncSetAttribute(KERNEL, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
                             if (e_ != cudaSuccess) return (int)e_; } \
-    return launch_pdl(qk_norm_rope_write_kernel<TI, TO, VEC>, grid, dim3(QKN_WARPS * 32), smem, stream, (const TI*)q, q_stride, \
-        (const TI*)k, k_stride, (const TI*)v, v_stride, (TO*)q_out, qo_stride, q_w, k_w, wb, eps, positions, inv_freq, rot_dims, \
-        slot_mapping, (TO*)k_cache, (TO*)v_cache, n_q, n_kv, d, dv, page_size, num_slots, err); } while (0)
+    return launch_pdl(KERNEL, grid, dim3(THREADS), smem, stream, (const TI_*)q, q_stride, (const TI_*)k, k_stride, (const TI_*)v, \
+        v_stride, (TO_*)q_out, qo_stride, q_w, k_w, wb, eps, positions, inv_freq, rot_dims, slot_mapping, (TO_*)k_cache, \
+        (TO_*)v_cache, n_q, n_kv, d, dv, page_size, num_slots, err, interleaved); } while (0)
+#define QKN_GO(TI, TO, VEC) do { \
+    typedef TI TI_; typedef TO TO_; \
+    auto row_kernel = qk_row_norm_rope_write_kernel<TI, TO, VEC>; \
+    auto head_kernel = qk_norm_rope_write_kernel<TI, TO, VEC>; \
+    if (whole_row) QKN_RUN(row_kernel, QKR_THREADS); \
+    QKN_RUN(head_kernel, QKN_WARPS * 32); } while (0)
 #define QKN_LAUNCH(TI, TO) do { if (vec) QKN_GO(TI, TO, true); else QKN_GO(TI, TO, false); } while (0)
   if (in_dtype == PHOTON_F32 && out_dtype == PHOTON_F32) QKN_LAUNCH(float, float);
   if (in_dtype == PHOTON_F32 && out_dtype == PHOTON_BF16) QKN_LAUNCH(float, bf16);

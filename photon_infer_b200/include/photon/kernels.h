@@ -89,7 +89,12 @@ PHOTON_EXPORT int photon_scale_bias_rows(float* x, float scale, const void* bias
 /* out[i] = act(x[i]) over total elements of one dtype (x may be out); act: PHOTON_ACT_SILU, _GELU_TANH or _GELU. */
 PHOTON_EXPORT int photon_activation(const void* x, void* out, int dtype, long total, int act, cudaStream_t stream);
 /* x [T, W] (row stride ldx, in place) *= sigmoid(g [T, W]) (row stride ldg, its own dtype), in 32-bit, rounded once. */
-PHOTON_EXPORT int photon_gate_mul(void* x, long ldx, int x_dtype, const void* g, long ldg, int g_dtype, int T, int W, cudaStream_t stream);
+PHOTON_EXPORT int photon_gate_mul(void* x, long ldx, int x_dtype, const void* g, long ldg, int g_dtype, int T, int W, int span, cudaStream_t stream);
+/* A sublayer between two norms: residual [*, H] (float, in place) += pw * y / sqrt(mean(y^2) + post_eps), then out [n, H] = w *
+ * residual / sqrt(mean(residual^2) + eps).  rows (may be null): only these rows are read, the residual stays as it is. */
+PHOTON_EXPORT int photon_add_normed_rmsnorm(const void* y, int y_dtype, const void* pw, int pw_dtype, float post_eps, float* residual,
+                              const void* w, int w_dtype, float eps, void* out, int out_dtype, const int* rows, int n, int H,
+                              cudaStream_t stream);
 /* residual [T, H] (float, in place) += (delta + delta2) + other + bias; delta, delta2 [T, H] of delta_dtype, other [T, H]
  * float, bias [H] of bias_dtype; each may be null. */
 PHOTON_EXPORT int photon_stream_add(float* residual, const void* delta, const void* delta2, int delta_dtype, const float* other,
@@ -115,7 +120,7 @@ PHOTON_EXPORT int photon_qk_norm_rope_write(const void* q, long q_stride, const 
                               int in_dtype, void* q_out, long qo_stride, int out_dtype, const void* q_w, const void* k_w,
                               int w_dtype, float eps, const int* positions, const double* inv_freq, int rot_dims,
                               const int* slot_mapping, void* k_cache, void* v_cache, int T, int n_q, int n_kv, int d, int dv,
-                              int page_size, long num_slots, int* err, cudaStream_t stream);
+                              int page_size, long num_slots, int whole_row, int interleaved, int* err, cudaStream_t stream);
 
 /* ------------------------------------------------------------------ attention.cu (float32 and any even head size) */
 /* Values are dv wide: v_cache [num_pages][n_kv][page_size][dv], out [T][n_q * dv]; v_cache == k_cache (dv <= d): the value
@@ -125,14 +130,14 @@ PHOTON_EXPORT int photon_paged_attention(const void* q, long q_stride, void* out
                            const void* v_cache, const int* block_table, int max_pages, const int* token_seq,
                            const int* positions, int T_, int n_q, int n_kv, int d, int dv, int page_size, int num_pages,
                            int window, float scale, int splits, float* part, int* err, cudaStream_t stream);
-/* The same with kept first keys (keys < keep_first stay visible behind the window), a sink (one more key with score 0 and
- * no value in the softmax's denominator) and bounded scores (s <- softcap * tanh(s / softcap); 0: off).  gate (may be
+/* The same with kept first keys (keys < keep_first stay visible behind the window), sinks (float [n_q], may be null:
+ * one more key with this score and no value in head h's softmax) and bounded scores (s <- softcap * tanh(s / softcap); 0: off).  gate (may be
  * null; here and in the two tensor-core kernels below): [T, n_q * dv] of the type of q, row stride gate_stride; every
  * output is multiplied by sigmoid(gate) before it is rounded. */
 PHOTON_EXPORT int photon_paged_attention_ex(const void* q, long q_stride, void* out, long out_stride, int dtype, const void* k_cache,
                               const void* v_cache, const int* block_table, int max_pages, const int* token_seq,
                               const int* positions, int T_, int n_q, int n_kv, int d, int dv, int page_size, int num_pages,
-                              int window, float scale, int splits, float* part, int* err, int keep_first, int sink,
+                              int window, float scale, int splits, float* part, int* err, int keep_first, const float* sinks,
                               float softcap, const void* gate, long gate_stride, cudaStream_t stream);
 
 /* ------------------------------------------------------------------ latent.cu: attention over a cached latent */
@@ -150,9 +155,11 @@ PHOTON_EXPORT int photon_latent_q_rope(const void* q, long q_stride, int dtype, 
                          int interleaved, const int* positions, const float* inv_freq, void* out, long out_stride, int out_head,
                          int out_off, int T_, cudaStream_t stream);
 /* out[t, h, :] = W[h] x[t, h, :] for every head: x [M][heads][K], out [M][heads][N] (row and head strides in elements),
- * W [heads][N][K]; gate [M][heads * N] (row stride gate_row, may be null): times sigmoid(gate). */
+ * W [heads][N][K]; gate [M][heads * N] (row stride gate_row, may be null): times sigmoid(gate);
+ * gate_heads != 0: gate is [M][heads]. */
 PHOTON_EXPORT int photon_head_linear(const void* x, long x_row, long x_head, const void* W, void* out, long o_row, long o_head,
-                       int dtype, int M, int heads, int N, int K, const void* gate, long gate_row, cudaStream_t stream);
+                       int dtype, int M, int heads, int N, int K, const void* gate, long gate_row, int gate_heads,
+                       cudaStream_t stream);
 
 /* A decode step's queries in one launch (bfloat16, M <= 16, dim a multiple of 8, else PHOTON_ERR_UNSUPPORTED): out[m, h, :N] =
  * W[h] q[m, h, :dim] and out[m, h, out_off ..] = the rotated last rot numbers of the head. */
@@ -165,31 +172,33 @@ PHOTON_EXPORT int photon_gather_rows(const void* cache, int dtype, const int* ta
                        int first, int count, int valid_lo, int valid_hi, void* out, int* err, cudaStream_t stream);
 /* probs [rows][ldp] = softmax(scale * scores [rows][ld]) over the keys that row r sees, zero elsewhere, up to column cols:
  * column c is the key at first_key + c, row r the token at first_pos + r / heads, which sees the keys up to its own
- * position, with window > 0 the last window of them. */
+ * position, with window > 0 the last window of them.  sinks float [heads] (may be null): exp(sinks[r % heads]) joins the
+ * row's denominator. */
 PHOTON_EXPORT int photon_causal_softmax_rows(const float* scores, long ld, void* probs, long ldp, int dtype, int rows, int heads,
-                               int first_pos, int first_key, int window, int cols, float scale, cudaStream_t stream);
+                               int first_pos, int first_key, int window, int cols, float scale, const float* sinks,
+                               cudaStream_t stream);
 
 /* Decoded tokens on the tensor cores (bfloat16; width and dv multiples of 16): token t sees the rows 0 .. positions[t] of
  * request token_seq[t], with window > 0 the last window of them; a row's value is its first dv numbers.  splits >=
  * ceil((largest position + 1) / 64) (with a window ceil((window - 1) / 64) + 1 are always enough); part: float
- * [T * heads * splits * (dv + 2)]. */
+ * [T * heads * splits * (dv + 2)]; sinks float [heads], may be null. */
 PHOTON_EXPORT int photon_latent_decode_attention(const void* q, long q_stride, const void* cache, const int* block_table,
                                    int max_pages, const int* token_seq, const int* positions, int T_, int heads, int width,
                                    int dv, int page_size, int num_pages, float scale, int window, int splits, float* part,
-                                   void* out, long out_stride, int* err, cudaStream_t stream);
+                                   void* out, long out_stride, const float* sinks, int* err, cudaStream_t stream);
 
 /* ------------------------------------------------------------------ attention_latent_tc.cu (-DLT_NU=, -DLT_NR=, -DLT_NV=: 64-wide
  * chunks of d, r, v; bfloat16): long prompt portions over an expanded latent */
 /* q [T][heads][d + r] (the unrotated parts), q_rot [T][heads][r], kv [rows][>= heads * (d + v)]: heads x d key numbers then
  * heads x v value numbers per row, rot_rows [rows][r]: the key part all heads share; out [T][heads * v], times sigmoid(gate)
- * where gate is not null.  seqs (host): S x (first token, tokens, position of the first token, position of the request's
+ * where gate is not null (gate_heads != 0: gate is [T][heads]); sinks float [heads], may be null.  seqs (host): S x (first token, tokens, position of the first token, position of the request's
  * first row, that row).  d, r, v multiples of 8, everything 16-byte aligned. */
 PHOTON_EXPORT int photon_attention_latent_tc_chunks(void);
 PHOTON_EXPORT int photon_attention_latent_tc_max_seqs(void);
 PHOTON_EXPORT int photon_attention_latent_tc(const void* q, long q_stride, const void* q_rot, const void* kv, long kv_stride,
                                const void* rot_rows, long rot_stride, void* out, long out_stride, const void* gate,
-                               long gate_stride, const int* seqs, int S, int T, int rows, int heads, int d, int r, int v,
-                               int window, float scale, int* err, cudaStream_t stream);
+                               long gate_stride, int gate_heads, const float* sinks, const int* seqs, int S, int T, int rows,
+                               int heads, int d, int r, int v, int window, float scale, int* err, cudaStream_t stream);
 
 /* ------------------------------------------------------------------ hyper.cu: parallel residual streams */
 /* out [n][H] = norm(u) * w + bias, u = sum_s win[s] X_s (win null: the sum), after the pending write
@@ -278,12 +287,17 @@ PHOTON_EXPORT int photon_conv_state(const void* x, long x_stride, int x_dtype, i
 /* S_t = keep_t S_(t-1) + take_t k_t v_t^T, o_t = S_t^T q_t per head (S [N][dv] in the request's state row).  mode 0: a
  * state-space layer (keep = exp(-exp(A_log) dt), take = dt = softplus(ga + dt_bias), out = o + D v; p0, p1, p2 = A_log,
  * dt_bias, D).  mode 1: a matrix memory with capped log gates and a running maximum (ga, gb the raw input and forget
- * gates, p0, p1 their biases; out = o / (max(|n . q|, exp(-m)) + 1e-6); n [H][N] and m [H] follow S in the state row). */
+ * gates, p0, p1 their biases; out = o / (max(|n . q|, exp(-m)) + 1e-6); n [H][N] and m [H] follow S in the state row).
+ * mode 2: a gate per row, S_t = S_(t-1) + k (v^T - S_(t-1)), k = (1 - p1) / (1 + exp(z + p0)) with the raw gates z in k and p0,
+ * p1 [qk_heads * N], queries silu(q); p0 null: q and k come from photon_linrec_gates. */
 PHOTON_EXPORT int photon_linrec(int mode, const float* q, long q_stride, const float* k, long k_stride, const float* v,
                      long v_stride, const float* ga, const float* gb, long g_stride, const float* p0, const float* p1,
                      const float* p2, float cap, float q_scale, const int* cu_tokens, const int* state_slots, float* state,
                      long state_stride, int num_slots, float* out, long out_stride, int S, int H, int qk_heads, int N, int dv,
                      int* err, cudaStream_t stream);
+/* Mode 2's inputs of a long portion: q_out = silu(q), k_out = (1 - lower) / (1 + exp(z + bias)); q, z float [T][C] views. */
+PHOTON_EXPORT int photon_linrec_gates(const float* q, long q_stride, const float* z, long z_stride, const float* bias,
+                           const float* lower, float* q_out, float* k_out, long out_stride, int T, int C, cudaStream_t stream);
 
 /* ------------------------------------------------------------------ attention_talk.cu: attention whose heads' scores are mixed */
 /* Bias (float, may be null) on q [T][H * d] and k [T][G * d] of in_dtype, rotation of the first rot_dims numbers of a head
@@ -346,14 +360,18 @@ PHOTON_EXPORT int photon_moe_route(const void* h, long h_stride, int dtype, cons
                      int H, int E, int top, int* ids, float* weights, int* counts, cudaStream_t stream);
 /* mode 1: softmax over all experts, groups of neighbours of which only the keep_groups best (by their largest score) may
  * be chosen from, weights = chosen scores / (their sum + 1e-20) * route_scale.  mode 2: scores are sigmoid(logit), a group's
- * score is the sum of its two largest, weights = chosen scores * route_scale.  Wsg [H] (may be null): shared_gate [T] =
+ * score is the sum of its two largest, weights = chosen scores * route_scale.  mode 3: softmax over all experts, chosen by
+ * score + correction [E] (may be null), weights = chosen scores * route_scale; the last `identity` outputs are identity
+ * experts (counts then has E - identity + 1 entries).  Wsg [H] (may be null): shared_gate [T] =
  * sigmoid(Wsg . h). */
 PHOTON_EXPORT int photon_moe_route_ex(const void* h, long h_stride, int dtype, const void* Wr, const void* bias, int bias_dtype, int T_,
                         int H, int E, int top, int* ids, float* weights, int* counts, int mode, int n_groups, int keep_groups,
-                        float route_scale, const void* Wsg, float* shared_gate, cudaStream_t stream);
+                        float route_scale, const void* Wsg, float* shared_gate, const float* correction, int identity,
+                        cudaStream_t stream);
 /* Stable sort of the n = T * top pairs by expert: offsets [E + 1], sorted [n], place [n], tiles [3 * max_tiles] of
- * photon_moe_tile_rows() rows at most (expert, first row, rows), num_tiles [1]. */
-PHOTON_EXPORT int photon_moe_align(const int* ids, const int* counts, int n, int E, int* offsets, int* sorted, int* place,
+ * photon_moe_tile_rows() rows at most (expert, first row, rows), num_tiles [1].  real = E - 1: the last bucket holds the pairs
+ * whose id is real or more (identity experts), without tiles; else real = E. */
+PHOTON_EXPORT int photon_moe_align(const int* ids, const int* counts, int n, int E, int real, int* offsets, int* sorted, int* place,
                      int* tiles, int* num_tiles, cudaStream_t stream);
 PHOTON_EXPORT int photon_moe_tile_rows(void);
 /* Grouped product over the sorted rows with W [E][N][K]; gather (may be null): sorted row r reads A row
@@ -369,40 +387,44 @@ PHOTON_EXPORT int photon_moe_glu(const void* gate_up, void* out, int dtype, int 
 /* out[t] = sum_j weights[t, j] * y[place[t, j]] (+ shared_out[t]) (weights null: all 1); y [n][H] float or bfloat16; place null: row t * top + j. */
 PHOTON_EXPORT int photon_moe_combine(const void* y, long ldy, int y_dtype, const int* place, const float* weights, int top,
                        const void* shared_out, void* out, int out_dtype, int T_, int H, cudaStream_t stream);
-/* shared_gate [T] (may be null) multiplies the shared expert's rows. */
+/* shared_gate [T] (may be null) multiplies the shared expert's rows.  ids [T][top] (may be null): a pair whose id is real or
+ * more adds row t of x [T][H] (out_dtype, row stride ldx) instead of a row of y. */
 PHOTON_EXPORT int photon_moe_combine_ex(const void* y, long ldy, int y_dtype, const int* place, const float* weights, int top,
-                          const void* shared_out, const float* shared_gate, void* out, int out_dtype, int T_, int H,
-                          cudaStream_t stream);
+                          const void* shared_out, const float* shared_gate, const int* ids, int real, const void* x, long ldx,
+                          void* out, int out_dtype, int T_, int H, cudaStream_t stream);
 /* out[r, :] = x[sorted[r] / div, :]: the pairs' input rows in sorted order. */
 PHOTON_EXPORT int photon_moe_gather(const void* x, long ldx, int dtype, const int* sorted, int div, void* out, int n, int H,
                       cudaStream_t stream);
 /* Few pairs (decode steps), bfloat16: out[p] = W[ids[p]] x[p / x_div], one matrix-vector product per pair, unsorted;
- * glu, weights (pair p's factor is weights[p]), limit and slope as photon_moe_gemm. */
-PHOTON_EXPORT int photon_moe_gemv(const void* x, long ldx, int x_div, const int* ids, int n, const void* W, void* out, long ldo,
+ * glu, weights (pair p's factor is weights[p]), limit and slope as photon_moe_gemm.  Pairs whose id is `experts` or more are
+ * skipped. */
+PHOTON_EXPORT int photon_moe_gemv(const void* x, long ldx, int x_div, const int* ids, int n, const void* W, int experts, void* out, long ldo,
                     int out_dtype, int N, int K, int glu, int act, const float* weights, float limit, float slope,
                     cudaStream_t stream);
 
-/* ------------------------------------------------------------------ attention_flash.cu (-DHEAD_DIM=d, d % 16 == 0, <= 128; bfloat16) */
+/* ------------------------------------------------------------------ attention_flash.cu (-DHEAD_DIM=d [-DVALUE_DIM=dv, default d], multiples of 16
+ * up to 128; bfloat16): v_cache rows, out and gate are dv wide */
 PHOTON_EXPORT int photon_flash_attention_head_dim(void);
 PHOTON_EXPORT int photon_flash_attention_max_groups(void);
 /* mode bit 0: requests with more than 16 rows (tokens x heads per key/value head); bit 1: the others, their keys
- * split over num_splits blocks (part_acc/part_ml: float scratch of T * n_q * num_splits * (d + 2); tickets: int
+ * split over num_splits blocks (part_acc/part_ml: float scratch of T * n_q * num_splits * (dv + 2); tickets: int
  * [S * n_kv], zero between launches) and over nsub groups of warps per block.  context_lens may be null. */
 PHOTON_EXPORT int photon_flash_attention(const void* q, long q_stride, void* out, long out_stride, const void* k_cache,
                            const void* v_cache, const int* block_table, int max_pages, const int* cu_tokens,
                            const int* positions, const int* context_lens, float* part_acc, float* part_ml, int* tickets,
                            int S, int max_tokens_per_seq, int n_q, int n_kv, int d, int page_size, int num_pages,
                            int window, float scale, int num_splits, int nsub, int mode, int* err, cudaStream_t stream);
-/* The same with kept first keys (with a window, keys < keep_first stay visible), a sink (one more key with score 0 and no
- * value) and bounded scores (softcap * tanh(score * scale / softcap); 0: off). */
+/* The same with kept first keys (with a window, keys < keep_first stay visible), sinks (float [n_q], may be null: one
+ * more key with this score and no value in head h's softmax) and bounded scores (softcap * tanh(score * scale / softcap); 0: off). */
 PHOTON_EXPORT int photon_flash_attention_ex(const void* q, long q_stride, void* out, long out_stride, const void* k_cache,
                               const void* v_cache, const int* block_table, int max_pages, const int* cu_tokens,
                               const int* positions, const int* context_lens, float* part_acc, float* part_ml, int* tickets,
                               int S, int max_tokens_per_seq, int n_q, int n_kv, int d, int page_size, int num_pages,
                               int window, float scale, int num_splits, int nsub, int mode, int* err, int keep_first,
-                              int sink, float softcap, const void* gate, long gate_stride, cudaStream_t stream);
+                              const float* sinks, float softcap, const void* gate, long gate_stride, cudaStream_t stream);
 
-/* ------------------------------------------------------------------ attention_tc.cu (-DHEAD_DIM=64|128; bfloat16; tcgen05) */
+/* ------------------------------------------------------------------ attention_tc.cu (-DHEAD_DIM=d [-DVALUE_DIM=dv, default d], multiples of 8 from 16 to
+ * 128; bfloat16; tcgen05): v_cache rows, out and gate are dv wide */
 PHOTON_EXPORT int photon_attention_tc_head_dim(void);
 /* Requests with more than 16 rows only; the others are left untouched. */
 PHOTON_EXPORT int photon_attention_tc(const void* q, long q_stride, void* out, long out_stride, const void* k_cache,
@@ -412,7 +434,7 @@ PHOTON_EXPORT int photon_attention_tc(const void* q, long q_stride, void* out, l
 PHOTON_EXPORT int photon_attention_tc_ex(const void* q, long q_stride, void* out, long out_stride, const void* k_cache,
                            const void* v_cache, const int* block_table, int max_pages, const int* cu_tokens,
                            const int* positions, int S, int max_tokens_per_seq, int T, int n_q, int n_kv, int d,
-                           int page_size, int num_pages, int window, float scale, int* err, int keep_first, int sink,
+                           int page_size, int num_pages, int window, float scale, int* err, int keep_first, const float* sinks,
                            float softcap, const void* gate, long gate_stride, cudaStream_t stream);
 
 /* ------------------------------------------------------------------ attention_decode.cu (-DHEAD_DIM=64|128; bfloat16; TMA) */

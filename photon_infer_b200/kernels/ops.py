@@ -140,6 +140,28 @@ def add_rmsnorm(delta: Optional[torch.Tensor], residual: torch.Tensor, weight: t
            "add_rmsnorm")
 
 
+def add_normed_rmsnorm(y: torch.Tensor, post_weight: torch.Tensor, post_eps: float, residual: torch.Tensor, weight: torch.Tensor,
+                       eps: float, out: torch.Tensor, rows: Optional[torch.Tensor] = None) -> None:
+    """A sublayer between two norms: ``residual += post_weight * y / rms(y)`` in float32 (in place; skipped when ``rows`` is
+    given), then ``out = weight * residual / rms(residual)``, each root mean square with an eps of its own inside the root.
+    With ``rows`` (int32 list) only those rows are read and ``out`` has one row per list entry."""
+    _cuda(y, post_weight, residual, weight, out, rows)
+    H = residual.shape[-1]
+    n = rows.numel() if rows is not None else residual.shape[0]
+    if residual.dtype != torch.float32 or not residual.is_contiguous() or y.shape != residual.shape or not y.is_contiguous():
+        raise PhotonError(ErrorCode.SHAPE_MISMATCH, "add_normed_rmsnorm: contiguous y [T, H] beside a contiguous float32 stream [T, H]")
+    if out.shape != (n, H) or not out.is_contiguous() or weight.numel() != H or post_weight.numel() != H \
+            or not weight.is_contiguous() or not post_weight.is_contiguous():
+        raise PhotonError(ErrorCode.SHAPE_MISMATCH, "add_normed_rmsnorm: out must be [rows, H] and both weights [H]")
+    if rows is not None:
+        _int32(rows, "rows")
+    f = _fn("elementwise", "photon_add_normed_rmsnorm",
+            [c_void_p, c_int, c_void_p, c_int, c_float, c_void_p, c_void_p, c_int, c_float, c_void_p, c_int, c_void_p, c_int, c_int,
+             c_void_p])
+    _check(f(_ptr(y), _dtype_code(y), _ptr(post_weight), _dtype_code(post_weight), float(post_eps), _ptr(residual), _ptr(weight),
+             _dtype_code(weight), float(eps), _ptr(out), _dtype_code(out), _ptr(rows), n, H, _stream()), "add_normed_rmsnorm")
+
+
 def _check_delta_scale(scale: Optional[torch.Tensor], delta, delta2, H: int) -> None:
     if scale is None:
         return
@@ -200,14 +222,15 @@ def activation(x: torch.Tensor, activation: str, out: Optional[torch.Tensor] = N
 
 
 def gate_mul(x: torch.Tensor, gate: torch.Tensor) -> None:
-    """``x [T, W] *= sigmoid(gate [T, W])`` in place; both may be views with a row stride, ``gate`` may be 32-bit
-    beside a bfloat16 ``x``."""
+    """``x [T, W] *= sigmoid(gate)`` in place; ``gate [T, W]``, or ``[T, W / n]`` with one number for ``n`` neighbouring columns
+    (a head's outputs).  Both may be views with a row stride, ``gate`` may be 32-bit beside a bfloat16 ``x``."""
     _cuda(x, gate)
-    if x.dim() != 2 or gate.shape != x.shape or x.stride(1) != 1 or gate.stride(1) != 1:
-        raise PhotonError(ErrorCode.SHAPE_MISMATCH, "gate_mul: x and gate [T, W] with contiguous rows")
-    f = _fn("elementwise", "photon_gate_mul", [c_void_p, c_long, c_int, c_void_p, c_long, c_int, c_int, c_int, c_void_p])
+    if x.dim() != 2 or gate.dim() != 2 or gate.shape[0] != x.shape[0] or gate.shape[1] < 1 or x.shape[1] % gate.shape[1] \
+            or x.stride(1) != 1 or gate.stride(1) != 1:
+        raise PhotonError(ErrorCode.SHAPE_MISMATCH, "gate_mul: x [T, W] and gate [T, W or a divisor of it] with contiguous rows")
+    f = _fn("elementwise", "photon_gate_mul", [c_void_p, c_long, c_int, c_void_p, c_long, c_int, c_int, c_int, c_int, c_void_p])
     _check(f(_ptr(x), x.stride(0), _dtype_code(x), _ptr(gate), gate.stride(0), _dtype_code(gate), x.shape[0], x.shape[1],
-             _stream()), "gate_mul")
+             x.shape[1] // gate.shape[1], _stream()), "gate_mul")
 
 
 def stream_add(residual: torch.Tensor, delta: Optional[torch.Tensor], delta2: Optional[torch.Tensor],
@@ -339,9 +362,10 @@ def qk_norm_rope_write(q: torch.Tensor, k: Optional[torch.Tensor], v: Optional[t
                        positions: torch.Tensor, inv_freq: Optional[torch.Tensor], rot_dims: int,
                        slot_mapping: Optional[torch.Tensor], k_cache: Optional[torch.Tensor],
                        v_cache: Optional[torch.Tensor], n_q: int, n_kv: int, head_dim: int, value_dim: int,
-                       err: Optional[torch.Tensor]) -> None:
-    """Per head ``y = x / sqrt(mean(x^2) + eps) [* weight]`` for ``q [T, n_q * d]`` and ``k [T, n_kv * d]``, then the
-    rotation of the first ``rot_dims`` numbers of every head (number ``j`` with ``j + rot_dims / 2``, angle
+                       err: Optional[torch.Tensor], whole_row: bool = False, interleaved: bool = False) -> None:
+    """Per head ``y = x / sqrt(mean(x^2) + eps) [* weight]`` for ``q [T, n_q * d]`` and ``k [T, n_kv * d]`` (``whole_row``: one
+    norm over all numbers of ``q`` and one over all of ``k``, with weights of those sizes), then the rotation of the first
+    ``rot_dims`` numbers of every head (number ``j`` with ``j + rot_dims / 2`` or, ``interleaved``, ``2j`` with ``2j + 1``; angle
     ``position * inv_freq[j]``, ``inv_freq`` float64), queries into ``q_out`` and keys and ``v [T, n_kv * dv]`` into the
     paged caches ``[pages, n_kv, page_size, d | dv]``.  The inputs are views with any row stride and may be 32-bit
     while ``q_out`` and the caches are bfloat16.  Caches None: only the queries (``k`` and ``v`` are not read)."""
@@ -369,19 +393,19 @@ def qk_norm_rope_write(q: torch.Tensor, k: Optional[torch.Tensor], v: Optional[t
                                  or rot_dims > d):
         raise PhotonError(ErrorCode.SHAPE_MISMATCH, "qk_norm_rope_write: inv_freq must be float64 [rot_dims / 2], rot_dims even, <= head_dim")
     wt = q_weight if q_weight is not None else k_weight
-    for w in (q_weight, k_weight):
-        if w is not None and (w.numel() != d or w.dtype != wt.dtype or not w.is_contiguous()):
-            raise PhotonError(ErrorCode.SHAPE_MISMATCH, "qk_norm_rope_write: norm weights must be [head_dim] of one dtype")
+    for w, heads in ((q_weight, n_q), (k_weight, n_kv)):
+        if w is not None and (w.numel() != (heads * d if whole_row else d) or w.dtype != wt.dtype or not w.is_contiguous()):
+            raise PhotonError(ErrorCode.SHAPE_MISMATCH, "qk_norm_rope_write: norm weights must be [head_dim] (or [heads * head_dim]) of one dtype")
     f = _fn("qk_norm", "photon_qk_norm_rope_write",
             [c_void_p, c_long, c_void_p, c_long, c_void_p, c_long, c_int, c_void_p, c_long, c_int, c_void_p, c_void_p, c_int,
              c_float, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int,
-             c_long, c_void_p, c_void_p])
+             c_long, c_int, c_int, c_void_p, c_void_p])
     _check(f(_ptr(q), q.stride(0), _ptr(k) if write else None, k.stride(0) if write else 0, _ptr(v) if write else None,
              v.stride(0) if write else 0, _dtype_code(q), _ptr(q_out), q_out.stride(0), _dtype_code(q_out), _ptr(q_weight),
              _ptr(k_weight), _dtype_code(wt) if wt is not None else F32, float(eps), _ptr(positions),
              _ptr(inv_freq) if rot_dims else None, int(rot_dims) if inv_freq is not None else 0, _ptr(slot_mapping),
-             _ptr(k_cache), _ptr(v_cache), T, n_q, n_kv, d, dv, page_size, num_slots, _ptr(err), _stream()),
-           "qk_norm_rope_write")
+             _ptr(k_cache), _ptr(v_cache), T, n_q, n_kv, d, dv, page_size, num_slots, int(whole_row), int(interleaved), _ptr(err),
+             _stream()), "qk_norm_rope_write")
 
 
 # ----------------------------------------------------------------------------- attention
@@ -394,6 +418,19 @@ def _check_gate(gate: Optional[torch.Tensor], q: torch.Tensor, out: torch.Tensor
         raise PhotonError(ErrorCode.SHAPE_MISMATCH, "attention: the gate must have the shape of the output and the type of q")
 
 
+def _check_sink(sink: Optional[torch.Tensor], heads: int) -> None:
+    if sink is None:
+        return
+    _cuda(sink)
+    if sink.dtype != torch.float32 or sink.numel() != heads or not sink.is_contiguous():
+        raise PhotonError(ErrorCode.SHAPE_MISMATCH, "attention: sinks must be contiguous float32, one per query head")
+
+
+def value_defines(head_dim: int, value_dim: Optional[int]) -> dict:
+    """Definitions that the tensor-core attention kernels are compiled with."""
+    return {"HEAD_DIM": head_dim} if value_dim in (None, head_dim) else {"HEAD_DIM": head_dim, "VALUE_DIM": int(value_dim)}
+
+
 def gate_fusable(gate: torch.Tensor) -> bool:
     """Whether the tensor-core attention kernels can take this gate into their epilogue (16-byte aligned rows)."""
     return gate.stride(1) == 1 and gate.data_ptr() % 16 == 0 and (gate.stride(0) * gate.element_size()) % 16 == 0
@@ -403,7 +440,7 @@ def paged_attention(q: torch.Tensor, out: torch.Tensor, k_cache: torch.Tensor, v
                     block_table: torch.Tensor, token_seq: torch.Tensor, positions: torch.Tensor,
                     n_q: int, n_kv: int, head_dim: int, window: Optional[int], scale: float,
                     err: Optional[torch.Tensor], value_dim: Optional[int] = None, splits: int = 1,
-                    keep_first: int = 0, sink: bool = False, softcap: Optional[float] = None,
+                    keep_first: int = 0, sink: Optional[torch.Tensor] = None, softcap: Optional[float] = None,
                     gate: Optional[torch.Tensor] = None) -> None:
     """General paged causal attention.  ``q`` is a ``[T, n_q * d]`` view (row stride free),
     ``out [T, n_q * dv]``; the token at position ``p`` of request ``token_seq[t]`` sees keys
@@ -411,11 +448,13 @@ def paged_attention(q: torch.Tensor, out: torch.Tensor, k_cache: torch.Tensor, v
     width of a value; ``v_cache is k_cache`` means that a key's value is the first ``value_dim`` numbers of
     its own row (attention over a cached latent).  ``splits`` > 1 shares every token's keys out over that many
     blocks (for decoded tokens with long contexts; the order of the sums then depends on ``splits``).
-    ``keep_first``: with a window, keys ``0 .. keep_first - 1`` stay visible as well.  ``sink``: the softmax has one
-    more key with score 0 and no value (``p_j = exp(s_j) / (1 + sum exp(s_i))``).  ``softcap``: scores become
+    ``keep_first``: with a window, keys ``0 .. keep_first - 1`` stay visible as well.  ``sink`` (float32
+    ``[n_q]``): a head's softmax has one more key with the score ``sink[h]``, which is neither scaled nor bounded, and no value
+    (``p_j = exp(s_j) / (exp(sink[h]) + sum exp(s_i))``).  ``softcap``: scores become
     ``softcap * tanh(score / softcap)`` after the scale.  ``gate`` (``[T, n_q * value_dim]`` of the type of ``q``, a
     view with any row stride): every output is multiplied by ``sigmoid(gate)`` before it is rounded."""
     _check_gate(gate, q, out)
+    _check_sink(sink, n_q)
     _cuda(q, out, k_cache, v_cache, block_table, token_seq, positions, err)
     T = q.shape[0]
     dv = head_dim if value_dim is None else int(value_dim)
@@ -433,14 +472,14 @@ def paged_attention(q: torch.Tensor, out: torch.Tensor, k_cache: torch.Tensor, v
         _int32(t, name)
     f = _fn("attention", "photon_paged_attention_ex",
             [c_void_p, c_long, c_void_p, c_long, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p,
-             c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_void_p, c_void_p, c_int, c_int,
+             c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_void_p, c_void_p, c_int, c_void_p,
              c_float, c_void_p, c_long, c_void_p])
     splits = max(1, min(int(splits), 64))
     part = torch.empty(T * n_q * splits * (dv + 2), dtype=torch.float32, device=q.device) if splits > 1 else None
     _check(f(_ptr(q), q.stride(0), _ptr(out), out.stride(0), _dtype_code(q), _ptr(k_cache), _ptr(v_cache),
              _ptr(block_table), block_table.shape[1], _ptr(token_seq), _ptr(positions), T, n_q, n_kv, head_dim, dv,
              k_cache.shape[2], k_cache.shape[0], int(window) if window else 0, float(scale), splits, _ptr(part), _ptr(err),
-             int(keep_first or 0), int(bool(sink)), float(softcap or 0.0), _ptr(gate), gate.stride(0) if gate is not None else 0,
+             int(keep_first or 0), _ptr(sink), float(softcap or 0.0), _ptr(gate), gate.stride(0) if gate is not None else 0,
              _stream()), "paged_attention")
     if splits > 1:
         global _launch_count
@@ -468,14 +507,15 @@ def reset_tickets(device) -> None:
         _skinny_buffers[key][1].zero_()
 
 
-def flash_attention_supported(dtype: torch.dtype, head_dim: int) -> bool:
-    """The tensor-core kernel takes bfloat16 and head sizes that are a multiple of 16 up to 128."""
-    return dtype == torch.bfloat16 and head_dim % 16 == 0 and 16 <= head_dim <= 128
+def flash_attention_supported(dtype: torch.dtype, head_dim: int, value_dim: Optional[int] = None) -> bool:
+    """The tensor-core kernel takes bfloat16 and heads (and values) that are a multiple of 16 up to 128 wide."""
+    fits = lambda d: d % 16 == 0 and 16 <= d <= 128
+    return dtype == torch.bfloat16 and fits(head_dim) and fits(value_dim or head_dim)
 
 
-def flash_attention_max_groups(head_dim: int) -> int:
+def flash_attention_max_groups(head_dim: int, value_dim: Optional[int] = None) -> int:
     """Groups of four warps that the split-key kernel can run in one block at this head size (4, 2 or 1)."""
-    lib = load_module("attention_flash", {"HEAD_DIM": head_dim})
+    lib = load_module("attention_flash", value_defines(head_dim, value_dim))
     return int(lib.photon_flash_attention_max_groups())
 
 
@@ -485,28 +525,33 @@ def flash_attention(q: torch.Tensor, out: torch.Tensor, k_cache: torch.Tensor, v
                     window: Optional[int], scale: float, num_splits: int, scratch: Optional[torch.Tensor],
                     rows_mode: bool, keys_mode: bool, err: Optional[torch.Tensor],
                     context_lens: Optional[torch.Tensor] = None, key_groups: int = 1, keep_first: int = 0,
-                    sink: bool = False, softcap: Optional[float] = None, gate: Optional[torch.Tensor] = None) -> None:
+                    sink: Optional[torch.Tensor] = None, softcap: Optional[float] = None, gate: Optional[torch.Tensor] = None,
+                    value_dim: Optional[int] = None) -> None:
     """Paged causal attention on the tensor cores.  ``cu_tokens [S + 1]`` gives each request's
     tokens in the step.  ``rows_mode``: run requests with more than 16 rows (tokens x heads per
     group); ``keys_mode``: run the others, their keys split over ``num_splits`` blocks.
-    ``scratch``: float32, at least ``T * n_q * num_splits * (head_dim + 2)`` when ``num_splits > 1``.
+    ``scratch``: float32, at least ``T * n_q * num_splits * (value_dim + 2)`` when ``num_splits > 1``.
     ``context_lens [S]`` (optional): tokens of each request after this step; the split-key kernel then
     derives positions from it (a request's tokens of the step are its last ones) and saves a round trip.
     ``key_groups``: 1, 2 or 4 groups of four warps per block of the split-key kernel, each walking its own
     share of the block's keys (``flash_attention_max_groups`` bounds it); their results are merged in shared
     memory, which is far cheaper than the merge of ``num_splits`` blocks through global memory.
-    ``keep_first``, ``sink``, ``softcap``, ``gate``: as in ``paged_attention``."""
+    ``keep_first``, ``sink``, ``softcap``, ``gate``, ``value_dim``: as in ``paged_attention``."""
     _check_gate(gate, q, out)
+    _check_sink(sink, n_q)
+    dv = value_dim or head_dim
     _cuda(q, out, k_cache, v_cache, block_table, cu_tokens, positions, scratch, err, context_lens)
     if context_lens is not None:
         _int32(context_lens, "context_lens")
         if context_lens.numel() < num_seqs:
             raise PhotonError(ErrorCode.SHAPE_MISMATCH, "flash_attention: context_lens must cover every request")
     T = q.shape[0]
-    if not flash_attention_supported(q.dtype, head_dim) or n_kv <= 0 or n_q % n_kv:
-        raise PhotonError(ErrorCode.UNSUPPORTED_SIZE, f"flash_attention: head_dim {head_dim} in {q.dtype} is not supported")
-    if q.shape[1] != n_q * head_dim or q.stride(1) != 1 or out.shape != (T, n_q * head_dim) or not out.is_contiguous():
-        raise PhotonError(ErrorCode.SHAPE_MISMATCH, "flash_attention: q and out must be [T, n_q * head_dim]")
+    if not flash_attention_supported(q.dtype, head_dim, dv) or n_kv <= 0 or n_q % n_kv:
+        raise PhotonError(ErrorCode.UNSUPPORTED_SIZE, f"flash_attention: heads of {head_dim} and {dv} in {q.dtype} are not supported")
+    if q.shape[1] != n_q * head_dim or q.stride(1) != 1 or out.shape != (T, n_q * dv) or not out.is_contiguous():
+        raise PhotonError(ErrorCode.SHAPE_MISMATCH, "flash_attention: q must be [T, n_q * head_dim], out [T, n_q * value_dim]")
+    if k_cache.shape[3] != head_dim or v_cache.shape[3] != dv:
+        raise PhotonError(ErrorCode.SHAPE_MISMATCH, "flash_attention: the caches' last dimension must be head_dim / value_dim")
     if out.dtype != q.dtype or k_cache.dtype != q.dtype or v_cache.dtype != q.dtype:
         raise PhotonError(ErrorCode.INVALID_ARGUMENT, "flash_attention: q, out and the caches must be bfloat16")
     for name, t in (("block_table", block_table), ("cu_tokens", cu_tokens), ("positions", positions)):
@@ -516,11 +561,11 @@ def flash_attention(q: torch.Tensor, out: torch.Tensor, k_cache: torch.Tensor, v
     part_acc = part_ml = tickets = None
     splits = int(num_splits) if keys_mode else 1
     if splits > 1:
-        need = T * n_q * splits * (head_dim + 2)
+        need = T * n_q * splits * (dv + 2)
         if scratch is None or scratch.dtype != torch.float32 or scratch.numel() < need or not scratch.is_contiguous():
             raise PhotonError(ErrorCode.INVALID_ARGUMENT, f"flash_attention: scratch must hold {need} float32 values")
         part_acc = scratch
-        part_ml = scratch[T * n_q * splits * head_dim:]
+        part_ml = scratch[T * n_q * splits * dv:]
         tickets = _attention_tickets(q.device)
         if tickets.numel() < num_seqs * n_kv:
             raise PhotonError(ErrorCode.UNSUPPORTED_SIZE, "flash_attention: too many requests for the ticket buffer")
@@ -528,14 +573,14 @@ def flash_attention(q: torch.Tensor, out: torch.Tensor, k_cache: torch.Tensor, v
     f = _fn("attention_flash", "photon_flash_attention_ex",
             [c_void_p, c_long, c_void_p, c_long, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p,
              c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_int,
-             c_int, c_void_p, c_int, c_int, c_float, c_void_p, c_long, c_void_p],
-            defines={"HEAD_DIM": head_dim})
+             c_int, c_void_p, c_int, c_void_p, c_float, c_void_p, c_long, c_void_p],
+            defines=value_defines(head_dim, value_dim))
     _check(f(_ptr(q), q.stride(0), _ptr(out), out.stride(0), _ptr(k_cache), _ptr(v_cache), _ptr(block_table),
              block_table.shape[1], _ptr(cu_tokens), _ptr(positions), _ptr(context_lens), _ptr(part_acc), _ptr(part_ml),
              _ptr(tickets),
              int(num_seqs), int(max_tokens_per_seq), n_q, n_kv, head_dim, k_cache.shape[2], k_cache.shape[0],
              int(window) if window else 0, float(scale), splits, int(key_groups) if keys_mode else 1, mode, _ptr(err),
-             int(keep_first or 0), int(bool(sink)), float(softcap or 0.0), _ptr(gate), gate.stride(0) if gate is not None else 0,
+             int(keep_first or 0), _ptr(sink), float(softcap or 0.0), _ptr(gate), gate.stride(0) if gate is not None else 0,
              _stream()), "flash_attention")
     if rows_mode and keys_mode:
         global _launch_count
@@ -650,10 +695,15 @@ def attention_decode(q: torch.Tensor, out: torch.Tensor, k_cache: torch.Tensor, 
 USE_ATTENTION_TC = os.environ.get("PHOTON_ATTENTION_TC", "1") != "0"
 
 
-def attention_tc_supported(dtype: torch.dtype, head_dim: int, group: int, page_size: int) -> bool:
-    """The tcgen05 kernel for prompt portions: bfloat16, head size 64 or 128, up to 128 heads per
-    key/value head and pages of 8, 16, 32 or a multiple of 64 tokens."""
-    return (dtype == torch.bfloat16 and head_dim in (64, 128) and 1 <= group <= 128
+def attention_tc_heads(head_dim: int, value_dim: Optional[int] = None) -> bool:
+    """Head and value widths of the tcgen05 kernel for prompt portions (its tiles are 64 or 128 wide, zeros behind a head)."""
+    return all(d % 8 == 0 and 16 <= d <= 128 for d in (head_dim, value_dim or head_dim))
+
+
+def attention_tc_supported(dtype: torch.dtype, head_dim: int, group: int, page_size: int, value_dim: Optional[int] = None) -> bool:
+    """The tcgen05 kernel for prompt portions: bfloat16, heads and values of up to 128 numbers (multiples of 8), up to 128
+    heads per key/value head and pages of 8, 16, 32 or a multiple of 64 tokens."""
+    return (dtype == torch.bfloat16 and attention_tc_heads(head_dim, value_dim) and 1 <= group <= 128
             and page_size % 8 == 0 and page_size >= 8 and (64 % page_size == 0 or page_size % 64 == 0))
 
 
@@ -661,36 +711,40 @@ def attention_tc(q: torch.Tensor, out: torch.Tensor, k_cache: torch.Tensor, v_ca
                  block_table: torch.Tensor, cu_tokens: torch.Tensor, positions: torch.Tensor,
                  num_seqs: int, max_tokens_per_seq: int, n_q: int, n_kv: int, head_dim: int,
                  window: Optional[int], scale: float, err: Optional[torch.Tensor], keep_first: int = 0,
-                 sink: bool = False, softcap: Optional[float] = None, gate: Optional[torch.Tensor] = None) -> None:
+                 sink: Optional[torch.Tensor] = None, softcap: Optional[float] = None, gate: Optional[torch.Tensor] = None,
+                 value_dim: Optional[int] = None) -> None:
     """Paged causal attention of the requests that bring more than 16 rows (tokens x heads per
     group) in this step, on the tcgen05 tensor cores; the rows of the other requests are left
-    untouched (``flash_attention`` with ``keys_mode`` takes them).  ``keep_first``, ``sink``, ``softcap``, ``gate``: as in
-    ``paged_attention`` (the gate's rows must start on 16-byte boundaries: ``gate_fusable``)."""
+    untouched (``flash_attention`` with ``keys_mode`` takes them).  ``keep_first``, ``sink``, ``softcap``, ``gate``,
+    ``value_dim``: as in ``paged_attention`` (the gate's rows must start on 16-byte boundaries: ``gate_fusable``)."""
     _check_gate(gate, q, out)
+    _check_sink(sink, n_q)
+    dv = value_dim or head_dim
     _cuda(q, out, k_cache, v_cache, block_table, cu_tokens, positions, err)
     T = q.shape[0]
-    if n_kv <= 0 or n_q % n_kv or not attention_tc_supported(q.dtype, head_dim, n_q // n_kv, k_cache.shape[2]):
+    if n_kv <= 0 or n_q % n_kv or not attention_tc_supported(q.dtype, head_dim, n_q // n_kv, k_cache.shape[2], dv):
         raise PhotonError(ErrorCode.UNSUPPORTED_SIZE,
-                          f"attention_tc: head_dim {head_dim}, {n_q}/{n_kv} heads, pages of {k_cache.shape[2]} in {q.dtype} is not supported")
-    if q.shape[1] != n_q * head_dim or q.stride(1) != 1 or out.shape != (T, n_q * head_dim) or not out.is_contiguous():
-        raise PhotonError(ErrorCode.SHAPE_MISMATCH, "attention_tc: q and out must be [T, n_q * head_dim]")
+                          f"attention_tc: {n_q}/{n_kv} heads of {head_dim} and {dv}, pages of {k_cache.shape[2]} in {q.dtype} is not supported")
+    if q.shape[1] != n_q * head_dim or q.stride(1) != 1 or out.shape != (T, n_q * dv) or not out.is_contiguous():
+        raise PhotonError(ErrorCode.SHAPE_MISMATCH, "attention_tc: q must be [T, n_q * head_dim], out [T, n_q * value_dim]")
     if out.dtype != q.dtype or k_cache.dtype != q.dtype or v_cache.dtype != q.dtype:
         raise PhotonError(ErrorCode.INVALID_ARGUMENT, "attention_tc: q, out and the caches must be bfloat16")
-    if not k_cache.is_contiguous() or not v_cache.is_contiguous() or k_cache.shape != v_cache.shape:
-        raise PhotonError(ErrorCode.INVALID_ARGUMENT, "attention_tc: the caches must be contiguous [pages, n_kv, page, d]")
+    if not k_cache.is_contiguous() or not v_cache.is_contiguous() or k_cache.shape[:3] != v_cache.shape[:3] \
+            or k_cache.shape[3] != head_dim or v_cache.shape[3] != dv:
+        raise PhotonError(ErrorCode.INVALID_ARGUMENT, "attention_tc: the caches must be contiguous [pages, n_kv, page, d | dv]")
     for name, t in (("block_table", block_table), ("cu_tokens", cu_tokens), ("positions", positions)):
         _int32(t, name)
     if cu_tokens.numel() < num_seqs + 1 or block_table.shape[0] < num_seqs:
         raise PhotonError(ErrorCode.SHAPE_MISMATCH, "attention_tc: cu_tokens and block_table must cover every request")
     f = _fn("attention_tc", "photon_attention_tc_ex",
             [c_void_p, c_long, c_void_p, c_long, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p,
-             c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_void_p, c_int, c_int, c_float,
+             c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_void_p, c_int, c_void_p, c_float,
              c_void_p, c_long, c_void_p],
-            defines={"HEAD_DIM": head_dim})
+            defines=value_defines(head_dim, value_dim))
     _check(f(_ptr(q), q.stride(0), _ptr(out), out.stride(0), _ptr(k_cache), _ptr(v_cache), _ptr(block_table),
              block_table.shape[1], _ptr(cu_tokens), _ptr(positions), int(num_seqs), int(max_tokens_per_seq), T,
              n_q, n_kv, head_dim, k_cache.shape[2], k_cache.shape[0], int(window) if window else 0, float(scale),
-             _ptr(err), int(keep_first or 0), int(bool(sink)), float(softcap or 0.0), _ptr(gate),
+             _ptr(err), int(keep_first or 0), _ptr(sink), float(softcap or 0.0), _ptr(gate),
              gate.stride(0) if gate is not None else 0, _stream()), "attention_tc")
 
 
@@ -1068,12 +1122,14 @@ def latent_decode_shares(max_context: int, window: Optional[int] = None) -> int:
 
 def latent_decode_attention(q: torch.Tensor, out: torch.Tensor, cache: torch.Tensor, block_table: torch.Tensor,
                             token_seq: torch.Tensor, positions: torch.Tensor, heads: int, width: int, value_dim: int,
-                            scale: float, max_context: int, err: Optional[torch.Tensor], window: Optional[int] = None) -> None:
+                            scale: float, max_context: int, err: Optional[torch.Tensor], window: Optional[int] = None,
+                            sink: Optional[torch.Tensor] = None) -> None:
     """Attention of decoded tokens (or of the few tokens of a short portion) over cached latent rows on the tensor
     cores: ``q [T, heads * width]``, ``cache [pages, 1, page_size, width]``, ``out [T, heads * value_dim]``; every token
     sees the rows up to its own position (with a ``window`` the last ``window`` of them), a row's value is its first
     ``value_dim`` numbers.  ``max_context``: an upper bound of the tokens' contexts (sizes the grid: one block per token
-    and 64 rows that it may see)."""
+    and 64 rows that it may see).  ``sink`` (float32 ``[heads]``): as in ``paged_attention``."""
+    _check_sink(sink, heads)
     _cuda(q, out, cache, block_table, token_seq, positions, err)
     T = q.shape[0]
     if not latent_decode_supported(q, width, value_dim) or q.shape[1] != heads * width or q.stride(1) != 1 \
@@ -1086,10 +1142,10 @@ def latent_decode_attention(q: torch.Tensor, out: torch.Tensor, cache: torch.Ten
     part = torch.empty(T * heads * splits * (value_dim + 2), dtype=torch.float32, device=q.device)
     f = _fn("latent", "photon_latent_decode_attention",
             [c_void_p, c_long, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int,
-             c_float, c_int, c_int, c_void_p, c_void_p, c_long, c_void_p, c_void_p])
+             c_float, c_int, c_int, c_void_p, c_void_p, c_long, c_void_p, c_void_p, c_void_p])
     _check(f(_ptr(q), q.stride(0), _ptr(cache), _ptr(block_table), block_table.shape[1], _ptr(token_seq), _ptr(positions), T,
              heads, width, value_dim, cache.shape[2], cache.shape[0], float(scale), int(window or 0), splits, _ptr(part), _ptr(out),
-             out.stride(0), _ptr(err), _stream()), "latent_decode_attention")
+             out.stride(0), _ptr(sink), _ptr(err), _stream()), "latent_decode_attention")
     global _launch_count
     _launch_count += 1
 
@@ -1101,7 +1157,8 @@ HEAD_LINEAR_LIBRARY_ROWS = 16
 def head_linear(x: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, gate: Optional[torch.Tensor] = None) -> None:
     """``out[t, h, :] = weight[h] @ x[t, h, :]`` for all heads at once: ``x [T, heads, K]`` and
     ``out [T, heads, N]`` are views with free row and head strides, ``weight [heads, N, K]`` is contiguous.  ``gate
-    [T, heads * N]`` (rows with a stride): every output is multiplied by ``sigmoid(gate)``.
+    [T, heads * N]``, or ``[T, heads]`` for one number per head (rows with a stride): every output is multiplied by
+    ``sigmoid(gate)``.
     float32 and few rows: this package's kernel (one chain of fused multiply-adds per output, the gate in its epilogue);
     many bfloat16 rows: the library's batched product, then the gate."""
     _cuda(x, weight, out, gate)
@@ -1110,8 +1167,8 @@ def head_linear(x: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, gate: 
     if weight.shape != (heads, N, K) or not weight.is_contiguous() or out.shape != (T, heads, N) \
             or x.stride(2) != 1 or out.stride(2) != 1 or x.dtype != weight.dtype or out.dtype != x.dtype:
         raise PhotonError(ErrorCode.SHAPE_MISMATCH, "head_linear: x [T, heads, K], weight [heads, N, K], out [T, heads, N]")
-    if gate is not None and (gate.shape != (T, heads * N) or gate.stride(1) != 1 or gate.dtype != x.dtype):
-        raise PhotonError(ErrorCode.SHAPE_MISMATCH, "head_linear: gate [T, heads * N] of the type of x")
+    if gate is not None and (gate.shape not in ((T, heads * N), (T, heads)) or gate.stride(1) != 1 or gate.dtype != x.dtype):
+        raise PhotonError(ErrorCode.SHAPE_MISMATCH, "head_linear: gate [T, heads * N] or [T, heads] of the type of x")
     if x.dtype == torch.bfloat16 and T >= HEAD_LINEAR_LIBRARY_ROWS:
         torch.bmm(x.transpose(0, 1), weight.transpose(1, 2), out=out.transpose(0, 1))
         if gate is not None:
@@ -1121,9 +1178,10 @@ def head_linear(x: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, gate: 
         return
     f = _fn("latent", "photon_head_linear",
             [c_void_p, c_long, c_long, c_void_p, c_void_p, c_long, c_long, c_int, c_int, c_int, c_int, c_int, c_void_p, c_long,
-             c_void_p])
+             c_int, c_void_p])
     _check(f(_ptr(x), x.stride(0), x.stride(1), _ptr(weight), _ptr(out), out.stride(0), out.stride(1), _dtype_code(x),
-             T, heads, N, K, _ptr(gate), gate.stride(0) if gate is not None else 0, _stream()), "head_linear")
+             T, heads, N, K, _ptr(gate), gate.stride(0) if gate is not None else 0,
+             int(gate is not None and gate.shape[1] != heads * N), _stream()), "head_linear")
 
 
 def latent_absorb_supported(q: torch.Tensor, dim: int, rot: int) -> bool:
@@ -1184,12 +1242,15 @@ def latent_prompt_defines(dtype: torch.dtype, d: int, r: int, v: int, kv_rank: i
 
 def latent_prompt_attention(q: torch.Tensor, q_rot: torch.Tensor, kv: torch.Tensor, rot_rows: torch.Tensor, out: torch.Tensor,
                             seqs, heads: int, d: int, r: int, v: int, window: Optional[int], scale: float,
-                            err: Optional[torch.Tensor], gate: Optional[torch.Tensor] = None) -> None:
+                            err: Optional[torch.Tensor], gate: Optional[torch.Tensor] = None,
+                            sink: Optional[torch.Tensor] = None) -> None:
     """Attention of long prompt portions over an expanded latent on the tcgen05 tensor cores.  ``q [T, heads * (d + r)]`` (its
     unrotated parts are read), ``q_rot [T, heads, r]``; ``kv [rows, heads * (d + v)]``: the heads' keys, then their values;
     ``rot_rows [rows, r]`` (a view): the key part that all heads share.  ``seqs``: per request ``(first token, tokens, position
     of the first token, position of its first row, that row)``.  ``out [T, heads * v]`` gets the rows of those tokens, times
-    ``sigmoid(gate)`` when a gate is given."""
+    ``sigmoid(gate)`` when a gate is given (``[T, heads * v]``, or ``[T, heads]`` for one number per head); ``sink`` (float32
+    ``[heads]``): as in ``paged_attention``."""
+    _check_sink(sink, heads)
     _cuda(q, q_rot, kv, rot_rows, out, err, gate)
     T, rows = q.shape[0], kv.shape[0]
     defines = latent_prompt_defines(q.dtype, d, r, v, 8)
@@ -1200,31 +1261,34 @@ def latent_prompt_attention(q: torch.Tensor, q_rot: torch.Tensor, kv: torch.Tens
             or out.shape != (T, heads * v) or out.stride(1) != 1 \
             or any(t.dtype != torch.bfloat16 for t in (q_rot, kv, rot_rows, out)):
         raise PhotonError(ErrorCode.SHAPE_MISMATCH, "latent_prompt_attention: q [T, heads * (d + r)], kv [rows, heads * (d + v)], all bfloat16")
-    if gate is not None and (gate.shape != (T, heads * v) or gate.stride(1) != 1 or gate.dtype != torch.bfloat16):
-        raise PhotonError(ErrorCode.SHAPE_MISMATCH, "latent_prompt_attention: gate [T, heads * v] bfloat16")
+    if gate is not None and (gate.shape not in ((T, heads * v), (T, heads)) or gate.stride(1) != 1 or gate.dtype != torch.bfloat16):
+        raise PhotonError(ErrorCode.SHAPE_MISMATCH, "latent_prompt_attention: gate [T, heads * v] or [T, heads] bfloat16")
     flat = [int(x) for s in seqs for x in s]
     host = (ctypes.c_int * len(flat))(*flat)
     f = _fn("attention_latent_tc", "photon_attention_latent_tc",
-            [c_void_p, c_long, c_void_p, c_void_p, c_long, c_void_p, c_long, c_void_p, c_long, c_void_p, c_long, c_void_p, c_int,
-             c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_void_p, c_void_p], defines=defines)
+            [c_void_p, c_long, c_void_p, c_void_p, c_long, c_void_p, c_long, c_void_p, c_long, c_void_p, c_long, c_int, c_void_p,
+             c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_void_p, c_void_p], defines=defines)
     _check(f(_ptr(q), q.stride(0), _ptr(q_rot), _ptr(kv), kv.stride(0), _ptr(rot_rows), rot_rows.stride(0), _ptr(out), out.stride(0),
-             _ptr(gate), gate.stride(0) if gate is not None else 0, ctypes.cast(host, c_void_p), len(flat) // 5, T, rows, heads, d, r,
+             _ptr(gate), gate.stride(0) if gate is not None else 0, int(gate is not None and gate.shape[1] != heads * v), _ptr(sink),
+             ctypes.cast(host, c_void_p), len(flat) // 5, T, rows, heads, d, r,
              v, int(window or 0), float(scale), _ptr(err), _stream()), "latent_prompt_attention")
 
 
 def causal_softmax_rows(scores: torch.Tensor, probs: torch.Tensor, heads: int, first_pos: int, scale: float,
-                        first_key: int = 0, window: Optional[int] = None) -> None:
+                        first_key: int = 0, window: Optional[int] = None, sink: Optional[torch.Tensor] = None) -> None:
     """``probs = softmax(scale * scores)`` row by row over the keys each row may see: column ``c`` is the key at position
     ``first_key + c``, row ``r`` belongs to the token at position ``first_pos + r // heads`` and sees the keys up to that
-    position (with a ``window`` the last ``window`` of them); zero elsewhere."""
+    position (with a ``window`` the last ``window`` of them); zero elsewhere.  ``sink`` (float32 ``[heads]``): ``exp(sink[r %
+    heads])`` joins the denominator of row ``r``."""
+    _check_sink(sink, int(heads))
     _cuda(scores, probs)
     rows, cols = scores.shape
     if scores.dtype != torch.float32 or scores.stride(1) != 1 or probs.shape != scores.shape or probs.stride(1) != 1:
         raise PhotonError(ErrorCode.SHAPE_MISMATCH, "causal_softmax_rows: scores float32 [rows, cols], probs of the same shape")
     f = _fn("latent", "photon_causal_softmax_rows",
-            [c_void_p, c_long, c_void_p, c_long, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_void_p])
+            [c_void_p, c_long, c_void_p, c_long, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_void_p, c_void_p])
     _check(f(_ptr(scores), scores.stride(0), _ptr(probs), probs.stride(0), _dtype_code(probs), rows, int(heads), int(first_pos),
-             int(first_key), int(window or 0), cols, float(scale), _stream()), "causal_softmax_rows")
+             int(first_key), int(window or 0), cols, float(scale), _ptr(sink), _stream()), "causal_softmax_rows")
 
 
 # ----------------------------------------------------------------------------- parallel residual streams
@@ -1558,18 +1622,40 @@ def conv_silu(x: torch.Tensor, taps_w: torch.Tensor, bias: Optional[torch.Tensor
                  int(conv_offset), state.shape[0], int(num_seqs), C, _stream()), "conv_state")
 
 
-LINREC_MODES = {"state_space": 0, "matrix_memory": 1}
+LINREC_MODES = {"state_space": 0, "matrix_memory": 1, "forget_write": 2}
 
 
-def linrec(mode: str, q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, gate_a: torch.Tensor, gate_b: Optional[torch.Tensor],
-           p0: torch.Tensor, p1: torch.Tensor, p2: Optional[torch.Tensor], cap: float, q_scale: float, cu_tokens: torch.Tensor,
+def linrec_gates(q: torch.Tensor, z: torch.Tensor, bias: torch.Tensor, lower: torch.Tensor, q_out: torch.Tensor,
+                 k_out: torch.Tensor) -> None:
+    """The inputs of a ``forget_write`` recurrence for all tokens side by side: ``q_out = silu(q)`` and the write gates ``k_out
+    = (1 - lower) sigmoid(-(z + bias))``; float32 ``[T, C]`` views with unit column stride."""
+    _cuda(q, z, bias, lower, q_out, k_out)
+    T, C = q.shape
+    for t, what in ((q, "q"), (z, "z"), (q_out, "q_out"), (k_out, "k_out")):
+        if t.dtype != torch.float32 or t.shape != (T, C) or t.stride(1) != 1:
+            raise PhotonError(ErrorCode.SHAPE_MISMATCH, f"linrec_gates: {what} must be a float32 [{T}, {C}] view")
+    for t in (bias, lower):
+        if t.dtype != torch.float32 or t.numel() != C or not t.is_contiguous():
+            raise PhotonError(ErrorCode.SHAPE_MISMATCH, f"linrec_gates: bias and lower must be float32 [{C}]")
+    if q_out.stride(0) != k_out.stride(0):
+        raise PhotonError(ErrorCode.SHAPE_MISMATCH, "linrec_gates: both outputs must have one row stride")
+    f = _fn("linrec", "photon_linrec_gates",
+            [c_void_p, c_long, c_void_p, c_long, c_void_p, c_void_p, c_void_p, c_void_p, c_long, c_int, c_int, c_void_p])
+    _check(f(_ptr(q), q.stride(0), _ptr(z), z.stride(0), _ptr(bias), _ptr(lower), _ptr(q_out), _ptr(k_out), q_out.stride(0), T, C,
+             _stream()), "linrec_gates")
+
+
+def linrec(mode: str, q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, gate_a: Optional[torch.Tensor], gate_b: Optional[torch.Tensor],
+           p0: Optional[torch.Tensor], p1: Optional[torch.Tensor], p2: Optional[torch.Tensor], cap: float, q_scale: float, cu_tokens: torch.Tensor,
            state_slots: torch.Tensor, state: torch.Tensor, out: torch.Tensor, num_seqs: int, heads: int, qk_heads: int,
            dim: int, vdim: int, err: Optional[torch.Tensor]) -> None:
     """The recurrence ``S <- keep S + take k v^T, o = S^T q`` over the tokens of a step, per request and head, with the
     state ``[heads, dim, vdim]`` (then, for ``matrix_memory``, ``n [heads, dim]`` and ``m [heads]``) at the start of the
     request's float32 state row.  ``state_space``: ``gate_a`` = raw step sizes ``[T, heads]``, ``p0, p1, p2`` = ``A_log``,
     ``dt_bias``, ``D``; the output is ``o + D v``.  ``matrix_memory``: ``gate_a, gate_b`` = raw input and forget gates, ``p0,
-    p1`` their biases, ``cap`` their bound; the output is ``o / (max(|n . q|, exp(-m)) + 1e-6)``.  All inputs float32 views
+    p1`` their biases, ``cap`` their bound; the output is ``o / (max(|n . q|, exp(-m)) + 1e-6)``.  ``forget_write``: a gate per
+    row of the state, ``S <- S + k (v^T - S)``; ``k`` holds the raw gates ``z`` and the write gate is ``(1 - p1) sigmoid(-(z +
+    p0))``, ``p0, p1 [qk_heads * dim]``, ``q`` enters as ``silu(q)``; with ``p0, p1`` None both come from ``linrec_gates``.  All inputs float32 views
     with unit column stride; ``out`` float32 ``[T, heads * vdim]``."""
     _cuda(q, k, v, gate_a, gate_b, p0, p1, p2, cu_tokens, state_slots, state, out, err)
     if mode not in LINREC_MODES:
@@ -1579,13 +1665,15 @@ def linrec(mode: str, q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, gate_a:
                        (gate_b, heads, "gate_b"), (out, heads * vdim, "out")):
         if t is not None and (t.dtype != torch.float32 or t.shape != (T, w) or t.stride(1) != 1):
             raise PhotonError(ErrorCode.SHAPE_MISMATCH, f"linrec: {what} must be a float32 [T, {w}] view")
-    if gate_b is not None and gate_b.stride(0) != gate_a.stride(0):
+    if gate_b is not None and (gate_a is None or gate_b.stride(0) != gate_a.stride(0)):
         raise PhotonError(ErrorCode.SHAPE_MISMATCH, "linrec: both gates must have one row stride")
-    if (mode == "matrix_memory") != (gate_b is not None):
-        raise PhotonError(ErrorCode.INVALID_ARGUMENT, "linrec: the matrix memory has two gates, the state-space layer one")
+    if (mode == "matrix_memory") != (gate_b is not None) or (mode == "forget_write") != (gate_a is None):
+        raise PhotonError(ErrorCode.INVALID_ARGUMENT, "linrec: the matrix memory has two gates per head, the state-space layer one, "
+                          "the forget-and-write layer none beside its rows' gates")
+    per = qk_heads * dim if mode == "forget_write" else heads
     for t, what in ((p0, "p0"), (p1, "p1"), (p2, "p2")):
-        if t is not None and (t.dtype != torch.float32 or t.numel() != heads or not t.is_contiguous()):
-            raise PhotonError(ErrorCode.SHAPE_MISMATCH, f"linrec: {what} must be float32 [heads]")
+        if t is not None and (t.dtype != torch.float32 or t.numel() != per or not t.is_contiguous()):
+            raise PhotonError(ErrorCode.SHAPE_MISMATCH, f"linrec: {what} must be float32 [{per}]")
     need = heads * dim * vdim + (heads * dim + heads if mode == "matrix_memory" else 0)
     if state.dtype != torch.float32 or state.dim() != 2 or not state.is_contiguous() or state.shape[1] < need:
         raise PhotonError(ErrorCode.SHAPE_MISMATCH, "linrec: state must be contiguous float32 [slots, row]")
@@ -1596,7 +1684,7 @@ def linrec(mode: str, q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, gate_a:
              c_float, c_float, c_void_p, c_void_p, c_void_p, c_long, c_int, c_void_p, c_long, c_int, c_int, c_int, c_int, c_int,
              c_void_p, c_void_p])
     _check(f(LINREC_MODES[mode], _ptr(q), q.stride(0), _ptr(k), k.stride(0), _ptr(v), v.stride(0), _ptr(gate_a), _ptr(gate_b),
-             gate_a.stride(0), _ptr(p0), _ptr(p1), _ptr(p2), float(cap), float(q_scale), _ptr(cu_tokens), _ptr(state_slots),
+             gate_a.stride(0) if gate_a is not None else 0, _ptr(p0), _ptr(p1), _ptr(p2), float(cap), float(q_scale), _ptr(cu_tokens), _ptr(state_slots),
              _ptr(state), state.stride(0), state.shape[0], _ptr(out), out.stride(0), int(num_seqs), heads, qk_heads, dim, vdim,
              _ptr(err), _stream()), "linrec")
 
@@ -1830,17 +1918,20 @@ def moe_tile_rows() -> int:
 
 def moe_route(h: torch.Tensor, w_router: torch.Tensor, bias: Optional[torch.Tensor], top: int,
               scoring: str = "softmax_chosen", groups: int = 1, keep_groups: int = 1, route_scale: float = 1.0,
-              w_shared_gate: Optional[torch.Tensor] = None):
+              w_shared_gate: Optional[torch.Tensor] = None, correction: Optional[torch.Tensor] = None, identity: int = 0):
     """Router logits in 32-bit and the ``top`` experts of every token.  ``scoring`` ``softmax_chosen``: the largest
     logits win and the weights are the softmax over the chosen logits.  ``softmax_all``: scores are the softmax
     over all experts; the experts form ``groups`` equal groups of neighbours, a group's score is its largest
     score and only experts of the ``keep_groups`` best groups can be chosen; the weights are the chosen scores
     over their sum (+ 1e-20) times ``route_scale``.  ``sigmoid``: scores are ``sigmoid(logit)``, a group's score is the
     sum of its two largest scores, and the weights are the chosen scores times ``route_scale`` (not divided by their
-    sum).  ``w_shared_gate [1, H]``: also returns ``sigmoid(w . h)``
+    sum).  ``softmax_raw``: scores are the softmax over all experts, the experts with the largest ``score + correction``
+    (float32 ``[E]``, may be None) are chosen, and the weights are the chosen scores without the correction times
+    ``route_scale``, not divided by their sum; the last ``identity`` of the ``E`` router outputs are identity experts, and
+    ``counts`` has ``E - identity + 1`` entries then, the last one for all of them.  ``w_shared_gate [1, H]``: also returns ``sigmoid(w . h)``
     per token.  Returns ``(ids int32 [T, top], weights float32 [T, top], counts int32 [E])`` or, with a gate,
     those and ``gate float32 [T]``."""
-    _cuda(h, w_router, bias, w_shared_gate)
+    _cuda(h, w_router, bias, w_shared_gate, correction)
     if scoring not in ROUTER_SCORING:
         raise PhotonError(ErrorCode.INVALID_ARGUMENT, f"moe_route: unknown scoring {scoring!r} ({', '.join(ROUTER_SCORING)})")
     T, H = h.shape
@@ -1849,7 +1940,9 @@ def moe_route(h: torch.Tensor, w_router: torch.Tensor, bias: Optional[torch.Tens
         raise PhotonError(ErrorCode.SHAPE_MISMATCH, "moe_route: h [T, H] and the router [E, H] of one dtype")
     ids = torch.empty((T, top), dtype=torch.int32, device=h.device)
     weights = torch.empty((T, top), dtype=torch.float32, device=h.device)
-    counts = torch.empty(E, dtype=torch.int32, device=h.device)
+    if correction is not None and (correction.dtype != torch.float32 or correction.numel() != E or not correction.is_contiguous()):
+        raise PhotonError(ErrorCode.SHAPE_MISMATCH, "moe_route: the correction must be contiguous float32 [E]")
+    counts = torch.empty(E - identity + 1 if identity else E, dtype=torch.int32, device=h.device)
     gate = None
     if w_shared_gate is not None:
         if w_shared_gate.numel() != H or w_shared_gate.dtype != w_router.dtype or not w_shared_gate.is_contiguous():
@@ -1857,24 +1950,27 @@ def moe_route(h: torch.Tensor, w_router: torch.Tensor, bias: Optional[torch.Tens
         gate = torch.empty(T, dtype=torch.float32, device=h.device)
     f = _fn("moe", "photon_moe_route_ex",
             [c_void_p, c_long, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p,
-             c_void_p, c_int, c_int, c_int, c_float, c_void_p, c_void_p, c_void_p])
+             c_void_p, c_int, c_int, c_int, c_float, c_void_p, c_void_p, c_void_p, c_int, c_void_p])
     _check(f(_ptr(h), h.stride(0), _dtype_code(h), _ptr(w_router), _ptr(bias),
              _dtype_code(bias) if bias is not None else F32, T, H, E, int(top), _ptr(ids), _ptr(weights), _ptr(counts),
              ROUTER_SCORING[scoring], int(groups), int(keep_groups), float(route_scale), _ptr(w_shared_gate), _ptr(gate),
-             _stream()), "moe_route")
+             _ptr(correction), int(identity), _stream()), "moe_route")
     if gate is not None:
         return ids, weights, counts, gate
     return ids, weights, counts
 
 
-ROUTER_SCORING = {"softmax_chosen": 0, "softmax_all": 1, "sigmoid": 2}
+ROUTER_SCORING = {"softmax_chosen": 0, "softmax_all": 1, "sigmoid": 2, "softmax_raw": 3}
 
 
-def moe_align(ids: torch.Tensor, counts: torch.Tensor):
-    """Sorts the (token, choice) pairs by expert on the device.  Returns ``(offsets [E + 1], sorted [n], place
+def moe_align(ids: torch.Tensor, counts: torch.Tensor, experts: Optional[int] = None):
+    """Sorts the (token, choice) pairs by expert on the device.  ``experts`` smaller by one than the number of counts: the
+    last bucket holds the pairs whose id is ``experts`` or more (identity experts); they come last and have no row tiles.
+    Returns ``(offsets [E + 1], sorted [n], place
     [n], tiles [max_tiles, 3], num_tiles [1], max_tiles)``."""
     _cuda(ids, counts)
     n, E = ids.numel(), counts.numel()
+    real = E if experts is None else int(experts)
     max_tiles = n // moe_tile_rows() + E
     dev = ids.device
     offsets = torch.empty(E + 1, dtype=torch.int32, device=dev)
@@ -1883,8 +1979,8 @@ def moe_align(ids: torch.Tensor, counts: torch.Tensor):
     tiles = torch.empty((max_tiles, 3), dtype=torch.int32, device=dev)
     num_tiles = torch.empty(1, dtype=torch.int32, device=dev)
     f = _fn("moe", "photon_moe_align",
-            [c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p])
-    _check(f(_ptr(ids), _ptr(counts), n, E, _ptr(offsets), _ptr(srt), _ptr(place), _ptr(tiles), _ptr(num_tiles),
+            [c_void_p, c_void_p, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p])
+    _check(f(_ptr(ids), _ptr(counts), n, E, real, _ptr(offsets), _ptr(srt), _ptr(place), _ptr(tiles), _ptr(num_tiles),
              _stream()), "moe_align")
     return offsets, srt, place, tiles, num_tiles, max_tiles
 
@@ -1938,12 +2034,18 @@ def moe_glu(gate_up: torch.Tensor, out: torch.Tensor, activation: str, srt: Opti
 
 
 def moe_combine(y: torch.Tensor, place: Optional[torch.Tensor], weights: Optional[torch.Tensor], shared_out: Optional[torch.Tensor],
-                out: torch.Tensor, shared_gate: Optional[torch.Tensor] = None) -> None:
+                out: torch.Tensor, shared_gate: Optional[torch.Tensor] = None, ids: Optional[torch.Tensor] = None,
+                experts: int = 0, x: Optional[torch.Tensor] = None) -> None:
     """``out[t] = sum_j weights[t, j] * y[place[t, j]] (+ shared_out[t])``, summed in 32-bit in the order of ``j``;
     ``place`` None: the rows of ``y`` stand in the order of the pairs.  ``shared_gate`` float32 ``[T]``: the shared
     expert's row of token ``t`` is multiplied by ``shared_gate[t]``.  ``weights`` None: a plain sum (the experts' inputs
-    carried the weights)."""
-    _cuda(y, place, weights, shared_out, out, shared_gate)
+    carried the weights).  ``ids [T, top]``: a pair whose id is ``experts`` or more belongs to an identity expert and adds row
+    ``t`` of ``x [T, H]`` (of the type of ``out``) instead of its row of ``y``."""
+    _cuda(y, place, weights, shared_out, out, shared_gate, ids, x)
+    if ids is not None:
+        _int32(ids, "ids")
+        if x is None or x.shape != out.shape or x.dtype != out.dtype or x.stride(1) != 1:
+            raise PhotonError(ErrorCode.SHAPE_MISMATCH, "moe_combine: identity experts need the tokens' rows, of the shape and type of out")
     T, H = out.shape[0], y.shape[1]
     top = weights.shape[1] if weights is not None else y.shape[0] // max(T, 1)
     if shared_gate is not None and (shared_out is None or shared_gate.dtype != torch.float32 or shared_gate.numel() != T):
@@ -1953,9 +2055,10 @@ def moe_combine(y: torch.Tensor, place: Optional[torch.Tensor], weights: Optiona
                                             or shared_out.dtype != out.dtype)):
         raise PhotonError(ErrorCode.SHAPE_MISMATCH, "moe_combine: y [n, H], out and shared_out contiguous [T, H]")
     f = _fn("moe", "photon_moe_combine_ex",
-            [c_void_p, c_long, c_int, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p])
+            [c_void_p, c_long, c_int, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_long, c_void_p, c_int,
+             c_int, c_int, c_void_p])
     _check(f(_ptr(y), y.stride(0), _dtype_code(y), _ptr(place), _ptr(weights), top, _ptr(shared_out), _ptr(shared_gate),
-             _ptr(out), _dtype_code(out), T, H, _stream()), "moe_combine")
+             _ptr(ids), int(experts), _ptr(x), x.stride(0) if x is not None else 0, _ptr(out), _dtype_code(out), T, H, _stream()), "moe_combine")
 
 
 def moe_gather(x: torch.Tensor, srt: torch.Tensor, div: int) -> torch.Tensor:
@@ -1978,7 +2081,8 @@ def moe_gemv(x: torch.Tensor, x_div: int, ids: torch.Tensor, weight: torch.Tenso
              activation: Optional[str] = None, weights: Optional[torch.Tensor] = None, limit: float = 0.0,
              slope: float = 1.0) -> None:
     """A decode step's few (token, choice) pairs: ``out[p] = weight[ids[p]] @ x[p // x_div]``, one matrix-vector
-    product per pair in the order of the pairs, the expert's rows streamed once.  bfloat16 in, bfloat16 or float32 out.
+    product per pair in the order of the pairs, the expert's rows streamed once; rows of pairs whose id is ``E`` or more
+    (identity experts) are left as they are.  bfloat16 in, bfloat16 or float32 out.
     ``weights`` float32 (one per pair): a factor on the pair's input row."""
     _cuda(x, ids, weight, out, weights)
     act = _expert_act(glu, activation)
@@ -1991,9 +2095,9 @@ def moe_gemv(x: torch.Tensor, x_div: int, ids: torch.Tensor, weight: torch.Tenso
     if out.shape != (n, N // 2 if glu else N) or out.stride(1) != 1:
         raise PhotonError(ErrorCode.SHAPE_MISMATCH, "moe_gemv: out [pairs, N or N / 2]")
     f = _fn("moe", "photon_moe_gemv",
-            [c_void_p, c_long, c_int, c_void_p, c_int, c_void_p, c_void_p, c_long, c_int, c_int, c_int, c_int, c_int, c_void_p, c_float,
+            [c_void_p, c_long, c_int, c_void_p, c_int, c_void_p, c_int, c_void_p, c_long, c_int, c_int, c_int, c_int, c_int, c_void_p, c_float,
              c_float, c_void_p])
-    _check(f(_ptr(x), x.stride(0), int(x_div), _ptr(ids), n, _ptr(weight), _ptr(out), out.stride(0), _dtype_code(out), N, K,
+    _check(f(_ptr(x), x.stride(0), int(x_div), _ptr(ids), n, _ptr(weight), E, _ptr(out), out.stride(0), _dtype_code(out), N, K,
              int(glu), act, _ptr(weights), float(limit), float(slope), _stream()), "moe_gemv")
 
 

@@ -33,11 +33,16 @@ class LayerSpec:
     connect1: Optional[PartSpec] = None
     connect2: Optional[PartSpec] = None
 
+    # norms on the mixer's and the feed-forward's output (with a block that has them, kind "sandwich")
+    post1: Optional[PartSpec] = None
+    post2: Optional[PartSpec] = None
+
     def optional_parts(self):
         """``(block parameter, part table, spec)`` of the optional parts that this layer has."""
         return [(key, table, ps) for key, table, ps in (("scale1", "scale", self.scale1), ("scale2", "scale", self.scale2),
                                                         ("connect1", "connection", self.connect1),
-                                                        ("connect2", "connection", self.connect2)) if ps is not None]
+                                                        ("connect2", "connection", self.connect2),
+                                                        ("post1", "norm", self.post1), ("post2", "norm", self.post2)) if ps is not None]
 
 
 @dataclasses.dataclass

@@ -47,7 +47,8 @@ class PagedAttention(Mixer):
             mods.extend(["gemm_skinny", "gemm_skinny_fused", "gemm_tc", "gemm_tc2"])
         if ops.flash_attention_supported(dtype, self.head_dim):
             mods.append(("attention_flash", {"HEAD_DIM": self.head_dim}))
-        if dtype == torch.bfloat16 and self.head_dim in (64, 128) and ops.USE_ATTENTION_TC and self.n_q // self.n_kv <= 128:
+        if dtype == torch.bfloat16 and ops.flash_attention_supported(dtype, self.head_dim) and ops.USE_ATTENTION_TC \
+                and self.n_q // self.n_kv <= 128:
             mods.append(("attention_tc", {"HEAD_DIM": self.head_dim}))
         if dtype == torch.bfloat16 and self.head_dim in (64, 128) and self.n_q // self.n_kv <= 16:
             mods.append(("attention_decode", {"HEAD_DIM": self.head_dim}))
@@ -156,15 +157,16 @@ class PagedAttention(Mixer):
 
 
 def attend_tensor_cores(mixer, q: torch.Tensor, out: torch.Tensor, ctx: StepContext, cache: LayerCache,
-                        keep_first: int = 0, sink: bool = False, softcap: Optional[float] = None,
+                        keep_first: int = 0, sink: Optional[torch.Tensor] = None, softcap: Optional[float] = None,
                         gate: Optional[torch.Tensor] = None) -> None:
-    """The tensor-core attention kernels for one step of ``mixer`` (anything with ``n_q``, ``n_kv``, ``head_dim``,
-    ``window``, ``scale`` and a ``_max_groups`` slot): requests with many rows walk their keys in one block per 128
+    """The tensor-core attention kernels for one step of ``mixer`` (anything with ``n_q``, ``n_kv``, ``head_dim``, optionally
+    ``value_dim``, ``window``, ``scale`` and a ``_max_groups`` slot): requests with many rows walk their keys in one block per 128
     rows, requests with few rows (decoded tokens) split their keys over blocks.  ``keep_first``, ``sink``,
     ``softcap``, ``gate``: the rules of ``ops.paged_attention``; the persistent kernel for long contexts has none of them."""
     self = mixer
-    extras = dict(keep_first=keep_first, sink=sink, softcap=softcap, gate=gate)
-    plain = not (keep_first or sink or softcap) and gate is None
+    value_dim = getattr(self, "value_dim", self.head_dim)
+    extras = dict(keep_first=keep_first, sink=sink, softcap=softcap, gate=gate, value_dim=value_dim)
+    plain = not (keep_first or softcap) and sink is None and gate is None and value_dim == self.head_dim
     group = ctx.groups[cache.group]
     gsize = self.n_q // self.n_kv
     # tensor cores: requests with many rows walk their keys in one block per 128 rows, requests
@@ -184,16 +186,16 @@ def attend_tensor_cores(mixer, q: torch.Tensor, out: torch.Tensor, ctx: StepCont
     decode_tma = plan is not None
     if keys_mode and not decode_tma:
         if self._max_groups is None:
-            self._max_groups = ops.flash_attention_max_groups(self.head_dim)
+            self._max_groups = ops.flash_attention_max_groups(self.head_dim, value_dim)
         splits, groups = choose_key_shares(sum(few) * self.n_kv, keys, self._max_groups, sms=ops.sm_count(q.device))
         # the kernel indexes its partial results by the token's place in the step, so beside a long prompt
         # portion every share costs T rows: no more shares than 64 MB of them
-        per_share = T * self.n_q * (self.head_dim + 2) * 4
+        per_share = T * self.n_q * (value_dim + 2) * 4
         splits = max(1, min(splits, (64 << 20) // per_share))
         if splits > 1:
-            scratch = torch.empty(T * self.n_q * splits * (self.head_dim + 2), dtype=torch.float32, device=q.device)
+            scratch = torch.empty(T * self.n_q * splits * (value_dim + 2), dtype=torch.float32, device=q.device)
     if rows_mode and ops.USE_ATTENTION_TC and \
-            ops.attention_tc_supported(q.dtype, self.head_dim, gsize, cache.k.shape[2]):
+            ops.attention_tc_supported(q.dtype, self.head_dim, gsize, cache.k.shape[2], value_dim):
         # prompt portions: tensor memory and TMA; the split-key kernel keeps the decoded tokens
         ops.attention_tc(q, out, cache.k, cache.v, group.block_table, ctx.cu_tokens, ctx.positions,
                          ctx.num_seqs, ctx.max_query_len, self.n_q, self.n_kv, self.head_dim, self.window,

@@ -29,7 +29,8 @@ class TensorSpec:
     and are held in the run dtype; ``"vector"`` tensors (norm weights) keep 32-bit
     storage when the file has it; ``"int"`` tensors are integer tables, held as int32.
     ``init`` tells the random-weights mode how to fill it: ``"normal"`` (N(0, std)),
-    ``"norm"`` (ones, or 1 + N(0, norm_std)), ``"eye"`` (identity + N(0, std)), ``"zeros"``.
+    ``"norm"`` (ones, or 1 + N(0, norm_std)), ``"eye"`` (identity + N(0, std)), ``"unit"``
+    (uniform between 0 and 1), ``"zeros"``.
     A dimension of ``-1`` in ``shape`` is a size that the configuration does not give: the weight file decides it
     (the loader accepts any size there), and the random-weights mode uses ``free_size``.
     """
@@ -184,8 +185,8 @@ class Normed:
 
     def materialize(self) -> torch.Tensor:
         """The normed rows as a 32-bit tensor, for a consumer that cannot take the norm into its own kernel."""
-        x = self.tensor if self.bias is None else self.tensor.to(torch.float32) + self.bias.to(torch.float32)
-        return self.norm.forward(x, torch.float32)
+        x = self.tensor.to(torch.float32)
+        return self.norm.forward(x if self.bias is None else x + self.bias.to(torch.float32), torch.float32)
 
 
 @dataclasses.dataclass

@@ -7,6 +7,8 @@ without a feed-forward adds the mixer's output alone.
 Output norm: ``x += norm1(mixer(x)); x += norm2(ff(x))``: the sublayers read the stream itself and the norms sit on
 their outputs.
 
+Sandwich: ``x += post1(mixer(norm1(x))); x += post2(ff(norm2(x)))``: a norm before and a norm behind every sublayer.
+
 Hyper pre-norm: pre-norm over several parallel residual streams, which each sublayer reads and writes through a connection
 of its own.
 
@@ -131,6 +133,35 @@ class OutputNormBlock(Block):
         return residual, Normed(self.feed_forward.forward(h2, ctx), self.norm2)
 
 
+class SandwichBlock(Block):
+    """A norm before and a norm behind every sublayer.  The norm behind it stays pending with the output (``Normed``), so that
+    one kernel does it, the residual sum and the norm of the next sublayer (``RMSNorm.add_forward``)."""
+
+    def __init__(self, norm1: Norm, mixer: Mixer, post1: Norm, norm2: Optional[Norm] = None, feed_forward: Optional[FeedForward] = None,
+                 post2: Optional[Norm] = None):
+        if not (norm2 is None) == (feed_forward is None) == (post2 is None):
+            raise ValueError("a block has a second pair of norms exactly when it has a feed-forward")
+        self.norm1, self._mixer, self.post1 = norm1, mixer, post1
+        self.norm2, self.feed_forward, self.post2 = norm2, feed_forward, post2
+
+    def parts(self) -> Dict[str, Part]:
+        p = {"norm1": self.norm1, "mixer": self._mixer, "post1": self.post1}
+        if self.feed_forward is not None:
+            p.update(norm2=self.norm2, feed_forward=self.feed_forward, post2=self.post2)
+        return p
+
+    def mixer(self) -> Mixer:
+        return self._mixer
+
+    def forward(self, residual: torch.Tensor, delta, ctx: StepContext, cache: LayerCache):
+        h = self.norm1.add_forward(delta, residual, ctx.dtype)
+        a = Normed(self._mixer.forward(h, ctx, cache), self.post1)
+        if self.feed_forward is None:
+            return residual, a
+        h2 = self.norm2.add_forward(a, residual, ctx.dtype)
+        return residual, Normed(self.feed_forward.forward(h2, ctx), self.post2)
+
+
 class HyperPreNormBlock(Block):
     """Pre-norm over several residual streams: a sublayer's norm gets ``sum_s in[s] X_s`` and its output is written back into
     all streams, mixed with each other at the same time (``parts/hyper.py``).  The write stays pending (``Connected``) for
@@ -165,4 +196,5 @@ class HyperPreNormBlock(Block):
 register_block("pre_norm", PreNormBlock)
 register_block("parallel", ParallelBlock)
 register_block("output_norm", OutputNormBlock)
+register_block("sandwich", SandwichBlock)
 register_block("hyper_pre_norm", HyperPreNormBlock)

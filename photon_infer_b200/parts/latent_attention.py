@@ -21,7 +21,10 @@ feature ``i`` paired with ``i + rot_dims / 2`` or (``rot_interleaved``) feature 
 unchanged.
 
 Variants, all by parameter.  ``window``: a token sees its own row and the ``window - 1`` before it.  ``output_gate``: the
-concatenated heads are multiplied by ``sigmoid(W_g h)`` before ``W_o``; ``W_g``'s rows ride in the fused down-projection.
+concatenated heads are multiplied by ``sigmoid(W_g h)`` before ``W_o`` (``head``: ``W_g`` has one row per head, whose gate
+multiplies all of the head's output); ``W_g``'s rows ride in the fused down-projection.  ``sink``: the softmax of head ``h``
+has one more key with no value and the learned score ``sink[h]``, which is not scaled: ``exp(sink[h])`` joins the denominator.
+``rot_scaling`` stretches the rotation's frequencies (``parts/rope.py``).
 ``own_kv`` False: the layer has no ``W_dkv``; it reads the cached rows of an earlier layer (the run list's ``kv_from``) with
 its own queries, ``W_uk``, ``W_uv``, window and everything else.  ``cache_window``: how many rows the cache must keep for
 this layer AND the layers that read its pages (``"own"``: this layer's window; None: everything).
@@ -37,6 +40,7 @@ from ..kernels import ops
 from .base import LayerCache, Mixer, PagedCacheSpec, StepContext, TensorSpec
 from .linear import project
 from .registry import register_mixer
+from .rope import scaled_frequencies
 
 
 class LatentAttention(Mixer):
@@ -44,7 +48,8 @@ class LatentAttention(Mixer):
 
     def __init__(self, hidden_size: int, heads: int, dim: int, rot_dim: int, vdim: int, kv_rank: int, q_rank: int,
                  scale: float, eps: float, rot_base: float, rot_dims: Optional[int] = None, window: Optional[int] = None,
-                 rot_interleaved: bool = False, cache_window="own", own_kv: bool = True, output_gate: bool = False):
+                 rot_interleaved: bool = False, cache_window="own", own_kv: bool = True, output_gate=False, sink: bool = False,
+                 rot_scaling: Optional[dict] = None):
         self.hidden_size, self.heads, self.dim, self.rot_dim, self.vdim = hidden_size, heads, dim, rot_dim, vdim
         self.kv_rank, self.q_rank = kv_rank, q_rank
         self.scale, self.eps = float(scale), float(eps)
@@ -57,11 +62,13 @@ class LatentAttention(Mixer):
         self.cache_window = self.window if cache_window == "own" else (int(cache_window) if cache_window else None)
         if self.cache_window is not None and (self.window is None or self.window > self.cache_window):
             raise ValueError("the cache must keep at least the rows that this layer's window sees")
-        self.own_kv, self.output_gate = bool(own_kv), bool(output_gate)
+        if output_gate not in (False, True, "head"):
+            raise ValueError("output_gate is False, True (a number per output) or 'head' (a number per head)")
+        self.own_kv, self.output_gate, self.sink = bool(own_kv), output_gate, bool(sink)
+        self.gate_width = 0 if not output_gate else heads * (vdim if output_gate is True else 1)
+        self.sinks: Optional[torch.Tensor] = None
         self.width = kv_rank + rot_dim          # one cached row
-        half = self.rot_dims // 2
-        self.inv_freq_host = torch.tensor([self.rot_base ** (-2.0 * i / self.rot_dims) for i in range(half)],
-                                          dtype=torch.float64).to(torch.float32)
+        self.inv_freq_host = scaled_frequencies(self.rot_dims, self.rot_base, rot_scaling).to(torch.float32)
         self.inv_freq: Optional[torch.Tensor] = None
         self.w_down = self.w_uq = self.w_absorb = self.w_uv = self.w_kv = self.w_o = None
         self.q_norm = self.kv_norm = None
@@ -88,13 +95,18 @@ class LatentAttention(Mixer):
             specs += [TensorSpec("dkv", (self.kv_rank + r, H)), TensorSpec("dkv.norm", (self.kv_rank,), role="vector", init="norm")]
         specs += [TensorSpec("uk", (n * d, self.kv_rank)), TensorSpec("uv", (n * v, self.kv_rank))]
         if self.output_gate:
-            specs.append(TensorSpec("g", (n * v, H)))
+            specs.append(TensorSpec("g", (self.gate_width, H)))
+        if self.sink:
+            specs.append(TensorSpec("sink", (n,), role="vector", init="normal"))
         return specs + [TensorSpec("o", (H, n * v))]
 
     def load(self, tensors: Dict[str, torch.Tensor]) -> None:
         n, d, v = self.heads, self.dim, self.vdim
         down = [tensors["dq"]] + ([tensors["dkv"]] if self.own_kv else []) + ([tensors["g"]] if self.output_gate else [])
+        if self.gate_width % 8:                 # rows of the product stay a multiple of 16 bytes
+            down.append(torch.zeros((-self.gate_width % 8, self.hidden_size), dtype=down[0].dtype, device=down[0].device))
         self.w_down = torch.cat(down, dim=0).contiguous()                                 # h is read once
+        self.sinks = tensors["sink"].to(torch.float32).contiguous() if self.sink else None
         self.q_norm = tensors["dq.norm"].contiguous()
         self.kv_norm = tensors["dkv.norm"].contiguous() if self.own_kv else None
         self.w_uq = tensors["uq"].contiguous()
@@ -117,7 +129,8 @@ class LatentAttention(Mixer):
         n, d, r, kr = self.heads, self.dim, self.rot_dim, self.kv_rank
         group = ctx.groups[cache.group]
         down = project(h, self.w_down)                                   # [T, q_rank (+ kv_rank + rot) (+ gate)]
-        gate = down[:, down.shape[1] - n * self.vdim:] if self.output_gate else None
+        at = self.q_rank + (self.width if self.own_kv else 0)
+        gate = down[:, at:at + self.gate_width] if self.output_gate else None
         store = self.own_kv and not cache.shared
         cq = torch.empty((T, self.q_rank), dtype=h.dtype, device=h.device)
         ops.latent_prep(down, self.q_rank, kr, r, self.rot_dims, self.q_norm, self.kv_norm, self.eps, ctx.positions,
@@ -199,9 +212,10 @@ class LatentAttention(Mixer):
         kv = project(latents[:, :kr], self.w_kv)                         # [rows, heads * (dim + vdim)]
         q_rot = torch.empty((T, n, r), dtype=q.dtype, device=q.device)
         ops.latent_q_rope(q, n, d, r, self.rot_dims, ctx.positions, self.inv_freq, q_rot, 0, interleaved=self.rot_interleaved)
-        fused = gate is not None and gate.data_ptr() % 16 == 0 and gate.stride(0) % 8 == 0      # 16-byte gates in the epilogue
+        # in the epilogue: one number per head, or gates that can be read 16 bytes at a time
+        fused = gate is not None and (self.output_gate == "head" or (gate.data_ptr() % 16 == 0 and gate.stride(0) % 8 == 0))
         ops.latent_prompt_attention(q, q_rot, kv, latents[:, kr:], o, seqs, n, d, r, self.vdim, self.window, self.scale,
-                                    ctx.error_flag, gate=gate if fused else None)
+                                    ctx.error_flag, gate=gate if fused else None, sink=self.sinks)
         if gate is not None and not fused:
             for t, m, *_ in seqs:
                 ops.gate_mul(o[t:t + m], gate[t:t + m])
@@ -244,7 +258,7 @@ class LatentAttention(Mixer):
             # bfloat16 with widths that fit the tensor cores' tiles: one block per token and 64 cached rows
             ops.latent_decode_attention(q2, o_lat[a:b], cache.k, group.block_table, token_seq, positions, n,
                                         self.width, self.kv_rank, self.scale, ctx.max_context_len, ctx.error_flag,
-                                        window=self.window)
+                                        window=self.window, sink=self.sinks)
             return
         splits = 1
         if q_lat.dtype == torch.bfloat16:
@@ -256,7 +270,7 @@ class LatentAttention(Mixer):
             splits = max(1, min(4 * ops.sm_count(q_lat.device) // max(1, (b - a) * chunks), tiles, 64))
         ops.paged_attention(q_lat[a:b].view(b - a, n * self.width), o_lat[a:b], cache.k, cache.k, group.block_table,
                             token_seq, positions, n, 1, self.width, self.window, self.scale,
-                            ctx.error_flag, value_dim=self.kv_rank, splits=splits)
+                            ctx.error_flag, value_dim=self.kv_rank, splits=splits, sink=self.sinks)
 
     def _dense(self, q, o, start: int, table: torch.Tensor, cache: LayerCache, ctx: StepContext) -> None:
         m, n, kr = q.shape[0], self.heads, self.kv_rank
@@ -277,7 +291,7 @@ class LatentAttention(Mixer):
             part = rows[lo - base:hi - base]
             scores = torch.mm(q[t0:t1].view((t1 - t0) * n, self.width), part.t(), out_dtype=torch.float32)
             probs = torch.empty(scores.shape, dtype=q.dtype, device=q.device)
-            ops.causal_softmax_rows(scores, probs, n, start + t0, self.scale, first_key=lo, window=w)
+            ops.causal_softmax_rows(scores, probs, n, start + t0, self.scale, first_key=lo, window=w, sink=self.sinks)
             torch.mm(probs, part[:, :kr], out=o[t0:t1].view((t1 - t0) * n, kr))
             t0 = t1
 

@@ -21,6 +21,11 @@ over their sum times ``route_scale``.  ``shared_gate``: the shared expert's outp
 ``sigmoid(W_sg h)``, one number per token (``shared.sg [1, H]``), computed with the router's logits in 32-bit.
 ``scoring`` ``sigmoid``: scores are ``sigmoid(logit)``, each expert by itself; a group's score is the sum of its two largest
 scores; the weights are the chosen scores times ``route_scale``, not divided by their sum.
+``scoring`` ``softmax_raw``: scores are the softmax over all experts, and the weights are the chosen scores times
+``route_scale``, not divided by their sum.  With ``correction`` (a learned vector, one number per router output) the experts
+with the largest ``score + correction`` are chosen; the weights leave it out.  ``identity``: the last ``identity`` router
+outputs are experts without matrices whose output is the token's own input row; their pairs pass no product (in the sorted
+order they come last) and the weighted sum adds the row.
 ``weight_input``: the weight multiplies the expert's input instead of its output, ``sum_j expert_j(w_j h)``; the first
 products are linear, so their 32-bit sums are scaled in the epilogue (or by the gated unit's kernel) and the outputs are
 added as they are.  ``activation`` ``clamped_swish`` (gated experts): ``g = min(W_gate x, act_limit)``,
@@ -49,8 +54,13 @@ class MoEFeedForward(FeedForward):
                  activation: str = "silu", shared_activation: Optional[str] = None, gated: bool = True,
                  router_bias: bool = True, scoring: str = "softmax_chosen", groups: int = 1, keep_groups: Optional[int] = None,
                  route_scale: float = 1.0, shared_gate: bool = False, weight_input: bool = False, act_limit: Optional[float] = None,
-                 act_slope: float = 1.0):
-        if not 1 <= top <= experts:
+                 act_slope: float = 1.0, correction: bool = False, identity: int = 0):
+        self.identity, self.correction = int(identity or 0), bool(correction)
+        if (self.identity or self.correction) and scoring != "softmax_raw":
+            raise ValueError("identity experts and a choice correction go with the scoring 'softmax_raw'")
+        if self.identity < 0 or (self.identity and weight_input):
+            raise ValueError("identity experts are weighted on their output")
+        if not 1 <= top <= experts + self.identity:
             raise ValueError("a token uses between one and all of the experts")
         if activation not in ops.ACTIVATIONS and activation not in ops.GATED_ACTIVATIONS:
             raise ValueError(f"unknown activation {activation!r}")
@@ -70,19 +80,25 @@ class MoEFeedForward(FeedForward):
         self.gated, self.router_bias, self.scoring = bool(gated), bool(router_bias), scoring
         self.groups = int(groups or 1)
         self.keep_groups = int(keep_groups) if keep_groups else self.groups
-        if experts % self.groups or not 1 <= self.keep_groups <= self.groups or self.keep_groups * (experts // self.groups) < top:
+        if scoring == "softmax_raw" and self.groups > 1:
+            raise ValueError("the scoring 'softmax_raw' has no groups of experts")
+        if self.groups > 1 and experts % self.groups or not 1 <= self.keep_groups <= self.groups or self.keep_groups * (experts + self.identity) // self.groups < top:
             raise ValueError("the experts must split into equal groups, and the kept groups must hold at least `top` experts")
         self.route_scale = float(route_scale)
         self.shared_gate = bool(shared_gate) and bool(shared_size)
         self.w_shared_gate = None
+        self.choice_correction: Optional[torch.Tensor] = None
         self.w_router = self.b_router = self.w_gate_up = self.w_down = None
         self.shared_gate_up = self.shared_down = None
 
     def tensor_specs(self) -> List[TensorSpec]:
         H, F = self.hidden_size, self.expert_size
-        specs = [TensorSpec("router", (self.experts, H))]
+        outputs = self.experts + self.identity
+        specs = [TensorSpec("router", (outputs, H))]
         if self.router_bias:
-            specs.append(TensorSpec("router.b", (self.experts,), role="vector", init="normal"))
+            specs.append(TensorSpec("router.b", (outputs,), role="vector", init="normal"))
+        if self.correction:
+            specs.append(TensorSpec("correction", (outputs,), role="vector", init="normal"))
         for e in range(self.experts):
             specs += ([TensorSpec(f"e{e}.gate", (F, H))] if self.gated else []) + \
                      [TensorSpec(f"e{e}.up", (F, H)), TensorSpec(f"e{e}.down", (H, F))]
@@ -98,6 +114,7 @@ class MoEFeedForward(FeedForward):
         E = self.experts
         self.w_router = tensors["router"].contiguous()
         self.b_router = tensors["router.b"].contiguous() if self.router_bias else None
+        self.choice_correction = tensors["correction"].to(torch.float32).contiguous() if self.correction else None
         # the first matrix of every expert: [gate rows; up rows] of a gated expert, the up rows of a plain one
         first = (lambda p: torch.cat([tensors[p + "gate"], tensors[p + "up"]], dim=0)) if self.gated else (lambda p: tensors[p + "up"])
         self.w_gate_up = torch.stack([first(f"e{e}.") for e in range(E)]).contiguous()
@@ -137,7 +154,7 @@ class MoEFeedForward(FeedForward):
                 shared_done = torch.cuda.Event()
                 shared_done.record(side)
         routed = ops.moe_route(h, self.w_router, self.b_router, self.top, self.scoring, self.groups, self.keep_groups,
-                               self.route_scale, self.w_shared_gate)
+                               self.route_scale, self.w_shared_gate, self.choice_correction, self.identity)
         ids, weights, counts = routed[:3]
         sgate = routed[3] if self.w_shared_gate is not None else None
         if shared_done is not None:
@@ -153,7 +170,8 @@ class MoEFeedForward(FeedForward):
         def combine(y, place):
             if shared_done is not None:
                 torch.cuda.current_stream().wait_event(shared_done)      # the shared expert's rows are there
-            ops.moe_combine(y, place, None if self.weight_input else weights, shared, out, sgate)
+            own = dict(ids=ids, experts=self.experts, x=h) if self.identity else {}
+            ops.moe_combine(y, place, None if self.weight_input else weights, shared, out, sgate, **own)
 
         if n <= GEMV_MAX_PAIRS and ops.moe_gemv_supported(h, self.w_gate_up) and self.expert_size % 8 == 0:
             # a decode step: nothing is sorted, every pair streams its expert's matrices once
@@ -163,11 +181,11 @@ class MoEFeedForward(FeedForward):
             ops.moe_gemv(act, 1, ids, self.w_down, y)
             combine(y, None)
             return out
-        offsets, srt, place, tiles, num_tiles, max_tiles = ops.moe_align(ids, counts)
+        offsets, srt, place, tiles, num_tiles, max_tiles = ops.moe_align(ids, counts, self.experts)
         if h.dtype == torch.bfloat16 and n >= GROUPED_LIBRARY_PAIRS and H % 8 == 0 and self.expert_size % 8 == 0:
             # many bfloat16 rows: the library's grouped product over the rows gathered in sorted order
             xs = ops.moe_gather(h, srt, self.top)
-            gate_up = torch._grouped_mm(xs, self.w_gate_up.transpose(1, 2), offs=offsets[1:])
+            gate_up = torch._grouped_mm(xs, self.w_gate_up.transpose(1, 2), offs=offsets[1:self.experts + 1])
             if glu:
                 act = torch.empty((n, self.expert_size), dtype=h.dtype, device=h.device)
                 if self.own_unit:
@@ -176,7 +194,7 @@ class MoEFeedForward(FeedForward):
                     ops.swiglu(gate_up, act, act_name)
             else:
                 act = ops.activation(gate_up, act_name)
-            y = torch._grouped_mm(act, self.w_down.transpose(1, 2), offs=offsets[1:])
+            y = torch._grouped_mm(act, self.w_down.transpose(1, 2), offs=offsets[1:self.experts + 1])
             combine(y, place)
             return out
         act = torch.empty((n, self.expert_size), dtype=h.dtype, device=h.device)

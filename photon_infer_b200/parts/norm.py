@@ -58,9 +58,17 @@ class RMSNorm(Norm):
 
     def add_forward(self, delta, residual, out_dtype):
         out = torch.empty(residual.shape, dtype=out_dtype, device=residual.device)
+        if self._fuses(delta):
+            ops.add_normed_rmsnorm(delta.tensor, delta.norm.weight, delta.norm.eps, residual, self.weight, self.eps, out)
+            return out
         d1, d2, sc = delta_terms(delta)
         ops.add_rmsnorm(d1, residual, self.weight, self.eps, out, delta2=d2, delta_scale=sc)
         return out
+
+    @staticmethod
+    def _fuses(delta) -> bool:
+        """A pending output that passes an RMS norm of its own: that norm, the sum and this norm are one kernel."""
+        return isinstance(delta, Normed) and isinstance(delta.norm, RMSNorm) and delta.bias is None
 
     def read_streams(self, delta, streams, w_in, out_dtype, rows=None):
         return _read_streams(self, False, delta, streams, w_in, out_dtype, rows)
@@ -69,6 +77,9 @@ class RMSNorm(Norm):
         if isinstance(delta, Connected):
             return self.read_streams(delta, residual, None, out_dtype, rows)[0]
         out = torch.empty((rows.numel(), residual.shape[1]), dtype=out_dtype, device=residual.device)
+        if self._fuses(delta):
+            ops.add_normed_rmsnorm(delta.tensor, delta.norm.weight, delta.norm.eps, residual, self.weight, self.eps, out, rows=rows)
+            return out
         d1, d2, sc = delta_terms(delta)
         ops.add_rmsnorm(d1, residual, self.weight, self.eps, out, rows=rows, delta2=d2, delta_scale=sc)
         return out

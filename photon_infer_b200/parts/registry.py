@@ -53,5 +53,5 @@ def create_part(table_name: str, kind: str, params: dict):
 
 
 def _ensure_builtin() -> None:
-    from . import (attention, block, delta_rule, diff_attention, gla, hyper, latent_attention, matrix_memory, mlp, moe,  # noqa: F401
+    from . import (attention, block, delta_rule, diff_attention, gla, hgrn2, hyper, latent_attention, matrix_memory, mlp, moe,  # noqa: F401
                    norm, normed_attention, rope, state_space, stream, talking_attention)                                       # (each registers itself)

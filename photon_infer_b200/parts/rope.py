@@ -24,11 +24,12 @@ from .base import PositionEncoding
 from .registry import register_position_encoding
 
 
-def inverse_frequencies(head_dim: int, theta: float, scaling: Optional[dict]) -> torch.Tensor:
-    """float64 arithmetic on the host, returned as float32 ``[head_dim / 2]``."""
+def scaled_frequencies(dims: int, base: float, scaling: Optional[dict] = None) -> torch.Tensor:
+    """Frequencies of the ``dims / 2`` pairs of ``dims`` rotated numbers, float64 ``[dims / 2]``; ``scaling`` as above (keys
+    ``factor``, ``low_freq_factor``, ``high_freq_factor``, ``original_max_position_embeddings``)."""
     out = []
-    for j in range(head_dim // 2):
-        f = float(theta) ** (-2.0 * j / head_dim)
+    for j in range(dims // 2):
+        f = float(base) ** (-2.0 * j / dims)
         if scaling is not None:
             factor = float(scaling["factor"])
             low = float(scaling["low_freq_factor"])
@@ -41,7 +42,12 @@ def inverse_frequencies(head_dim: int, theta: float, scaling: Optional[dict]) ->
                 s = (orig / lam - low) / (high - low)
                 f = (1.0 - s) * f / factor + s * f
         out.append(f)
-    return torch.tensor(out, dtype=torch.float64).to(torch.float32)
+    return torch.tensor(out, dtype=torch.float64)
+
+
+def inverse_frequencies(head_dim: int, theta: float, scaling: Optional[dict]) -> torch.Tensor:
+    """float64 arithmetic on the host, returned as float32 ``[head_dim / 2]``."""
+    return scaled_frequencies(head_dim, theta, scaling).to(torch.float32)
 
 
 class RotaryEncoding(PositionEncoding):

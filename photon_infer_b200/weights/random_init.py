@@ -23,6 +23,10 @@ from ..parts.base import TensorSpec
 from .safetensors_io import write_safetensors
 
 
+#: Numbers of the init "unit" are uniform between 0 and this: bounds of gates stay below 1 in bfloat16 as well.
+UNIT_BELOW = 0.95
+
+
 def _generator(seed: int, name: str) -> torch.Generator:
     digest = hashlib.sha256(f"{seed}:{name}".encode()).digest()
     g = torch.Generator(device="cpu")
@@ -44,6 +48,8 @@ def random_tensor(spec: TensorSpec, name: str, seed: int, init_std: float, norm_
             t += norm_std * torch.randn(shape, generator=g, dtype=torch.float32)
     elif spec.init == "normal":
         t = init_std * torch.randn(shape, generator=g, dtype=torch.float32)
+    elif spec.init == "unit":
+        t = UNIT_BELOW * torch.rand(shape, generator=g, dtype=torch.float32)
     elif spec.init == "eye":
         t = torch.eye(*shape, dtype=torch.float32) + init_std * torch.randn(shape, generator=g, dtype=torch.float32)
     else:
@@ -102,6 +108,8 @@ def random_tensors_on_device(declared: Dict[str, TensorSpec], run_dtype: torch.d
                 t += norm_std * torch.randn(shape, generator=g, dtype=dtype, device=dev)
         elif spec.init == "normal":
             t = torch.empty(shape, dtype=dtype, device=dev).normal_(0.0, init_std, generator=g)
+        elif spec.init == "unit":
+            t = UNIT_BELOW * torch.rand(shape, generator=g, dtype=dtype, device=dev)
         elif spec.init == "eye":
             t = torch.empty(shape, dtype=dtype, device=dev).normal_(0.0, init_std, generator=g) + torch.eye(*shape, dtype=dtype, device=dev)
         else:

@@ -594,3 +594,107 @@ def milozen_plain_logits(folder: str, ids: Sequence[int]) -> torch.Tensor:
         cfg, tensors = milozen_plain_model(folder)
         _milozen_cache[key] = milozen_plain.forward(cfg, tensors, list(ids))
     return _milozen_cache[key]
+
+
+# ----------------------------------------------------------------------------- Fezavik
+
+def _vatt(heads, kv_heads, dim, vdim, scale, size=None, rot=None):
+    m = dict(heads=heads, kv_heads=kv_heads, dim=dim, vdim=vdim, scale=scale)
+    if rot is not None:
+        m["rot"] = rot
+    if size is not None:
+        m["mask"] = dict(size=size)
+    return dict(type="attention", mixer=m)
+
+
+def _vlat(heads, dim, rot_dim, vdim, kv_rank, q_rank, scale, size=None, base=10000.0, dims=None):
+    m = dict(heads=heads, dim=dim, rot_dim=rot_dim, vdim=vdim, kv_rank=kv_rank, q_rank=q_rank, scale=scale,
+             rot=dict(base=base, dims=rot_dim if dims is None else dims))
+    if size is not None:
+        m["mask"] = dict(size=size)
+    return dict(type="latent_attention", mixer=m)
+
+
+def _vgrn(heads, dim, vdim):
+    return dict(type="hgrn2", mixer=dict(heads=heads, dim=dim, vdim=vdim))
+
+
+def _vmoe(experts, top, ff, identity=0):
+    r = dict(experts=experts, top=top)
+    if identity:
+        r["identity"] = identity
+    return dict(mlp=dict(kind="moe", router=r, expert=dict(ff=ff)))
+
+
+_NONE = dict(mlp=None)
+_stretch = lambda factor, low, high, original: dict(factor=factor, low=low, high=high, original=original)
+
+# Tiny Fezavik configurations that differ in every size, in the order of the layers and in which optional pieces they have.
+TINY_FEZAVIK: Dict[str, dict] = {
+    # each kind of mixer; heads that fit the tensor cores' tiles, values wider than keys; a layer without a feed-forward
+    "fv_a": dict(
+        config=dict(architecture="Fezavik", vocab=150, width=64, norm=dict(eps=1e-5),
+                    layers=[dict(_vatt(6, 2, 16, 32, 0.3, 40, dict(base=5000.0, dims=8, scaling=_stretch(4.0, 1.0, 4.0, 64))), **_vmoe(6, 2, 32, 2)),
+                            dict(_vgrn(2, 12, 20), **_vmoe(4, 3, 24, 3)),
+                            dict(_vlat(3, 16, 8, 20, 24, 40, 0.3, 17, 500.0), **_NONE),
+                            dict(_vatt(3, 3, 32, 16, 0.2, 9, dict(base=300.0, dims=32)), **_vmoe(5, 4, 16, 1))]),
+        seed=61, init_std=0.1, norm_std=0.1, block_size=16),
+    # rows of 16s in the latent (tensor-core decoding in bfloat16), heads of 64 with values of 80; pages of 8
+    "fv_b": dict(
+        config=dict(architecture="Fezavik", vocab=210, width=96, norm=dict(eps=1e-6),
+                    layers=[dict(_vlat(4, 32, 16, 24, 48, 64, 0.2, 70), **_vmoe(8, 3, 24, 4)),
+                            dict(_vgrn(3, 32, 48), **_NONE),
+                            dict(_vatt(4, 2, 64, 80, 0.1, 33, dict(base=10000.0, dims=48, scaling=_stretch(8.0, 0.5, 3.0, 128))), **_vmoe(3, 3, 16)),
+                            dict(_vlat(18, 8, 32, 8, 64, 32, 0.25, None, 1e6, 20), **_vmoe(5, 5, 16, 1))]),
+        seed=62, init_std=0.08, norm_std=0.15, block_size=8),
+    # sizes that are multiples of nothing; windows of three keys and of one; a single expert beside identity experts
+    "fv_c": dict(
+        config=dict(architecture="Fezavik", vocab=77, width=50, norm=dict(eps=2e-5),
+                    layers=[dict(_vatt(5, 1, 10, 7, 0.4, 3, dict(base=50.0, dims=6)), **_vmoe(7, 3, 14, 2)),
+                            dict(_vgrn(3, 9, 33), **_vmoe(1, 2, 18, 3)),
+                            dict(_vlat(5, 7, 6, 9, 13, 11, 0.4, 1, 50.0), **_NONE),
+                            dict(_vgrn(1, 21, 5), **_vmoe(2, 1, 10))]),
+        seed=63, init_std=0.12, norm_std=0.05, block_size=16),
+    # wide heads: 128 x 128 of state, attention heads of 128, a wide latent; windows longer than most requests; pages of 32
+    "fv_d": dict(
+        config=dict(architecture="Fezavik", vocab=90, width=32, norm=dict(eps=1e-5),
+                    layers=[dict(_vgrn(1, 128, 128), **_vmoe(2, 2, 16, 2)),
+                            dict(_vlat(2, 64, 64, 128, 256, 24, 0.09, 100, 300000.0), **_vmoe(4, 1, 24, 4)),
+                            dict(_vatt(2, 1, 128, 128, 0.09, 160, dict(base=1e5, dims=64, scaling=_stretch(2.0, 1.0, 2.0, 32))), **_NONE)]),
+        seed=64, init_std=0.15, norm_std=0.1, block_size=32),
+    # no window and no rotation anywhere; more experts than a warp has lanes, no identity experts
+    "fv_e": dict(
+        config=dict(architecture="Fezavik", vocab=131, width=48, norm=dict(eps=1e-5),
+                    layers=[dict(_vatt(8, 4, 24, 8, 0.25), **_vmoe(40, 5, 8)),
+                            dict(_vlat(2, 16, 16, 24, 32, 20, 0.2, None, 777.0), **_vmoe(33, 2, 8, 30)),
+                            dict(_vgrn(4, 40, 8), **_vmoe(3, 2, 36, 1)),
+                            dict(_vatt(2, 2, 48, 96, 0.2), **_NONE)]),
+        seed=65, init_std=0.1, norm_std=0.1, block_size=16),
+}
+
+
+def make_fezavik_folder(path: str, name: str, dtype: str = "bfloat16") -> str:
+    from photon_infer_b200.weights import write_random_model
+    t = TINY_FEZAVIK[name]
+    write_random_model(path, t["config"], seed=t["seed"], init_std=t["init_std"], norm_std=t["norm_std"], dtype=dtype)
+    return path
+
+
+_fezavik_cache: Dict[tuple, torch.Tensor] = {}
+_fezavik_models: Dict[str, tuple] = {}
+
+
+def fezavik_plain_model(folder: str):
+    from plain import fezavik_plain
+    if folder not in _fezavik_models:
+        _fezavik_models[folder] = fezavik_plain.read_folder(folder)
+    return _fezavik_models[folder]
+
+
+def fezavik_plain_logits(folder: str, ids: Sequence[int]) -> torch.Tensor:
+    from plain import fezavik_plain
+    key = (folder, tuple(ids))
+    if key not in _fezavik_cache:
+        cfg, tensors = fezavik_plain_model(folder)
+        _fezavik_cache[key] = fezavik_plain.forward(cfg, tensors, list(ids))
+    return _fezavik_cache[key]

@@ -222,6 +222,7 @@ class _Step:
         nq, nkv, d, dv = self.dims
         ctx = self.ctx()
         q = torch.cat(self.q).reshape(-1, nq * d).to(DEV)
+        sink = torch.zeros(nq, device=DEV) if sink else None               # the extra key's score is 0
         out = torch.full((q.shape[0], nq * dv), float("nan"), dtype=self.dtype, device=DEV)
         if gate is not None:
             wide = torch.zeros(q.shape[0], nq * dv + 16, dtype=self.dtype, device=DEV)     # a view with a row stride, 16-byte aligned rows
