@@ -29,7 +29,10 @@ with a relu gate), beside a Llama decoder with the same window and the Finelix d
 the Pebodra decoder (norms on the sublayers' outputs; differential attention, some layers reading another layer's keys
 and values; state-space and matrix-memory layers; PolyNorm and routed feed-forwards), beside the same two.  ``--design milozen``
 does it for the Milozen decoder (parallel residual streams; attention over a cached latent with a window and an output
-gate, some layers reading another layer's latent; experts with bounded activations), beside the same two.
+gate, some layers reading another layer's latent; experts with bounded activations), beside the same two.  ``--design
+fezavik`` does it for the Fezavik decoder (norms around every sublayer; attention normed over whole projections with a window
+and a learned sink; latent attention with a sink and head gates; a recurrence whose forget gate also writes; experts with a
+choice correction and identity experts), beside Llama and the three designs that hold its mixers' closest relatives.
 
 ``--impl reference`` runs lumia431/photon_infer itself where it could be built (``baseline/``); else it
 prints an ``unavailable`` line.
@@ -380,7 +383,7 @@ def main() -> int:
     ap.add_argument("--layers-3b", type=int, default=0, help="fewer layers for the 3B workload (0: all 28)")
     ap.add_argument("--layers-8b", type=int, default=0, help="fewer layers for the 8B workload (0: all 32)")
     ap.add_argument("--batch-8b", type=int, default=8)
-    ap.add_argument("--design", default=None, choices=["finelix", "fekopel", "lerosun", "pebodra", "milozen"],
+    ap.add_argument("--design", default=None, choices=["finelix", "fekopel", "lerosun", "pebodra", "milozen", "fezavik"],
                     help="compare this design with a Llama decoder of equal size instead of running the headline")
     ap.add_argument("--design-sizes", default="2048,4096", help="widths to run with --design")
     args = ap.parse_args()

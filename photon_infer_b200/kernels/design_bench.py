@@ -1,8 +1,10 @@
-"""Prefill and decode throughput of another design (the Finelix, the Fekopel, the Lerosun, the Pebodra or the Milozen
-decoder) beside a Llama decoder of equal width, depth and feed-forward size (``python bench.py --design
-finelix|fekopel|lerosun|pebodra|milozen``), with the parts of a layer timed alone against their rooflines.  The Lerosun and
+"""Prefill and decode throughput of another design (the Finelix, the Fekopel, the Lerosun, the Pebodra, the Milozen or the
+Fezavik decoder) beside a Llama decoder of equal width, depth and feed-forward size (``python bench.py --design
+finelix|fekopel|lerosun|pebodra|milozen|fezavik``), with the parts of a layer timed alone against their rooflines.  The Lerosun and
 the Pebodra decoder also run beside the Finelix decoder, the other design with a recurrent mixer (a matrix of state per
-head) and routed experts next to attention, and so does the Milozen decoder, which shares latent attention with it.
+head) and routed experts next to attention, and so does the Milozen decoder, which shares latent attention with it.  The
+Fezavik decoder, whose three mixers each have a counterpart in another design, also runs beside Finelix (a recurrence with a
+decay per channel, experts), Milozen (latent attention with a window and a gate) and Fekopel (normed queries and keys, a sink).
 
 Random weights drawn on the device, synthetic token ids, bfloat16.  Per size:
 
@@ -120,6 +122,26 @@ def milozen_config(width: int, layers: int) -> dict:
                         for i in range(layers)])
 
 
+FEZAVIK_WINDOW = 1024
+
+
+def fezavik_config(width: int, layers: int) -> dict:
+    """Layers in the order attention, recurrence, latent attention, recurrence: heads of 128, four query heads per key/value
+    head, half of a head rotated by stretched frequencies; a recurrence with heads of 128 x 128; a latent of 512 + 64 with heads
+    of 128 + 64; windows of 1,024 keys.  16 experts of width and 4 identity experts, 2 per token, in every layer."""
+    heads = width // 128
+    mlp = dict(kind="moe", router=dict(experts=16, top=2, identity=4), expert=dict(ff=width))
+    mask = dict(size=FEZAVIK_WINDOW)
+    scaling = dict(factor=8.0, low=1.0, high=4.0, original=512)
+    att = dict(type="attention", mixer=dict(heads=heads, kv_heads=max(1, width // 512), dim=128, vdim=128, scale=128 ** -0.5, mask=mask,
+                                            rot=dict(base=10000.0, dims=64, scaling=scaling)), mlp=mlp)
+    lat = dict(type="latent_attention", mixer=dict(heads=heads, dim=128, rot_dim=64, vdim=128, kv_rank=512, q_rank=max(768, width * 3 // 8),
+                                                   scale=192 ** -0.5, mask=mask, rot=dict(base=10000.0, dims=64)), mlp=mlp)
+    rec = dict(type="hgrn2", mixer=dict(heads=heads, dim=128, vdim=128), mlp=mlp)
+    return dict(architecture="Fezavik", vocab=32000, width=width, norm=dict(eps=1e-5),
+                layers=[(att, rec, lat, rec)[i % 4] for i in range(layers)])
+
+
 def llama_config(width: int, layers: int, window=None) -> dict:
     cfg = dict(architectures=["LlamaForCausalLM"], hidden_size=width, intermediate_size=4 * width, num_hidden_layers=layers,
                num_attention_heads=width // 128, num_key_value_heads=max(1, width // 512), head_dim=128, vocab_size=32000,
@@ -177,11 +199,22 @@ def _time_graph(fn, reps: int = 8) -> float:
     return min(times) * 1e3
 
 
-def _part_bytes(part, kind: str, rows: int) -> int:
+def _pairs_with_products(part, h: torch.Tensor) -> int:
+    """(Token, choice) pairs of a routed feed-forward that go through an expert's matrices (the others chose an identity expert)."""
+    n = h.shape[0] * part.top
+    if not part.identity:
+        return n
+    from . import ops
+    ids = ops.moe_route(h, part.w_router, part.b_router, part.top, part.scoring, part.groups, part.keep_groups, part.route_scale,
+                        None, part.choice_correction, part.identity)[0]
+    return int((ids < part.experts).sum())
+
+
+def _part_bytes(part, kind: str, pairs: int) -> int:
     if kind == "moe":
         # a step reads the router, the shared expert and the experts that were chosen (all of them at most)
         expert = (part.w_gate_up[0].numel() + part.w_down[0].numel()) * part.w_down.element_size()
-        used = min(part.experts, rows * part.top)
+        used = min(part.experts, pairs)
         rest = part.weight_bytes() - part.experts * expert
         return rest + used * expert
     return part.weight_bytes()
@@ -190,7 +223,7 @@ def _part_bytes(part, kind: str, rows: int) -> int:
 def _mixer_numbers(m, kind: str, tokens: int, contexts) -> tuple:
     """(bytes of cache or state a step over ``contexts`` moves, floating-point operations of ``tokens`` rows)."""
     w = m.weight_bytes()
-    if kind == "gla":
+    if kind in ("gla", "hgrn2"):
         state = len(contexts) * m.heads * m.dim * m.vdim * 4 * 2
         flops = tokens * (w // 2) * 2 + 5 * tokens * m.heads * m.dim * m.vdim
         return state, flops
@@ -240,6 +273,7 @@ def _parts(runner, hbm_peak: float, tf_peak: float) -> Dict[str, dict]:
     from ..parts.matrix_memory import MatrixMemoryMixer
     from ..parts.state_space import StateSpaceMixer
     from ..parts.gla import GatedLinearAttention
+    from ..parts.hgrn2 import Hgrn2Mixer
     from ..parts.latent_attention import LatentAttention
     from ..parts.moe import MoEFeedForward
     from ..parts.normed_attention import NormedAttention
@@ -270,9 +304,10 @@ def _parts(runner, hbm_peak: float, tf_peak: float) -> Dict[str, dict]:
             m = block.mixer()
             kind = {GatedLinearAttention: "gla", LatentAttention: "latent", PagedAttention: "attention",
                     NormedAttention: "normed", TalkingAttention: "talking", GatedDeltaRule: "delta",
-                    DifferentialAttention: "diff", StateSpaceMixer: "ssm", MatrixMemoryMixer: "memory"}.get(type(m))
-            if kind == "normed":                     # the two kinds of layer are timed apart
-                kind_name = "normed_gated" if m.output_gate else "normed_sink"
+                    DifferentialAttention: "diff", StateSpaceMixer: "ssm", MatrixMemoryMixer: "memory",
+                    Hgrn2Mixer: "hgrn2"}.get(type(m))
+            if kind == "normed":                     # the kinds of layer are timed apart
+                kind_name = "normed_row" if m.norm_scope == "row" else "normed_gated" if m.output_gate else "normed_sink"
             elif kind == "latent":                   # a layer with a latent of its own, and one that reads another's rows
                 kind_name = "latent" if m.own_kv else "latent_reader"
             elif kind == "diff":                     # a layer that owns its keys and values, and one that reads another's
@@ -285,13 +320,18 @@ def _parts(runner, hbm_peak: float, tf_peak: float) -> Dict[str, dict]:
                 fkind = "polynorm"
             lc = runner._layer_caches[i]
             streams = getattr(block, "connect1", None)
-            norm_name = "norm" if streams is None else "streams"
+            behind = getattr(block, "post1", None)       # a norm behind the sublayer as well
+            norm_name = "streams" if streams is not None else "norm" if behind is None else "sandwich"
             if (norm_name, phase) not in seen and hasattr(block, "norm2") and not model.spec.layers[e.layer].block.kind == "output_norm":
                 seen.add((norm_name, phase))
                 y = torch.randn(T, H, device=model.device).to(model.dtype)
                 if streams is None:
                     x = torch.randn(T, H, device=model.device)
-                    step = lambda: block.norm1.add_forward(y, x, model.dtype)
+                    pending = y
+                    if behind is not None:
+                        from ..parts.base import Normed
+                        pending = Normed(y, behind)
+                    step = lambda: block.norm1.add_forward(pending, x, model.dtype)
                     moved = T * H * (2 * 4 + 2 * 2)
                 else:
                     from ..parts.base import Connected
@@ -310,10 +350,11 @@ def _parts(runner, hbm_peak: float, tf_peak: float) -> Dict[str, dict]:
             if fkind and (fkind, phase) not in seen:
                 seen.add((fkind, phase))
                 us = timer(lambda: ff.forward(h, ctx))
-                wb = _part_bytes(ff, fkind, T)
+                pairs = _pairs_with_products(ff, h) if fkind == "moe" else 0
+                wb = _part_bytes(ff, fkind, pairs)
                 if fkind == "moe":
                     expert = (ff.w_gate_up[0].numel() + ff.w_down[0].numel())
-                    active = (ff.weight_bytes() // ff.w_down.element_size() - ff.experts * expert) + ff.top * expert
+                    active = (ff.weight_bytes() // ff.w_down.element_size() - ff.experts * expert) + pairs / T * expert
                 else:
                     active = ff.weight_bytes() // ff.w_down.element_size()
                 frac = wb / (us * 1e-6) / (hbm_peak * 1e9) if phase == "decode" else 2 * T * active / (us * 1e-6) / (tf_peak * 1e12)
@@ -373,7 +414,7 @@ def run_design_comparison(design: str, args, hbm_peak: float, tf_peak: float, pe
     layers = {2048: 8, 4096: 4}
     make, window = {"finelix": (finelix_config, None), "fekopel": (fekopel_config, FEKOPEL_WINDOW),
                     "lerosun": (lerosun_config, LEROSUN_WINDOW), "pebodra": (pebodra_config, PEBODRA_WINDOW),
-                    "milozen": (milozen_config, MILOZEN_WINDOW)}[design]
+                    "milozen": (milozen_config, MILOZEN_WINDOW), "fezavik": (fezavik_config, FEZAVIK_WINDOW)}[design]
     line = {"design": design, "dtype": args.dtype, "data": "synthetic", "peaks": peak_src,
             "workload": {"prefill_tokens": PREFILL, "decode_batch": BATCH, "decode_context": PROMPT, "steps": steps,
                          "warmup": warmup}, "sizes": {}}
@@ -381,8 +422,10 @@ def run_design_comparison(design: str, args, hbm_peak: float, tf_peak: float, pe
         n_layers = layers.get(width, 4)
         point = {"layers": n_layers}
         models = [(design, make(width, n_layers)), ("llama", llama_config(width, n_layers, window))]
-        if design in ("lerosun", "pebodra", "milozen"):
+        if design in ("lerosun", "pebodra", "milozen", "fezavik"):
             models.append(("finelix", finelix_config(width, n_layers)))
+        if design == "fezavik":
+            models += [("milozen", milozen_config(width, n_layers)), ("fekopel", fekopel_config(width, n_layers))]
         for name, cfg in models:
             print(f"[bench] {name} width {width}, {n_layers} layers", file=sys.stderr, flush=True)
             model = random_model(cfg, args.dtype, seed=0)

@@ -665,18 +665,28 @@ TINY_FEZAVIK: Dict[str, dict] = {
     # no window and no rotation anywhere; more experts than a warp has lanes, no identity experts
     "fv_e": dict(
         config=dict(architecture="Fezavik", vocab=131, width=48, norm=dict(eps=1e-5),
-                    layers=[dict(_vatt(8, 4, 24, 8, 0.25), **_vmoe(40, 5, 8)),
+                    layers=[dict(_vatt(8, 4, 24, 8, 0.25), **_vmoe(40, 2, 8)),
                             dict(_vlat(2, 16, 16, 24, 32, 20, 0.2, None, 777.0), **_vmoe(33, 2, 8, 30)),
                             dict(_vgrn(4, 40, 8), **_vmoe(3, 2, 36, 1)),
                             dict(_vatt(2, 2, 48, 96, 0.2), **_NONE)]),
-        seed=65, init_std=0.1, norm_std=0.1, block_size=16),
+        seed=65, init_std=0.1, norm_std=0.1, block_size=16, correction_scale=8),
 }
 
 
 def make_fezavik_folder(path: str, name: str, dtype: str = "bfloat16") -> str:
+    """Random weights; the routers' are six times as large (and the choice's corrections, where the routers have many outputs,
+    eight times), so that few choices between experts are close calls: a norm stands behind the experts, so that another choice
+    changes the layer's output by as much as the output itself."""
     from photon_infer_b200.weights import write_random_model
+    from photon_infer_b200.weights.safetensors_io import SafetensorsFile, write_safetensors
     t = TINY_FEZAVIK[name]
     write_random_model(path, t["config"], seed=t["seed"], init_std=t["init_std"], norm_std=t["norm_std"], dtype=dtype)
+    file = os.path.join(path, "model.safetensors")
+    stored = SafetensorsFile(file)
+    tensors = {k: stored.read(k) for k in stored.entries}
+    stored.close()
+    factor = {"router": 6, "correction": t.get("correction_scale", 1)}
+    write_safetensors(file, {k: factor.get(k.rsplit(".", 1)[-1], 1) * v for k, v in tensors.items()})
     return path
 
 

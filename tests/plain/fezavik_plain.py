@@ -154,9 +154,9 @@ def route(h, w, top, forced=None):
 def moe_ff(h, w, mlp, forced=None):
     ids, weights = route(h, w, mlp["router"]["top"], forced)
     out = torch.zeros_like(h)
-    for t in range(h.shape[0]):
-        for e, s in zip(ids[t].tolist(), weights[t]):
-            out[t] += s * (expert(h[t][None], w, e)[0] if e < mlp["router"]["experts"] else h[t])
+    for e in torch.unique(ids).tolist():
+        t, j = (ids == e).nonzero(as_tuple=True)                # the tokens that use it, and as which of their choices
+        out[t] += weights[t, j, None] * (expert(h[t], w, e) if e < mlp["router"]["experts"] else h[t])
     return out
 
 
@@ -204,7 +204,7 @@ def read_folder(folder):
         if name == "__metadata__":
             continue
         a, b = info["data_offsets"]
-        tensors[name] = torch.frombuffer(bytearray(data[a:b]), dtype=_DT[info["dtype"]]).reshape(info["shape"]).clone()
+        tensors[name] = t64(torch.frombuffer(bytearray(data[a:b]), dtype=_DT[info["dtype"]]).reshape(info["shape"]))
     return cfg, tensors
 
 
