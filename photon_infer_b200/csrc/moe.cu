@@ -25,17 +25,18 @@
 // ---------------------------------------------------------------- router
 // A block owns `tok` consecutive tokens (at most its number of warps, at most 8): a warp takes every nwarp-th row of
 // the router and forms that row's logit for all of the block's tokens at once, so the row is read once per block.
-// Then warp i chooses for token i.  A logit's sum has the same order whatever `tok` is.  Measured on B200 with 2,048
+// Then warp i chooses for token i.  A logit's sum has the same order whatever `tok` and the number of warps are.  Measured on B200 with 2,048
 // tokens, 16 experts, rows of 2,048 (the call with its memset): one token per block 57 us, two 47, four 41, eight 59
 // (256 blocks, each walking its rows in sequence, are too few); 8 tokens: one per block 22 us, eight in one block 61.
+// Few tokens (TOK 1): one per block, a warp per row (up to 32), four loads of the row in flight.
 #define MOE_ROUTE_TOK 8
-template <typename T>
-__global__ void moe_route_kernel(const T* __restrict__ h, long h_stride, const T* __restrict__ Wr,
+template <typename T, int TOK>
+__global__ void __launch_bounds__(TOK == 1 ? 1024 : 256) moe_route_kernel(const T* __restrict__ h, long h_stride, const T* __restrict__ Wr,
                                  const void* __restrict__ bias, int bias_bf16, int H, int E, int top,
                                  int* __restrict__ ids, float* __restrict__ weights, int* __restrict__ counts, int T_,
                                  int mode, int n_groups, int keep_groups, float route_scale,
                                  const T* __restrict__ Wsg, float* __restrict__ shared_gate, int tok,
-                                 const float* __restrict__ correction, int real) {
+                                 const float* __restrict__ correction, int real, const float* __restrict__ given) {
   extern __shared__ float logits[];                     // per token: E (+ 1: the shared expert's gate) + n_groups flags (mode 3: + E)
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nwarp = blockDim.x >> 5;
   const int t0 = blockIdx.x * tok;
@@ -44,17 +45,24 @@ __global__ void moe_route_kernel(const T* __restrict__ h, long h_stride, const T
   constexpr int V = 16 / sizeof(T);                      // elements of a 16-byte load
   const bool vec = (H % V == 0) && ((uintptr_t)h % 16 == 0) && (h_stride % V == 0) && ((uintptr_t)Wr % 16 == 0) &&
                    ((uintptr_t)Wsg % 16 == 0);
-  for (int e = warp; e < E + (Wsg ? 1 : 0); e += nwarp) {
+  if (given) {                                           // the logits come from a product of their own
+    for (int i = threadIdx.x; i < ntok * E; i += blockDim.x) {
+      const int u = i / E, e = i - u * E;
+      logits[u * LS + e] = given[(size_t)(t0 + u) * E + e] + (bias ? load_w(bias, bias_bf16, e) : 0.f);
+    }
+  }
+  for (int e = given ? E + warp : warp; e < E + (Wsg ? 1 : 0); e += nwarp) {
     const T* w = e < E ? Wr + (size_t)e * H : Wsg;
-    float acc[MOE_ROUTE_TOK];
+    float acc[TOK];
 #pragma unroll
-    for (int i = 0; i < MOE_ROUTE_TOK; ++i) acc[i] = 0.f;
+    for (int i = 0; i < TOK; ++i) acc[i] = 0.f;
     if (vec) {
+#pragma unroll (TOK == 1 ? 4 : 1)
       for (int k = lane * V; k < H; k += 32 * V) {
         const uint4 wv = *reinterpret_cast<const uint4*>(w + k);
         const T* wp = reinterpret_cast<const T*>(&wv);
 #pragma unroll
-        for (int i = 0; i < MOE_ROUTE_TOK; ++i) {
+        for (int i = 0; i < TOK; ++i) {
           if (i < ntok) {
             const uint4 xv = *reinterpret_cast<const uint4*>(h + (size_t)(t0 + i) * h_stride + k);
             const T* xp = reinterpret_cast<const T*>(&xv);
@@ -67,13 +75,13 @@ __global__ void moe_route_kernel(const T* __restrict__ h, long h_stride, const T
       for (int k = lane; k < H; k += 32) {
         const float wk = to_f32(w[k]);
 #pragma unroll
-        for (int i = 0; i < MOE_ROUTE_TOK; ++i)
+        for (int i = 0; i < TOK; ++i)
           if (i < ntok) acc[i] = fmaf(to_f32(h[(size_t)(t0 + i) * h_stride + k]), wk, acc[i]);
       }
     }
     const float add = (bias && e < E) ? load_w(bias, bias_bf16, e) : 0.f;
 #pragma unroll
-    for (int i = 0; i < MOE_ROUTE_TOK; ++i) {
+    for (int i = 0; i < TOK; ++i) {
       if (i < ntok) {
         const float v = warp_sum(acc[i]);
         if (lane == 0) logits[i * LS + e] = v + add;
@@ -250,7 +258,7 @@ PHOTON_API int photon_moe_route(const void* h, long h_stride, int dtype, const v
                                 int T_, int H, int E, int top, int* ids, float* weights, int* counts,
                                 cudaStream_t stream) {
   return photon_moe_route_ex(h, h_stride, dtype, Wr, bias, bias_dtype, T_, H, E, top, ids, weights, counts, 0, 1, 1, 1.0f,
-                             nullptr, nullptr, nullptr, 0, stream);
+                             nullptr, nullptr, nullptr, 0, nullptr, stream);
 }
 
 // mode 0: as above.  mode 1: scores are the softmax over all experts; with n_groups > 1 the experts form that many
@@ -260,12 +268,13 @@ PHOTON_API int photon_moe_route(const void* h, long h_stride, int dtype, const v
 // by their sum.  mode 3: scores are the softmax over all experts, those with the largest score + correction [E] (may be
 // null) are chosen, the weights are the chosen scores without the correction times route_scale, not divided by their sum.
 // identity (mode 3): the last `identity` of the E router outputs are identity experts; counts has E - identity + 1 entries
-// then, the last of which counts all their pairs.  Wsg (may be null): one more row
+// then, the last of which counts all their pairs.  logits float [T][E] (may be null): z without the bias, from a product of
+// its own (Wr is not read).  Wsg (may be null): one more row
 // [H] of the router's type; shared_gate [T] then gets sigmoid(Wsg . h), the gate of a shared expert.
 PHOTON_API int photon_moe_route_ex(const void* h, long h_stride, int dtype, const void* Wr, const void* bias, int bias_dtype,
                                    int T_, int H, int E, int top, int* ids, float* weights, int* counts, int mode,
                                    int n_groups, int keep_groups, float route_scale, const void* Wsg, float* shared_gate,
-                                   const float* correction, int identity, cudaStream_t stream) {
+                                   const float* correction, int identity, const float* logits, cudaStream_t stream) {
   if (T_ <= 0) return 0;
   if (E <= 0 || top <= 0 || top > E || H <= 0) return PHOTON_ERR_ARGUMENT;
   if (mode < 0 || mode > 3) return PHOTON_ERR_ARGUMENT;
@@ -273,23 +282,21 @@ PHOTON_API int photon_moe_route_ex(const void* h, long h_stride, int dtype, cons
   if (n_groups < 1 || keep_groups < 1 || keep_groups > n_groups || E % n_groups) return PHOTON_ERR_ARGUMENT;
   if (mode != 0 && n_groups > 1 && (long)keep_groups * (E / n_groups) < top) return PHOTON_ERR_ARGUMENT;
   if ((Wsg == nullptr) != (shared_gate == nullptr)) return PHOTON_ERR_ARGUMENT;
-  const int warps = E >= 8 ? 8 : (E >= 4 ? 4 : 2);
   // few tokens (a decode step): one per block, so that every token's logits form on an SM of their own
-  const int tok = T_ >= 64 ? (warps < 4 ? warps : 4) : 1;
+  const bool few = T_ < 64;
+  const int warps = few ? (E + 1 < 32 ? (E + 1 < 2 ? 2 : E + 1) : 32) : (E >= 8 ? 8 : (E >= 4 ? 4 : 2));
+  const int tok = few ? 1 : (warps < 4 ? warps : 4);
   const size_t smem = (size_t)tok * (E + 1 + n_groups + (mode == 3 ? E : 0)) * sizeof(float);
   const int buckets = identity > 0 ? E - identity + 1 : E, real = identity > 0 ? E - identity : E;
   if (smem > 48 * 1024) return PHOTON_ERR_UNSUPPORTED;
   cudaError_t e = cudaMemsetAsync(counts, 0, (size_t)buckets * sizeof(int), stream);
   if (e != cudaSuccess) return (int)e;
   const int blocks = (T_ + tok - 1) / tok;
-  if (dtype == PHOTON_BF16)
-    moe_route_kernel<bf16><<<blocks, warps * 32, smem, stream>>>((const bf16*)h, h_stride, (const bf16*)Wr, bias,
-                                                                bias_dtype == PHOTON_BF16, H, E, top, ids, weights, counts, T_,
-                                                                mode, n_groups, keep_groups, route_scale, (const bf16*)Wsg, shared_gate, tok, correction, real);
-  else
-    moe_route_kernel<float><<<blocks, warps * 32, smem, stream>>>((const float*)h, h_stride, (const float*)Wr, bias,
-                                                                 bias_dtype == PHOTON_BF16, H, E, top, ids, weights, counts, T_,
-                                                                 mode, n_groups, keep_groups, route_scale, (const float*)Wsg, shared_gate, tok, correction, real);
+#define MOE_ROUTE(T, TOK) moe_route_kernel<T, TOK><<<blocks, warps * 32, smem, stream>>>((const T*)h, h_stride, (const T*)Wr, bias, \
+      bias_dtype == PHOTON_BF16, H, E, top, ids, weights, counts, T_, mode, n_groups, keep_groups, route_scale, (const T*)Wsg, shared_gate, \
+      tok, correction, real, logits)
+  if (dtype == PHOTON_BF16) { if (few) MOE_ROUTE(bf16, 1); else MOE_ROUTE(bf16, MOE_ROUTE_TOK); }
+  else { if (few) MOE_ROUTE(float, 1); else MOE_ROUTE(float, MOE_ROUTE_TOK); }
   return launch_status();
 }
 
@@ -472,12 +479,44 @@ PHOTON_API int photon_moe_gemm(const void* A, long lda, int dtype, const int* ga
 }
 
 // ---------------------------------------------------------------- weighted sum of the chosen experts
+__device__ __forceinline__ void moe_load4(const float* p, float* f) { const float4 r = *reinterpret_cast<const float4*>(p); f[0] = r.x; f[1] = r.y; f[2] = r.z; f[3] = r.w; }
+__device__ __forceinline__ void moe_load4(const bf16* p, float* f) {
+  const uint2 r = *reinterpret_cast<const uint2*>(p);
+  const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&r.x)), b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&r.y));
+  f[0] = a.x; f[1] = a.y; f[2] = b.x; f[3] = b.y;
+}
+__device__ __forceinline__ void moe_store4(float* p, const float* f) { *reinterpret_cast<float4*>(p) = make_float4(f[0], f[1], f[2], f[3]); }
+__device__ __forceinline__ void moe_store4(bf16* p, const float* f) {
+  __nv_bfloat162 a = __floats2bfloat162_rn(f[0], f[1]), b = __floats2bfloat162_rn(f[2], f[3]);
+  *reinterpret_cast<uint2*>(p) = make_uint2(*reinterpret_cast<uint32_t*>(&a), *reinterpret_cast<uint32_t*>(&b));
+}
+
 template <typename TY, typename TO>
 __global__ void moe_combine_kernel(const TY* __restrict__ y, long ldy, const int* __restrict__ place,
                                    const float* __restrict__ weights, int top, const TO* __restrict__ shared_out,
                                    TO* __restrict__ out, int H, const float* __restrict__ shared_gate,
-                                   const int* __restrict__ ids, int real, const TO* __restrict__ x, long ldx) {
+                                   const int* __restrict__ ids, int real, const TO* __restrict__ x, long ldx, int vec) {
   const int t = blockIdx.x;
+  if (vec) {
+    for (int i = (blockIdx.y * blockDim.x + threadIdx.x) * 4; i < H; i += gridDim.y * blockDim.x * 4) {
+      float acc[4] = {0.f, 0.f, 0.f, 0.f}, f[4];
+      for (int j = 0; j < top; ++j) {
+        const float w = weights ? weights[(size_t)t * top + j] : 1.0f;
+        if (ids && ids[(size_t)t * top + j] >= real) moe_load4(x + (size_t)t * ldx + i, f);
+        else moe_load4(y + (size_t)(place ? place[(size_t)t * top + j] : t * top + j) * ldy + i, f);
+#pragma unroll
+        for (int e = 0; e < 4; ++e) acc[e] = fmaf(w, f[e], acc[e]);
+      }
+      if (shared_out) {
+        const float sg = shared_gate ? shared_gate[t] : 1.0f;
+        moe_load4(shared_out + (size_t)t * H + i, f);
+#pragma unroll
+        for (int e = 0; e < 4; ++e) acc[e] += shared_gate ? sg * f[e] : f[e];
+      }
+      moe_store4(out + (size_t)t * H + i, acc);
+    }
+    return;
+  }
   for (int i = threadIdx.x; i < H; i += blockDim.x) {
     float acc = 0.f;
     for (int j = 0; j < top; ++j) {
@@ -507,24 +546,28 @@ PHOTON_API int photon_moe_combine_ex(const void* y, long ldy, int y_dtype, const
                                      long ldx, void* out, int out_dtype, int T_, int H, cudaStream_t stream) {
   if (T_ <= 0) return 0;
   if (ids != nullptr && x == nullptr) return PHOTON_ERR_ARGUMENT;
+  const uintptr_t ya = y_dtype == PHOTON_F32 ? 15 : 7, oa = out_dtype == PHOTON_F32 ? 15 : 7;       // four numbers at a time
+  const int vec = H % 4 == 0 && ldy % 4 == 0 && ldx % 4 == 0 && ((uintptr_t)y & ya) == 0 && ((uintptr_t)out & oa) == 0 &&
+                  ((uintptr_t)shared_out & oa) == 0 && ((uintptr_t)x & oa) == 0;
   const int threads = H >= 1024 ? 256 : 128;
-  if (out_dtype == PHOTON_BF16 && y_dtype == PHOTON_F32)
-    moe_combine_kernel<float, bf16><<<T_, threads, 0, stream>>>((const float*)y, ldy, place, weights, top, (const bf16*)shared_out, (bf16*)out, H, shared_gate, ids, real, (const bf16*)x, ldx);
-  else if (out_dtype == PHOTON_BF16 && y_dtype == PHOTON_BF16)
-    moe_combine_kernel<bf16, bf16><<<T_, threads, 0, stream>>>((const bf16*)y, ldy, place, weights, top, (const bf16*)shared_out, (bf16*)out, H, shared_gate, ids, real, (const bf16*)x, ldx);
-  else if (out_dtype == PHOTON_F32 && y_dtype == PHOTON_F32)
-    moe_combine_kernel<float, float><<<T_, threads, 0, stream>>>((const float*)y, ldy, place, weights, top, (const float*)shared_out, (float*)out, H, shared_gate, ids, real, (const float*)x, ldx);
-  else
-    return PHOTON_ERR_ARGUMENT;
+  const int cols = vec ? (H / 4 + threads - 1) / threads : 1;                 // few tokens: a token's columns over several blocks
+  const dim3 grid(T_, T_ < 64 && cols > 1 ? (cols < 16 ? cols : 16) : 1);
+#define MOE_COMBINE(TY, TO) moe_combine_kernel<TY, TO><<<grid, threads, 0, stream>>>((const TY*)y, ldy, place, weights, top, \
+      (const TO*)shared_out, (TO*)out, H, shared_gate, ids, real, (const TO*)x, ldx, vec)
+  if (out_dtype == PHOTON_BF16 && y_dtype == PHOTON_F32) MOE_COMBINE(float, bf16);
+  else if (out_dtype == PHOTON_BF16 && y_dtype == PHOTON_BF16) MOE_COMBINE(bf16, bf16);
+  else if (out_dtype == PHOTON_F32 && y_dtype == PHOTON_F32) MOE_COMBINE(float, float);
+  else return PHOTON_ERR_ARGUMENT;
   return launch_status();
 }
 
 // ---------------------------------------------------------------- rows in sorted order
 // out[r, :] = x[sorted[r] / div, :]: the input rows of the (token, choice) pairs, expert by expert, as the
-// library's grouped product wants them.
+// library's grouped product wants them.  used (may be null): rows from *used on (identity experts) are left as they are.
 template <typename T>
 __global__ void moe_gather_kernel(const T* __restrict__ x, long ldx, const int* __restrict__ sorted, int div,
-                                  T* __restrict__ out, int H) {
+                                  T* __restrict__ out, int H, const int* __restrict__ used) {
+  if (used && (int)blockIdx.x >= *used) return;
   const T* src = x + (size_t)(sorted[blockIdx.x] / div) * ldx;
   T* dst = out + (size_t)blockIdx.x * H;
   if (H % (16 / sizeof(T)) == 0 && (uintptr_t)src % 16 == 0 && (uintptr_t)dst % 16 == 0) {
@@ -537,11 +580,11 @@ __global__ void moe_gather_kernel(const T* __restrict__ x, long ldx, const int* 
 }
 
 PHOTON_API int photon_moe_gather(const void* x, long ldx, int dtype, const int* sorted, int div, void* out, int n, int H,
-                                 cudaStream_t stream) {
+                                 const int* used, cudaStream_t stream) {
   if (n <= 0) return 0;
   if (div <= 0) return PHOTON_ERR_ARGUMENT;
-  if (dtype == PHOTON_BF16) moe_gather_kernel<bf16><<<n, 128, 0, stream>>>((const bf16*)x, ldx, sorted, div, (bf16*)out, H);
-  else moe_gather_kernel<float><<<n, 128, 0, stream>>>((const float*)x, ldx, sorted, div, (float*)out, H);
+  if (dtype == PHOTON_BF16) moe_gather_kernel<bf16><<<n, 128, 0, stream>>>((const bf16*)x, ldx, sorted, div, (bf16*)out, H, used);
+  else moe_gather_kernel<float><<<n, 128, 0, stream>>>((const float*)x, ldx, sorted, div, (float*)out, H, used);
   return launch_status();
 }
 
@@ -550,8 +593,9 @@ PHOTON_API int photon_moe_gather(const void* x, long ldx, int dtype, const int* 
 template <typename T>
 __global__ void moe_glu_kernel(const T* __restrict__ gate_up, T* __restrict__ out, int I, int act,
                                const int* __restrict__ sorted, const float* __restrict__ weights, float limit, float slope,
-                               int vec) {
+                               int vec, const int* __restrict__ used) {
   const size_t r = blockIdx.x;
+  if (used && (int)r >= *used) return;
   const float f = weights ? weights[sorted[r]] : 1.0f;
   const T* g = gate_up + r * 2 * I;
   const T* u = g + I;
@@ -574,9 +618,10 @@ __global__ void moe_glu_kernel(const T* __restrict__ gate_up, T* __restrict__ ou
   }
 }
 
-// sorted [n] (pair index of each row) goes with weights [pairs]; weights null: no factors.  act: PHOTON_ACT_*.
+// sorted [n] (pair index of each row) goes with weights [pairs]; weights null: no factors.  act: PHOTON_ACT_*.  used: as
+// photon_moe_gather.
 PHOTON_API int photon_moe_glu(const void* gate_up, void* out, int dtype, int n, int I, int act, const int* sorted,
-                              const float* weights, float limit, float slope, cudaStream_t stream) {
+                              const float* weights, float limit, float slope, const int* used, cudaStream_t stream) {
   if (n <= 0 || I <= 0) return 0;
   if (weights && !sorted) return PHOTON_ERR_ARGUMENT;
   const int N = dtype == PHOTON_BF16 ? 8 : 4;
@@ -584,9 +629,9 @@ PHOTON_API int photon_moe_glu(const void* gate_up, void* out, int dtype, int n, 
   const int threads = 128, per = threads * (vec ? N : 1);
   const dim3 grid(n, (I + per - 1) / per < 8 ? (I + per - 1) / per : 8);
   if (dtype == PHOTON_BF16)
-    moe_glu_kernel<bf16><<<grid, threads, 0, stream>>>((const bf16*)gate_up, (bf16*)out, I, act, sorted, weights, limit, slope, vec);
+    moe_glu_kernel<bf16><<<grid, threads, 0, stream>>>((const bf16*)gate_up, (bf16*)out, I, act, sorted, weights, limit, slope, vec, used);
   else
-    moe_glu_kernel<float><<<grid, threads, 0, stream>>>((const float*)gate_up, (float*)out, I, act, sorted, weights, limit, slope, vec);
+    moe_glu_kernel<float><<<grid, threads, 0, stream>>>((const float*)gate_up, (float*)out, I, act, sorted, weights, limit, slope, vec, used);
   return launch_status();
 }
 

@@ -124,10 +124,11 @@ qk_norm_rope_write_kernel(const TI* q, long q_stride, const TI* k, long k_stride
 }
 
 // The norm over the whole projection: one block per token.  The row (q, then k) waits in shared memory as 32-bit numbers
-// while its two sums of squares form; the sines and cosines of the token's position are computed once for all heads.
-#define QKR_THREADS 256
+// while its two sums of squares form; beside that one more warp computes the sines and cosines of the token's position, once
+// for all heads.
+#define QKR_THREADS 256                                // and the warp for the angles
 template <typename TI, typename TO, bool VEC>
-__global__ void __launch_bounds__(QKR_THREADS)
+__global__ void __launch_bounds__(QKR_THREADS + 32)
 qk_row_norm_rope_write_kernel(const TI* q, long q_stride, const TI* k, long k_stride, const TI* v, long v_stride,
                               TO* q_out, long qo_stride, const void* __restrict__ q_w, const void* __restrict__ k_w,
                               int w_bf16, float eps, const int* __restrict__ positions,
@@ -142,12 +143,16 @@ qk_row_norm_rope_write_kernel(const TI* q, long q_stride, const TI* k, long k_st
   float* cs = xs + ((nq + nk + 3) & ~3);
   float* sn = cs + half;
   pdl_wait();
-  const double pos = (double)positions[t];
-  for (int j = tid; j < half; j += QKR_THREADS) {
-    double s, c;
-    sincos(pos * inv_freq[j], &s, &c);
-    cs[j] = (float)c;
-    sn[j] = (float)s;
+  if (warp == QKR_THREADS / 32) {
+    const double pos = (double)positions[t];
+    for (int j = lane; j < half; j += 32) {
+      double s, c;
+      sincos(pos * inv_freq[j], &s, &c);
+      cs[j] = (float)c;
+      sn[j] = (float)s;
+    }
+    __syncthreads();
+    return;
   }
   float sq = 0.f, sk = 0.f;
   const TI* qr = q + (size_t)t * q_stride;
@@ -206,8 +211,30 @@ qk_row_norm_rope_write_kernel(const TI* q, long q_stride, const TI* k, long k_st
     const int off = is_q ? i : i - nq, h = off / d, j = off - h * d;      // a head's first number is a multiple of STEP
     TO* dst = is_q ? q_out + (size_t)t * qo_stride + off : k_cache + (((size_t)page * n_kv + h) * page_size + at) * d + j;
     float f[STEP];
+    const void* w = is_q ? q_w : k_w;
+    const float inv = is_q ? qinv : kinv;
+    if constexpr (VEC) {
+      // whole quads of neighbours, or quads that are not rotated; the rest number by number
+      if (j >= rot_dims || (interleaved && j + 3 < rot_dims)) {
+        float wv[4] = {1.f, 1.f, 1.f, 1.f};
+        if (w) { if (w_bf16) qkn_load4((const bf16*)w + off, wv); else qkn_load4((const float*)w + off, wv); }
+        qkn_load4(xs + i, f);
 #pragma unroll
-    for (int u = 0; u < STEP; ++u) f[u] = value(i - j, j + u, is_q ? qinv : kinv, is_q ? q_w : k_w, h * d);
+        for (int u = 0; u < 4; ++u) f[u] = f[u] * inv * wv[u];
+        if (j < rot_dims) {
+          const float c0 = cs[j >> 1], s0 = sn[j >> 1], c1 = cs[(j >> 1) + 1], s1 = sn[(j >> 1) + 1];
+          const float a = f[0], b = f[2];
+          f[0] = a * c0 - f[1] * s0;
+          f[1] = f[1] * c0 + a * s0;
+          f[2] = b * c1 - f[3] * s1;
+          f[3] = f[3] * c1 + b * s1;
+        }
+        qkn_store4(dst, f);
+        continue;
+      }
+    }
+#pragma unroll
+    for (int u = 0; u < STEP; ++u) f[u] = value(i - j, j + u, inv, w, h * d);
     if constexpr (VEC) qkn_store4(dst, f); else *dst = from_f32<TO>(f[0]);
   }
   if (slot >= 0) {
@@ -246,7 +273,7 @@ PHOTON_API int photon_qk_norm_rope_write(const void* q, long q_stride, const voi
   const uintptr_t ia = in_dtype == PHOTON_F32 ? 16 : 8, oa = out_dtype == PHOTON_F32 ? 16 : 8;   // bytes of four elements
   const bool vec = d % 4 == 0 && dv % 4 == 0 && q_stride % 4 == 0 && k_stride % 4 == 0 && v_stride % 4 == 0 && qo_stride % 4 == 0 &&
                    (uintptr_t)q % ia == 0 && (uintptr_t)k % ia == 0 && (uintptr_t)v % ia == 0 && (uintptr_t)q_out % oa == 0 &&
-                   (uintptr_t)k_cache % oa == 0 && (uintptr_t)v_cache % oa == 0;
+                   (uintptr_t)k_cache % oa == 0 && (uintptr_t)v_cache % oa == 0 && (uintptr_t)q_w % 16 == 0 && (uintptr_t)k_w % 16 == 0;
 #define QKN_RUN(KERNEL, THREADS) do { \
     if (smem > 48 * 1024) { cudaError_t e_ = cudaFuncSetAttribute(KERNEL, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
                             if (e_ != cudaSuccess) return (int)e_; } \
@@ -257,7 +284,7 @@ PHOTON_API int photon_qk_norm_rope_write(const void* q, long q_stride, const voi
     typedef TI TI_; typedef TO TO_; \
     auto row_kernel = qk_row_norm_rope_write_kernel<TI, TO, VEC>; \
     auto head_kernel = qk_norm_rope_write_kernel<TI, TO, VEC>; \
-    if (whole_row) QKN_RUN(row_kernel, QKR_THREADS); \
+    if (whole_row) QKN_RUN(row_kernel, QKR_THREADS + 32); \
     QKN_RUN(head_kernel, QKN_WARPS * 32); } while (0)
 #define QKN_LAUNCH(TI, TO) do { if (vec) QKN_GO(TI, TO, true); else QKN_GO(TI, TO, false); } while (0)
   if (in_dtype == PHOTON_F32 && out_dtype == PHOTON_F32) QKN_LAUNCH(float, float);

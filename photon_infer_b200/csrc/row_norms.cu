@@ -97,6 +97,55 @@ group_rmsnorm_kernel(const TX* x, long x_stride, const float* gate, long gate_st
   }
 }
 
+// The plain form (no gate, no bias, no stream): a warp per part, the part in registers, QUADS groups of four numbers a lane.
+template <typename T> __device__ __forceinline__ void rn_load4(const T* p, float* f);
+template <> __device__ __forceinline__ void rn_load4<float>(const float* p, float* f) { const float4 r = *reinterpret_cast<const float4*>(p); f[0] = r.x; f[1] = r.y; f[2] = r.z; f[3] = r.w; }
+template <> __device__ __forceinline__ void rn_load4<bf16>(const bf16* p, float* f) {
+  const uint2 r = *reinterpret_cast<const uint2*>(p);
+  const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&r.x)), b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&r.y));
+  f[0] = a.x; f[1] = a.y; f[2] = b.x; f[3] = b.y;
+}
+__device__ __forceinline__ void rn_store4(float* p, const float* f) { *reinterpret_cast<float4*>(p) = make_float4(f[0], f[1], f[2], f[3]); }
+__device__ __forceinline__ void rn_store4(bf16* p, const float* f) {
+  __nv_bfloat162 a = __floats2bfloat162_rn(f[0], f[1]), b = __floats2bfloat162_rn(f[2], f[3]);
+  *reinterpret_cast<uint2*>(p) = make_uint2(*reinterpret_cast<uint32_t*>(&a), *reinterpret_cast<uint32_t*>(&b));
+}
+
+template <typename TX, typename TO, int QUADS>
+__global__ void __launch_bounds__(RN_THREADS)
+part_rmsnorm_kernel(const TX* __restrict__ x, long x_stride, const void* __restrict__ w, int w_bf16, TO* __restrict__ out, long out_stride,
+                    int gs, int groups, long parts, float eps) {
+  const int lane = threadIdx.x & 31;
+  const long part = (long)blockIdx.x * (RN_THREADS / 32) + (threadIdx.x >> 5);
+  if (part >= parts) return;
+  const long r = part / groups;
+  const int c0 = (int)(part - r * groups) * gs;
+  const TX* xr = x + r * x_stride + c0;
+  float v[QUADS][4];
+  float ss = 0.f;
+#pragma unroll
+  for (int u = 0; u < QUADS; ++u) {
+    const int i = (u * 32 + lane) * 4;
+#pragma unroll
+    for (int e = 0; e < 4; ++e) v[u][e] = 0.f;
+    if (i < gs) rn_load4<TX>(xr + i, v[u]);
+#pragma unroll
+    for (int e = 0; e < 4; ++e) ss += v[u][e] * v[u][e];
+  }
+  ss = warp_sum(ss);
+  const float inv = 1.0f / sqrtf(ss / (float)gs + eps);
+#pragma unroll
+  for (int u = 0; u < QUADS; ++u) {
+    const int i = (u * 32 + lane) * 4;
+    if (i < gs) {
+      float y[4];
+#pragma unroll
+      for (int e = 0; e < 4; ++e) y[e] = v[u][e] * inv * load_w(w, w_bf16, c0 + i + e);
+      rn_store4(out + r * out_stride + c0 + i, y);
+    }
+  }
+}
+
 // x [T][H] of x_dtype with row stride x_stride (elements); null with a residual: the stream's rows are only copied out.
 // gate: float [T][H] with row stride gate_stride, needed when gate_mode is 1 or 2.  residual: float [T][H] contiguous
 // or null.  w [H] of w_dtype.  out [T][H] of out_dtype with row stride out_stride, may be null when a residual is given.
@@ -114,7 +163,15 @@ PHOTON_API int photon_group_rmsnorm(const void* x, long x_stride, int x_dtype, c
   const size_t smem = (size_t)H * sizeof(float);
   if (smem > 200 * 1024) return PHOTON_ERR_UNSUPPORTED;
   const int wb = w_dtype == PHOTON_BF16;
+  const int gs = H / groups;
+  const uintptr_t ia = x_dtype == PHOTON_F32 ? 15 : 7, oa = out_dtype == PHOTON_F32 ? 15 : 7;      // four numbers at a time
+  const bool plain = x != nullptr && out != nullptr && residual == nullptr && gate_mode == 0 && x_bias == nullptr && groups >= RN_THREADS / 32 &&
+                     gs % 4 == 0 && gs <= 512 && x_stride % 4 == 0 && out_stride % 4 == 0 && ((uintptr_t)x & ia) == 0 && ((uintptr_t)out & oa) == 0;
+  const long parts = (long)T * groups;
+  const unsigned pblocks = (unsigned)((parts + RN_THREADS / 32 - 1) / (RN_THREADS / 32));
+#define RN_PART(TX, TO, Q) part_rmsnorm_kernel<TX, TO, Q><<<pblocks, RN_THREADS, 0, stream>>>((const TX*)x, x_stride, w, wb, (TO*)out, out_stride, gs, groups, parts, eps)
 #define RN_GO(TX, TO) do { \
+    if (plain) { if (gs <= 128) RN_PART(TX, TO, 1); else if (gs <= 256) RN_PART(TX, TO, 2); else RN_PART(TX, TO, 4); return launch_status(); } \
     if (smem > 48 * 1024) { cudaError_t e_ = cudaFuncSetAttribute(group_rmsnorm_kernel<TX, TO>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
                             if (e_ != cudaSuccess) return (int)e_; } \
     group_rmsnorm_kernel<TX, TO><<<T, RN_THREADS, smem, stream>>>((const TX*)x, x_stride, gate, gate_stride, gate_mode, residual, \

@@ -362,12 +362,12 @@ PHOTON_EXPORT int photon_moe_route(const void* h, long h_stride, int dtype, cons
  * be chosen from, weights = chosen scores / (their sum + 1e-20) * route_scale.  mode 2: scores are sigmoid(logit), a group's
  * score is the sum of its two largest, weights = chosen scores * route_scale.  mode 3: softmax over all experts, chosen by
  * score + correction [E] (may be null), weights = chosen scores * route_scale; the last `identity` outputs are identity
- * experts (counts then has E - identity + 1 entries).  Wsg [H] (may be null): shared_gate [T] =
+ * experts (counts then has E - identity + 1 entries).  logits float [T][E] (may be null): the product Wr h, formed before.  Wsg [H] (may be null): shared_gate [T] =
  * sigmoid(Wsg . h). */
 PHOTON_EXPORT int photon_moe_route_ex(const void* h, long h_stride, int dtype, const void* Wr, const void* bias, int bias_dtype, int T_,
                         int H, int E, int top, int* ids, float* weights, int* counts, int mode, int n_groups, int keep_groups,
                         float route_scale, const void* Wsg, float* shared_gate, const float* correction, int identity,
-                        cudaStream_t stream);
+                        const float* logits, cudaStream_t stream);
 /* Stable sort of the n = T * top pairs by expert: offsets [E + 1], sorted [n], place [n], tiles [3 * max_tiles] of
  * photon_moe_tile_rows() rows at most (expert, first row, rows), num_tiles [1].  real = E - 1: the last bucket holds the pairs
  * whose id is real or more (identity experts), without tiles; else real = E. */
@@ -383,7 +383,7 @@ PHOTON_EXPORT int photon_moe_gemm(const void* A, long lda, int dtype, const int*
                     int act, const float* weights, float limit, float slope, cudaStream_t stream);
 /* out [n][I] = act(w gate) * (w up), gate_up [n][2 I] of one dtype; row r's factor w = weights[sorted[r]] (weights null: 1). */
 PHOTON_EXPORT int photon_moe_glu(const void* gate_up, void* out, int dtype, int n, int I, int act, const int* sorted,
-                   const float* weights, float limit, float slope, cudaStream_t stream);
+                   const float* weights, float limit, float slope, const int* used, cudaStream_t stream);
 /* out[t] = sum_j weights[t, j] * y[place[t, j]] (+ shared_out[t]) (weights null: all 1); y [n][H] float or bfloat16; place null: row t * top + j. */
 PHOTON_EXPORT int photon_moe_combine(const void* y, long ldy, int y_dtype, const int* place, const float* weights, int top,
                        const void* shared_out, void* out, int out_dtype, int T_, int H, cudaStream_t stream);
@@ -392,9 +392,10 @@ PHOTON_EXPORT int photon_moe_combine(const void* y, long ldy, int y_dtype, const
 PHOTON_EXPORT int photon_moe_combine_ex(const void* y, long ldy, int y_dtype, const int* place, const float* weights, int top,
                           const void* shared_out, const float* shared_gate, const int* ids, int real, const void* x, long ldx,
                           void* out, int out_dtype, int T_, int H, cudaStream_t stream);
-/* out[r, :] = x[sorted[r] / div, :]: the pairs' input rows in sorted order. */
+/* out[r, :] = x[sorted[r] / div, :]: the pairs' input rows in sorted order; used (device, may be null; here and in
+ * photon_moe_glu): only rows r < *used. */
 PHOTON_EXPORT int photon_moe_gather(const void* x, long ldx, int dtype, const int* sorted, int div, void* out, int n, int H,
-                      cudaStream_t stream);
+                      const int* used, cudaStream_t stream);
 /* Few pairs (decode steps), bfloat16: out[p] = W[ids[p]] x[p / x_div], one matrix-vector product per pair, unsorted;
  * glu, weights (pair p's factor is weights[p]), limit and slope as photon_moe_gemm.  Pairs whose id is `experts` or more are
  * skipped. */

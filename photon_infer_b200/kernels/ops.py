@@ -1918,7 +1918,8 @@ def moe_tile_rows() -> int:
 
 def moe_route(h: torch.Tensor, w_router: torch.Tensor, bias: Optional[torch.Tensor], top: int,
               scoring: str = "softmax_chosen", groups: int = 1, keep_groups: int = 1, route_scale: float = 1.0,
-              w_shared_gate: Optional[torch.Tensor] = None, correction: Optional[torch.Tensor] = None, identity: int = 0):
+              w_shared_gate: Optional[torch.Tensor] = None, correction: Optional[torch.Tensor] = None, identity: int = 0,
+              logits: Optional[torch.Tensor] = None):
     """Router logits in 32-bit and the ``top`` experts of every token.  ``scoring`` ``softmax_chosen``: the largest
     logits win and the weights are the softmax over the chosen logits.  ``softmax_all``: scores are the softmax
     over all experts; the experts form ``groups`` equal groups of neighbours, a group's score is its largest
@@ -1928,10 +1929,13 @@ def moe_route(h: torch.Tensor, w_router: torch.Tensor, bias: Optional[torch.Tens
     sum).  ``softmax_raw``: scores are the softmax over all experts, the experts with the largest ``score + correction``
     (float32 ``[E]``, may be None) are chosen, and the weights are the chosen scores without the correction times
     ``route_scale``, not divided by their sum; the last ``identity`` of the ``E`` router outputs are identity experts, and
-    ``counts`` has ``E - identity + 1`` entries then, the last one for all of them.  ``w_shared_gate [1, H]``: also returns ``sigmoid(w . h)``
+    ``counts`` has ``E - identity + 1`` entries then, the last one for all of them.  ``logits`` (float32 ``[T, E]``): ``W_r h`` from a
+    product of its own; the kernel then only chooses.  ``w_shared_gate [1, H]``: also returns ``sigmoid(w . h)``
     per token.  Returns ``(ids int32 [T, top], weights float32 [T, top], counts int32 [E])`` or, with a gate,
     those and ``gate float32 [T]``."""
-    _cuda(h, w_router, bias, w_shared_gate, correction)
+    _cuda(h, w_router, bias, w_shared_gate, correction, logits)
+    if logits is not None and (logits.dtype != torch.float32 or logits.shape != (h.shape[0], w_router.shape[0]) or not logits.is_contiguous()):
+        raise PhotonError(ErrorCode.SHAPE_MISMATCH, "moe_route: logits must be contiguous float32 [T, E]")
     if scoring not in ROUTER_SCORING:
         raise PhotonError(ErrorCode.INVALID_ARGUMENT, f"moe_route: unknown scoring {scoring!r} ({', '.join(ROUTER_SCORING)})")
     T, H = h.shape
@@ -1950,11 +1954,11 @@ def moe_route(h: torch.Tensor, w_router: torch.Tensor, bias: Optional[torch.Tens
         gate = torch.empty(T, dtype=torch.float32, device=h.device)
     f = _fn("moe", "photon_moe_route_ex",
             [c_void_p, c_long, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p,
-             c_void_p, c_int, c_int, c_int, c_float, c_void_p, c_void_p, c_void_p, c_int, c_void_p])
+             c_void_p, c_int, c_int, c_int, c_float, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p])
     _check(f(_ptr(h), h.stride(0), _dtype_code(h), _ptr(w_router), _ptr(bias),
              _dtype_code(bias) if bias is not None else F32, T, H, E, int(top), _ptr(ids), _ptr(weights), _ptr(counts),
              ROUTER_SCORING[scoring], int(groups), int(keep_groups), float(route_scale), _ptr(w_shared_gate), _ptr(gate),
-             _ptr(correction), int(identity), _stream()), "moe_route")
+             _ptr(correction), int(identity), _ptr(logits), _stream()), "moe_route")
     if gate is not None:
         return ids, weights, counts, gate
     return ids, weights, counts
@@ -2019,8 +2023,9 @@ def _expert_act(glu: bool, activation: Optional[str]) -> int:
 
 
 def moe_glu(gate_up: torch.Tensor, out: torch.Tensor, activation: str, srt: Optional[torch.Tensor] = None,
-            weights: Optional[torch.Tensor] = None, limit: float = 0.0, slope: float = 1.0) -> None:
-    """The gated unit of the routed experts on rows in sorted order: ``gate_up [n, 2 I]`` -> ``out [n, I]``; with
+            weights: Optional[torch.Tensor] = None, limit: float = 0.0, slope: float = 1.0, used: Optional[torch.Tensor] = None) -> None:
+    """The gated unit of the routed experts on rows in sorted order: ``gate_up [n, 2 I]`` -> ``out [n, I]`` (``used``: as in
+    ``moe_gather``); with
     ``weights`` float32 (one per pair) and ``srt`` the sums of row ``r`` are multiplied by ``weights[srt[r]]`` first."""
     _cuda(gate_up, out, srt, weights)
     n, I2 = gate_up.shape
@@ -2028,9 +2033,10 @@ def moe_glu(gate_up: torch.Tensor, out: torch.Tensor, activation: str, srt: Opti
         raise PhotonError(ErrorCode.SHAPE_MISMATCH, "moe_glu: gate_up [n, 2 I] and out [n, I] of one dtype")
     if weights is not None and (srt is None or weights.numel() != n or weights.dtype != torch.float32 or not weights.is_contiguous()):
         raise PhotonError(ErrorCode.INVALID_ARGUMENT, "moe_glu: input factors are float32, one per pair, and need the sorted list")
-    f = _fn("moe", "photon_moe_glu", [c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_float, c_float, c_void_p])
+    f = _fn("moe", "photon_moe_glu", [c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_float, c_float,
+                                      c_void_p, c_void_p])
     _check(f(_ptr(gate_up), _ptr(out), _dtype_code(out), n, I2 // 2, _expert_act(True, activation), _ptr(srt), _ptr(weights),
-             float(limit), float(slope), _stream()), "moe_glu")
+             float(limit), float(slope), _ptr(_used_rows(used)), _stream()), "moe_glu")
 
 
 def moe_combine(y: torch.Tensor, place: Optional[torch.Tensor], weights: Optional[torch.Tensor], shared_out: Optional[torch.Tensor],
@@ -2061,13 +2067,22 @@ def moe_combine(y: torch.Tensor, place: Optional[torch.Tensor], weights: Optiona
              _ptr(ids), int(experts), _ptr(x), x.stride(0) if x is not None else 0, _ptr(out), _dtype_code(out), T, H, _stream()), "moe_combine")
 
 
-def moe_gather(x: torch.Tensor, srt: torch.Tensor, div: int) -> torch.Tensor:
-    """``out[r] = x[srt[r] // div]``: the pairs' input rows in sorted order."""
+def _used_rows(used: Optional[torch.Tensor]) -> Optional[torch.Tensor]:
+    """``used``: int32 ``[1]`` on the device, the number of sorted rows that belong to experts with matrices."""
+    if used is not None:
+        _cuda(used)
+        if used.dtype != torch.int32 or used.numel() != 1:
+            raise PhotonError(ErrorCode.SHAPE_MISMATCH, "the number of used rows must be one int32")
+    return used
+
+
+def moe_gather(x: torch.Tensor, srt: torch.Tensor, div: int, used: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """``out[r] = x[srt[r] // div]``: the pairs' input rows in sorted order; with ``used`` only the first ``used[0]`` of them."""
     _cuda(x, srt)
     n, H = srt.numel(), x.shape[1]
     out = torch.empty((n, H), dtype=x.dtype, device=x.device)
-    f = _fn("moe", "photon_moe_gather", [c_void_p, c_long, c_int, c_void_p, c_int, c_void_p, c_int, c_int, c_void_p])
-    _check(f(_ptr(x), x.stride(0), _dtype_code(x), _ptr(srt), int(div), _ptr(out), n, H, _stream()), "moe_gather")
+    f = _fn("moe", "photon_moe_gather", [c_void_p, c_long, c_int, c_void_p, c_int, c_void_p, c_int, c_int, c_void_p, c_void_p])
+    _check(f(_ptr(x), x.stride(0), _dtype_code(x), _ptr(srt), int(div), _ptr(out), n, H, _ptr(_used_rows(used)), _stream()), "moe_gather")
     return out
 
 

@@ -153,8 +153,11 @@ class MoEFeedForward(FeedForward):
                 shared_early = self._shared(h)
                 shared_done = torch.cuda.Event()
                 shared_done.record(side)
+        logits = None
+        if self.scoring == "softmax_raw" and T >= ROUTER_PRODUCT_ROWS and h.dtype == torch.bfloat16:
+            logits = project(h, self.w_router, out_dtype=torch.float32)     # bfloat16 operands, 32-bit sums, as in the router's kernel
         routed = ops.moe_route(h, self.w_router, self.b_router, self.top, self.scoring, self.groups, self.keep_groups,
-                               self.route_scale, self.w_shared_gate, self.choice_correction, self.identity)
+                               self.route_scale, self.w_shared_gate, self.choice_correction, self.identity, logits)
         ids, weights, counts = routed[:3]
         sgate = routed[3] if self.w_shared_gate is not None else None
         if shared_done is not None:
@@ -184,12 +187,13 @@ class MoEFeedForward(FeedForward):
         offsets, srt, place, tiles, num_tiles, max_tiles = ops.moe_align(ids, counts, self.experts)
         if h.dtype == torch.bfloat16 and n >= GROUPED_LIBRARY_PAIRS and H % 8 == 0 and self.expert_size % 8 == 0:
             # many bfloat16 rows: the library's grouped product over the rows gathered in sorted order
-            xs = ops.moe_gather(h, srt, self.top)
+            used = offsets[self.experts:self.experts + 1] if self.identity else None      # rows that reach a product
+            xs = ops.moe_gather(h, srt, self.top, used)
             gate_up = torch._grouped_mm(xs, self.w_gate_up.transpose(1, 2), offs=offsets[1:self.experts + 1])
             if glu:
                 act = torch.empty((n, self.expert_size), dtype=h.dtype, device=h.device)
-                if self.own_unit:
-                    ops.moe_glu(gate_up, act, act_name, srt=srt, **unit)
+                if self.own_unit or self.identity:
+                    ops.moe_glu(gate_up, act, act_name, srt=srt, used=used, **unit)
                 else:
                     ops.swiglu(gate_up, act, act_name)
             else:
@@ -218,6 +222,8 @@ def _side_stream(device) -> "torch.cuda.Stream":
     return _side_streams[key]
 
 
+#: From this many bfloat16 rows on the router's logits are a matrix product of their own (scoring ``softmax_raw``).
+ROUTER_PRODUCT_ROWS = 256
 #: Up to this many (token, choice) pairs a bfloat16 step runs one matrix-vector product per pair.
 GEMV_MAX_PAIRS = 64
 #: From this many pairs on a bfloat16 step hands the sorted rows to the library's grouped product.
