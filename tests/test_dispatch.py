@@ -42,7 +42,9 @@ def test_tcgen05_attention_sizes():
     for page in (8, 16, 32, 64, 128, 256):
         assert ops.attention_tc_supported(bf, 128, 4, page)
     assert not ops.attention_tc_supported(bf, 64, 129, 16)        # more rows per token than a tile holds
-    assert not ops.attention_tc_supported(bf, 96, 4, 16)          # heads of 64 or 128 only
+    assert ops.attention_tc_supported(bf, 96, 4, 16) and ops.attention_tc_supported(bf, 40, 4, 16, 88)     # zeros behind the head
+    assert not ops.attention_tc_supported(bf, 92, 4, 16)          # heads and values are multiples of 8 ..
+    assert not ops.attention_tc_supported(bf, 64, 4, 16, 136)     # .. of at most 128
     assert not ops.attention_tc_supported(bf, 64, 4, 4)           # a TMA box needs pages of 8 tokens or more
     assert not ops.attention_tc_supported(bf, 64, 4, 24)          # pages must divide 64 or be a multiple of it
     assert not ops.attention_tc_supported(bf, 64, 4, 96)

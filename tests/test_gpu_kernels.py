@@ -845,7 +845,9 @@ def test_attention_tcgen05_far_key_and_page_edges():
 def test_attention_tcgen05_refuses_other_sizes():
     from photon_infer_b200.errors import PhotonError
     from photon_infer_b200.kernels import ops
-    assert not ops.attention_tc_supported(torch.bfloat16, 80, 4, 16)
+    assert not ops.attention_tc_supported(torch.bfloat16, 84, 4, 16)
+    assert not ops.attention_tc_supported(torch.bfloat16, 136, 4, 16)
+    assert not ops.attention_tc_supported(torch.bfloat16, 64, 4, 16, 200)
     assert not ops.attention_tc_supported(torch.bfloat16, 64, 129, 16)
     assert not ops.attention_tc_supported(torch.bfloat16, 64, 4, 4)
     assert not ops.attention_tc_supported(torch.float32, 64, 4, 16)
