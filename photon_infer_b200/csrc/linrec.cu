@@ -409,14 +409,13 @@ static int linrec_launch(int rpl, dim3 grid, cudaStream_t stream, const float* q
 }
 
 // ---------------------------------------------------------------- a gate per row (mode 2)
-// A lane owns R rows x 2 columns of one (request, head)'s state, as pairs of neighbouring rows for the packed 32-bit
+// A lane owns R rows x 4 columns of one (request, head)'s state, as pairs of neighbouring rows for the packed 32-bit
 // instructions of sm_100 (a pair is two IEEE operations); L lanes share the columns, lane i of them holding the rows
-// (j L + i) 4 .. + 3, j < R / 4 (N <= L R).  A block of eight warps owns 16 * 32 / L neighbouring columns.  Per token a pair takes d = v -
-// S, S += k d, o += q S; the lanes' shares of the read-outs meet by shuffles in one tree over the lanes, so every token's
-// arithmetic is the same chain wherever its step starts.
-#ifndef LRR_C
+// (j L + i) 4 .. + 3, j < R / 4 (N <= L R).  A block of four warps owns 16 * 32 / L neighbouring columns.  Per token a pair takes
+// d = v - S, S += k d, o += q S; the lanes' shares of the read-outs meet by shuffles in one tree over the lanes, so every
+// token's arithmetic is the same chain wherever its step starts.  (Two columns a lane and eight warps take the same time for
+// one request of 2,048 tokens and 16 heads of 128 x 128, and a tenth more for 32 heads.)
 #define LRR_C 4                 // columns of a lane: 2 or 4
-#endif
 #define LRR_THREADS (512 / LRR_C)
 typedef unsigned long long lr_pair;
 struct alignas(LRR_C * 4) LrCols { float x[LRR_C]; };   // the lane's columns of one row
